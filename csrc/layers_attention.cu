@@ -1,0 +1,323 @@
+// Attention in the latent space of latent attention: the cached latent row is key and value of every head at once, the queries
+// arrive multiplied into that space.  A tile is up to BM consecutive (token, head) rows of one request; rows of a tile share every
+// latent row they read.  Scores and softmax weights stay in fp32: for the tensor cores a weight is split into two bf16 parts (the
+// rounded value and the rest), whose products with the latent rows are summed.
+//
+//   latent_attn_mma_kernel   bf16 latents up to 512 wide: mma.sync m16n8k16, latent tiles double-buffered with cp.async
+//   latent_attn_kernel       any width, bf16 or fp32 storage
+//   latent_combine_kernel    joins the key ranges of a split launch
+#include "layers.cuh"
+
+namespace dlp {
+
+__device__ __forceinline__ void mma16816(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+                 : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+__device__ __forceinline__ void ldsm_x4(uint32_t (&r)[4], const void* p) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_u32(p)));
+}
+__device__ __forceinline__ void ldsm_x2(uint32_t (&r)[2], const void* p) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x2.shared.b16 {%0,%1}, [%2];" : "=r"(r[0]), "=r"(r[1]) : "r"(smem_u32(p)));
+}
+__device__ __forceinline__ void ldsm_x4_t(uint32_t (&r)[4], const void* p) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_u32(p)));
+}
+__device__ __forceinline__ void cp_async16(void* dst, const void* src, bool ok) {
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(dst)), "l"(src), "r"(ok ? 16 : 0) : "memory");
+}
+__device__ __forceinline__ void cp_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+template <int N> __device__ __forceinline__ void cp_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
+// (x, y) -> packed bf16 pair and the packed remainder
+__device__ __forceinline__ void split_bf16(float x, float y, uint32_t& hi, uint32_t& lo) {
+    const __nv_bfloat162 h = __floats2bfloat162_rn(x, y);
+    const __nv_bfloat162 l = __floats2bfloat162_rn(x - __low2float(h), y - __high2float(h));
+    hi = *reinterpret_cast<const uint32_t*>(&h);
+    lo = *reinterpret_cast<const uint32_t*>(&l);
+}
+
+struct KeyRange { int len, lo, hi; };      // keys visible to the tile's last row; the part of them this split reads
+__device__ __forceinline__ KeyRange tile_keys(const LatentArgs& a, int row_last, int split, int step) {
+    KeyRange k;
+    k.len = min(a.pos[row_last / a.H] + 1, a.max_pages * a.page_size);
+    const int per = ((k.len + a.n_splits - 1) / a.n_splits + step - 1) / step * step;
+    k.lo = min(k.len, split * per);
+    k.hi = min(k.len, k.lo + per);
+    return k;
+}
+
+template <int MW, int RMAX>
+__global__ void __launch_bounds__(256, 1) latent_attn_mma_kernel(const LatentArgs a) {
+    constexpr int BM = 16 * MW, BN = 64, NW = 8 / MW, KPW = BN / NW, LS = BN + 4;
+    constexpr int NPAIR = (RMAX / 16 + NW - 1) / NW;      // 16-column output blocks of a warp
+    extern __shared__ __align__(16) uint8_t la_smem[];
+    const int Rc = a.Rc, LD = Rc + 8;
+    __nv_bfloat16* qs = reinterpret_cast<__nv_bfloat16*>(la_smem);
+    __nv_bfloat16* cs = qs + BM * LD;                     // [2][BN][LD]
+    float* S = reinterpret_cast<float*>(cs + 2 * BN * LD);
+    float* s_alpha = S + BM * LS;
+    float* s_l = s_alpha + BM;
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, mw = warp / NW, nw = warp % NW, g = lane >> 2, c = lane & 3;
+    const int tile = blockIdx.x, split = blockIdx.y;
+    pdl_wait();
+    const int row0 = a.tile_row0[tile], rows = a.tile_rows[tile];
+    if (rows <= 0) return;
+    const KeyRange kr = tile_keys(a, row0 + rows - 1, split, BN);
+    const int* bt = a.block_table + (size_t)a.tok_slot[row0 / a.H] * a.max_pages;
+    const __nv_bfloat16* cache = reinterpret_cast<const __nv_bfloat16*>(a.cache);
+    const int chunks = Rc / 8;
+    auto load_tile = [&](int k0, int b) {
+        for (int i = tid; i < BN * chunks; i += 256) {
+            const int kk = i / chunks, ch = i - kk * chunks, key = k0 + kk;
+            const bool ok = key < kr.hi;
+            const int kc = ok ? key : 0;
+            const size_t src = ((size_t)bt[kc / a.page_size] * a.page_size + kc % a.page_size) * Rc + ch * 8;
+            cp_async16(cs + ((size_t)b * BN + kk) * LD + ch * 8, cache + src, ok);
+        }
+        cp_commit();
+    };
+    const int n_tiles = (kr.hi - kr.lo + BN - 1) / BN;
+    if (n_tiles > 0) load_tile(kr.lo, 0);
+    {
+        const uint4* q = reinterpret_cast<const uint4*>(reinterpret_cast<const __nv_bfloat16*>(a.q) + (size_t)row0 * Rc);
+        for (int i = tid; i < BM * chunks; i += 256) {
+            const int r = i / chunks, ch = i - r * chunks;
+            *reinterpret_cast<uint4*>(qs + r * LD + ch * 8) = r < rows ? q[(size_t)r * chunks + ch] : make_uint4(0, 0, 0, 0);
+        }
+    }
+    constexpr int TPR = 256 / BM;                          // softmax threads per row
+    const int sr = tid / TPR, sub = tid % TPR;
+    const int my_pos = sr < rows ? a.pos[(row0 + sr) / a.H] : -1;
+    float m_run = -INFINITY, l_run = 0.f;
+    float acc[NPAIR][2][4] = {};
+    for (int it = 0; it < n_tiles; ++it) {
+        const int k0 = kr.lo + it * BN, b = it & 1;
+        if (it + 1 < n_tiles) { load_tile(k0 + BN, b ^ 1); cp_wait<1>(); } else { cp_wait<0>(); }
+        __syncthreads();
+        const __nv_bfloat16* ct = cs + (size_t)b * BN * LD;
+        {   // scores: 16 rows x KPW keys per warp
+            float sacc[KPW / 8][4] = {};
+            for (int k = 0; k < Rc; k += 16) {
+                uint32_t af[4];
+                ldsm_x4(af, qs + (mw * 16 + (lane & 15)) * LD + k + (lane >> 4) * 8);
+#pragma unroll
+                for (int j = 0; j < KPW / 8; ++j) {
+                    uint32_t bf[2];
+                    ldsm_x2(bf, ct + (nw * KPW + j * 8 + (lane & 7)) * LD + k + ((lane >> 3) & 1) * 8);
+                    mma16816(sacc[j], af, bf[0], bf[1]);
+                }
+            }
+#pragma unroll
+            for (int j = 0; j < KPW / 8; ++j)
+#pragma unroll
+                for (int e = 0; e < 4; ++e)
+                    S[(mw * 16 + g + (e >> 1) * 8) * LS + nw * KPW + j * 8 + c * 2 + (e & 1)] = sacc[j][e] * a.scale;
+        }
+        __syncthreads();
+        {   // running softmax
+            float* row = S + sr * LS;
+            float v[BN / TPR], mx = m_run;
+#pragma unroll
+            for (int i = 0; i < BN / TPR; ++i) {
+                const int kk = i * TPR + sub, key = k0 + kk;
+                v[i] = (key <= my_pos && key < kr.hi) ? row[kk] : -INFINITY;
+                mx = fmaxf(mx, v[i]);
+            }
+#pragma unroll
+            for (int x = 1; x < TPR; x <<= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, x));
+            const float ms = mx == -INFINITY ? 0.f : mx;
+            const float alpha = m_run == -INFINITY ? 0.f : expf(m_run - ms);
+            float sum = 0.f;
+#pragma unroll
+            for (int i = 0; i < BN / TPR; ++i) {
+                const float p = expf(v[i] - ms);
+                sum += p;
+                row[i * TPR + sub] = p;
+            }
+#pragma unroll
+            for (int x = 1; x < TPR; x <<= 1) sum += __shfl_xor_sync(0xffffffffu, sum, x);
+            l_run = l_run * alpha + sum;
+            m_run = mx;
+            if (sub == 0) s_alpha[sr] = alpha;
+        }
+        __syncthreads();
+        {   // context: 16 rows x this warp's 16-column blocks
+            const float a0 = s_alpha[mw * 16 + g], a1 = s_alpha[mw * 16 + g + 8];
+#pragma unroll
+            for (int j = 0; j < NPAIR; ++j)
+#pragma unroll
+                for (int n = 0; n < 2; ++n) { acc[j][n][0] *= a0; acc[j][n][1] *= a0; acc[j][n][2] *= a1; acc[j][n][3] *= a1; }
+#pragma unroll
+            for (int kk = 0; kk < BN / 16; ++kk) {
+                uint32_t hi[4], lo[4];
+                const float* r0 = S + (mw * 16 + g) * LS + kk * 16 + c * 2;
+                const float* r1 = r0 + 8 * LS;
+                split_bf16(r0[0], r0[1], hi[0], lo[0]);
+                split_bf16(r1[0], r1[1], hi[1], lo[1]);
+                split_bf16(r0[8], r0[9], hi[2], lo[2]);
+                split_bf16(r1[8], r1[9], hi[3], lo[3]);
+#pragma unroll
+                for (int j = 0; j < NPAIR; ++j) {
+                    const int col = (j * NW + nw) * 16;
+                    if (col < Rc) {
+                        uint32_t bf[4];
+                        ldsm_x4_t(bf, ct + (kk * 16 + (lane & 15)) * LD + col + (lane >> 4) * 8);
+                        mma16816(acc[j][0], hi, bf[0], bf[1]);
+                        mma16816(acc[j][1], hi, bf[2], bf[3]);
+                        mma16816(acc[j][0], lo, bf[0], bf[1]);
+                        mma16816(acc[j][1], lo, bf[2], bf[3]);
+                    }
+                }
+            }
+        }
+        __syncthreads();      // the next load overwrites this tile's buffer two iterations on, S in the next one
+    }
+    pdl_launch_dependents();
+    if (sub == 0) {
+        s_l[sr] = l_run;
+        if (a.n_splits > 1 && sr < rows) {
+            float* ml = a.part_ml + ((size_t)split * a.T * a.H + row0 + sr) * 2;
+            ml[0] = m_run;
+            ml[1] = l_run;
+        }
+    }
+    __syncthreads();
+#pragma unroll
+    for (int half = 0; half < 2; ++half) {
+        const int r = mw * 16 + g + half * 8;
+        if (r >= rows) continue;
+        const float inv = s_l[r] > 0.f ? 1.f / s_l[r] : 0.f;
+        const size_t row = (size_t)row0 + r;
+#pragma unroll
+        for (int j = 0; j < NPAIR; ++j)
+#pragma unroll
+            for (int n = 0; n < 2; ++n) {
+                const int col = (j * NW + nw) * 16 + n * 8 + c * 2;
+                if (col >= Rc) continue;
+                const float x = acc[j][n][half * 2], y = acc[j][n][half * 2 + 1];
+                if (a.n_splits > 1)
+                    *reinterpret_cast<float2*>(a.part_o + ((size_t)split * a.T * a.H + row) * Rc + col) = make_float2(x, y);
+                else
+                    *reinterpret_cast<__nv_bfloat162*>(reinterpret_cast<__nv_bfloat16*>(a.out) + row * Rc + col) = __floats2bfloat162_rn(x * inv, y * inv);
+            }
+    }
+}
+
+// ---- any width, any storage: one CTA per (token, head) row and key range --------------------------------------------
+template <typename WT>
+__global__ void __launch_bounds__(128) latent_attn_kernel(const LatentArgs a) {
+    extern __shared__ __align__(16) uint8_t la_smem[];
+    float* q = reinterpret_cast<float*>(la_smem);         // [Rc]
+    float* acc = q + a.Rc;                                // [Rc]
+    float* s = acc + a.Rc;                                // [64]
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const int row = blockIdx.x, t = row / a.H, split = blockIdx.y, Rc = a.Rc;
+    pdl_wait();
+    const KeyRange kr = tile_keys(a, row, split, 64);
+    const int* bt = a.block_table + (size_t)a.tok_slot[t] * a.max_pages;
+    const WT* cache = reinterpret_cast<const WT*>(a.cache);
+    for (int r = tid; r < Rc; r += 128) {
+        q[r] = (float)reinterpret_cast<const WT*>(a.q)[(size_t)row * Rc + r];
+        acc[r] = 0.f;
+    }
+    float m = -INFINITY, l = 0.f;
+    for (int k0 = kr.lo; k0 < kr.hi; k0 += 64) {
+        __syncthreads();
+        const int n = min(64, kr.hi - k0);
+        for (int kk = warp; kk < 64; kk += 4) {
+            float d = 0.f;
+            if (kk < n) {
+                const int key = k0 + kk;
+                const WT* cr = cache + ((size_t)bt[key / a.page_size] * a.page_size + key % a.page_size) * Rc;
+                for (int r = lane; r < Rc; r += 32) d = fmaf(q[r], (float)cr[r], d);
+            }
+            d = warp_sum(d);
+            if (lane == 0) s[kk] = kk < n ? d * a.scale : -INFINITY;
+        }
+        __syncthreads();
+        const float s0 = s[lane], s1 = s[lane + 32];
+        const float mn = fmaxf(m, warp_max(fmaxf(s0, s1)));
+        const float p0 = expf(s0 - mn), p1 = expf(s1 - mn), alpha = m == -INFINITY ? 0.f : expf(m - mn);
+        l = l * alpha + warp_sum(p0 + p1);
+        m = mn;
+        __syncthreads();
+        if (warp == 0) { s[lane] = p0; s[lane + 32] = p1; }
+        __syncthreads();
+        for (int r = tid; r < Rc; r += 128) {
+            float v = acc[r] * alpha;
+            for (int kk = 0; kk < n; ++kk) {
+                const int key = k0 + kk;
+                v = fmaf(s[kk], (float)cache[((size_t)bt[key / a.page_size] * a.page_size + key % a.page_size) * Rc + r], v);
+            }
+            acc[r] = v;
+        }
+    }
+    pdl_launch_dependents();
+    if (a.n_splits > 1) {
+        const size_t o = (size_t)split * a.T * a.H + row;
+        for (int r = tid; r < Rc; r += 128) a.part_o[o * Rc + r] = acc[r];
+        if (tid == 0) { a.part_ml[o * 2] = m; a.part_ml[o * 2 + 1] = l; }
+    } else {
+        const float inv = l > 0.f ? 1.f / l : 0.f;
+        for (int r = tid; r < Rc; r += 128) reinterpret_cast<WT*>(a.out)[(size_t)row * Rc + r] = (WT)(acc[r] * inv);
+    }
+}
+
+template <typename WT>
+__global__ void __launch_bounds__(128) latent_combine_kernel(const LatentArgs a) {
+    pdl_wait();
+    const int row = blockIdx.x;
+    const size_t stride = (size_t)a.T * a.H;
+    float m = -INFINITY, l = 0.f;
+    for (int s = 0; s < a.n_splits; ++s) m = fmaxf(m, a.part_ml[(s * stride + row) * 2]);
+    for (int s = 0; s < a.n_splits; ++s) {
+        const float ms = a.part_ml[(s * stride + row) * 2];
+        l += ms == -INFINITY ? 0.f : a.part_ml[(s * stride + row) * 2 + 1] * expf(ms - m);
+    }
+    const float inv = l > 0.f ? 1.f / l : 0.f;
+    for (int r = threadIdx.x; r < a.Rc; r += 128) {
+        float v = 0.f;
+        for (int s = 0; s < a.n_splits; ++s) {
+            const float ms = a.part_ml[(s * stride + row) * 2];
+            if (ms != -INFINITY) v = fmaf(a.part_o[(s * stride + row) * a.Rc + r], expf(ms - m), v);
+        }
+        reinterpret_cast<WT*>(a.out)[(size_t)row * a.Rc + r] = (WT)(v * inv);
+    }
+    pdl_launch_dependents();
+}
+
+template <int MW, int RMAX>
+static int launch_latent_mma(const LatentArgs& a, cudaStream_t s) {
+    constexpr int BM = 16 * MW;
+    const size_t smem = (size_t)(BM + 128) * (a.Rc + 8) * 2 + (size_t)BM * 68 * 4 + BM * 8;
+    DLP_REQUIRE(smem <= 227 * 1024, "latent_attention: %zu bytes of shared memory", smem);
+    auto kern = latent_attn_mma_kernel<MW, RMAX>;
+    if (first_use_on_device((const void*)kern)) DLP_CHECK_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024));
+    DLP_CHECK_CUDA(launch_pdl(kern, dim3(a.n_tiles, a.n_splits), dim3(256), smem, s, a));
+    return 0;
+}
+
+int latent_attention(const LatentArgs& a, int f32, cudaStream_t s) {
+    DLP_REQUIRE(a.q && a.cache && a.block_table && a.tok_slot && a.pos && a.out && a.tile_row0 && a.tile_rows, "latent_attention: null argument");
+    DLP_REQUIRE(a.H > 0 && a.Rc > 0 && a.Rc % 32 == 0 && a.T > 0 && a.n_tiles > 0 && a.page_size > 0 && a.max_pages > 0, "latent_attention: bad shape");
+    DLP_REQUIRE(a.n_splits >= 1 && a.n_splits <= 64 && (a.n_splits == 1 || (a.part_o && a.part_ml)), "latent_attention: %d key ranges", a.n_splits);
+    int rc = 0;
+    if (!f32 && a.Rc <= 512) {
+        DLP_REQUIRE(a.bm == 16 || a.bm == 32 || a.bm == 64, "latent_attention: tile of %d rows", a.bm);
+        if (a.Rc <= 128) rc = a.bm == 16 ? launch_latent_mma<1, 128>(a, s) : a.bm == 32 ? launch_latent_mma<2, 128>(a, s) : launch_latent_mma<4, 128>(a, s);
+        else rc = a.bm == 16 ? launch_latent_mma<1, 512>(a, s) : a.bm == 32 ? launch_latent_mma<2, 512>(a, s) : launch_latent_mma<4, 512>(a, s);
+    } else {
+        const size_t smem = (size_t)(2 * a.Rc + 64) * 4;
+        DLP_REQUIRE(smem <= 48 * 1024, "latent_attention: latent of %d", a.Rc);
+        DLP_CHECK_CUDA(f32 ? launch_pdl(latent_attn_kernel<float>, dim3(a.T * a.H, a.n_splits), dim3(128), smem, s, a)
+                           : launch_pdl(latent_attn_kernel<__nv_bfloat16>, dim3(a.T * a.H, a.n_splits), dim3(128), smem, s, a));
+    }
+    if (rc) return rc;
+    if (a.n_splits > 1) {
+        if (f32) DLP_CHECK_CUDA(launch_pdl(latent_combine_kernel<float>, dim3(a.T * a.H), dim3(128), 0, s, a));
+        else DLP_CHECK_CUDA(launch_pdl(latent_combine_kernel<__nv_bfloat16>, dim3(a.T * a.H), dim3(128), 0, s, a));
+    }
+    return 0;
+}
+
+}  // namespace dlp

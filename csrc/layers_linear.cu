@@ -1,0 +1,444 @@
+// Matrix products of the layer-list models and the row preparation around them.
+//
+//   matvec_kernel        decode (1..4 rows): weights streamed once; the residual sum and the norms in front of a product run in the
+//                        prologue, GEGLU in the epilogue.  Any N, any K whose padded form is a multiple of 8.
+//   stage_rows_kernel    the same row preparation as one launch, for the tcgen05 GEMM sizes.
+//   sgemm_kernel         fp32 storage, any number of rows (no reduced-precision product).
+//   head_matmul_kernel   one small matrix per head (latent attention's key absorption and value expansion), mma.sync m16n8k16.
+#include "layers.cuh"
+
+namespace dlp {
+
+template <typename T> struct Act;
+template <> struct Act<__nv_bfloat16> {
+    static constexpr int VEC = 8;
+    static __device__ __forceinline__ float to_f(__nv_bfloat16 v) { return __bfloat162float(v); }
+    static __device__ __forceinline__ __nv_bfloat16 from_f(float v) { return __float2bfloat16_rn(v); }
+};
+template <> struct Act<float> {
+    static constexpr int VEC = 4;
+    static __device__ __forceinline__ float to_f(float v) { return v; }
+    static __device__ __forceinline__ float from_f(float v) { return v; }
+};
+
+__device__ __forceinline__ float gelu_tanh_f(float z) {
+    return 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
+}
+
+// ---- row preparation ------------------------------------------------------------------------------------
+// NT rows starting at t0, all threads of the block.  `put(t, k, v)` receives every value of the padded row.  `sums` holds
+// stage_scratch(NT, groups) floats; ends with a barrier.
+__host__ __device__ inline int stage_parts(int rows, int groups, int nwarps) {
+    const int tg = rows * groups;
+    return tg >= nwarps ? 1 : (nwarps + tg - 1) / tg;
+}
+__host__ __device__ inline int stage_scratch(int rows, int groups, int nwarps) { return rows * groups * (stage_parts(rows, groups, nwarps) + 1); }
+
+template <typename XT>
+__device__ __forceinline__ float stage_x0(const RowStage& p, int t, int k) {
+    return p.x_f32 ? reinterpret_cast<const float*>(p.x)[(size_t)t * p.ldx + k] : Act<XT>::to_f(reinterpret_cast<const XT*>(p.x)[(size_t)t * p.ldx + k]);
+}
+
+// reciprocal root mean square of every (row, group) of f(t, k) -> sums[rows * groups * parts + t * groups + g]; returns that base
+template <typename F>
+__device__ __forceinline__ float* stage_rms(int rows, int groups, int K, float eps, float* sums, F f) {
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5;
+    const int parts = stage_parts(rows, groups, nw), gs = K / groups, per = ((gs + parts - 1) / parts + 31) / 32 * 32;
+    for (int i = warp; i < rows * groups * parts; i += nw) {
+        const int tg = i / parts, part = i - tg * parts, t = tg / groups, g = tg - t * groups;
+        const int lo = part * per, hi = min(gs, lo + per);
+        float a = 0.f;
+#pragma unroll 4
+        for (int k = lo + lane; k < hi; k += 32) {
+            const float v = f(t, g * gs + k);
+            a = fmaf(v, v, a);
+        }
+        a = warp_sum(a);
+        if (lane == 0) sums[i] = a;
+    }
+    __syncthreads();
+    float* rs = sums + rows * groups * parts;
+    for (int i = threadIdx.x; i < rows * groups; i += blockDim.x) {
+        float a = 0.f;
+        for (int j = 0; j < parts; ++j) a += sums[i * parts + j];
+        rs[i] = 1.f / sqrtf(a / (float)gs + eps);
+    }
+    __syncthreads();
+    return rs;
+}
+
+template <typename XT, int NT, typename Put>
+__device__ __forceinline__ void stage_rows_dev(const RowStage& p, int t0, int rows, float* sums, bool store_h, Put put) {
+    const float* rs1 = nullptr;
+    const float* rs2 = nullptr;
+    const int gs1 = p.y ? p.K / p.groups1 : 1, gs2 = p.w2 ? p.K / p.groups2 : 1;
+    if (p.y) rs1 = stage_rms(rows, p.groups1, p.K, p.eps, sums, [&](int t, int k) { return p.y[(size_t)(t0 + t) * p.ldy + k]; });
+    auto base = [&](int t, int k) {
+        float v = stage_x0<XT>(p, t0 + t, k);
+        if (p.y) v += p.y[(size_t)(t0 + t) * p.ldy + k] * rs1[t * p.groups1 + k / gs1] * p.w1[k];
+        return v;
+    };
+    if (p.w2) rs2 = stage_rms(rows, p.groups2, p.K, p.eps, sums + (p.y ? stage_scratch(rows, p.groups1, blockDim.x >> 5) : 0), base);
+    for (int t = 0; t < rows; ++t) {
+#pragma unroll 4
+        for (int k = threadIdx.x; k < p.Kp; k += blockDim.x) {
+            float v = 0.f;
+            if (k < p.K) {
+                v = base(t, k);
+                if (store_h && p.h_out) p.h_out[(size_t)(t0 + t) * p.ldh + k] = v;
+                if (p.w2) v *= rs2[t * p.groups2 + k / gs2] * p.w2[k % p.w2_mod];
+            }
+            put(t, k, v);
+        }
+    }
+    __syncthreads();
+}
+static size_t stage_bytes(const RowStage& p, int rows, int nwarps) {
+    return ((size_t)(p.y ? stage_scratch(rows, p.groups1, nwarps) : 0) + (p.w2 ? stage_scratch(rows, p.groups2, nwarps) : 0)) * 4 + 16;
+}
+
+template <typename XT>
+__global__ void __launch_bounds__(256) stage_rows_kernel(const RowStage p, XT* xb, int ldxb) {
+    extern __shared__ __align__(16) float st_sums[];
+    pdl_wait();
+    const int t0 = blockIdx.x;
+    stage_rows_dev<XT, 1>(p, t0, 1, st_sums, true, [&](int, int k, float v) { xb[(size_t)t0 * ldxb + k] = Act<XT>::from_f(v); });
+    pdl_launch_dependents();
+}
+
+// ---- decode mat-vec ------------------------------------------------------------------------------------------
+// A unit is two weight rows x (32 * VEC * U) columns: U 16-byte loads per row and lane.  A block owns a contiguous range of row
+// pairs, its warps take the units in a fixed order and always hold the next unit's loads while they reduce the current one.  The
+// first unit is requested before the dependency wait: weights do not depend on the previous kernel.
+template <typename WT, int NT>
+__global__ void __launch_bounds__(512, 1) matvec_kernel(const RowStage st, const WT* __restrict__ w, int ldw, int N, void* out, int ldo, int out_mode, int T) {
+    constexpr int VEC = Act<WT>::VEC, U = 4, COLS = 32 * VEC * U;
+    extern __shared__ __align__(16) uint8_t mv_smem[];
+    WT* xs = reinterpret_cast<WT*>(mv_smem);
+    const int K = st.Kp;
+    size_t off = ((size_t)NT * K * sizeof(WT) + 15) & ~size_t(15);
+    float* sums = reinterpret_cast<float*>(mv_smem + off);
+    const int KC = (K + COLS - 1) / COLS;
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5;
+    const int pairs = (N + 1) / 2;
+    const int p_lo = (int)((long long)pairs * blockIdx.x / gridDim.x), p_hi = (int)((long long)pairs * (blockIdx.x + 1) / gridDim.x);
+    const int units = (p_hi - p_lo) * KC;
+    uint4 buf[2][2][U];
+    auto issue = [&](int u, int b) {
+        const int pr = u / KC, c = u - pr * KC, row = (p_lo + pr) * 2;
+        const WT* r0 = w + (size_t)row * ldw + c * COLS + lane * VEC;
+        const WT* r1 = w + (size_t)min(row + 1, N - 1) * ldw + c * COLS + lane * VEC;
+#pragma unroll
+        for (int i = 0; i < U; ++i) {
+            const bool ok = c * COLS + i * 32 * VEC + lane * VEC < K;
+            buf[b][0][i] = ok ? ldg_nc_v4(r0 + i * 32 * VEC) : make_uint4(0, 0, 0, 0);
+            buf[b][1][i] = ok ? ldg_nc_v4(r1 + i * 32 * VEC) : make_uint4(0, 0, 0, 0);
+        }
+    };
+    int u = warp;
+    if (u < units) issue(u, 0);
+    pdl_wait();
+    stage_rows_dev<WT, NT>(st, 0, T, sums, blockIdx.x == 0, [&](int t, int k, float v) { xs[(size_t)t * K + k] = Act<WT>::from_f(v); });
+    float* part = sums;      // [units][2][NT]: the staging scratch is free again
+    auto reduce = [&](int u, int b) {
+        const int pr = u / KC, c = u - pr * KC;
+        float acc[2][NT];
+#pragma unroll
+        for (int m = 0; m < 2; ++m)
+#pragma unroll
+            for (int t = 0; t < NT; ++t) acc[m][t] = 0.f;
+#pragma unroll
+        for (int i = 0; i < U; ++i) {
+            const int k = c * COLS + i * 32 * VEC + lane * VEC;
+            if (k < K) {
+                float wf[2][VEC];
+#pragma unroll
+                for (int m = 0; m < 2; ++m) {
+                    const uint32_t ww[4] = {buf[b][m][i].x, buf[b][m][i].y, buf[b][m][i].z, buf[b][m][i].w};
+#pragma unroll
+                    for (int j = 0; j < 4; ++j) {
+                        if (VEC == 8) {
+                            const float2 f = bf2_to_f2(ww[j]);
+                            wf[m][(2 * j) % VEC] = f.x;
+                            wf[m][(2 * j + 1) % VEC] = f.y;
+                        } else {
+                            wf[m][j] = __uint_as_float(ww[j]);
+                        }
+                    }
+                }
+#pragma unroll
+                for (int t = 0; t < NT; ++t) {
+                    if (t >= T) break;
+                    const uint4 xv = *reinterpret_cast<const uint4*>(xs + (size_t)t * K + k);
+                    const uint32_t xw[4] = {xv.x, xv.y, xv.z, xv.w};
+#pragma unroll
+                    for (int j = 0; j < 4; ++j) {
+                        if (VEC == 8) {
+                            const float2 f = bf2_to_f2(xw[j]);
+#pragma unroll
+                            for (int m = 0; m < 2; ++m) {
+                                acc[m][t] = fmaf(wf[m][(2 * j) % VEC], f.x, acc[m][t]);
+                                acc[m][t] = fmaf(wf[m][(2 * j + 1) % VEC], f.y, acc[m][t]);
+                            }
+                        } else {
+#pragma unroll
+                            for (int m = 0; m < 2; ++m) acc[m][t] = fmaf(wf[m][j], __uint_as_float(xw[j]), acc[m][t]);
+                        }
+                    }
+                }
+            }
+        }
+#pragma unroll
+        for (int m = 0; m < 2; ++m)
+#pragma unroll
+            for (int t = 0; t < NT; ++t) {
+                const float v = warp_sum(acc[m][t]);
+                if (lane == 0) part[((size_t)u * 2 + m) * NT + t] = v;
+            }
+    };
+    // two register sets, unrolled by hand so that the set index is a constant
+    while (u < units) {
+        if (u + nw < units) issue(u + nw, 1);
+        reduce(u, 0);
+        u += nw;
+        if (u >= units) break;
+        if (u + nw < units) issue(u + nw, 0);
+        reduce(u, 1);
+        u += nw;
+    }
+    pdl_launch_dependents();
+    __syncthreads();
+    const int np = p_hi - p_lo;
+    for (int i = threadIdx.x; i < np * NT; i += blockDim.x) {
+        const int pr = i / NT, t = i - pr * NT;
+        if (t >= T) continue;
+        float a0 = 0.f, a1 = 0.f;
+        for (int c = 0; c < KC; ++c) {
+            a0 += part[((size_t)(pr * KC + c) * 2) * NT + t];
+            a1 += part[((size_t)(pr * KC + c) * 2 + 1) * NT + t];
+        }
+        const int row = (p_lo + pr) * 2;
+        if (out_mode == LO_GEGLU) {
+            reinterpret_cast<WT*>(out)[(size_t)t * ldo + (row >> 1)] = Act<WT>::from_f(gelu_tanh_f(a0) * a1);
+        } else {
+            float* o = reinterpret_cast<float*>(out) + (size_t)t * ldo + row;
+            o[0] = a0;
+            if (row + 1 < N) o[1] = a1;
+        }
+    }
+}
+
+template <typename WT, int NT>
+static int launch_matvec(const RowStage& st, const void* w, int ldw, int N, void* out, int ldo, int out_mode, int T, cudaStream_t s) {
+    constexpr int COLS = 32 * Act<WT>::VEC * 4;
+    const int pairs = (N + 1) / 2, KC = (st.Kp + COLS - 1) / COLS;
+    const int grid = pairs < sm_count() ? pairs : sm_count();
+    const size_t xbytes = ((size_t)NT * st.Kp * sizeof(WT) + 15) & ~size_t(15);
+    const size_t part = (size_t)((pairs + grid - 1) / grid) * KC * 2 * NT * 4, stg = stage_bytes(st, T, 16);
+    const size_t smem = xbytes + (part > stg ? part : stg);
+    DLP_REQUIRE(smem <= 227 * 1024, "matvec: %d rows of width %d need %zu bytes of shared memory", T, st.Kp, smem);
+    auto kern = matvec_kernel<WT, NT>;
+    if (first_use_on_device((const void*)kern))
+        DLP_CHECK_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024));
+    DLP_CHECK_CUDA(launch_pdl(kern, dim3(grid), dim3(512), smem, s, st, (const WT*)w, ldw, N, out, ldo, out_mode, T));
+    return 0;
+}
+
+static int check_stage(const RowStage& st, const char* who) {
+    DLP_REQUIRE(st.x && st.K > 0 && st.Kp >= st.K, "%s: bad input row", who);
+    DLP_REQUIRE(!st.y || (st.w1 && st.groups1 > 0 && st.K % st.groups1 == 0), "%s: %d norm groups do not divide the width %d", who, st.groups1, st.K);
+    DLP_REQUIRE(!st.w2 || (st.w2_mod > 0 && st.groups2 > 0 && st.K % st.groups2 == 0), "%s: %d norm groups do not divide the width %d", who, st.groups2, st.K);
+    return 0;
+}
+
+int matvec(const RowStage& st, const void* w, int ldw, int N, void* out, int ldo, int out_mode, int T, int f32, cudaStream_t s) {
+    int rc = check_stage(st, "matvec");
+    if (rc) return rc;
+    DLP_REQUIRE(w && out && N > 0 && T >= 1 && T <= 4, "matvec: bad argument (T=%d N=%d)", T, N);
+    DLP_REQUIRE(st.Kp % 8 == 0 && ldw % 8 == 0 && ldw >= st.Kp, "matvec: row length %d / stride %d must be multiples of 8", st.Kp, ldw);
+    DLP_REQUIRE(out_mode == LO_F32 || (out_mode == LO_GEGLU && N % 2 == 0), "matvec: output mode %d", out_mode);
+    if (f32) {
+        if (T == 1) return launch_matvec<float, 1>(st, w, ldw, N, out, ldo, out_mode, T, s);
+        if (T == 2) return launch_matvec<float, 2>(st, w, ldw, N, out, ldo, out_mode, T, s);
+        return launch_matvec<float, 4>(st, w, ldw, N, out, ldo, out_mode, T, s);
+    }
+    if (T == 1) return launch_matvec<__nv_bfloat16, 1>(st, w, ldw, N, out, ldo, out_mode, T, s);
+    if (T == 2) return launch_matvec<__nv_bfloat16, 2>(st, w, ldw, N, out, ldo, out_mode, T, s);
+    return launch_matvec<__nv_bfloat16, 4>(st, w, ldw, N, out, ldo, out_mode, T, s);
+}
+
+int stage_rows(const RowStage& st, void* xb, int ldxb, int T, int f32, cudaStream_t s) {
+    int rc = check_stage(st, "stage_rows");
+    if (rc) return rc;
+    DLP_REQUIRE(xb && T > 0 && ldxb >= st.Kp, "stage_rows: bad argument");
+    const size_t smem = stage_bytes(st, 1, 8);
+    DLP_REQUIRE(smem <= 48 * 1024, "stage_rows: too many norm groups");
+    if (f32) DLP_CHECK_CUDA(launch_pdl(stage_rows_kernel<float>, dim3(T), dim3(256), smem, s, st, (float*)xb, ldxb));
+    else DLP_CHECK_CUDA(launch_pdl(stage_rows_kernel<__nv_bfloat16>, dim3(T), dim3(256), smem, s, st, (__nv_bfloat16*)xb, ldxb));
+    return 0;
+}
+
+// ---- fp32 matrix product ---------------------------------------------------------------------------------
+__global__ void __launch_bounds__(256) sgemm_kernel(const float* __restrict__ x, int ldx, const float* __restrict__ w, int ldw, int N, int K, float* out, int ldo,
+                                                    int out_mode, int T) {
+    __shared__ float xs[16][68], ws[16][68];
+    const int n0 = blockIdx.x * 64, t0 = blockIdx.y * 64, tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
+    float acc[4][4] = {};
+    pdl_wait();
+    for (int k0 = 0; k0 < K; k0 += 16) {
+        for (int i = threadIdx.x; i < 64 * 16; i += 256) {
+            const int r = i >> 4, k = i & 15;
+            xs[k][r] = (t0 + r < T && k0 + k < K) ? x[(size_t)(t0 + r) * ldx + k0 + k] : 0.f;
+            ws[k][r] = (n0 + r < N && k0 + k < K) ? w[(size_t)(n0 + r) * ldw + k0 + k] : 0.f;
+        }
+        __syncthreads();
+#pragma unroll
+        for (int k = 0; k < 16; ++k) {
+            float a[4], b[4];
+#pragma unroll
+            for (int i = 0; i < 4; ++i) { a[i] = xs[k][ty * 4 + i]; b[i] = ws[k][tx * 4 + i]; }
+#pragma unroll
+            for (int i = 0; i < 4; ++i)
+#pragma unroll
+                for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(a[i], b[j], acc[i][j]);
+        }
+        __syncthreads();
+    }
+    pdl_launch_dependents();
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        const int t = t0 + ty * 4 + i;
+        if (t >= T) continue;
+        if (out_mode == LO_GEGLU) {
+#pragma unroll
+            for (int j = 0; j < 4; j += 2) {
+                const int n = n0 + tx * 4 + j;
+                if (n < N) out[(size_t)t * ldo + (n >> 1)] = gelu_tanh_f(acc[i][j]) * acc[i][j + 1];
+            }
+        } else {
+#pragma unroll
+            for (int j = 0; j < 4; ++j)
+                if (n0 + tx * 4 + j < N) out[(size_t)t * ldo + n0 + tx * 4 + j] = acc[i][j];
+        }
+    }
+}
+
+int sgemm(const float* x, int ldx, const float* w, int ldw, int N, int K, void* out, int ldo, int out_mode, int T, cudaStream_t s) {
+    DLP_REQUIRE(x && w && out && N > 0 && K > 0 && T > 0, "sgemm: bad argument");
+    DLP_REQUIRE(out_mode == LO_F32 || (out_mode == LO_GEGLU && N % 2 == 0), "sgemm: output mode %d", out_mode);
+    DLP_CHECK_CUDA(launch_pdl(sgemm_kernel, dim3((N + 63) / 64, (T + 63) / 64), dim3(256), 0, s, x, ldx, w, ldw, N, K, (float*)out, ldo, out_mode, T));
+    return 0;
+}
+
+// ---- one matrix per head: out[t, h, n] = sum_k x[t, h, k] W[h][n][k]  (* sigmoid(gate[t, h])) ---------------
+// A is 16 * MT tokens of one head (shared memory), B comes straight from global memory, 16 bytes per lane: the k index inside a
+// 32-wide block is permuted the same way on both operands, so that a lane's eight k values are contiguous.
+__device__ __forceinline__ void mma_bf16(float (&c)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0, uint32_t b1) {
+    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+                 : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
+}
+
+template <int MT>
+__global__ void __launch_bounds__(128) head_matmul_kernel(const void* x, int x_f32, int ldx, int x_head, int kx, const __nv_bfloat16* __restrict__ w, int Kp, int N,
+                                                          int n_rows, __nv_bfloat16* out, int ldo, int out_head, const float* gate, int ldg, int T) {
+    extern __shared__ __align__(16) uint8_t hm_smem[];
+    __nv_bfloat16* xs = reinterpret_cast<__nv_bfloat16*>(hm_smem);
+    const int ldxs = Kp + 8, h = blockIdx.y, t0 = blockIdx.z * 16 * MT;
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, g = lane >> 2, c = lane & 3;
+    pdl_wait();
+    for (int i = threadIdx.x; i < 16 * MT * Kp; i += 128) {
+        const int t = i / Kp, k = i - t * Kp;
+        float v = 0.f;
+        if (t0 + t < T && k < kx) {
+            const size_t o = (size_t)(t0 + t) * ldx + (size_t)h * x_head + k;
+            v = x_f32 ? reinterpret_cast<const float*>(x)[o] : __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(x)[o]);
+        }
+        xs[t * ldxs + k] = __float2bfloat16_rn(v);
+    }
+    __syncthreads();
+    const int n0 = blockIdx.x * 64 + warp * 16;
+    float acc[MT][2][4] = {};
+    const __nv_bfloat16* wr[2];
+    bool ok[2];
+#pragma unroll
+    for (int j = 0; j < 2; ++j) {
+        const int n = n0 + j * 8 + g;
+        ok[j] = n < n_rows;
+        wr[j] = w + ((size_t)h * n_rows + (ok[j] ? n : 0)) * Kp + c * 8;
+    }
+#pragma unroll 4
+    for (int k = 0; k < Kp; k += 32) {
+        uint4 b[2];
+#pragma unroll
+        for (int j = 0; j < 2; ++j) b[j] = ok[j] ? ldg_nc_v4(wr[j] + k) : make_uint4(0, 0, 0, 0);
+#pragma unroll
+        for (int m = 0; m < MT; ++m) {
+            const uint4 lo = *reinterpret_cast<const uint4*>(xs + (m * 16 + g) * ldxs + k + c * 8);
+            const uint4 hi = *reinterpret_cast<const uint4*>(xs + (m * 16 + g + 8) * ldxs + k + c * 8);
+#pragma unroll
+            for (int j = 0; j < 2; ++j) {
+                mma_bf16(acc[m][j], lo.x, hi.x, lo.y, hi.y, b[j].x, b[j].y);
+                mma_bf16(acc[m][j], lo.z, hi.z, lo.w, hi.w, b[j].z, b[j].w);
+            }
+        }
+    }
+    pdl_launch_dependents();
+#pragma unroll
+    for (int m = 0; m < MT; ++m)
+#pragma unroll
+        for (int r = 0; r < 2; ++r) {
+            const int t = t0 + m * 16 + g + r * 8;
+            if (t >= T) continue;
+            const float sc = gate ? 1.f / (1.f + expf(-gate[(size_t)t * ldg + h])) : 1.f;
+#pragma unroll
+            for (int j = 0; j < 2; ++j)
+#pragma unroll
+                for (int e = 0; e < 2; ++e) {
+                    const int n = n0 + j * 8 + c * 2 + e;
+                    if (n < N) out[(size_t)t * ldo + (size_t)h * out_head + n] = __float2bfloat16_rn(acc[m][j][r * 2 + e] * sc);
+                }
+        }
+}
+
+__global__ void __launch_bounds__(128) head_matmul_f32_kernel(const float* x, int ldx, int x_head, int kx, const float* __restrict__ w, int Kp, int N, int n_rows,
+                                                              float* out, int ldo, int out_head, const float* gate, int ldg) {
+    extern __shared__ __align__(16) float hf_x[];
+    const int h = blockIdx.y, t = blockIdx.z, n = blockIdx.x * 128 + threadIdx.x;
+    pdl_wait();
+    for (int k = threadIdx.x; k < Kp; k += 128) hf_x[k] = k < kx ? x[(size_t)t * ldx + (size_t)h * x_head + k] : 0.f;
+    __syncthreads();
+    pdl_launch_dependents();
+    if (n >= N) return;
+    const float* wr = w + ((size_t)h * n_rows + n) * Kp;
+    float a = 0.f;
+    for (int k = 0; k < Kp; ++k) a = fmaf(hf_x[k], wr[k], a);
+    if (gate) a *= 1.f / (1.f + expf(-gate[(size_t)t * ldg + h]));
+    out[(size_t)t * ldo + (size_t)h * out_head + n] = a;
+}
+
+// w is [H][n_rows][Kp] with zero padding along k; x holds kx values per head
+int head_matmul(const void* x, int x_f32, int ldx, int x_head, int kx, const void* w, int Kp, int H, int N, int n_rows, void* out, int ldo, int out_head,
+                const float* gate, int ldg, int T, int f32, cudaStream_t s) {
+    DLP_REQUIRE(x && w && out && H > 0 && N > 0 && N <= n_rows && T > 0 && kx <= Kp && Kp % 32 == 0, "head_matmul: bad argument (Kp=%d N=%d)", Kp, N);
+    if (f32) {
+        for (int t = 0; t < T; t += 32768) {     // grid.z limit
+            const int n = T - t < 32768 ? T - t : 32768;
+            DLP_CHECK_CUDA(launch_pdl(head_matmul_f32_kernel, dim3((N + 127) / 128, H, n), dim3(128), Kp * 4, s, (const float*)x + (size_t)t * ldx, ldx, x_head, kx,
+                                      (const float*)w, Kp, N, n_rows, (float*)out + (size_t)t * ldo, ldo, out_head, gate ? gate + (size_t)t * ldg : nullptr, ldg));
+        }
+        return 0;
+    }
+    const int mt = T <= 16 ? 1 : 4;
+    const size_t smem = (size_t)16 * mt * (Kp + 8) * 2;
+    DLP_REQUIRE(smem <= 227 * 1024, "head_matmul: inner size %d", Kp);
+    dim3 grid((N + 63) / 64, H, (T + 16 * mt - 1) / (16 * mt));
+    auto k1 = head_matmul_kernel<1>;
+    auto k4 = head_matmul_kernel<4>;
+    if (first_use_on_device((const void*)k1)) DLP_CHECK_CUDA(cudaFuncSetAttribute(k1, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024));
+    if (first_use_on_device((const void*)k4)) DLP_CHECK_CUDA(cudaFuncSetAttribute(k4, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024));
+    DLP_CHECK_CUDA(launch_pdl(mt == 1 ? k1 : k4, grid, dim3(128), smem, s, x, x_f32, ldx, x_head, kx, (const __nv_bfloat16*)w, Kp, N, n_rows, (__nv_bfloat16*)out, ldo,
+                              out_head, gate, ldg, T));
+    return 0;
+}
+
+}  // namespace dlp

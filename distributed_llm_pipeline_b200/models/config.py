@@ -12,6 +12,14 @@ from typing import Any
 
 
 @dataclass(frozen=True)
+class LayerSpec:
+    """One entry of a layer list: the token mixer with its sizes and constants, and the feed-forward (None: the layer has none)."""
+    type: str
+    mixer: dict[str, Any]
+    mlp: dict[str, Any] | None = None
+
+
+@dataclass(frozen=True)
 class ModelConfig:
     name: str = "llama"
     arch: str = "llama"
@@ -76,6 +84,9 @@ class ModelConfig:
     post_norm: bool = False
     pre_norm: bool = True
     qk_norm_full: bool = False
+    # layer-list models (models/layered.py): every layer is described on its own; the head / feed-forward fields above do not apply
+    layers: tuple[LayerSpec, ...] = ()
+    norm_groups: int = 1           # the norm divides each of this many equal parts of the vector by its own root mean square
 
     @property
     def generic(self) -> bool:

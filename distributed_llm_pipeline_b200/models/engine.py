@@ -1,0 +1,373 @@
+"""Engine core: sequences, paged cache, recurrent state, batched decode under CUDA graphs, sampling records, generation loop.
+
+Parity: the part of `llama_context` (`llama.cpp/src/llama-context.cpp:1042-1104,1375-1724`) that does not depend on what a layer
+computes.  A model family supplies the step body: `_decode_body`, `prefill`, and the buffers behind them (models/llama.py for GGUF
+families, models/layered.py for layer-list models).
+"""
+from __future__ import annotations
+
+import os
+from dataclasses import dataclass, field
+
+import torch
+
+from ..ops import api as ops
+
+
+@dataclass
+class Sequence:
+    sid: int
+    length: int = 0
+    pages: list[int] = field(default_factory=list)
+
+
+class PagedKVCache:
+    """Fixed-size pages + a host-side free list and block table.  A layer keeps any number of named planes, each
+    [n_pages, heads, page, dim]: `k` and `v` for softmax attention, one `c` plane of latent rows for latent attention."""
+
+    def __init__(self, planes: dict[str, dict[int, tuple[int, int]]], n_pages: int, page_size: int, max_seqs: int,
+                 max_pages_per_seq: int, device, dtype=torch.float16):
+        self.page_size = page_size
+        self.n_pages = n_pages
+        self.max_pages = max_pages_per_seq
+        self.planes = {name: {il: torch.zeros(n_pages, heads, page_size, dim, dtype=dtype, device=device) for il, (heads, dim) in per.items()}
+                       for name, per in planes.items()}
+        self.free = list(range(n_pages - 1, -1, -1))
+        self.block_table = torch.zeros(max_seqs, max_pages_per_seq, dtype=torch.int32, device=device)
+        self.block_table_host = torch.zeros(max_seqs, max_pages_per_seq, dtype=torch.int32)
+        if torch.device(device).type == "cuda":
+            self.block_table_host = self.block_table_host.pin_memory()
+
+    @property
+    def k(self):
+        return self.planes["k"]
+
+    @property
+    def v(self):
+        return self.planes["v"]
+
+    def each_plane(self):
+        """(layer, name, tensor) in a fixed order: by layer, then by plane."""
+        for il in sorted({il for per in self.planes.values() for il in per}):
+            for name, per in self.planes.items():
+                if il in per:
+                    yield il, name, per[il]
+
+    def ensure(self, seq: Sequence, new_len: int):
+        need = (new_len + self.page_size - 1) // self.page_size
+        if need > self.max_pages:
+            raise RuntimeError(f"sequence {seq.sid}: context {new_len} exceeds n_ctx")
+        grew = False
+        while len(seq.pages) < need:
+            if not self.free:
+                raise RuntimeError("KV cache exhausted (no free pages)")
+            pg = self.free.pop()
+            self.block_table_host[seq.sid, len(seq.pages)] = pg
+            seq.pages.append(pg)
+            grew = True
+        if grew:
+            self.block_table[seq.sid].copy_(self.block_table_host[seq.sid], non_blocking=True)
+
+    def release(self, seq: Sequence):
+        self.free.extend(reversed(seq.pages))
+        seq.pages.clear()
+        seq.length = 0
+
+    def bytes(self) -> int:
+        return sum(t.numel() * t.element_size() for _, _, t in self.each_plane())
+
+
+class RecurrentState:
+    """fp32 state of the recurrent layers: one slot per sequence in every layer's tensor [max_seqs, *shape].  A state stands for all
+    tokens seen so far; it cannot be cut back to an earlier token, only cleared, copied, saved and restored whole."""
+
+    def __init__(self, shapes: dict[int, tuple[int, ...]], max_seqs: int, device):
+        self.layers = {il: torch.zeros(max_seqs, *shape, dtype=torch.float32, device=device) for il, shape in shapes.items()}
+
+    def __bool__(self):
+        return bool(self.layers)
+
+    def clear(self, sid: int):
+        for t in self.layers.values():
+            t[sid].zero_()
+
+    def copy(self, src: int, dst: int):
+        for t in self.layers.values():
+            t[dst].copy_(t[src])
+
+    def save(self, sids) -> list[torch.Tensor]:
+        idx = torch.as_tensor(list(sids), dtype=torch.long)
+        return [t[idx.to(t.device)].clone() for t in self.layers.values()]
+
+    def restore(self, sids, saved: list[torch.Tensor]):
+        idx = torch.as_tensor(list(sids), dtype=torch.long)
+        for t, v in zip(self.layers.values(), saved):
+            t[idx.to(t.device)] = v
+
+    def bytes(self) -> int:
+        return sum(t.numel() * 4 for t in self.layers.values())
+
+
+class NullComm:
+    """Single-rank communicator (tp = pp = 1)."""
+    tp_size = 1
+    tp_rank = 0
+
+    def allreduce_delta(self, delta, il, which):
+        return delta
+
+    def allgather_logits(self, logits, vocab_range, vocab_size):
+        return logits
+
+    fused = False
+
+
+class EngineCore:
+    def _init_core(self, weights, n_ctx: int, max_seqs: int, page_size: int, max_batch_tokens: int, comm, first_stage: bool, last_stage: bool, device):
+        """Everything that does not depend on the model family; the caller allocates `kv`, `rstate` and the activation buffers."""
+        self.w = weights
+        self.cfg = weights.cfg
+        self.device = dev = device
+        self.comm = comm or NullComm()
+        self.first_stage, self.last_stage = first_stage, last_stage
+        self.n_ctx, self.max_seqs, self.page_size = n_ctx, max_seqs, page_size
+        self.max_tokens = max(max_batch_tokens, max_seqs)
+        self.max_rows = M = self.max_tokens + 8   # head-room: the sequence-parallel path pads T up to a multiple of tp
+        self.rstate = RecurrentState({}, max_seqs, dev)
+        self.seqs: dict[int, Sequence] = {}
+        self._free_sids = list(range(max_seqs - 1, -1, -1))
+        i32 = torch.int32
+        self.fused_tp = self.sp_ok = False
+        self._greedy_now = False
+        self.tokens = torch.zeros(M, dtype=i32, device=dev)
+        self.pos = torch.zeros(M, dtype=i32, device=dev)
+        self.slot = torch.zeros(M, dtype=i32, device=dev)
+        self.kv_len = torch.zeros(M, dtype=i32, device=dev)
+        self.active = torch.zeros(max_seqs, dtype=i32, device=dev)   # sequence slot of each decode batch row
+        self._active_host: list[int] = []
+        self.seq_len_dev = torch.zeros(max_seqs, dtype=i32, device=dev)
+        self.next_tok = torch.zeros(max_seqs, dtype=i32, device=dev)
+        self.step_ctr = torch.zeros(1, dtype=i32, device=dev)
+        # per-sequence sampler records (dlp_sample_params: top_k, top_p, min_p, temp, seed, draw counter) read by the device sampler
+        self.samp = torch.zeros(max_seqs, ops.SAMPLE_REC_WORDS, dtype=i32, device=dev)
+        self._samp_host: dict[int, tuple] = {}      # what each record currently holds
+        self._seq_sampling: dict[int, tuple] = {}   # per-sequence overrides of self.sampling (set_seq_sampling)
+        self.max_graphs = int(os.environ.get("DLP_MAX_GRAPHS", str(max(24, 4 * max_seqs + 8))))   # (batch sizes x attention variants x greedy)
+        self._graphs: dict[tuple, torch.cuda.CUDAGraph] = {}
+        self._graph_launches: dict[tuple, int] = {}    # kernels inside each captured graph
+        self.launches_replayed = 0                      # kernels launched through graph replays so far
+        self.sampling = dict(top_k=40, top_p=0.95, min_p=0.05, temp=0.0, seed=0)
+        self.cvec: dict[int, torch.Tensor] = {}     # layer -> fp32 [E] added to the residual stream after that layer
+        self.eval_callback = None      # fn(name, layer, tensor) called after every layer (eager paths only; disables graphs)
+        self._variant = None           # launch variant of the decode step; part of the graph key
+
+    # ---- what a family may override ---------------------------------------------------------------
+    mixed_batches = False       # True: `step` runs prompt portions and decoded tokens of several sequences in one forward
+    can_shift = True            # the cached tokens can slide to earlier positions (context shift)
+
+    def _graph_ok(self) -> bool:
+        return True
+
+    def _choose_variant(self, max_len: int):
+        """Pick the launch variant of the next decode step from the longest context (cached tokens + 1)."""
+
+    def _companion_variants(self) -> list:
+        """Variants to capture together with the current one."""
+        return []
+
+    def _decode_body(self, B: int, sample: bool):
+        raise NotImplementedError
+
+    # ---- sequence management ------------------------------------------------------------------
+    def alloc_seq(self) -> int:
+        if not self._free_sids:
+            raise RuntimeError("no free sequence slots")
+        sid = self._free_sids.pop()
+        self.seqs[sid] = Sequence(sid)
+        return sid
+
+    def free_seq(self, sid: int):
+        self.kv.release(self.seqs.pop(sid))
+        self._free_sids.append(sid)
+        self._seq_sampling.pop(sid, None)
+        self._samp_host.pop(sid, None)
+
+    def set_seq_sampling(self, sid: int, top_k: int = 40, top_p: float = 0.95, min_p: float = 0.05, temp: float = 0.0, seed: int = 0):
+        """Sampler parameters of one sequence for the device sampler; also restarts that sequence's random stream, so a request
+        with a given seed draws the same tokens whatever ran before it (the reference keeps one seeded RNG per slot,
+        `common/sampling.cpp:179-311`).  Sequences without their own record follow `self.sampling`."""
+        self._seq_sampling[sid] = (int(top_k), float(top_p), float(min_p), float(temp), int(seed))
+        self._samp_host.pop(sid, None)
+
+    def _sync_sampling(self, sids):
+        for sid in sids:
+            s = self.sampling
+            want = self._seq_sampling.get(sid) or (s["top_k"], s["top_p"], s["min_p"], s["temp"], s["seed"])
+            if self._samp_host.get(sid) != want:
+                self.samp[sid].copy_(ops.pack_sample_record(*want))
+                self._samp_host[sid] = want
+
+    def seq_len(self, sid: int) -> int:
+        return self.seqs[sid].length
+
+    def reusable(self, sid: int, n: int) -> int:
+        """How many of the first `n` cached tokens of a sequence can be kept when the rest is dropped: all of them from a paged cache,
+        none with a recurrent state (which only stands for its whole sequence)."""
+        return n if not self.rstate or n == self.seqs[sid].length else 0
+
+    def truncate_seq(self, sid: int, new_len: int):
+        """Keep only the first `new_len` cached tokens of a sequence (prompt-prefix reuse, rollback after errors).
+        Parity: `llama_memory_seq_rm(seq, p0=new_len, p1=-1)` (`llama-kv-cache.cpp:224-320`); pages past the cut
+        return to the free list."""
+        seq = self.seqs[sid]
+        new_len = max(0, min(new_len, seq.length))
+        if self.reusable(sid, new_len) != new_len:
+            raise RuntimeError(f"sequence {sid}: a recurrent state cannot be cut back from {seq.length} to {new_len} tokens")
+        if self.rstate and new_len == 0:
+            self.rstate.clear(sid)
+        keep_pages = (new_len + self.page_size - 1) // self.page_size
+        while len(seq.pages) > keep_pages:
+            self.kv.free.append(seq.pages.pop())
+        seq.length = new_len
+        self.seq_len_dev[sid] = new_len
+
+    def copy_seq(self, src: int, dst: int, n: int | None = None):
+        """Copy the first `n` cached tokens (default: all) of sequence `src` into `dst` (which is overwritten).
+        Parity: `llama_memory_seq_cp` (`llama-kv-cache.cpp:322-392`) - used for prompt sharing between slots / beams."""
+        s, d = self.seqs[src], self.seqs[dst]
+        n = s.length if n is None else min(n, s.length)
+        if self.rstate and n not in (0, s.length):
+            raise NotImplementedError("a recurrent state can only be copied whole")
+        self.truncate_seq(dst, 0)
+        self.kv.ensure(d, n)
+        npg = (n + self.page_size - 1) // self.page_size
+        if npg:
+            sp = torch.tensor(s.pages[:npg], dtype=torch.long, device=self.device)
+            dp = torch.tensor(d.pages[:npg], dtype=torch.long, device=self.device)
+            for _, _, t in self.kv.each_plane():
+                t[dp] = t[sp]
+        if self.rstate and n:
+            self.rstate.copy(src, dst)
+        d.length = n
+        self.seq_len_dev[dst] = n
+
+    def _advance_inputs(self, sid: int, T: int):
+        """Grow the sequence's pages for T more tokens; positions and cache slots of those tokens (host int32)."""
+        seq = self.seqs[sid]
+        self.kv.ensure(seq, seq.length + T)
+        pos = torch.arange(seq.length, seq.length + T, dtype=torch.int32)
+        pages = torch.tensor(seq.pages, dtype=torch.int32)
+        slot = pages[(pos // self.page_size).long()] * self.page_size + pos % self.page_size
+        return pos, slot.to(torch.int32)
+
+    # ---- decode -----------------------------------------------------------------------------------
+    @torch.no_grad()
+    def decode(self, sids: list[int], tokens=None, hidden_in: torch.Tensor | None = None, sample: bool = True,
+               use_graph: bool = True):
+        """One token for each sequence in `sids` (any subset of slots; batch row i belongs to sids[i]).
+        tokens: host ints / tensor, or None to feed back the previously sampled tokens (device resident).
+        Returns next-token ids (device int32 [B]) when sampling, else logits [B, vocab]; or hidden states."""
+        B = len(sids)
+        for sid in sids:
+            seq = self.seqs[sid]
+            self.kv.ensure(seq, seq.length + 1)
+        if sids != self._active_host:
+            self.active[:B].copy_(torch.tensor(sids, dtype=torch.int32), non_blocking=False)
+            self._active_host = list(sids)
+        if tokens is not None and self.first_stage:
+            self.next_tok[:B].copy_(torch.as_tensor(tokens, dtype=torch.int32), non_blocking=True)
+        if hidden_in is not None:
+            self.h[:B].copy_(hidden_in)
+        graphable = (use_graph and self.eval_callback is None and self.device.type == "cuda" and self._graph_ok()
+                     and not getattr(self.comm, "no_graph", False)    # (the sequence-parallel path is capturable too: its epochs are
+                     and not (self.sp_ok and B > 4 and os.environ.get("DLP_SP_GRAPH", "1") == "0"))   # positions inside the pass on top of a device-side counter; DLP_SP_GRAPH=0: A/B)
+        self._choose_variant(max(self.seqs[sid].length for sid in sids) + 1)
+        if sample and self.last_stage:
+            self._sync_sampling(sids)
+        # all rows greedy on the fused tensor-parallel path: sharded arg-max instead of gathering the logits (host-side fact, so
+        # it is part of the graph key; at most one extra graph per batch size)
+        self._greedy_now = bool(sample and self.last_stage and self.fused_tp and (B in (1, 2, 4) or (self.sp_ok and 4 < B <= 64)) and
+                                os.environ.get("DLP_TP_ARGMAX", "1") == "1" and all(self._samp_host[sid][3] <= 0 for sid in sids))
+        if graphable:
+            # only the batch size, the output kind and the attention variant shape the graph (sampler parameters are device data)
+            key = (B, sample, self._variant, self._greedy_now)
+            g = self._graphs.pop(key, None)
+            if g is None:
+                while len(self._graphs) + 2 > self.max_graphs:    # least recently used graphs go first
+                    old = next(iter(self._graphs))
+                    del self._graphs[old]
+                    self._graph_launches.pop(old, None)
+                want = self._variant
+                for other in self._companion_variants():   # captured now as well: the switch between them must not stall a later step
+                    self._variant = other
+                    self._capture(B, sample, key[:2] + (other,) + key[3:])
+                self._variant = want
+                g = self._capture(B, sample, key)
+                self._graphs.pop(key)
+            self._graphs[key] = g      # most recently used last
+            g.replay()
+            self.launches_replayed += self._graph_launches.get(key, 0)
+        else:
+            self._decode_body(B, sample)
+        for sid in sids:
+            self.seqs[sid].length += 1
+        if not self.last_stage:
+            return self.h[:B]
+        return self.next_tok[:B] if sample else self.logits_full[:B]
+
+    def _capture(self, B: int, sample: bool, key=None):
+        # warm-up (also lets every kernel set its attributes), then roll back the bookkeeping it advanced
+        saved = self.seq_len_dev.clone()
+        saved_ctr = self.step_ctr.clone()
+        saved_h = self.h[:B].clone()   # non-first stages consume their input hidden state in place: the warm-up must not eat it
+        saved_tok = self.next_tok.clone()   # the warm-up samples into next_tok: the pending input token must survive it
+        saved_samp = self.samp.clone()      # ... and advances the draw counters
+        saved_state = self.rstate.save(self._active_host[:B])   # ... and the recurrent states
+        s = torch.cuda.Stream()
+        s.wait_stream(torch.cuda.current_stream())
+        with torch.cuda.stream(s):
+            self._decode_body(B, sample)
+        torch.cuda.current_stream().wait_stream(s)
+        self.seq_len_dev.copy_(saved)
+        self.step_ctr.copy_(saved_ctr)
+        self.h[:B].copy_(saved_h)
+        self.next_tok.copy_(saved_tok)
+        self.samp.copy_(saved_samp)
+        self.rstate.restore(self._active_host[:B], saved_state)
+        g = torch.cuda.CUDAGraph()
+        n0 = ops.launch_count
+        with torch.cuda.graph(g):
+            self._decode_body(B, sample)
+        self.launches_per_graph = getattr(self, "launches_per_graph", {})
+        self.launches_per_graph[(B, sample)] = ops.launch_count - n0
+        self._graph_launches[key or (B, sample)] = ops.launch_count - n0
+        self.seq_len_dev.copy_(saved)
+        self.step_ctr.copy_(saved_ctr)
+        self._graphs[key or (B, sample)] = g
+        return g
+
+    # ---- convenience ------------------------------------------------------------------------------
+    @torch.no_grad()
+    def generate(self, prompt: list[int], n_predict: int, sid: int | None = None, stop_ids: tuple[int, ...] = ()):
+        """Greedy / sampled generation for one sequence (slot 0 path); returns the generated ids."""
+        own = sid is None
+        if own:
+            sid = self.alloc_seq()
+        logits = self.prefill(sid, prompt)
+        s = self.sampling
+        if s["temp"] <= 0:
+            tok = ops.argmax(logits[None])
+        else:   # first token from the prefill logits: same per-sequence record (and random stream) as the decode steps
+            self._sync_sampling([sid])
+            tok = ops.sample_dev(logits[None], self.samp, torch.tensor([sid], dtype=torch.int32, device=self.device),
+                                 torch.empty(1, dtype=torch.int32, device=self.device))
+        self.next_tok[:1].copy_(tok)
+        out = [int(tok[0])]
+        for _ in range(n_predict - 1):
+            if out[-1] in stop_ids:
+                break
+            nt = self.decode([sid])
+            out.append(int(nt[0]))
+        if own:
+            self.free_seq(sid)
+        return out

@@ -13,109 +13,41 @@ PP activation hand-off (see parallel/).
 from __future__ import annotations
 
 import math
-from dataclasses import dataclass, field
-
 import os
 
 import torch
 
 from ..ops import api as ops
-from .config import ModelConfig
+from .engine import EngineCore, NullComm, PagedKVCache, Sequence  # noqa: F401 (Sequence, NullComm: part of this module's surface)
 from .reference import limit_to_groups, rope_attn_scale, rope_inv_freq
 from .weights import ModelWeights
 
 
-@dataclass
-class Sequence:
-    sid: int
-    length: int = 0
-    pages: list[int] = field(default_factory=list)
-
-
-class PagedKVCache:
-    """Fixed-size pages [n_pages, Hkv, page, D] per layer + a host-side free list and block table."""
-
-    def __init__(self, cfg: ModelConfig, layers, n_head_kv: int, n_pages: int, page_size: int, max_seqs: int,
-                 max_pages_per_seq: int, device):
-        self.page_size = page_size
-        self.n_pages = n_pages
-        self.max_pages = max_pages_per_seq
-        shape = (n_pages, n_head_kv, page_size, cfg.head_dim)
-        self.k = {il: torch.zeros(shape, dtype=torch.float16, device=device) for il in layers}
-        self.v = {il: torch.zeros(shape, dtype=torch.float16, device=device) for il in layers}
-        self.free = list(range(n_pages - 1, -1, -1))
-        self.block_table = torch.zeros(max_seqs, max_pages_per_seq, dtype=torch.int32, device=device)
-        self.block_table_host = torch.zeros(max_seqs, max_pages_per_seq, dtype=torch.int32)
-        if torch.device(device).type == "cuda":
-            self.block_table_host = self.block_table_host.pin_memory()
-
-    def ensure(self, seq: Sequence, new_len: int):
-        need = (new_len + self.page_size - 1) // self.page_size
-        if need > self.max_pages:
-            raise RuntimeError(f"sequence {seq.sid}: context {new_len} exceeds n_ctx")
-        grew = False
-        while len(seq.pages) < need:
-            if not self.free:
-                raise RuntimeError("KV cache exhausted (no free pages)")
-            pg = self.free.pop()
-            self.block_table_host[seq.sid, len(seq.pages)] = pg
-            seq.pages.append(pg)
-            grew = True
-        if grew:
-            self.block_table[seq.sid].copy_(self.block_table_host[seq.sid], non_blocking=True)
-
-    def release(self, seq: Sequence):
-        self.free.extend(reversed(seq.pages))
-        seq.pages.clear()
-        seq.length = 0
-
-    def bytes(self) -> int:
-        return sum(t.numel() * 2 for t in self.k.values()) * 2
-
-
-class NullComm:
-    """Single-rank communicator (tp = pp = 1)."""
-    tp_size = 1
-    tp_rank = 0
-
-    def allreduce_delta(self, delta, il, which):
-        return delta
-
-    def allgather_logits(self, logits, vocab_range, vocab_size):
-        return logits
-
-    fused = False
-
-
-class LlamaEngine:
+class LlamaEngine(EngineCore):
     def __init__(self, weights: ModelWeights, n_ctx: int = 4096, max_seqs: int = 8, page_size: int = 64,
                  max_batch_tokens: int = 2048, n_pages: int | None = None, comm=None, first_stage: bool = True,
                  last_stage: bool = True, attn_splits: int | None = None):
-        self.w = weights
-        self.cfg = cfg = weights.cfg
+        cfg = weights.cfg
         dev = (weights.tok_embd or weights.lm_head or next(iter(weights.layers.values())).wqkv).device
-        self.device = dev
-        self.comm = comm or NullComm()
-        self.first_stage, self.last_stage = first_stage, last_stage
-        self.n_ctx, self.max_seqs, self.page_size = n_ctx, max_seqs, page_size
-        self.max_tokens = max(max_batch_tokens, max_seqs)
+        self._init_core(weights, n_ctx, max_seqs, page_size, max_batch_tokens, comm, first_stage, last_stage, dev)
         self.Hq, self.Hkv, self.D = weights.n_head_local, weights.n_head_kv_local, cfg.head_dim
         self.E, self.F = cfg.n_embd, weights.n_ff_local
         if dev.type == "cuda" and self.D not in (64, 128):
             raise NotImplementedError(f"head dimension {self.D}: the attention kernels are built for 64 and 128 (phi-2 has 80, gemma 256)")
+        if dev.type == "cuda":
+            ops.need_full_library()
         max_pages = (n_ctx + page_size - 1) // page_size
         if n_pages is None:
             n_pages = max_pages * max_seqs
-        self.kv = PagedKVCache(cfg, weights.layer_range, self.Hkv, n_pages, page_size, max_seqs, max_pages, dev)
+        per_layer = {il: (self.Hkv, cfg.head_dim) for il in weights.layer_range}
+        self.kv = PagedKVCache({"k": per_layer, "v": per_layer}, n_pages, page_size, max_seqs, max_pages, dev)
         self.inv_freq = rope_inv_freq(cfg, weights.rope_freqs.cpu() if weights.rope_freqs is not None else None).to(dev)
         if cfg.rope_dim < cfg.head_dim:     # partial rotary: zero angles for the dims left alone (Wq / Wk rows were re-ordered at load, models/weights.py)
             self.inv_freq = torch.cat([self.inv_freq, torch.zeros(cfg.head_dim // 2 - cfg.rope_dim // 2, dtype=self.inv_freq.dtype, device=dev)])
         # layers without rotary encoding (smollm3: every 4th) run the same kernels on a zero-angle table: the rotation is the identity
         self.inv_freq_off = torch.zeros_like(self.inv_freq) if cfg.no_rope_step > 0 else None
         self.attn_scale = rope_attn_scale(cfg)
-        self.seqs: dict[int, Sequence] = {}
-        self._free_sids = list(range(max_seqs - 1, -1, -1))
-        M = self.max_tokens + 8   # head-room: the sequence-parallel path pads T up to a multiple of tp
+        M = self.max_rows
         f16, f32, i32 = torch.float16, torch.float32, torch.int32
         qkv_dim = (self.Hq + 2 * self.Hkv) * self.D
         self.h = torch.zeros(M, self.E, dtype=f32, device=dev)
@@ -124,8 +56,6 @@ class LlamaEngine:
             raise NotImplementedError(f"the {cfg.arch} family runs the generic layer path: tensor parallelism through --tp-impl nccl")
         if cfg.generic and cfg.is_moe and (cfg.norm_type != "rms" or cfg.parallel_residual or cfg.post_norm or not cfg.pre_norm):
             raise NotImplementedError("routed experts on the generic layer path need the sequential pre-RMSNorm block form")
-        self.sp_ok = False
-        self._greedy_now = False
         if self.fused_tp:
             if not self.comm.ready:
                 self.comm.setup(self.E, 2 * len(weights.layer_range))
@@ -150,20 +80,6 @@ class LlamaEngine:
         self.up32 = torch.zeros(M, self.F, dtype=f32, device=dev) if cfg.ffn_act != "swiglu" else None
         self.xn2 = torch.zeros(M, self.E, dtype=f16, device=dev) if cfg.post_norm or any(
             lw.attn_norm2 is not None or (cfg.parallel_residual and lw.ffn_norm is not None) for lw in weights.layers.values()) else None
-        self.tokens = torch.zeros(M, dtype=i32, device=dev)
-        self.pos = torch.zeros(M, dtype=i32, device=dev)
-        self.slot = torch.zeros(M, dtype=i32, device=dev)
-        self.kv_len = torch.zeros(M, dtype=i32, device=dev)
-        self.active = torch.zeros(max_seqs, dtype=i32, device=dev)   # sequence slot of each decode batch row
-        self._active_host: list[int] = []
-        self.seq_len_dev = torch.zeros(max_seqs, dtype=i32, device=dev)
-        self.next_tok = torch.zeros(max_seqs, dtype=i32, device=dev)
-        self.step_ctr = torch.zeros(1, dtype=i32, device=dev)
-        # per-sequence sampler records (dlp_sample_params: top_k, top_p, min_p, temp, seed, draw counter) read by the device sampler
-        self.samp = torch.zeros(max_seqs, ops.SAMPLE_REC_WORDS, dtype=i32, device=dev)
-        self._samp_host: dict[int, tuple] = {}      # what each record currently holds
-        self._seq_sampling: dict[int, tuple] = {}   # per-sequence overrides of self.sampling (set_seq_sampling)
-        self.max_graphs = int(os.environ.get("DLP_MAX_GRAPHS", str(max(24, 4 * max_seqs + 8))))   # (batch sizes x attention variants x greedy)
         v0, v1 = weights.vocab_range
         self.logits = torch.zeros(max(max_seqs, 1), v1 - v0, dtype=f32, device=dev) if last_stage else None
         if last_stage and self.comm.tp_size > 1 and hasattr(self.comm, "reserve_logits") and (v1 - v0) != cfg.vocab_size:
@@ -174,8 +90,6 @@ class LlamaEngine:
                         torch.zeros(max_seqs * self.Hq * ns * 2, dtype=f32, device=dev),
                         torch.zeros(max_seqs * self.Hq, dtype=i32, device=dev)) if ns > 1 else None
         self.scratch = None  # fp16 decode buffer for block-quantised weights on the GEMM path (allocated lazily)
-        self._graphs: dict[tuple, torch.cuda.CUDAGraph] = {}
-        self.sampling = dict(top_k=40, top_p=0.95, min_p=0.05, temp=0.0, seed=0)
         # decode attention in one launch (RoPE + KV write + split-KV + cluster combine); plain-llama layers with full-width RoPE
         self.attn_onepass = (dev.type == "cuda" and os.environ.get("DLP_ATTN_ONEPASS", "1") == "1" and cfg.rope_dim == self.D
                              and not cfg.qkv_bias and not cfg.qk_norm)
@@ -183,74 +97,24 @@ class LlamaEngine:
         # the cluster launch only pays once the context spans more than one 64-key split; below this many keys the two-kernel
         # path (RoPE kernel + attention) is used (profiles/r1_attn_onepass_ab.txt).  The host knows every sequence length, so the choice is part of the graph key.
         self.attn_onepass_min = int(os.environ.get("DLP_ATTN_ONEPASS_MIN", "64"))
-        self._onepass_now = False
-        self._graph_launches: dict[tuple, int] = {}    # kernels inside each captured graph
-        self.launches_replayed = 0                      # kernels launched through graph replays so far
+        self._variant = False
         self.rope_cs = (torch.zeros(max_seqs, self.D // 2, 2, dtype=f32, device=dev)
                         if self.attn_onepass and os.environ.get("DLP_ROPE_TABLE", "1") == "1" else None)
-        self.cvec: dict[int, torch.Tensor] = {}     # layer -> fp32 [E] added to the residual stream after that layer
-        self.eval_callback = None      # fn(name, layer, tensor) called after every layer (eager paths only; disables graphs)
 
-    # ---- sequence management ------------------------------------------------------------------
-    def alloc_seq(self) -> int:
-        if not self._free_sids:
-            raise RuntimeError("no free sequence slots")
-        sid = self._free_sids.pop()
-        self.seqs[sid] = Sequence(sid)
-        return sid
+    # the decode step has two attention variants (one-launch cluster kernel or RoPE + attention): `_variant` is True for the former
+    @property
+    def _onepass_now(self) -> bool:
+        return bool(self._variant)
 
-    def free_seq(self, sid: int):
-        self.kv.release(self.seqs.pop(sid))
-        self._free_sids.append(sid)
-        self._seq_sampling.pop(sid, None)
-        self._samp_host.pop(sid, None)
+    def _choose_variant(self, max_len: int):
+        self._variant = self.attn_onepass and max_len >= self.attn_onepass_min
 
-    def set_seq_sampling(self, sid: int, top_k: int = 40, top_p: float = 0.95, min_p: float = 0.05, temp: float = 0.0, seed: int = 0):
-        """Sampler parameters of one sequence for the device sampler; also restarts that sequence's random stream, so a request
-        with a given seed draws the same tokens whatever ran before it (the reference keeps one seeded RNG per slot,
-        `common/sampling.cpp:179-311`).  Sequences without their own record follow `self.sampling`."""
-        self._seq_sampling[sid] = (int(top_k), float(top_p), float(min_p), float(temp), int(seed))
-        self._samp_host.pop(sid, None)
+    def _companion_variants(self) -> list:
+        return [not self._variant] if self.attn_onepass else []
 
-    def _sync_sampling(self, sids):
-        for sid in sids:
-            s = self.sampling
-            want = self._seq_sampling.get(sid) or (s["top_k"], s["top_p"], s["min_p"], s["temp"], s["seed"])
-            if self._samp_host.get(sid) != want:
-                self.samp[sid].copy_(ops.pack_sample_record(*want))
-                self._samp_host[sid] = want
-
-    def seq_len(self, sid: int) -> int:
-        return self.seqs[sid].length
-
-    def truncate_seq(self, sid: int, new_len: int):
-        """Keep only the first `new_len` cached tokens of a sequence (prompt-prefix reuse, rollback after errors).
-        Parity: `llama_memory_seq_rm(seq, p0=new_len, p1=-1)` (`llama-kv-cache.cpp:224-320`); pages past the cut
-        return to the free list."""
-        seq = self.seqs[sid]
-        new_len = max(0, min(new_len, seq.length))
-        keep_pages = (new_len + self.page_size - 1) // self.page_size
-        while len(seq.pages) > keep_pages:
-            self.kv.free.append(seq.pages.pop())
-        seq.length = new_len
-        self.seq_len_dev[sid] = new_len
-
-    def copy_seq(self, src: int, dst: int, n: int | None = None):
-        """Copy the first `n` cached tokens (default: all) of sequence `src` into `dst` (which is overwritten).
-        Parity: `llama_memory_seq_cp` (`llama-kv-cache.cpp:322-392`) - used for prompt sharing between slots / beams."""
-        s, d = self.seqs[src], self.seqs[dst]
-        n = s.length if n is None else min(n, s.length)
-        self.truncate_seq(dst, 0)
-        self.kv.ensure(d, n)
-        npg = (n + self.page_size - 1) // self.page_size
-        if npg:
-            sp = torch.tensor(s.pages[:npg], dtype=torch.long, device=self.device)
-            dp = torch.tensor(d.pages[:npg], dtype=torch.long, device=self.device)
-            for il in self.w.layer_range:
-                self.kv.k[il][dp] = self.kv.k[il][sp]
-                self.kv.v[il][dp] = self.kv.v[il][sp]
-        d.length = n
-        self.seq_len_dev[dst] = n
+    def _graph_ok(self) -> bool:
+        moe_lw = next((lw for lw in self.w.layers.values() if lw.router is not None), None)
+        return moe_lw is None or self._moe_grouped_ok(moe_lw)      # routing through the host: no graph
 
     def shift_seq(self, sid: int, n_keep: int, n_discard: int):
         """Context shift: drop cached tokens [n_keep, n_keep + n_discard) and slide the rest down, re-rotating their keys by
@@ -845,114 +709,3 @@ class LlamaEngine:
             self.logits_full = lg  # full-vocab logits (gathered across TP ranks); static across graph replays
             if sample:   # records are indexed by sequence slot through the row -> slot map: nothing of a request is baked in
                 ops.sample_dev(lg, self.samp, self.active[:B], self.next_tok[:B])
-
-    @torch.no_grad()
-    def decode(self, sids: list[int], tokens=None, hidden_in: torch.Tensor | None = None, sample: bool = True,
-               use_graph: bool = True):
-        """One token for each sequence in `sids` (any subset of slots; batch row i belongs to sids[i]).
-        tokens: host ints / tensor, or None to feed back the previously sampled tokens (device resident).
-        Returns next-token ids (device int32 [B]) when sampling, else logits [B, vocab]; or hidden states."""
-        B = len(sids)
-        for sid in sids:
-            seq = self.seqs[sid]
-            self.kv.ensure(seq, seq.length + 1)
-        if sids != self._active_host:
-            self.active[:B].copy_(torch.tensor(sids, dtype=torch.int32), non_blocking=False)
-            self._active_host = list(sids)
-        if tokens is not None and self.first_stage:
-            self.next_tok[:B].copy_(torch.as_tensor(tokens, dtype=torch.int32), non_blocking=True)
-        if hidden_in is not None:
-            self.h[:B].copy_(hidden_in)
-        moe_lw = next((lw for lw in self.w.layers.values() if lw.router is not None), None)
-        moe_host = moe_lw is not None and not self._moe_grouped_ok(moe_lw)   # routing through the host: no graph
-        graphable = (use_graph and self.eval_callback is None and self.device.type == "cuda" and not moe_host
-                     and not getattr(self.comm, "no_graph", False)    # (the sequence-parallel path is capturable too: its epochs are
-                     and not (self.sp_ok and B > 4 and os.environ.get("DLP_SP_GRAPH", "1") == "0"))   # positions inside the pass on top of a device-side counter; DLP_SP_GRAPH=0: A/B)
-        self._onepass_now = self.attn_onepass and max(self.seqs[sid].length for sid in sids) + 1 >= self.attn_onepass_min
-        if sample and self.last_stage:
-            self._sync_sampling(sids)
-        # all rows greedy on the fused tensor-parallel path: sharded arg-max instead of gathering the logits (host-side fact, so
-        # it is part of the graph key; at most one extra graph per batch size)
-        self._greedy_now = bool(sample and self.last_stage and self.fused_tp and (B in (1, 2, 4) or (self.sp_ok and 4 < B <= 64)) and
-                                os.environ.get("DLP_TP_ARGMAX", "1") == "1" and all(self._samp_host[sid][3] <= 0 for sid in sids))
-        if graphable:
-            # only the batch size, the output kind and the attention variant shape the graph (sampler parameters are device data)
-            key = (B, sample, self._onepass_now, self._greedy_now)
-            g = self._graphs.pop(key, None)
-            if g is None:
-                while len(self._graphs) + 2 > self.max_graphs:    # least recently used graphs go first
-                    old = next(iter(self._graphs))
-                    del self._graphs[old]
-                    self._graph_launches.pop(old, None)
-                if self.attn_onepass:   # capture the other attention variant now as well: the switch at 64 keys must not stall
-                    want = self._onepass_now
-                    self._onepass_now = not want
-                    self._capture(B, sample, key[:2] + (not want,) + key[3:])
-                    self._onepass_now = want
-                g = self._capture(B, sample, key)
-                self._graphs.pop(key)
-            self._graphs[key] = g      # most recently used last
-            g.replay()
-            self.launches_replayed += self._graph_launches.get(key, 0)
-        else:
-            self._decode_body(B, sample)
-        for sid in sids:
-            self.seqs[sid].length += 1
-        if not self.last_stage:
-            return self.h[:B]
-        return self.next_tok[:B] if sample else self.logits_full[:B]
-
-    def _capture(self, B: int, sample: bool, key=None):
-        # warm-up (also lets every kernel set its attributes), then roll back the bookkeeping it advanced
-        saved = self.seq_len_dev.clone()
-        saved_ctr = self.step_ctr.clone()
-        saved_h = self.h[:B].clone()   # non-first stages consume their input hidden state in place: the warm-up must not eat it
-        saved_tok = self.next_tok.clone()   # the warm-up samples into next_tok: the pending input token must survive it
-        saved_samp = self.samp.clone()      # ... and advances the draw counters
-        s = torch.cuda.Stream()
-        s.wait_stream(torch.cuda.current_stream())
-        with torch.cuda.stream(s):
-            self._decode_body(B, sample)
-        torch.cuda.current_stream().wait_stream(s)
-        self.seq_len_dev.copy_(saved)
-        self.step_ctr.copy_(saved_ctr)
-        self.h[:B].copy_(saved_h)
-        self.next_tok.copy_(saved_tok)
-        self.samp.copy_(saved_samp)
-        g = torch.cuda.CUDAGraph()
-        n0 = ops.launch_count
-        with torch.cuda.graph(g):
-            self._decode_body(B, sample)
-        self.launches_per_graph = getattr(self, "launches_per_graph", {})
-        self.launches_per_graph[(B, sample)] = ops.launch_count - n0
-        self._graph_launches[key or (B, sample)] = ops.launch_count - n0
-        self.seq_len_dev.copy_(saved)
-        self.step_ctr.copy_(saved_ctr)
-        self._graphs[key or (B, sample)] = g
-        return g
-
-    # ---- convenience ------------------------------------------------------------------------------
-    @torch.no_grad()
-    def generate(self, prompt: list[int], n_predict: int, sid: int | None = None, stop_ids: tuple[int, ...] = ()):
-        """Greedy / sampled generation for one sequence (slot 0 path); returns the generated ids."""
-        own = sid is None
-        if own:
-            sid = self.alloc_seq()
-        logits = self.prefill(sid, prompt)
-        s = self.sampling
-        if s["temp"] <= 0:
-            tok = ops.argmax(logits[None])
-        else:   # first token from the prefill logits: same per-sequence record (and random stream) as the decode steps
-            self._sync_sampling([sid])
-            tok = ops.sample_dev(logits[None], self.samp, torch.tensor([sid], dtype=torch.int32, device=self.device),
-                                 torch.empty(1, dtype=torch.int32, device=self.device))
-        self.next_tok[:1].copy_(tok)
-        out = [int(tok[0])]
-        for _ in range(n_predict - 1):
-            if out[-1] in stop_ids:
-                break
-            nt = self.decode([sid])
-            out.append(int(nt[0]))
-        if own:
-            self.free_seq(sid)
-        return out

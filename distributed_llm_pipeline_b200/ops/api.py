@@ -40,6 +40,11 @@ def _count(n: int = 1):
     launch_count += n
 
 
+def need_full_library():
+    """Load the library with every kernel (a process may so far have loaded the layer-list part only)."""
+    _lib.load_full()
+
+
 def native(t: torch.Tensor) -> bool:
     return t.is_cuda
 

@@ -14,8 +14,10 @@ import threading
 _HERE = os.path.dirname(os.path.abspath(__file__))
 _REPO = os.path.dirname(os.path.dirname(_HERE))
 LIB_PATH = os.path.join(_HERE, "libdlp_b200.so")
+LAYERS_LIB_PATH = os.path.join(_HERE, "libdlp_b200_layers.so")      # the part a layer-list model runs (csrc/build.sh layers)
 
 _lib = None
+_lib_layers = None
 _lock = threading.Lock()
 
 
@@ -24,17 +26,22 @@ class dlp_weight(C.Structure):
                 ("wtype", C.c_int32), ("N", C.c_int32), ("K", C.c_int32), ("reserved", C.c_int32)]
 
 
-def build(force: bool = False) -> str:
-    """Compile the CUDA sources for sm_100a (cross-compiles without a GPU)."""
-    script = os.path.join(_REPO, "csrc", "build.sh")
-    if force and os.path.isdir(os.path.join(_REPO, "csrc", "build")):
-        for f in os.listdir(os.path.join(_REPO, "csrc", "build")):
+def build(force: bool = False, part: str = "all") -> str:
+    """Compile the CUDA sources for sm_100a (cross-compiles without a GPU).  One build at a time per checkout."""
+    import fcntl
+    csrc = os.path.join(_REPO, "csrc")
+    script = os.path.join(csrc, "build.sh")
+    if force and os.path.isdir(os.path.join(csrc, "build")):
+        for f in os.listdir(os.path.join(csrc, "build")):
             if f.endswith(".o"):
-                os.remove(os.path.join(_REPO, "csrc", "build", f))
-    res = subprocess.run(["bash", script], capture_output=True, text=True)
+                os.remove(os.path.join(csrc, "build", f))
+    os.makedirs(os.path.join(csrc, "build"), exist_ok=True)
+    with open(os.path.join(csrc, "build", ".lock"), "w") as lk:
+        fcntl.flock(lk, fcntl.LOCK_EX)
+        res = subprocess.run(["bash", script, part], capture_output=True, text=True)
     if res.returncode != 0:
-        raise RuntimeError(f"building libdlp_b200.so failed:\n{res.stdout}\n{res.stderr}")
-    return LIB_PATH
+        raise RuntimeError(f"building the kernel library ({part}) failed:\n{res.stdout}\n{res.stderr}")
+    return LIB_PATH if part == "all" else LAYERS_LIB_PATH
 
 
 def _declare(lib):
@@ -67,6 +74,14 @@ def _declare(lib):
         "dlp_sample": (i32, [vp, i32, i32, i32, i32, f32, f32, f32, u32, vp, vp, vp]),
         "dlp_f32_to_f16": (i32, [vp, vp, sz, vp]),
         "dlp_moe_route": (i32, [vp, i32, i32, i32, vp, vp, vp]),
+        "dlp_layers_matvec": (i32, [vp, vp, i32, i32, vp, i32, i32, i32, i32, vp]),
+        "dlp_layers_stage_rows": (i32, [vp, vp, i32, i32, i32, vp]),
+        "dlp_layers_linear": (i32, [vp, i32, vp, i32, i32, i32, vp, i32, i32, i32, i32, vp, sz, vp]),
+        "dlp_layers_head_matmul": (i32, [vp, i32, i32, i32, i32, vp, i32, i32, i32, i32, vp, i32, i32, vp, i32, i32, i32, vp]),
+        "dlp_layers_embed": (i32, [vp, i32, vp, vp, i32, i32, i32, i32, vp]),
+        "dlp_layers_latent_write": (i32, [vp, i32, vp, f32, i32, i32, vp, vp, i32, i32, vp]),
+        "dlp_layers_hgrn2": (i32, [vp, i32, vp]),
+        "dlp_layers_latent_attention": (i32, [vp, i32, vp]),
         "dlp_gemv_moe": (i32, [W, W, vp, vp, f32, vp, i32, i32, vp, i32, vp, vp]),
     }
     for name, (res, args) in sigs.items():
@@ -82,18 +97,40 @@ def available() -> bool:
 
 
 def load():
-    """Return the loaded library, building it first if the `.so` is absent and nvcc exists."""
+    """Return the loaded library (whichever part is loaded already), building the whole one first if it is absent and nvcc exists."""
+    return _lib or _lib_layers or load_full()
+
+
+def load_full():
+    """The library with every kernel: what GGUF models need."""
     global _lib
+    if _lib is None:
+        with _lock:
+            if _lib is None:
+                if not os.path.exists(LIB_PATH):
+                    build()
+                lib = C.CDLL(LIB_PATH, mode=C.RTLD_GLOBAL)
+                _declare(lib)
+                _lib = lib
+    return _lib
+
+
+def load_layers():
+    """A library with the kernels of layer-list models: the whole one when it is there, else the part (built at first use)."""
+    global _lib_layers
     if _lib is not None:
         return _lib
-    with _lock:
-        if _lib is None:
-            if not os.path.exists(LIB_PATH):
-                build()
-            lib = C.CDLL(LIB_PATH, mode=C.RTLD_GLOBAL)
-            _declare(lib)
-            _lib = lib
-    return _lib
+    if os.path.exists(LIB_PATH):
+        return load_full()
+    if _lib_layers is None:
+        with _lock:
+            if _lib_layers is None:
+                if not os.path.exists(LAYERS_LIB_PATH):
+                    build(part="layers")
+                lib = C.CDLL(LAYERS_LIB_PATH, mode=C.RTLD_LOCAL)
+                _declare(lib)
+                _lib_layers = lib
+    return _lib_layers
 
 
 class DlpError(RuntimeError):

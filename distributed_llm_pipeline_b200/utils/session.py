@@ -3,8 +3,9 @@
 Parity: llama.cpp session files and per-sequence state (`llama_state_seq_save_file` / `llama_state_save_file`,
 `llama.cpp/src/llama-context.cpp:2311-2509`; KV part `llama-kv-cache.cpp:1490-1980`) and the server's
 `/slots/:id?action=save|restore|erase` (`tools/server/server.cpp:196-197`).  File layout (little endian):
-  magic "DLPS" | u32 version | u32 json_len | json header | K/V payload: for each local layer, K then V,
-  [n_tokens, Hkv, D] fp16 (token-major, i.e. gathered out of the pages - the file does not depend on the page layout)
+  magic "DLPS" | u32 version | u32 json_len | json header | cache payload: for each local layer its planes (K then V; the latent rows
+  of latent attention), [n_tokens, heads, dim] in the cache's type (token-major, i.e. gathered out of the pages - the file does not
+  depend on the page layout) | the fp32 state of every recurrent layer
 The header records the model fingerprint (arch, dims, layer range, TP shard) and the token ids; restore refuses a
 mismatching model and works into a fragmented page pool (pages are allocated wherever the free list has them).
 """
@@ -13,7 +14,6 @@ from __future__ import annotations
 import json
 import struct
 
-import numpy as np
 import torch
 
 MAGIC = b"DLPS"
@@ -22,9 +22,13 @@ VERSION = 1
 
 def _fingerprint(eng) -> dict:
     c = eng.cfg
-    return {"arch": c.arch, "n_embd": c.n_embd, "n_layer": c.n_layer, "n_head_kv_local": eng.Hkv, "head_dim": c.head_dim,
-            "layers": [eng.w.layer_range.start, eng.w.layer_range.stop], "tp_rank": eng.w.tp_rank, "tp_size": eng.w.tp_size,
-            "vocab": c.vocab_size}
+    fp = {"arch": c.arch, "n_embd": c.n_embd, "n_layer": c.n_layer, "n_head_kv_local": getattr(eng, "Hkv", 0), "head_dim": c.head_dim,
+          "layers": [eng.w.layer_range.start, eng.w.layer_range.stop], "tp_rank": eng.w.tp_rank, "tp_size": eng.w.tp_size,
+          "vocab": c.vocab_size}
+    if c.layers:
+        fp["planes"] = [[il, name, list(t.shape[1:2] + t.shape[3:]), str(t.dtype)] for il, name, t in eng.kv.each_plane()]
+        fp["states"] = [[il, list(t.shape[1:])] for il, t in eng.rstate.layers.items()]
+    return fp
 
 
 def save_sequence(eng, sid: int, path: str, tokens: list[int] | None = None) -> int:
@@ -36,11 +40,12 @@ def save_sequence(eng, sid: int, path: str, tokens: list[int] | None = None) -> 
     hj = json.dumps(hdr).encode()
     with open(path, "wb") as f:
         f.write(MAGIC + struct.pack("<II", VERSION, len(hj)) + hj)
-        for il in eng.w.layer_range:
-            for cache in (eng.kv.k[il], eng.kv.v[il]):
-                # [pages, Hkv, page, D] -> [tokens, Hkv, D]
-                t = cache[pages].permute(0, 2, 1, 3).reshape(-1, eng.Hkv, eng.D)[:n].contiguous()
-                f.write(t.cpu().numpy().astype("<f2", copy=False).tobytes())
+        for _, _, cache in eng.kv.each_plane():
+            # [pages, heads, page, dim] -> [tokens, heads, dim]
+            t = cache[pages].permute(0, 2, 1, 3).reshape(-1, cache.shape[1], cache.shape[3])[:n].contiguous()
+            f.write(t.cpu().view(torch.uint8).numpy().tobytes())
+        for st in eng.rstate.layers.values():
+            f.write(st[sid].contiguous().cpu().numpy().tobytes())
         return f.tell()
 
 
@@ -64,16 +69,20 @@ def load_sequence(eng, sid: int, path: str) -> dict:
         ps = eng.page_size
         npg = (n + ps - 1) // ps
         pages = torch.tensor(seq.pages[:npg], dtype=torch.long, device=eng.device)
-        per = n * eng.Hkv * eng.D
-        for il in eng.w.layer_range:
-            for cache in (eng.kv.k[il], eng.kv.v[il]):
-                raw = np.frombuffer(f.read(per * 2), dtype="<f2")
-                if raw.size != per:
-                    raise ValueError(f"{path}: truncated session file")
-                t = torch.from_numpy(raw.copy()).view(n, eng.Hkv, eng.D)
-                pad = torch.zeros(npg * ps, eng.Hkv, eng.D, dtype=torch.float16)
-                pad[:n] = t
-                cache[pages] = pad.view(npg, ps, eng.Hkv, eng.D).permute(0, 2, 1, 3).to(eng.device)
+        def payload(nbytes):
+            raw = f.read(nbytes)
+            if len(raw) != nbytes:
+                raise ValueError(f"{path}: truncated session file")
+            return torch.frombuffer(bytearray(raw), dtype=torch.uint8) if nbytes else torch.empty(0, dtype=torch.uint8)
+
+        for _, _, cache in eng.kv.each_plane():
+            heads, dim = cache.shape[1], cache.shape[3]
+            t = payload(n * heads * dim * cache.element_size()).view(cache.dtype).view(n, heads, dim)
+            pad = torch.zeros(npg * ps, heads, dim, dtype=cache.dtype)
+            pad[:n] = t
+            cache[pages] = pad.view(npg, ps, heads, dim).permute(0, 2, 1, 3).to(eng.device)
+        for st in eng.rstate.layers.values():
+            st[sid] = payload(st[sid].numel() * 4).view(torch.float32).view(st.shape[1:]).to(eng.device)
         seq.length = n
         eng.seq_len_dev[sid] = n
     return hdr

@@ -347,6 +347,38 @@ int dlp_ipc_import(const void* handle64, void** ptr);
 int dlp_ipc_close(void* ptr);
 int dlp_memcpy_d2h(void* dst, const void* src, size_t bytes);
 
+/* ---- layer-list models: recurrent mixers, latent attention, norms behind the sublayers (csrc/layers_*.cu) ----
+ * f32 = 0: bf16 weights / activations / caches, fp32 accumulation; f32 = 1: fp32 throughout.  Residual stream, norms, recurrent
+ * state, attention scores and weights are fp32 in both. */
+typedef struct {              /* how a row is formed in front of a matrix product (csrc/layers.cuh RowStage) */
+    const void* x; int32_t x_f32, ldx;
+    const float* y; int32_t ldy;               /* x += gnorm(y; groups1) * w1 */
+    const float* w1; int32_t groups1;
+    float* h_out; int32_t ldh;
+    const float* w2; int32_t groups2, w2_mod;  /* then gnorm(.; groups2) * w2[k % w2_mod] */
+    float eps; int32_t K, Kp;
+} dlp_row_stage;
+typedef struct {
+    const float* proj; int32_t ldp; const float* fbias; const float* lower; float* state;
+    const int32_t* cu; const int32_t* seg_slot; const int32_t* pos; float* out; int32_t ldo, H, D, V, n_seg;
+} dlp_hgrn2_args;
+typedef struct {
+    const void* q; const void* cache; const int32_t* block_table; const int32_t* tok_slot; const int32_t* pos;
+    const int32_t* tile_row0; const int32_t* tile_rows; void* out; float* part_o; float* part_ml;
+    int32_t max_pages, page_size, H, Rc, T, n_tiles, bm, n_splits; float scale;
+} dlp_latent_args;
+/* decode product, 1..4 rows: out_mode 0 = fp32, 1 = GEGLU of interleaved (gate, up) rows -> activation type */
+int dlp_layers_matvec(const dlp_row_stage* st, const void* w, int ldw, int N, void* out, int ldo, int out_mode, int T, int f32, void* stream);
+int dlp_layers_stage_rows(const dlp_row_stage* st, void* xb, int ldxb, int T, int f32, void* stream);
+/* any number of rows: bf16 through the tcgen05 GEMM (ws: split-K workspace as for dlp_linear_ws), fp32 through an fp32 kernel */
+int dlp_layers_linear(const void* x, int ldx, const void* w, int ldw, int N, int K, void* out, int ldo, int out_mode, int T, int f32, void* ws, size_t ws_bytes, void* stream);
+int dlp_layers_head_matmul(const void* x, int x_f32, int ldx, int x_head, int kx, const void* w, int Kp, int H, int N, int n_rows, void* out, int ldo, int out_head,
+                           const float* gate, int ldg, int T, int f32, void* stream);
+int dlp_layers_embed(const void* table, int ld, const int32_t* ids, float* h, int E, int T, int vocab, int f32, void* stream);
+int dlp_layers_latent_write(const float* proj, int ldp, const float* w, float eps, int R, int Rc, const int32_t* slot, void* cache, int T, int f32, void* stream);
+int dlp_layers_hgrn2(const dlp_hgrn2_args* a, int impl, void* stream);   /* impl 0: token scan, 1: chunks on the tensor cores */
+int dlp_layers_latent_attention(const dlp_latent_args* a, int f32, void* stream);
+
 #ifdef __cplusplus
 }
 #endif
