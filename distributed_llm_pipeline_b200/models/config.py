@@ -18,6 +18,16 @@ class LayerSpec:
     mixer: dict[str, Any]
     mlp: dict[str, Any] | None = None
 
+    def n_params(self, width: int) -> int:
+        m = self.mixer
+        if self.type == "hgrn2":
+            hd, hv = m["heads"] * m["dim"], m["heads"] * m["vdim"]
+            n = width * (2 * hd + 2 * hv) + 2 * hd + m["vdim"]
+        else:       # latent_attention
+            hd, hv, r = m["heads"] * m["dim"], m["heads"] * m["vdim"], m["kv_rank"]
+            n = width * (hd + r + m["heads"] + hv) + r * (hd + hv) + r
+        return n + width + (3 * width * self.mlp["ff"] + width if self.mlp else 0)
+
 
 @dataclass(frozen=True)
 class ModelConfig:
@@ -126,6 +136,8 @@ class ModelConfig:
         return self.n_expert > 0
 
     def n_params(self) -> int:
+        if self.layers:
+            return 2 * self.vocab_size * self.n_embd + self.n_embd + sum(s.n_params(self.n_embd) for s in self.layers)
         attn = self.n_embd * (self.q_dim + 2 * self.kv_dim) + self.q_dim * self.n_embd
         ffn = 3 * self.n_embd * self.n_ff * max(1, self.n_expert) + (self.n_embd * self.n_expert if self.is_moe else 0)
         emb = self.vocab_size * self.n_embd * (1 if self.tie_embeddings else 2)

@@ -155,6 +155,8 @@ class EngineCore:
         self.max_graphs = int(os.environ.get("DLP_MAX_GRAPHS", str(max(24, 4 * max_seqs + 8))))   # (batch sizes x attention variants x greedy)
         self._graphs: dict[tuple, torch.cuda.CUDAGraph] = {}
         self._graph_launches: dict[tuple, int] = {}    # kernels inside each captured graph
+        self._graph_logits: dict[tuple, torch.Tensor] = {}     # full-vocabulary logits each captured graph leaves behind
+        self.logits_full = None
         self.launches_replayed = 0                      # kernels launched through graph replays so far
         self.sampling = dict(top_k=40, top_p=0.95, min_p=0.05, temp=0.0, seed=0)
         self.cvec: dict[int, torch.Tensor] = {}     # layer -> fp32 [E] added to the residual stream after that layer
@@ -168,7 +170,7 @@ class EngineCore:
     def _graph_ok(self) -> bool:
         return True
 
-    def _choose_variant(self, max_len: int):
+    def _choose_variant(self, B: int, max_len: int):
         """Pick the launch variant of the next decode step from the longest context (cached tokens + 1)."""
 
     def _companion_variants(self) -> list:
@@ -184,6 +186,7 @@ class EngineCore:
             raise RuntimeError("no free sequence slots")
         sid = self._free_sids.pop()
         self.seqs[sid] = Sequence(sid)
+        self.seq_len_dev[sid] = 0        # a decode step may be the sequence's first: the device-side length starts over with the slot
         return sid
 
     def free_seq(self, sid: int):
@@ -281,7 +284,7 @@ class EngineCore:
         graphable = (use_graph and self.eval_callback is None and self.device.type == "cuda" and self._graph_ok()
                      and not getattr(self.comm, "no_graph", False)    # (the sequence-parallel path is capturable too: its epochs are
                      and not (self.sp_ok and B > 4 and os.environ.get("DLP_SP_GRAPH", "1") == "0"))   # positions inside the pass on top of a device-side counter; DLP_SP_GRAPH=0: A/B)
-        self._choose_variant(max(self.seqs[sid].length for sid in sids) + 1)
+        self._choose_variant(B, max(self.seqs[sid].length for sid in sids) + 1)
         if sample and self.last_stage:
             self._sync_sampling(sids)
         # all rows greedy on the fused tensor-parallel path: sharded arg-max instead of gathering the logits (host-side fact, so
@@ -297,6 +300,7 @@ class EngineCore:
                     old = next(iter(self._graphs))
                     del self._graphs[old]
                     self._graph_launches.pop(old, None)
+                    self._graph_logits.pop(old, None)
                 want = self._variant
                 for other in self._companion_variants():   # captured now as well: the switch between them must not stall a later step
                     self._variant = other
@@ -306,6 +310,7 @@ class EngineCore:
                 self._graphs.pop(key)
             self._graphs[key] = g      # most recently used last
             g.replay()
+            self.logits_full = self._graph_logits.get(key)      # the rows this graph writes (another batch size may have been captured since)
             self.launches_replayed += self._graph_launches.get(key, 0)
         else:
             self._decode_body(B, sample)
@@ -341,6 +346,7 @@ class EngineCore:
         self.launches_per_graph = getattr(self, "launches_per_graph", {})
         self.launches_per_graph[(B, sample)] = ops.launch_count - n0
         self._graph_launches[key or (B, sample)] = ops.launch_count - n0
+        self._graph_logits[key or (B, sample)] = self.logits_full
         self.seq_len_dev.copy_(saved)
         self.step_ctr.copy_(saved_ctr)
         self._graphs[key or (B, sample)] = g

@@ -1,0 +1,384 @@
+"""Step of layer-list models on the engine core: mixers of different kinds in one model, norms behind the sublayers.
+
+The residual stream is fp32.  A sublayer's output `y` is not added at once: it stays pending, and the next matrix product forms
+`h + norm(y)` while it prepares its input rows (in the mat-vec prologue for up to four rows, in one row kernel in front of the GEMM
+for more).  One forward takes any mix of prompt portions and single tokens of different sequences: projections run over all rows,
+mixers over the segments.
+"""
+from __future__ import annotations
+
+from dataclasses import dataclass
+
+import torch
+
+from ..ops import api as ops
+from ..ops import layers as lops
+from ..ops.weights import DeviceWeight
+from ..gguf.constants import GGMLType
+from .engine import EngineCore, PagedKVCache, RecurrentState
+from .mixers import MIXERS, MLPS, Dense, LatentAttention, Rows, pad_to
+from .modeldir import ModelDir, open_model_dir
+from .weights import ModelWeights
+
+DTYPES = {"bf16": torch.bfloat16, "bfloat16": torch.bfloat16, "f32": torch.float32, "float32": torch.float32}
+MATVEC_ROWS = 4
+
+
+@dataclass
+class LayeredLayer:
+    mixer: object
+    norm1: torch.Tensor
+    mlp: object | None = None
+    norm2: torch.Tensor | None = None
+
+    def weights(self):
+        return self.mixer.weights() + (self.mlp.weights() if self.mlp is not None else [])
+
+
+class LayeredWeights(ModelWeights):
+    def nbytes(self) -> int:
+        return sum(w.nbytes for lw in self.layers.values() for w in lw.weights()) + self.tok_embd.nbytes + self.lm_head.nbytes
+
+
+def load_layered_weights(src: str | ModelDir, device, dtype="bf16", progress=None) -> LayeredWeights:
+    """Weights of a model folder on the device, in the storage type `dtype` (bf16 | f32); norms, biases and gate bounds are fp32."""
+    from .weights import LoadCancelled
+    d = open_model_dir(src) if isinstance(src, str) else src
+    dt = DTYPES[dtype] if isinstance(dtype, str) else dtype
+    cfg, f, dev = d.cfg, d.tensors, torch.device(device)
+
+    def f32(name, n):
+        t = f.tensor(name).to(device=dev, dtype=torch.float32).contiguous()
+        if t.shape != (n,):
+            raise ValueError(f"{name} has the shape {tuple(t.shape)}, expected ({n},)")
+        return t
+    layers = {}
+    for il, spec in enumerate(cfg.layers):
+        if progress is not None and progress(il / cfg.n_layer) is False:
+            raise LoadCancelled("load cancelled")
+        p = f"l{il}."
+        lw = LayeredLayer(MIXERS[spec.type](spec.mixer, lambda n: f.tensor(p + "mix." + n), dev, dt), f32(p + "norm1", cfg.n_embd))
+        if spec.mlp is not None:
+            lw.mlp = MLPS[spec.mlp["kind"]](spec.mlp, lambda n: f.tensor(p + "mlp." + n), dev, dt)
+            lw.norm2 = f32(p + "norm2", cfg.n_embd)
+        layers[il] = lw
+
+    def table(name):
+        w = Dense.make(f.tensor(name), dev, dt)
+        if w.N != cfg.vocab_size or w.K != cfg.n_embd:
+            raise ValueError(f"{name} is [{w.N}, {w.K}], expected [{cfg.vocab_size}, {cfg.n_embd}]")
+        return DeviceWeight(GGMLType.F32 if dt == torch.float32 else GGMLType.BF16, w.N, w.K, [w.t])
+    emb, head = table("embed"), table("head")
+    out_norm = f32("final.norm", cfg.n_embd)
+    if progress is not None and progress(1.0) is False:
+        raise LoadCancelled("load cancelled")
+    return LayeredWeights(cfg, layers, range(cfg.n_layer), 0, 1, emb, out_norm, head, (0, cfg.vocab_size), None)
+
+
+@dataclass
+class TileTable:
+    """(token, head) row tiles of one latent-attention shape."""
+    row0: torch.Tensor
+    rows: torch.Tensor
+    n: int
+    bm: int
+    n_splits: int
+
+
+@dataclass
+class Batch:
+    """Device-side description of one forward: T rows, grouped into segments (one per sequence)."""
+    T: int
+    n_seg: int
+    cu: torch.Tensor            # [n_seg + 1] row range of every segment
+    seg_slot: torch.Tensor      # [n_seg] sequence slot
+    tok_slot: torch.Tensor      # [T] sequence slot of every row
+    pos: torch.Tensor           # [T]
+    slot: torch.Tensor          # [T] cache row
+    tiles: dict[int, TileTable]
+
+
+class LayeredEngine(EngineCore):
+    mixed_batches = True
+    can_shift = False           # a recurrent state has no positions to slide
+
+    def __init__(self, weights: LayeredWeights, n_ctx: int = 4096, max_seqs: int = 8, page_size: int = 64, max_batch_tokens: int = 2048,
+                 n_pages: int | None = None, comm=None, first_stage: bool = True, last_stage: bool = True):
+        cfg = weights.cfg
+        if comm is not None and comm.tp_size > 1 or not (first_stage and last_stage):
+            raise NotImplementedError(f"{cfg.arch}: layer-list models run on one GPU (no tensor-parallel or pipeline split)")
+        dev = weights.tok_embd.device
+        self._init_core(weights, n_ctx, max_seqs, page_size, max_batch_tokens, comm, True, True, dev)
+        if dev.type == "cuda":
+            lops.load_library()
+        self.dtype = weights.tok_embd.planes[0].dtype
+        self.E = cfg.n_embd
+        mixers = {il: lw.mixer for il, lw in weights.layers.items()}
+        max_pages = (n_ctx + page_size - 1) // page_size
+        planes: dict[str, dict] = {}
+        for il, m in mixers.items():
+            for name, shape in m.planes.items():
+                planes.setdefault(name, {})[il] = shape
+        self.kv = PagedKVCache(planes, max_pages * max_seqs if n_pages is None else n_pages, page_size, max_seqs, max_pages, dev, dtype=self.dtype)
+        self.rstate = RecurrentState({il: m.state for il, m in mixers.items() if m.state is not None}, max_seqs, dev)
+        M, f32 = self.max_rows, torch.float32
+        self.hb = [torch.zeros(M, self.E, dtype=f32, device=dev) for _ in range(2)]      # residual stream; the mat-vec path alternates
+        self.h = self.hb[0]
+        self.cur = 0
+        self.y = torch.zeros(M, self.E, dtype=f32, device=dev)
+        sizes = {"proj": M * max(m.w_in.N for m in mixers.values()), "xb": M * max([pad_to(self.E, 8)] + [w.Kp for lw in weights.layers.values() for w in lw.weights()]),
+                 "act": M * max([8] + [lw.mlp.w_down.Kp for lw in weights.layers.values() if lw.mlp is not None])}
+        for m in mixers.values():
+            for name, n in m.buffers(M).items():
+                sizes[name] = max(sizes.get(name, 0), n)
+        types = {"proj": f32, "o": f32}
+        self._flat = {n: torch.zeros(sz, dtype=types.get(n, self.dtype), device=dev) for n, sz in sizes.items()}
+        self.logits = torch.zeros(max_seqs, cfg.vocab_size, dtype=f32, device=dev)
+        lat = [m for m in mixers.values() if isinstance(m, LatentAttention)]
+        self._latent_heads = sorted({m.H for m in lat})
+        self._split_ctas = 296                                       # two CTAs per SM: the key range is split until they are there
+        self.latent_ws = None
+        if lat:
+            rows = self._split_ctas * 64
+            self.latent_ws = (torch.zeros(rows * max(m.Rc for m in lat), dtype=f32, device=dev), torch.zeros(rows * 2, dtype=f32, device=dev))
+        self._variant = 1                                            # key ranges per decode query
+        self._decode_batches: dict[tuple, Batch] = {}
+
+    def buf(self, name: str, rows: int, cols: int, dtype=None) -> torch.Tensor:
+        return self._flat[name][:rows * cols].view(rows, cols)
+
+    # ---- matrix products -------------------------------------------------------------------------------
+    def _product(self, r: Rows, w: Dense, out: torch.Tensor, T: int, geglu: bool = False) -> torch.Tensor:
+        cfg = self.cfg
+        if T <= MATVEC_ROWS:
+            st = lops.row_stage(r.x, r.K, w.Kp, cfg.rms_eps, r.y, r.w1, cfg.norm_groups, r.h_out, r.w2, r.groups2)
+            return lops.matvec(st, w.t, out, T, geglu)
+        x = r.x
+        if r.y is not None or r.w2 is not None or x.dtype != self.dtype or x.shape[1] != w.Kp:
+            st = lops.row_stage(r.x, r.K, w.Kp, cfg.rms_eps, r.y, r.w1, cfg.norm_groups, r.h_out, r.w2, r.groups2)
+            x = lops.stage_rows(st, self.buf("xb", T, w.Kp), T)
+        return lops.linear(x[:T], w.t, out, geglu)
+
+    def _residual(self, T: int, pending) -> Rows:
+        """Rows of the residual stream with the pending sublayer output folded in on the way."""
+        if pending is None:
+            return Rows(self.hb[self.cur][:T], self.E)
+        src = self.hb[self.cur][:T]
+        if T <= MATVEC_ROWS:        # every block of the mat-vec reads the old rows: the new ones go to the other buffer
+            self.cur ^= 1
+        return Rows(src, self.E, y=self.y[:T], w1=pending, h_out=self.hb[self.cur][:T])
+
+    def _settle(self, T: int, pending):
+        """Fold the pending output into the residual stream now; returns the rows [T, E] fp32."""
+        if pending is not None:
+            h = self.hb[self.cur][:T]
+            st = lops.row_stage(h, self.E, self.E, self.cfg.rms_eps, self.y[:T], pending, self.cfg.norm_groups, h)
+            lops.stage_rows(st, self.buf("xb", T, self.E), T)
+        return self.hb[self.cur][:T]
+
+    # ---- one forward over a batch ------------------------------------------------------------------------
+    def _forward(self, ids: torch.Tensor, b: Batch):
+        """Embedding and all layers; returns the norm weight of the output still pending in self.y (None: nothing pending)."""
+        T = b.T
+        self.cur = 0
+        lops.embed(self.w.tok_embd.planes[0], ids, self.hb[0], T)
+        pending = None
+        for il, lw in self.w.layers.items():
+            m = lw.mixer
+            proj = self._product(self._residual(T, pending), m.w_in, self.buf("proj", T, m.w_in.N), T)
+            self._product(m.mix(self, il, proj, b), m.w_out, self.y[:T], T)
+            pending = lw.norm1
+            if lw.mlp is not None:
+                g = lw.mlp
+                act = self._product(self._residual(T, pending), g.w_gu, self.buf("act", T, g.w_down.Kp), T, geglu=True)
+                self._product(Rows(act, g.w_down.K), g.w_down, self.y[:T], T)
+                pending = lw.norm2
+            if self.eval_callback is not None or il in self.cvec:
+                h = self._settle(T, pending)
+                pending = None
+                if il in self.cvec:
+                    h.add_(self.cvec[il])
+                if self.eval_callback is not None:
+                    self.eval_callback("l_out", il, h)
+        return pending
+
+    def _head_rows(self, r: Rows, n: int, out: torch.Tensor) -> torch.Tensor:
+        r.w2, r.groups2 = self.w.out_norm, self.cfg.norm_groups
+        head = self.w.lm_head
+        return self._product(r, Dense(head.planes[0], head.K), out, n)
+
+    # ---- batch descriptions ---------------------------------------------------------------------------------
+    def _n_splits(self, n_tiles: int, max_len: int) -> int:
+        want, n = min(self._split_ctas // max(1, n_tiles), (max_len + 255) // 256, 32), 1
+        while n * 2 <= want:
+            n *= 2
+        return n
+
+    def _tile_lists(self, H: int, lens: list[int], bm: int):
+        row0, rows, base = [], [], 0
+        for n in lens:
+            for i in range(0, n * H, bm):
+                row0.append(base + i)
+                rows.append(min(bm, n * H - i))
+            base += n * H
+        return row0, rows
+
+    def _decode_batch(self, B: int) -> Batch:
+        b = self._decode_batches.get((B, self._variant))
+        if b is None:
+            dev, i32 = self.device, torch.int32
+            tiles = {}
+            for H in self._latent_heads:
+                bm = lops.latent_tile_rows(H, B)
+                row0, rows = self._tile_lists(H, [1] * B, bm)
+                tiles[H] = TileTable(torch.tensor(row0, dtype=i32, device=dev), torch.tensor(rows, dtype=i32, device=dev), len(row0), bm, min(self._variant, max(1, self._split_ctas // len(row0))))
+            b = Batch(B, B, torch.arange(B + 1, dtype=i32, device=dev), self.active, self.active, self.pos, self.slot, tiles)
+            self._decode_batches[(B, self._variant)] = b
+        return b
+
+    def _mixed_batch(self, parts: list[tuple[int, list[int]]]) -> tuple[torch.Tensor, Batch]:
+        """Grow every sequence by its tokens and upload the description in one copy."""
+        lens = [len(t) for _, t in parts]
+        T, n = sum(lens), len(parts)
+        cols: list[torch.Tensor] = [torch.cat([torch.as_tensor(t, dtype=torch.int32) for _, t in parts])]
+        pos, slot = zip(*(self._advance_inputs(sid, len(t)) for sid, t in parts))
+        cols += [torch.cat(pos), torch.cat(slot), torch.cat([torch.full((len(t),), sid, dtype=torch.int32) for sid, t in parts]),
+                 torch.tensor([0] + torch.tensor(lens).cumsum(0).tolist(), dtype=torch.int32), torch.tensor([sid for sid, _ in parts], dtype=torch.int32)]
+        shapes = []
+        for H in self._latent_heads:
+            bm = lops.latent_tile_rows(H, T)
+            row0, rows = self._tile_lists(H, lens, bm)
+            cols += [torch.tensor(row0, dtype=torch.int32), torch.tensor(rows, dtype=torch.int32)]
+            shapes.append((H, bm, len(row0)))
+        dev = iter(torch.cat(cols).to(self.device).split([c.numel() for c in cols]))
+        ids, pos_d, slot_d, tok_slot, cu, seg_slot = (next(dev) for _ in range(6))
+        longest = max(self.seqs[sid].length + len(t) for sid, t in parts)
+        tiles = {H: TileTable(next(dev), next(dev), nt, bm, self._n_splits(nt, longest)) for H, bm, nt in shapes}
+        return ids, Batch(T, n, cu, seg_slot, tok_slot, pos_d, slot_d, tiles)
+
+    def _run_mixed(self, parts: list[tuple[int, list[int]]]):
+        """Forward over one mixed batch; updates the sequence lengths.  Returns the pending norm weight (see _forward)."""
+        ids, b = self._mixed_batch(parts)
+        pending = self._forward(ids, b)
+        for sid, t in parts:
+            self.seqs[sid].length += len(t)
+        lens = torch.tensor([[sid, self.seqs[sid].length] for sid, _ in parts], dtype=torch.int32).to(self.device)
+        self.seq_len_dev[lens[:, 0].long()] = lens[:, 1]
+        return pending
+
+    # ---- public ---------------------------------------------------------------------------------------------
+    @torch.no_grad()
+    def step(self, entries, want=None) -> torch.Tensor:
+        """Append tokens to several sequences in one batch.  entries: [(sid, tokens)], every sequence at most once, portions of any length
+        beside single tokens; want: for every entry the places among its tokens whose logits are returned (default: the last one).
+        Returns fp32 logits [wanted, vocab] in the order of the entries.  A batch of single tokens is a decode step and runs as one
+        (captured graph); more tokens than the engine's batch holds run as several forwards."""
+        entries = [(sid, [int(t) for t in toks]) for sid, toks in entries]
+        if want is None:
+            want = [[len(t) - 1] for _, t in entries]
+        if len({sid for sid, _ in entries}) != len(entries) or any(not t for _, t in entries):
+            raise ValueError("step: every sequence may appear once, with at least one token")
+        if any(not 0 <= p < len(t) for (_, t), w in zip(entries, want) for p in w):
+            raise ValueError("step: a wanted place outside its tokens")
+        self._reserve([(sid, len(t)) for sid, t in entries])
+        if all(len(t) == 1 for _, t in entries):
+            lg = self.decode([sid for sid, _ in entries], [t[0] for _, t in entries], sample=False)
+            rows = [i for i, w in enumerate(want) for _ in w]
+            return lg[torch.tensor(rows, dtype=torch.long, device=self.device)].clone()
+        out = torch.empty(sum(len(w) for w in want), self.cfg.vocab_size, dtype=torch.float32, device=self.device)
+        offs = [0]
+        for w in want:
+            offs.append(offs[-1] + len(w))
+        done = [0] * len(entries)
+        while any(d < len(t) for d, (_, t) in zip(done, entries)):
+            room, parts, rows, dst = self.max_tokens, [], [], []
+            for i, (sid, toks) in enumerate(entries):
+                n = min(room, len(toks) - done[i])
+                if n <= 0:
+                    continue
+                base = self.max_tokens - room
+                for j, p in enumerate(want[i]):
+                    if done[i] <= p < done[i] + n:
+                        rows.append(base + p - done[i])
+                        dst.append(offs[i] + j)
+                parts.append((sid, toks[done[i]:done[i] + n]))
+                done[i] += n
+                room -= n
+            pending = self._run_mixed(parts)
+            if rows:
+                h = self._settle(sum(len(t) for _, t in parts), pending)
+                for k in range(0, len(rows), self.max_rows):
+                    idx = torch.tensor(rows[k:k + self.max_rows], dtype=torch.long, device=self.device)
+                    lg = self._head_rows(Rows(h[idx], self.E), len(idx), torch.empty(len(idx), self.cfg.vocab_size, dtype=torch.float32, device=self.device))
+                    out[torch.tensor(dst[k:k + self.max_rows], dtype=torch.long, device=self.device)] = lg
+        return out
+
+    def _reserve(self, grow):
+        """Refuse a batch that the pool cannot hold before anything of it is appended."""
+        need = 0
+        for sid, n in grow:
+            seq = self.seqs[sid]
+            if seq.length + n > self.n_ctx:
+                raise RuntimeError(f"sequence {sid}: context {seq.length + n} exceeds n_ctx")
+            need += max(0, (seq.length + n + self.page_size - 1) // self.page_size - len(seq.pages))
+        if need > len(self.kv.free):
+            raise RuntimeError("KV cache exhausted (no free pages)")
+
+    @torch.no_grad()
+    def prefill(self, sid: int, tokens, hidden_in=None, chunk: int | None = None, all_logits: bool = False):
+        """Append `tokens` to one sequence; logits [vocab] of the last token, or [T, vocab] of all of them."""
+        toks = [int(t) for t in torch.as_tensor(tokens).tolist()]
+        chunk = min(chunk or len(toks), len(toks))
+        outs = []
+        for c0 in range(0, len(toks), chunk):
+            part = toks[c0:c0 + chunk]
+            outs.append(self.step([(sid, part)], [list(range(len(part))) if all_logits else [len(part) - 1]]))
+        return torch.cat(outs) if all_logits else outs[-1][-1]
+
+    @torch.no_grad()
+    def embed(self, tokens, pooling: str = "mean", normalize: bool = True) -> torch.Tensor:
+        """Pooled final-norm hidden states of `tokens` (`mean` | `last` | `cls` | `none`), in a scratch sequence slot."""
+        if pooling not in ("mean", "last", "cls", "none"):
+            raise ValueError(f"unknown pooling {pooling!r}")
+        tokens = list(tokens)
+        if len(tokens) > self.max_tokens:
+            raise ValueError(f"{len(tokens)} tokens exceed the batch limit {self.max_tokens}")
+        sid = self.alloc_seq()
+        try:
+            h = self._settle(len(tokens), self._run_mixed([(sid, tokens)]))
+            st = lops.row_stage(h, self.E, self.E, self.cfg.rms_eps, w2=self.w.out_norm, groups2=self.cfg.norm_groups)
+            xn = lops.stage_rows(st, self.buf("xb", len(tokens), self.E), len(tokens)).float()
+        finally:
+            self.free_seq(sid)
+        e = {"mean": lambda: xn.mean(0), "last": lambda: xn[-1], "cls": lambda: xn[0], "none": lambda: xn}[pooling]()
+        return torch.nn.functional.normalize(e, dim=-1) if normalize else e.clone()
+
+    def _choose_variant(self, B: int, max_len: int):
+        if self._latent_heads:
+            H = self._latent_heads[-1]
+            bm = lops.latent_tile_rows(H, B)
+            self._variant = self._n_splits(B * ((H + bm - 1) // bm), max_len)
+
+    def _decode_body(self, B: int, sample: bool):
+        ops.advance(self.seq_len_dev, self.active, self.pos, self.slot, self.kv_len, self.kv.block_table, self.page_size, B)
+        pending = self._forward(self.next_tok, self._decode_batch(B))
+        lg = self._head_rows(self._residual(B, pending), B, self.logits[:B])
+        self.logits_full = lg
+        if sample:
+            ops.sample_dev(lg, self.samp, self.active[:B], self.next_tok[:B])
+
+    def set_control_vector(self, src, scale: float = 1.0, layer_range: tuple[int, int] | None = None):
+        """{layer: vector [width]} added to the residual stream behind that layer; None clears."""
+        self.cvec = {}
+        self._graphs.clear()
+        lo, hi = layer_range or (0, self.cfg.n_layer)
+        for il, v in (src or {}).items():
+            if lo <= il < hi:
+                if v.numel() != self.E:
+                    raise ValueError(f"control vector for layer {il} has {v.numel()} elements, the model is {self.E} wide")
+                self.cvec[il] = (v.float() * scale).to(self.device)
+
+    def memory_breakdown(self) -> dict:
+        act = sum(t.numel() * t.element_size() for t in [*self.hb, self.y, self.logits, *self._flat.values(), *(self.latent_ws or ())])
+        return {"model": self.w.nbytes(), "kv_cache": self.kv.bytes(), "recurrent_state": self.rstate.bytes(), "compute": act, "graphs": len(self._graphs),
+                "device": str(self.device)}

@@ -106,7 +106,7 @@ class LlamaEngine(EngineCore):
     def _onepass_now(self) -> bool:
         return bool(self._variant)
 
-    def _choose_variant(self, max_len: int):
+    def _choose_variant(self, B: int, max_len: int):
         self._variant = self.attn_onepass and max_len >= self.attn_onepass_min
 
     def _companion_variants(self) -> list:

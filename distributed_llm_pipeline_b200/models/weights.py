@@ -150,9 +150,20 @@ class LoadCancelled(RuntimeError):
 
 def load_weights(src: str | GGUFModelFiles, device, layer_range: range | None = None, tp_rank: int = 0, tp_size: int = 1,
                  first_stage: bool = True, last_stage: bool = True, shard_vocab: bool = True,
-                 lora: list[LoraAdapter] | None = None, progress=None) -> ModelWeights:
-    """`progress(fraction) -> bool` is called before every layer and once at the end (1.0); returning False abandons the load with
+                 lora: list[LoraAdapter] | None = None, progress=None, dtype: str | None = None) -> ModelWeights:
+    """`src`: a GGUF file (or the opened one), or a model folder (models/modeldir.py); `dtype` is the storage type of a folder's
+    weights (bf16 | f32; GGUF tensors keep the type of the file).
+    `progress(fraction) -> bool` is called before every layer and once at the end (1.0); returning False abandons the load with
     `LoadCancelled` (`llama_model_params.progress_callback`, the reference's test-model-load-cancel.cpp)."""
+    from .modeldir import ModelDir, is_model_dir, open_model_dir
+    if is_model_dir(src) or isinstance(src, ModelDir):
+        d = open_model_dir(src) if not isinstance(src, ModelDir) else src
+        if tp_size != 1 or lora or (layer_range is not None and layer_range != range(d.cfg.n_layer)) or not (first_stage and last_stage):
+            raise NotImplementedError(f"{d.cfg.arch}: layer-list models load whole, on one GPU and without adapters")
+        from .layered import load_layered_weights
+        return load_layered_weights(d, device, dtype or "bf16", progress)
+    if dtype is not None:
+        raise ValueError("a storage type can be chosen for model folders only: GGUF tensors keep the type of the file")
     f = open_gguf(src) if isinstance(src, str) else src
     lora = lora or []
     cfg = config_from_gguf(f.metadata, f.tensors)

@@ -35,6 +35,10 @@ class LatentArgs(C.Structure):
                 ("bm", C.c_int32), ("n_splits", C.c_int32), ("scale", C.c_float)]
 
 
+def load_library():
+    _lib.load_layers()
+
+
 def _need_cuda(t: torch.Tensor, what: str):
     if not t.is_cuda:
         raise RuntimeError(f"{what}: layer-list models run on a CUDA device only")
