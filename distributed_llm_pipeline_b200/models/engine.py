@@ -254,6 +254,22 @@ class EngineCore:
         d.length = n
         self.seq_len_dev[dst] = n
 
+    @property
+    def can_rollback(self) -> bool:
+        """Cached tokens can be dropped from the end (rejected drafts): not with a recurrent state."""
+        return not self.rstate
+
+    def pages_needed(self, sid: int, n: int) -> int:
+        """Free pages that `n` more tokens of a sequence would take."""
+        seq = self.seqs[sid]
+        return max(0, (seq.length + n + self.page_size - 1) // self.page_size - len(seq.pages))
+
+    def sample_rows(self, logits: torch.Tensor, sids: list[int]) -> list[int]:
+        """Draw one token per row with the device sampler's record of each row's sequence (the same stream as the decode steps)."""
+        self._sync_sampling(sids)
+        rows = torch.tensor(sids, dtype=torch.int32, device=self.device)
+        return ops.sample_dev(logits.contiguous(), self.samp, rows, torch.empty(len(sids), dtype=torch.int32, device=self.device)).tolist()
+
     def _advance_inputs(self, sid: int, T: int):
         """Grow the sequence's pages for T more tokens; positions and cache slots of those tokens (host int32)."""
         seq = self.seqs[sid]

@@ -320,7 +320,7 @@ class LayeredEngine(EngineCore):
             seq = self.seqs[sid]
             if seq.length + n > self.n_ctx:
                 raise RuntimeError(f"sequence {sid}: context {seq.length + n} exceeds n_ctx")
-            need += max(0, (seq.length + n + self.page_size - 1) // self.page_size - len(seq.pages))
+            need += self.pages_needed(sid, n)
         if need > len(self.kv.free):
             raise RuntimeError("KV cache exhausted (no free pages)")
 

@@ -1008,6 +1008,7 @@ def add_parallel_args(ap):
     ap.add_argument("--workers", type=int, default=0, help="launch this many local dlp-worker stages and use them (implies --rpc)")
     ap.add_argument("--worker-base-port", type=int, default=50052)
     ap.add_argument("--no-warmup", action="store_true", help="skip the start-up warm-up (kernel set-up + decode-graph capture per batch size)")
+    ap.add_argument("--dtype", default=os.environ.get("DLP_ARG_DTYPE"), choices=["bf16", "f32"], help="storage type of a model folder's weights and cache")
     ap.add_argument("--mlock", action="store_true", help="pin the model file's pages in RAM")
     ap.add_argument("--no-mmap", action="store_true", help="read the model file into memory instead of mapping it")
     ap.add_argument("--direct-io", action="store_true", help="read the model file with O_DIRECT (implies --no-mmap)")
@@ -1018,8 +1019,8 @@ def add_parallel_args(ap):
 
 def build_service(model: str, device: str = "cuda", n_ctx: int = 2048, n_slots: int = 4, n_batch: int = 2048, page_size: int = 64,
                   lora=None, pp: int = 1, tp: int = 1, tp_impl: str = "fused", tensor_split=None, rpc: str | None = None,
-                  workers: int = 0, worker_base_port: int = 50052, model_draft: str | None = None, draft_max: int = 16):
-    """Load a GGUF checkpoint and return (scheduler, model_info, startup_logs).
+                  workers: int = 0, worker_base_port: int = 50052, model_draft: str | None = None, draft_max: int = 16, dtype: str | None = None):
+    """Load a GGUF checkpoint or a model folder and return (scheduler, model_info, startup_logs).
 
     model_draft: a second, smaller checkpoint with the same vocabulary, loaded on the front-end process's device; greedy requests
     are then decoded by draft-and-verify blocks (`llama-server -md`, tools/server/server-context.cpp:2029-2068).
@@ -1031,13 +1032,16 @@ def build_service(model: str, device: str = "cuda", n_ctx: int = 2048, n_slots: 
 
     from ..gguf import open_gguf
     from ..models.llama import LlamaEngine
+    from ..models.modeldir import ModelDir, make_engine, open_model
     from ..models.weights import load_weights
-    from ..utils.tokenizer import Tokenizer
+    from ..utils.tokenizer import Tokenizer, tokenizer_for
     dev = device if (device != "cuda" or torch.cuda.is_available()) else "cpu"
-    f = open_gguf(model)
-    tok = Tokenizer(f.metadata)
+    f = open_model(model)
+    tok = tokenizer_for(f)
     t0 = time.time()
     info_extra = {}
+    if isinstance(f, ModelDir) and (workers or rpc or pp * tp > 1 or model_draft):
+        raise NotImplementedError(f"{f.cfg.arch}: a model folder is served by one GPU process (no workers, pipeline or tensor split, draft model)")
     if workers or rpc:
         from ..parallel.rpc import LocalWorkerPool, RpcEngine
         pool = None
@@ -1078,8 +1082,8 @@ def build_service(model: str, device: str = "cuda", n_ctx: int = 2048, n_slots: 
         logs.append(f"kv cache: {eng_local.kv.n_pages} pages x {eng_local.page_size} tokens per rank ({eng_local.kv.bytes() / 2**20:.1f} MiB), {n_slots} slots, n_ctx {n_ctx}\n")
         info_extra = {"pp": pp, "tp": tp}
     else:
-        w = load_weights(f, dev, lora=lora)
-        eng = LlamaEngine(w, n_ctx=n_ctx, max_seqs=n_slots + 1, page_size=page_size if dev != "cpu" else 16, max_batch_tokens=n_batch)
+        w = load_weights(f, dev, lora=lora, dtype=dtype)
+        eng = make_engine(w, n_ctx=n_ctx, max_seqs=n_slots + 1, page_size=page_size if dev != "cpu" else 16, max_batch_tokens=n_batch)
         cfg = w.cfg
         logs = [
             f"load: {os.path.basename(model)} | arch {cfg.arch} | {cfg.n_layer} layers | n_embd {cfg.n_embd} | vocab {cfg.vocab_size}\n",
@@ -1111,7 +1115,8 @@ def service_kwargs(a) -> dict:
     from ..utils.args import apply_loader_flags
     apply_loader_flags(a)
     return dict(pp=a.pp, tp=a.tp, tp_impl=a.tp_impl, tensor_split=a.tensor_split, rpc=a.rpc, workers=a.workers,
-                worker_base_port=a.worker_base_port, model_draft=getattr(a, "model_draft", None), draft_max=getattr(a, "draft_max", 16))
+                worker_base_port=a.worker_base_port, model_draft=getattr(a, "model_draft", None), draft_max=getattr(a, "draft_max", 16),
+                dtype=getattr(a, "dtype", None))
 
 
 def maybe_reexec(a, module: str, argv):

@@ -237,6 +237,8 @@ class Scheduler:
             slot.sid = eng.alloc_seq()
         keep = self._lcp(slot.cache_tokens, req.prompt_ids) if req.cache_prompt else 0
         keep = min(keep, len(req.prompt_ids) - 1)  # always evaluate at least the last prompt token
+        if hasattr(eng, "reusable"):               # a recurrent state keeps its whole prefix or nothing
+            keep = eng.reusable(slot.sid, keep)
         eng.truncate_seq(slot.sid, keep)
         slot.cache_tokens = slot.cache_tokens[:keep]
         slot.n_past = keep
@@ -284,6 +286,9 @@ class Scheduler:
         self.metrics.g["kv_pages_free"] = len(self.eng.kv.free)
         if not active:
             return False
+        if getattr(self.eng, "mixed_batches", False) and any(s.state == SlotState.PROMPT for s in active):
+            self._mixed_step(active)
+            return True
         # 1) prompt chunks, sharing the n_batch budget
         budget = self.n_batch
         for s in active:
@@ -358,6 +363,64 @@ class Scheduler:
                     self._accept(s, int(t))
         return True
 
+    def _mixed_step(self, active: list[Slot]):
+        """One forward for everything: a token of every generating slot beside prompt portions, sharing the n_batch budget."""
+        eng = self.eng
+        entries, want, free, budget = [], [], len(eng.kv.free), self.n_batch
+        for s in sorted(active, key=lambda s: s.state != SlotState.GENERATING):      # decoded tokens first: they always run
+            if s.req.cancelled:
+                self._finish(s, "cancelled")
+                continue
+            part = [s.next_token] if s.state == SlotState.GENERATING else s.req.prompt_ids[s.n_past:s.n_past + max(0, budget)]
+            if not part:
+                continue
+            need = eng.pages_needed(s.sid, len(part))
+            if need > free:
+                self._fail(s, "KV cache exhausted (no free pages)")
+                free = len(eng.kv.free) - sum(eng.pages_needed(e.sid, len(p)) for e, p in entries)
+                continue
+            free -= need
+            budget -= len(part)
+            entries.append((s, part))
+            last = s.state == SlotState.GENERATING or s.n_past + len(part) == len(s.req.prompt_ids)
+            want.append([len(part) - 1] if last else [])
+        if not entries:
+            return
+        t0 = time.time()
+        try:
+            logits = eng.step([(s.sid, part) for s, part in entries], want)
+        except RuntimeError as e:
+            for s, _ in entries:
+                self._fail(s, str(e))
+            return
+        rows = [s for (s, _), w in zip(entries, want) if w]
+        # the first token of a request comes from the host sampler, later ones from where a plain decode step would draw them
+        dev = [i for i, s in enumerate(rows) if s.state == SlotState.GENERATING and self._device_samplable(s)]
+        host = [i for i in range(len(rows)) if i not in dev]
+        new: dict[int, int] = {}
+        if dev:
+            for i in dev:
+                rows[i].sampler.accept(rows[i].next_token)
+            new.update(zip(dev, eng.sample_rows(logits[dev], [rows[i].sid for i in dev])))
+        if host:
+            new.update(zip(host, self._sample_rows(logits[host], [rows[i] for i in host])))
+        dt = time.time() - t0
+        n_gen = sum(s.state == SlotState.GENERATING for s, _ in entries)
+        self.metrics.add(n_decode_total=1, n_busy_slots_total=len(entries), tokens_predicted_total=n_gen, tokens_predicted_seconds_total=dt if n_gen else 0.0)
+        for s, part in entries:
+            s.cache_tokens.extend(part)
+            s.n_past += len(part)
+            self.metrics.c["n_tokens_max"] = max(self.metrics.c["n_tokens_max"], s.n_past)
+            if s.state == SlotState.PROMPT:
+                s.req.n_prompt_processed += len(part)
+                self.metrics.add(prompt_tokens_total=len(part))
+        for i, s in enumerate(rows):
+            if s.state == SlotState.PROMPT:
+                self.metrics.add(prompt_seconds_total=time.time() - s.req.t_start, tokens_predicted_total=1)
+                s.req.t_first_token = time.time()
+                s.state = SlotState.GENERATING
+            self._accept(s, int(new[i]))
+
     def _speculate(self, s: Slot) -> bool:
         """Draft-and-verify step for one slot (`server-context.cpp` speculative path with the n-gram "lookup" drafter of
         `common/ngram-cache.cpp`): the pending token plus up to n_draft drafted tokens go through ONE forward that returns logits
@@ -365,7 +428,8 @@ class Scheduler:
         normal batched decode step instead (no draft found, sampling is not greedy, engine cannot return all logits)."""
         req = s.req
         n_draft = req.n_draft if req.n_draft > 0 else (self.n_draft_default if req.n_draft == 0 else 0)     # n_draft < 0: off for this request
-        if n_draft <= 0 or req.n_probs > 0 or not req.sampling.greedy or req.sampling.host_only or not hasattr(self.eng, "copy_seq"):
+        if n_draft <= 0 or req.n_probs > 0 or not req.sampling.greedy or req.sampling.host_only or not hasattr(self.eng, "copy_seq") \
+                or not getattr(self.eng, "can_rollback", True):
             return False
         from .speculative import ModelDrafter, NgramDrafter
         history = s.cache_tokens + [s.next_token]
@@ -475,7 +539,7 @@ class Scheduler:
             req.stop_type = "limit"
             self._finish(s, "length")
         elif s.n_past + 1 >= self.eng.n_ctx:
-            if self.context_shift and hasattr(self.eng, "shift_seq"):
+            if self.context_shift and hasattr(self.eng, "shift_seq") and getattr(self.eng, "can_shift", True):
                 # keep the first n_keep tokens, drop half of the rest (server-context.cpp:1944-2003)
                 n_keep = (req.n_keep if req.n_keep >= 0 else len(req.prompt_ids)) + (1 if self.tok.add_bos else 0)     # n_keep does not count BOS
                 n_keep = min(n_keep, self.eng.n_ctx - 4)

@@ -101,6 +101,8 @@ def generate_speculative(engine, prompt: list[int], n_predict: int, drafter=None
     decoding of `engine` up to floating-point ties between the GEMM and mat-vec paths)."""
     drafter = drafter or NgramDrafter()
     stats = stats if stats is not None else SpecStats()
+    if not getattr(engine, "can_rollback", True):
+        raise NotImplementedError("draft-and-verify needs a cache that can drop rejected tokens; this model keeps a recurrent state")
     sid = engine.alloc_seq()
     drafter.start(prompt)
     try:

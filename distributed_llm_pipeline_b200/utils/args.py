@@ -25,7 +25,8 @@ class Opt:
 
 
 COMMON = [
-    Opt(("-m", "--model"), "GGUF checkpoint (first shard of a split set)", env="DLP_ARG_MODEL"),
+    Opt(("-m", "--model"), "GGUF checkpoint (first shard of a split set), or a model folder (config.json + model.safetensors)", env="DLP_ARG_MODEL"),
+    Opt(("--dtype",), "storage type of a model folder's weights and cache: bf16 | f32", None, str, "DLP_ARG_DTYPE", choices=("bf16", "f32")),
     Opt(("-c", "--ctx-size"), "context length per sequence", 2048, int, "DLP_ARG_CTX_SIZE"),
     Opt(("-b", "--batch-size"), "max tokens per scheduling step (logical batch)", 2048, int, "DLP_ARG_BATCH"),
     Opt(("-ub", "--ubatch-size"), "prefill chunk size (physical batch)", 512, int, "DLP_ARG_UBATCH"),

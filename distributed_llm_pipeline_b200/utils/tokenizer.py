@@ -153,6 +153,9 @@ class Tokenizer:
     @classmethod
     def from_gguf(cls, src):
         from ..gguf import open_gguf
+        from ..models.modeldir import is_model_dir, open_model_dir
+        if is_model_dir(src):
+            return tokenizer_for(open_model_dir(src))
         f = open_gguf(src) if isinstance(src, str) else src
         return cls(f.metadata)
 
@@ -326,6 +329,34 @@ class Tokenizer:
         if self.model in ("llama", "bert", "t5") and strip_leading_space and self.add_space_prefix and s.startswith(" "):
             s = s[1:]
         return s
+
+
+class IdTokenizer(Tokenizer):
+    """Vocabulary of a model folder without a tokenizer: text is token numbers separated by white space or commas, both ways."""
+
+    def __init__(self, n_vocab: int):
+        super().__init__({"tokenizer.ggml.model": "ids", "tokenizer.ggml.tokens": [f"{i} " for i in range(n_vocab)], "tokenizer.ggml.add_bos_token": False})
+        self.bos_id = self.eos_id = -1
+        self.stop_ids = set()
+
+    def encode(self, text: str, add_bos: bool | None = None, parse_special: bool = True) -> list[int]:
+        ids = []
+        for piece in re.split(r"[\s,]+", text.strip()):
+            if not piece:
+                continue
+            if not piece.isdecimal() or int(piece) >= self.n_vocab:
+                raise ValueError(f"{piece!r} is not a token number below {self.n_vocab}")
+            ids.append(int(piece))
+        return ids or [0]
+
+    def token_bytes(self, tid: int) -> bytes:
+        return self.tokens[tid].encode() if 0 <= tid < self.n_vocab else b""
+
+
+def tokenizer_for(model) -> Tokenizer:
+    """Tokenizer of an opened model: the GGUF vocabulary, or token numbers for a model folder (which carries none)."""
+    cfg = getattr(model, "cfg", None)
+    return IdTokenizer(cfg.vocab_size) if cfg is not None and cfg.layers else Tokenizer(model.metadata)
 
 
 class StreamDecoder:

@@ -54,12 +54,15 @@ def main(argv=None):
             log.info(line)
         tok = Tokenizer.from_gguf(a.model)
     else:
-        from distributed_llm_pipeline_b200.gguf import open_gguf
         from distributed_llm_pipeline_b200.models.llama import LlamaEngine
+        from distributed_llm_pipeline_b200.models.modeldir import ModelDir, make_engine, open_model
         from distributed_llm_pipeline_b200.models.weights import load_weights
+        from distributed_llm_pipeline_b200.utils.tokenizer import tokenizer_for
         dev = a.device if (a.device != "cuda" or torch.cuda.is_available()) else "cpu"
-        f = open_gguf(a.model)
-        if a.fit and dev != "cpu":
+        f = open_model(a.model)
+        if isinstance(f, ModelDir) and (a.model_draft or a.lookup):
+            sys.exit(f"dlp-cli: {f.cfg.arch} keeps a recurrent state that cannot drop rejected drafts: no -md / --lookup")
+        if a.fit and dev != "cpu" and not isinstance(f, ModelDir):
             from distributed_llm_pipeline_b200.models.config import config_from_gguf
             from distributed_llm_pipeline_b200.utils.fit import fit_params
             fr = fit_params(f, config_from_gguf(f.metadata, f.tensors), a.ctx_size, a.parallel, torch.cuda.mem_get_info()[0])
@@ -67,10 +70,10 @@ def main(argv=None):
             if not fr.fits:
                 sys.exit(f"dlp-cli: {fr.note}")
             a.ctx_size, a.parallel = fr.n_ctx, fr.n_slots
-        w = load_weights(f, dev, lora=lora_from_args(a))
-        eng = LlamaEngine(w, n_ctx=a.ctx_size, max_seqs=a.parallel, page_size=64 if dev != "cpu" else 16,
+        w = load_weights(f, dev, lora=lora_from_args(a), dtype=a.dtype)
+        eng = make_engine(w, n_ctx=a.ctx_size, max_seqs=a.parallel, page_size=64 if dev != "cpu" else 16,
                           max_batch_tokens=min(a.batch_size, a.ubatch_size))
-        tok = Tokenizer(f.metadata)
+        tok = tokenizer_for(f)
         log.info(f"load_tensors: offloaded {w.cfg.n_layer + 1}/{w.cfg.n_layer + 1} layers to GPU ({dev}), {w.nbytes() / 2**20:.1f} MiB")
     log.info(f"model loaded in {time.time() - t0:.2f} s | n_ctx {a.ctx_size} | slots {a.parallel}")
     prompt = open(a.file).read() if a.file else a.prompt
@@ -83,7 +86,7 @@ def main(argv=None):
         a.single_turn, chat_mode = True, False
     messages: list[dict] = [{"role": "system", "content": system}] if system else []
     if chat_mode:       # the conversation goes through the model's chat template (llama-cli's conversation mode)
-        from distributed_llm_pipeline_b200.gguf import open_gguf as _open
+        from distributed_llm_pipeline_b200.models.modeldir import open_model as _open
         from distributed_llm_pipeline_b200.serving.orchestrator import apply_chat_template
         md = _open(a.model).metadata
         chat_meta = {"tokenizer.chat_template": md.get("tokenizer.chat_template", ""), "bos_token": "", "eos_token": ""}
