@@ -356,7 +356,17 @@ def main():
     ap.add_argument("--emulate-tp", type=int, default=0, help="1 GPU only: time rank 0 of an N-way tensor-parallel step (profiling aid)")
     ap.add_argument("--no-tp-check", action="store_true", help="skip the fused-vs-NCCL greedy token comparison")
     ap.add_argument("--tp-impl", default=os.environ.get("DLP_TP_IMPL", "fused"), choices=["fused", "nccl"])
+    ap.add_argument("--layers", nargs="?", const="2048,4096", default=None, metavar="SIZES",
+                    help="instead of the headline workload: layer-list models beside a Llama of equal size, and each kernel against its roofline (tools/layers_bench.py)")
     args = ap.parse_args()
+    if args.layers:
+        sys.path.insert(0, os.path.join(REPO, "tools"))
+        import layers_bench
+        clocks = ClockSampler(0)
+        clocks.start()
+        res = layers_bench.main(["--sizes", args.layers])
+        print(json.dumps({**res, "clocks": clocks.stop()}), flush=True)
+        return
     args.warmup = max(args.warmup, 3)
     res = run_reference(args) if args.impl == "reference" else run_ours(args)
     if res:

@@ -7,7 +7,7 @@
 
 using namespace dlp;
 
-static_assert(sizeof(dlp_row_stage) == sizeof(RowStage) && sizeof(dlp_hgrn2_args) == sizeof(Hgrn2Args) && sizeof(dlp_latent_args) == sizeof(LatentArgs), "argument layout");
+static_assert(sizeof(dlp_row_stage) == sizeof(RowStage) && sizeof(dlp_hgrn2_args) == sizeof(Hgrn2Args) && sizeof(dlp_hgrn2_chunks) == sizeof(Hgrn2Chunks) && sizeof(dlp_latent_args) == sizeof(LatentArgs), "argument layout");
 
 extern "C" {
 
@@ -37,8 +37,9 @@ int dlp_layers_embed(const void* table, int ld, const int32_t* ids, float* h, in
 int dlp_layers_latent_write(const float* proj, int ldp, const float* w, float eps, int R, int Rc, const int32_t* slot, void* cache, int T, int f32, void* stream) {
     return latent_write(proj, ldp, w, eps, R, Rc, slot, cache, T, f32, (cudaStream_t)stream);
 }
-int dlp_layers_hgrn2(const dlp_hgrn2_args* a, int impl, void* stream) {
-    DLP_REQUIRE(a && impl == 0, "dlp_layers_hgrn2: bad argument");
+int dlp_layers_hgrn2(const dlp_hgrn2_args* a, const dlp_hgrn2_chunks* chunks, void* stream) {
+    DLP_REQUIRE(a, "dlp_layers_hgrn2: null argument");
+    if (chunks) return hgrn2_chunked(*reinterpret_cast<const Hgrn2Args*>(a), *reinterpret_cast<const Hgrn2Chunks*>(chunks), (cudaStream_t)stream);
     return hgrn2_scan(*reinterpret_cast<const Hgrn2Args*>(a), (cudaStream_t)stream);
 }
 int dlp_layers_latent_attention(const dlp_latent_args* a, int f32, void* stream) {

@@ -44,14 +44,37 @@ struct Hgrn2Args {
     const float* fbias;   // [H*D]
     const float* lower;   // [H*D]
     float* state;         // [slots, H, D, V]
-    const int* cu;        // [n_seg + 1] token range of every segment
+    const int* seg;       // [n_seg][2] token range of every segment
     const int* seg_slot;  // [n_seg] state slot
     const int* pos;       // [T] (a segment that starts at position 0 starts from the zero state)
     float* out;           // [T, ldo]
     int ldo, H, D, V, n_seg;
 };
+// Long segments in chunks of HGRN2_CHUNK tokens (layers_hgrn2.cu); `a.seg` / `a.seg_slot` list those segments only.
+constexpr int HGRN2_CHUNK = 64;
+struct Hgrn2Chunks {
+    const int* chunk;     // [n_chunks][2] first token, number of tokens (chunks of a segment follow each other)
+    const int* first;     // [n_seg + 1] first chunk of every segment
+    float* states;        // [n_chunks, H, D, V] workspace: what a chunk adds to the state, then the state a chunk starts from
+    float* decay;         // [n_chunks, H, D] workspace
+    int n_chunks, pad;
+};
 int hgrn2_scan(const Hgrn2Args& a, cudaStream_t s);
-int hgrn2_chunked(const Hgrn2Args& a, cudaStream_t s);
+int hgrn2_chunked(const Hgrn2Args& a, const Hgrn2Chunks& c, cudaStream_t s);
+
+#ifdef __CUDACC__
+// 1 - f = (1 - l) sigmoid(-z) is formed on its own: the difference would lose its digits where f is close to one.
+__device__ __forceinline__ void hgrn2_gate(float z, float l, float& f, float& k) {
+    const float e = expf(-fabsf(z)), hi = 1.f / (1.f + e), lo = e * hi;     // sigmoid(|z|), sigmoid(-|z|)
+    const float sp = z >= 0.f ? hi : lo, sn = z >= 0.f ? lo : hi;
+    f = l + (1.f - l) * sp;
+    k = (1.f - l) * sn;
+}
+__device__ __forceinline__ float silu_exact(float z) {
+    const float e = expf(-fabsf(z)), hi = 1.f / (1.f + e);
+    return z * (z >= 0.f ? hi : e * hi);
+}
+#endif
 
 struct LatentArgs {
     const void* q;            // [T, H, Rc] absorbed queries

@@ -1,0 +1,373 @@
+// HGRN2 over long segments: chunks of 64 tokens in parallel, fp32 gates and state, the products on the tensor cores.
+//
+//   f_t = l + (1 - l) sigmoid(z_t),  k_t = 1 - f_t,  S_t = diag(f_t) S_{t-1} + k_t v_t^T,  o_t = S_t^T q_t
+//
+//   hgrn2_chunk_state   what one chunk adds to the state, U = sum_s (prod_{u > s} f_u * k_s) v_s^T, and its total decay prod f
+//   hgrn2_chunk_scan    S <- decay * S + U over the chunks of a segment; leaves the state every chunk starts from
+//   hgrn2_chunk_out     o_t = (prod_{u <= t} f_u * q_t)^T S_start + sum_{s <= t} (q_t . prod_{s < u <= t} f_u . k_s) v_s
+//
+// A decay between two tokens is always a product of gates that lie between them, never a quotient of cumulative products, so strong
+// forgetting can only underflow to zero.  The 64 x 64 token weights are built from 16 x 16 blocks: below the diagonal the decay splits
+// into a factor up to the end of the key's block, whole blocks, and a factor from the start of the query's block; on the diagonal it is
+// a running product.  fp32 operands enter the tensor cores as two bf16 parts (value and remainder); v is rounded to bf16 once.
+#include "layers.cuh"
+#include "mma.cuh"
+
+namespace dlp {
+
+constexpr int HC = HGRN2_CHUNK;
+
+struct ChunkIn { int t0, n; };
+__device__ __forceinline__ ChunkIn chunk_in(const Hgrn2Chunks& c, int i) { return {c.chunk[2 * i], c.chunk[2 * i + 1]}; }
+
+// gate values of 16 consecutive tokens of one channel (tokens past the chunk's end leave the state alone)
+__device__ __forceinline__ void load_gates(const Hgrn2Args& a, const ChunkIn& c, int h, int d, int r0, float (&f)[16], float (&k)[16]) {
+    const int HD = a.H * a.D;
+    const bool ok = d < a.D;
+    const float b = ok ? a.fbias[h * a.D + d] : 0.f, l = ok ? a.lower[h * a.D + d] : 0.f;
+    float z[16];
+#pragma unroll
+    for (int r = 0; r < 16; ++r) z[r] = (ok && r0 + r < c.n) ? a.proj[(size_t)(c.t0 + r0 + r) * a.ldp + HD + h * a.D + d] : 0.f;
+#pragma unroll
+    for (int r = 0; r < 16; ++r) {
+        f[r] = 1.f;
+        k[r] = 0.f;
+        if (ok && r0 + r < c.n) hgrn2_gate(z[r] + b, l, f[r], k[r]);
+    }
+}
+template <int VP, int NTH>
+__device__ __forceinline__ void load_values(const Hgrn2Args& a, const ChunkIn& c, int h, int v0, __nv_bfloat16* sv) {
+    constexpr int LDV = VP + 8;
+    for (int i = threadIdx.x; i < HC * VP; i += NTH) {
+        const int s = i / VP, v = i - s * VP;
+        const bool ok = s < c.n && v0 + v < a.V;
+        sv[s * LDV + v] = __float2bfloat16_rn(ok ? a.proj[(size_t)(c.t0 + s) * a.ldp + 2 * a.H * a.D + h * a.V + v0 + v] : 0.f);
+    }
+}
+__device__ __forceinline__ void split_one(float x, __nv_bfloat16& hi, __nv_bfloat16& lo) {
+    hi = __float2bfloat16_rn(x);
+    lo = __float2bfloat16_rn(x - __bfloat162float(hi));
+}
+
+template <int DP, int VP>
+__global__ void __launch_bounds__(4 * DP) hgrn2_chunk_state_kernel(const Hgrn2Args a, const Hgrn2Chunks cc) {
+    constexpr int NTH = 4 * DP, LDK = DP + 8, LDV = VP + 8, MT = DP / 16, CG = NTH / 32 / MT, NP = VP / 16 / CG;
+    extern __shared__ __align__(16) uint8_t hc_smem[];
+    __nv_bfloat16* khi = reinterpret_cast<__nv_bfloat16*>(hc_smem);       // [64][LDK]
+    __nv_bfloat16* klo = khi + HC * LDK;
+    __nv_bfloat16* sv = klo + HC * LDK;                                   // [64][LDV]
+    float* sg = reinterpret_cast<float*>(sv + HC * LDV);                  // [4][DP]
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, d = tid % DP, q = tid / DP;
+    const int ch = blockIdx.x, h = blockIdx.y, v0 = blockIdx.z * VP;
+    pdl_wait();
+    const ChunkIn c = chunk_in(cc, ch);
+    float f[16], k[16];
+    load_gates(a, c, h, d, q * 16, f, k);
+    load_values<VP, NTH>(a, c, h, v0, sv);
+    float w = 1.f;
+#pragma unroll
+    for (int r = 15; r >= 0; --r) {      // decay from the token to the end of its block
+        k[r] *= w;
+        w *= f[r];
+    }
+    sg[q * DP + d] = w;
+    __syncthreads();
+    float rest = 1.f;
+    for (int j = q + 1; j < 4; ++j) rest *= sg[j * DP + d];
+#pragma unroll
+    for (int r = 0; r < 16; ++r) split_one(k[r] * rest, khi[(q * 16 + r) * LDK + d], klo[(q * 16 + r) * LDK + d]);
+    if (q == 0 && d < a.D && blockIdx.z == 0) cc.decay[((size_t)ch * a.H + h) * a.D + d] = w * rest;
+    __syncthreads();
+    const int mt = warp % MT, cg = warp / MT;
+    float acc[NP][2][4] = {};
+#pragma unroll
+    for (int ks = 0; ks < HC / 16; ++ks) {
+        uint32_t ah[4], al[4];
+        const int off = (ks * 16 + (lane & 7) + (lane >> 4) * 8) * LDK + mt * 16 + ((lane >> 3) & 1) * 8;
+        ldsm_x4_t(ah, khi + off);
+        ldsm_x4_t(al, klo + off);
+#pragma unroll
+        for (int j = 0; j < NP; ++j) {
+            uint32_t bf[4];
+            ldsm_x4_t(bf, sv + (ks * 16 + (lane & 15)) * LDV + (cg * NP + j) * 16 + (lane >> 4) * 8);
+            mma16816(acc[j][0], ah, bf[0], bf[1]);
+            mma16816(acc[j][1], ah, bf[2], bf[3]);
+            mma16816(acc[j][0], al, bf[0], bf[1]);
+            mma16816(acc[j][1], al, bf[2], bf[3]);
+        }
+    }
+    float* u = cc.states + ((size_t)ch * a.H + h) * a.D * a.V;
+#pragma unroll
+    for (int j = 0; j < NP; ++j)
+#pragma unroll
+        for (int n = 0; n < 2; ++n)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                const int dd = mt * 16 + (lane >> 2) + (e >> 1) * 8, v = v0 + (cg * NP + j) * 16 + n * 8 + (lane & 3) * 2 + (e & 1);
+                if (dd < a.D && v < a.V) u[(size_t)dd * a.V + v] = acc[j][n][e];
+            }
+    pdl_launch_dependents();
+}
+
+__global__ void __launch_bounds__(256) hgrn2_chunk_scan_kernel(const Hgrn2Args a, const Hgrn2Chunks cc) {
+    pdl_wait();
+    const int seg = blockIdx.z, h = blockIdx.y, e = blockIdx.x * 256 + threadIdx.x, n = a.D * a.V;
+    if (e < n) {
+        const int c0 = cc.first[seg], c1 = cc.first[seg + 1], d = e / a.V;
+        float* st = a.state + ((size_t)a.seg_slot[seg] * a.H + h) * n + e;
+        float S = a.pos[a.seg[2 * seg]] == 0 ? 0.f : *st;
+        float* u = cc.states + ((size_t)c0 * a.H + h) * n + e;
+        const float* g = cc.decay + ((size_t)c0 * a.H + h) * a.D + d;
+        const size_t su = (size_t)a.H * n, sg = (size_t)a.H * a.D;
+        constexpr int P = 8;                    // chunks in flight
+        float ub[P], gb[P];
+#pragma unroll
+        for (int i = 0; i < P; ++i)
+            if (c0 + i < c1) { ub[i] = u[i * su]; gb[i] = g[i * sg]; }
+        for (int c = c0; c < c1; c += P) {
+#pragma unroll
+            for (int i = 0; i < P; ++i) {
+                if (c + i >= c1) break;
+                u[i * su] = S;
+                S = fmaf(gb[i], S, ub[i]);
+                if (c + P + i < c1) { ub[i] = u[(P + i) * su]; gb[i] = g[(P + i) * sg]; }
+            }
+            u += P * su;
+            g += P * sg;
+        }
+        *st = S;
+    }
+    pdl_launch_dependents();
+}
+
+template <int DP, int VP>
+struct OutCfg {
+    static constexpr int NTH = 4 * DP, PARTS = NTH / HC, CPP = DP / PARTS;      // diagonal blocks: PARTS threads per key token, CPP channels each
+    static_assert(CPP == 16, "channel groups of the diagonal blocks");
+    static constexpr int LDF = DP;
+    static constexpr int LDK = DP + 8, LDV = VP + 8, LDA = HC + 4;
+    static constexpr int F_BYTES = HC * LDF * 4;
+    static constexpr int QH_BYTES = 2 * HC * LDK * 2;
+    static constexpr int K_BYTES = F_BYTES > QH_BYTES ? F_BYTES : QH_BYTES;     // k rows, later the decayed queries
+    static constexpr int V_BYTES = HC * LDV * 2, A_BYTES = HC * LDA * 4, G_BYTES = 4 * DP * 4;
+    static constexpr int QT_BYTES = 2 * 48 * LDK * 2, KT_BYTES = 2 * 96 * LDK * 2, S_BYTES = 2 * DP * LDV * 2;
+    static constexpr int X_BYTES = QT_BYTES + KT_BYTES > S_BYTES ? QT_BYTES + KT_BYTES : S_BYTES;   // block factors, later the state
+    static constexpr int SMEM = 2 * F_BYTES + K_BYTES + V_BYTES + A_BYTES + G_BYTES + X_BYTES;
+};
+
+// place of channel group `part`, 16-byte piece i inside a row of the diagonal operands: the groups a warp reads together fall into
+// different banks
+__device__ __forceinline__ int diag_piece(int part, int i) { return part * 16 + ((i ^ ((part >> 1) & 3)) << 2); }
+
+template <int DP, int VP>
+__global__ void __launch_bounds__(4 * DP, 1) hgrn2_chunk_out_kernel(const Hgrn2Args a, const Hgrn2Chunks cc) {
+    using C = OutCfg<DP, VP>;
+    constexpr int NTH = C::NTH, LDK = C::LDK, LDV = C::LDV, LDA = C::LDA, LDF = C::LDF, NW = NTH / 32, CG = NW / 4, NP = (VP / 16 + CG - 1) / CG;
+    extern __shared__ __align__(16) uint8_t hc_smem[];
+    float* sq = reinterpret_cast<float*>(hc_smem);
+    float* sf = sq + HC * LDF;
+    float* sk = sf + HC * LDF;
+    uint8_t* p = reinterpret_cast<uint8_t*>(sk) + C::K_BYTES;
+    __nv_bfloat16* sv = reinterpret_cast<__nv_bfloat16*>(p);
+    float* sA = reinterpret_cast<float*>(p + C::V_BYTES);
+    float* sg = reinterpret_cast<float*>(p + C::V_BYTES + C::A_BYTES);
+    uint8_t* x = p + C::V_BYTES + C::A_BYTES + C::G_BYTES;
+    __nv_bfloat16 *qthi = reinterpret_cast<__nv_bfloat16*>(x), *qtlo = qthi + 48 * LDK;
+    __nv_bfloat16 *kthi = qtlo + 48 * LDK, *ktlo = kthi + 96 * LDK;
+    __nv_bfloat16 *shi = reinterpret_cast<__nv_bfloat16*>(x), *slo = shi + DP * LDV;
+    __nv_bfloat16 *qhhi = reinterpret_cast<__nv_bfloat16*>(sk), *qhlo = qhhi + HC * LDK;
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, cq = lane & 3, d = tid % DP, q = tid / DP;
+    const int ch = blockIdx.x, h = blockIdx.y, v0 = blockIdx.z * VP;
+    pdl_wait();
+    const ChunkIn c = chunk_in(cc, ch);
+    float qt[16];               // query times the decay from the start of its block
+    {
+        float f[16], k[16];
+#pragma unroll
+        for (int r = 0; r < 16; ++r) {
+            const int t = q * 16 + r;
+            qt[r] = (d < a.D && t < c.n) ? a.proj[(size_t)(c.t0 + t) * a.ldp + h * a.D + d] : 0.f;
+        }
+        load_gates(a, c, h, d, q * 16, f, k);
+        load_values<VP, NTH>(a, c, h, v0, sv);
+        for (int i = tid; i < HC * LDA; i += NTH) sA[i] = 0.f;
+        const int o = diag_piece(d >> 4, (d & 15) >> 2) + (d & 3);
+        float w = 1.f;
+#pragma unroll
+        for (int r = 0; r < 16; ++r) {
+            const int t = q * 16 + r;
+            qt[r] = silu_exact(qt[r]);
+            sq[t * LDF + o] = qt[r];
+            sf[t * LDF + o] = f[r];
+            sk[t * LDF + o] = k[r];
+            w *= f[r];
+            qt[r] *= w;
+            if (q > 0) split_one(qt[r], qthi[(t - 16) * LDK + d], qtlo[(t - 16) * LDK + d]);
+        }
+        sg[q * DP + d] = w;
+        w = 1.f;
+#pragma unroll
+        for (int r = 15; r >= 0; --r) {     // key times the decay to the end of its block
+            k[r] *= w;
+            w *= f[r];
+        }
+        __syncthreads();
+        const float g1 = sg[DP + d], g2 = sg[2 * DP + d];
+        // key rows by (query block, key block): 0 (1,0)  1 (2,1)  2 (3,2)  3 (2,0)  4 (3,1)  5 (3,0)
+#pragma unroll
+        for (int r = 0; r < 16; ++r) {
+            if (q < 3) split_one(k[r], kthi[(q * 16 + r) * LDK + d], ktlo[(q * 16 + r) * LDK + d]);
+            if (q < 2) split_one(k[r] * (q == 0 ? g1 : g2), kthi[((3 + q) * 16 + r) * LDK + d], ktlo[((3 + q) * 16 + r) * LDK + d]);
+            if (q == 0) split_one(k[r] * g1 * g2, kthi[(80 + r) * LDK + d], ktlo[(80 + r) * LDK + d]);
+        }
+        float pre = 1.f;
+        for (int j = 0; j < q; ++j) pre *= sg[j * DP + d];
+#pragma unroll
+        for (int r = 0; r < 16; ++r) qt[r] *= pre;
+    }
+    {   // diagonal blocks: thread (key token s, channel group) runs over the queries of the block
+        const int s = tid / C::PARTS, part = tid % C::PARTS, b0 = s & ~15;
+        float w[C::CPP];
+#pragma unroll
+        for (int i = 0; i < C::CPP; ++i) w[i] = sk[s * LDF + diag_piece(part, i >> 2) + (i & 3)];
+#pragma unroll 1
+        for (int t = b0; t < b0 + 16; ++t) {
+            float acc = 0.f;
+            const bool later = t > s;
+#pragma unroll
+            for (int i = 0; i < C::CPP / 4; ++i) {
+                const float4 qv = *reinterpret_cast<const float4*>(sq + t * LDF + diag_piece(part, i));
+                const float4 fv = *reinterpret_cast<const float4*>(sf + t * LDF + diag_piece(part, i));
+                w[4 * i] *= later ? fv.x : 1.f;
+                w[4 * i + 1] *= later ? fv.y : 1.f;
+                w[4 * i + 2] *= later ? fv.z : 1.f;
+                w[4 * i + 3] *= later ? fv.w : 1.f;
+                acc = fmaf(qv.x, w[4 * i], acc);
+                acc = fmaf(qv.y, w[4 * i + 1], acc);
+                acc = fmaf(qv.z, w[4 * i + 2], acc);
+                acc = fmaf(qv.w, w[4 * i + 3], acc);
+            }
+#pragma unroll
+            for (int i = 1; i < C::PARTS; i <<= 1) acc += __shfl_xor_sync(0xffffffffu, acc, i);
+            if (part == 0 && t >= s) sA[t * LDA + s] = acc;
+        }
+    }
+    __syncthreads();
+    if (warp < 6) {     // blocks below the diagonal
+        constexpr int QI[6] = {1, 2, 3, 2, 3, 3}, KJ[6] = {0, 1, 2, 0, 1, 0};
+        int qi = 1, kj = 0;
+#pragma unroll
+        for (int i = 0; i < 6; ++i)
+            if (warp == i) { qi = QI[i]; kj = KJ[i]; }
+        float acc[2][4] = {};
+#pragma unroll
+        for (int ks = 0; ks < DP / 16; ++ks) {
+            uint32_t ah[4], al[4], bh[4], bl[4];
+            const int ao = ((qi - 1) * 16 + (lane & 15)) * LDK + ks * 16 + (lane >> 4) * 8;
+            const int bo = (warp * 16 + (lane & 7) + (lane >> 4) * 8) * LDK + ks * 16 + ((lane >> 3) & 1) * 8;
+            ldsm_x4(ah, qthi + ao);
+            ldsm_x4(al, qtlo + ao);
+            ldsm_x4(bh, kthi + bo);
+            ldsm_x4(bl, ktlo + bo);
+#pragma unroll
+            for (int n = 0; n < 2; ++n) {
+                mma16816(acc[n], ah, bh[2 * n], bh[2 * n + 1]);
+                mma16816(acc[n], ah, bl[2 * n], bl[2 * n + 1]);
+                mma16816(acc[n], al, bh[2 * n], bh[2 * n + 1]);
+            }
+        }
+#pragma unroll
+        for (int n = 0; n < 2; ++n)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) sA[(qi * 16 + g + (e >> 1) * 8) * LDA + kj * 16 + n * 8 + cq * 2 + (e & 1)] = acc[n][e];
+    }
+    __syncthreads();
+    // the block factors and the key rows are done with: state and decayed queries take their place
+#pragma unroll
+    for (int r = 0; r < 16; ++r) split_one(qt[r], qhhi[(q * 16 + r) * LDK + d], qhlo[(q * 16 + r) * LDK + d]);
+    {
+        const float* S = cc.states + ((size_t)ch * a.H + h) * a.D * a.V;
+#pragma unroll 8
+        for (int i = tid; i < DP * VP; i += NTH) {
+            const int dd = i / VP, v = i - dd * VP;
+            split_one((dd < a.D && v0 + v < a.V) ? S[(size_t)dd * a.V + v0 + v] : 0.f, shi[dd * LDV + v], slo[dd * LDV + v]);
+        }
+    }
+    __syncthreads();
+    const int mt = warp & 3, cg = warp >> 2;
+    float acc[NP][2][4] = {};
+#pragma unroll 2
+    for (int ks = 0; ks < DP / 16; ++ks) {
+        uint32_t ah[4], al[4];
+        const int ao = (mt * 16 + (lane & 15)) * LDK + ks * 16 + (lane >> 4) * 8;
+        ldsm_x4(ah, qhhi + ao);
+        ldsm_x4(al, qhlo + ao);
+#pragma unroll
+        for (int j = 0; j < NP; ++j) {
+            const int col = (cg * NP + j) * 16;
+            uint32_t bh[4], bl[4];
+            ldsm_x4_t(bh, shi + (ks * 16 + (lane & 15)) * LDV + col + (lane >> 4) * 8);
+            ldsm_x4_t(bl, slo + (ks * 16 + (lane & 15)) * LDV + col + (lane >> 4) * 8);
+#pragma unroll
+            for (int n = 0; n < 2; ++n) {
+                mma16816(acc[j][n], ah, bh[2 * n], bh[2 * n + 1]);
+                mma16816(acc[j][n], ah, bl[2 * n], bl[2 * n + 1]);
+                mma16816(acc[j][n], al, bh[2 * n], bh[2 * n + 1]);
+            }
+        }
+    }
+    for (int ks = 0; ks <= mt; ++ks) {       // tokens of the chunk itself, up to the query's block
+        uint32_t hi[4], lo[4];
+        const float* r0 = sA + (mt * 16 + g) * LDA + ks * 16 + cq * 2;
+        const float* r1 = r0 + 8 * LDA;
+        split_bf16(r0[0], r0[1], hi[0], lo[0]);
+        split_bf16(r1[0], r1[1], hi[1], lo[1]);
+        split_bf16(r0[8], r0[9], hi[2], lo[2]);
+        split_bf16(r1[8], r1[9], hi[3], lo[3]);
+#pragma unroll
+        for (int j = 0; j < NP; ++j) {
+            uint32_t bf[4];
+            ldsm_x4_t(bf, sv + (ks * 16 + (lane & 15)) * LDV + (cg * NP + j) * 16 + (lane >> 4) * 8);
+            mma16816(acc[j][0], hi, bf[0], bf[1]);
+            mma16816(acc[j][1], hi, bf[2], bf[3]);
+            mma16816(acc[j][0], lo, bf[0], bf[1]);
+            mma16816(acc[j][1], lo, bf[2], bf[3]);
+        }
+    }
+#pragma unroll
+    for (int j = 0; j < NP; ++j)
+#pragma unroll
+        for (int n = 0; n < 2; ++n)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                const int t = mt * 16 + g + (e >> 1) * 8, v = v0 + (cg * NP + j) * 16 + n * 8 + cq * 2 + (e & 1);
+                if (t < c.n && v < a.V) a.out[(size_t)(c.t0 + t) * a.ldo + h * a.V + v] = acc[j][n][e];
+            }
+    pdl_launch_dependents();
+}
+
+template <int P>
+static int launch_chunked(const Hgrn2Args& a, const Hgrn2Chunks& c, cudaStream_t s) {
+    constexpr int NTH = 4 * P;
+    constexpr size_t sm1 = (size_t)(2 * HC * (P + 8) + HC * (P + 8)) * 2 + 4 * P * 4;
+    constexpr size_t sm3 = OutCfg<P, P>::SMEM;
+    static_assert(sm3 <= 227 * 1024, "chunk staging");
+    auto k1 = hgrn2_chunk_state_kernel<P, P>;
+    auto k3 = hgrn2_chunk_out_kernel<P, P>;
+    if (first_use_on_device((const void*)k1)) DLP_CHECK_CUDA(cudaFuncSetAttribute(k1, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)sm1));
+    if (first_use_on_device((const void*)k3)) DLP_CHECK_CUDA(cudaFuncSetAttribute(k3, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)sm3));
+    const dim3 grid(c.n_chunks, a.H, (a.V + P - 1) / P);
+    DLP_CHECK_CUDA(launch_pdl(k1, grid, dim3(NTH), sm1, s, a, c));
+    DLP_CHECK_CUDA(launch_pdl(hgrn2_chunk_scan_kernel, dim3((a.D * a.V + 255) / 256, a.H, a.n_seg), dim3(256), 0, s, a, c));
+    DLP_CHECK_CUDA(launch_pdl(k3, grid, dim3(NTH), sm3, s, a, c));
+    return 0;
+}
+
+int hgrn2_chunked(const Hgrn2Args& a, const Hgrn2Chunks& c, cudaStream_t s) {
+    DLP_REQUIRE(a.proj && a.fbias && a.lower && a.state && a.seg && a.seg_slot && a.pos && a.out, "hgrn2_chunked: null argument");
+    DLP_REQUIRE(c.chunk && c.first && c.states && c.decay && c.n_chunks > 0, "hgrn2_chunked: no chunk table");
+    DLP_REQUIRE(a.H > 0 && a.H <= 65535 && a.D > 0 && a.D <= 128 && a.V > 0 && a.n_seg > 0 && a.n_seg <= 65535, "hgrn2_chunked: bad shape (D=%d)", a.D);
+    return a.D <= 64 && a.V <= 64 ? launch_chunked<64>(a, c, s) : launch_chunked<128>(a, c, s);
+}
+
+}  // namespace dlp

@@ -6,6 +6,7 @@
 //   sgemm_kernel         fp32 storage, any number of rows (no reduced-precision product).
 //   head_matmul_kernel   one small matrix per head (latent attention's key absorption and value expansion), mma.sync m16n8k16.
 #include "layers.cuh"
+#include "mma.cuh"
 
 namespace dlp {
 
@@ -333,11 +334,6 @@ int sgemm(const float* x, int ldx, const float* w, int ldw, int N, int K, void* 
 // ---- one matrix per head: out[t, h, n] = sum_k x[t, h, k] W[h][n][k]  (* sigmoid(gate[t, h])) ---------------
 // A is 16 * MT tokens of one head (shared memory), B comes straight from global memory, 16 bytes per lane: the k index inside a
 // 32-wide block is permuted the same way on both operands, so that a lane's eight k values are contiguous.
-__device__ __forceinline__ void mma_bf16(float (&c)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0, uint32_t b1) {
-    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-                 : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
-}
-
 template <int MT>
 __global__ void __launch_bounds__(128) head_matmul_kernel(const void* x, int x_f32, int ldx, int x_head, int kx, const __nv_bfloat16* __restrict__ w, int Kp, int N,
                                                           int n_rows, __nv_bfloat16* out, int ldo, int out_head, const float* gate, int ldg, int T) {
@@ -377,8 +373,8 @@ __global__ void __launch_bounds__(128) head_matmul_kernel(const void* x, int x_f
             const uint4 hi = *reinterpret_cast<const uint4*>(xs + (m * 16 + g + 8) * ldxs + k + c * 8);
 #pragma unroll
             for (int j = 0; j < 2; ++j) {
-                mma_bf16(acc[m][j], lo.x, hi.x, lo.y, hi.y, b[j].x, b[j].y);
-                mma_bf16(acc[m][j], lo.z, hi.z, lo.w, hi.w, b[j].z, b[j].w);
+                mma16816(acc[m][j], {lo.x, hi.x, lo.y, hi.y}, b[j].x, b[j].y);
+                mma16816(acc[m][j], {lo.z, hi.z, lo.w, hi.w}, b[j].z, b[j].w);
             }
         }
     }

@@ -48,17 +48,7 @@ int latent_write(const float* proj, int ldp, const float* w, float eps, int R, i
 
 // ---- HGRN2 -------------------------------------------------------------------------------------------------------
 //   f = l + (1 - l) sigmoid(z),  S <- diag(f) S + (1 - f) v^T,  o = S^T silu(q)
-// 1 - f = (1 - l) sigmoid(-z) is formed on its own: the difference would lose its digits where f is close to one.
-__device__ __forceinline__ void hgrn2_gate(float z, float l, float& f, float& k) {
-    const float e = expf(-fabsf(z)), hi = 1.f / (1.f + e), lo = e * hi;     // sigmoid(|z|), sigmoid(-|z|)
-    const float sp = z >= 0.f ? hi : lo, sn = z >= 0.f ? lo : hi;
-    f = l + (1.f - l) * sp;
-    k = (1.f - l) * sn;
-}
-__device__ __forceinline__ float silu_exact(float z) {
-    const float e = expf(-fabsf(z)), hi = 1.f / (1.f + e);
-    return z * (z >= 0.f ? hi : e * hi);
-}
+// (gate: hgrn2_gate in layers.cuh)
 
 // One CTA = one (segment, head, slice of 128 / RG value columns); a thread keeps RPT state rows of one column.  Tokens are staged
 // CT at a time; a row group's values sit RPT + 4 floats apart so that the RG groups of a warp read different banks.
@@ -74,7 +64,7 @@ __global__ void __launch_bounds__(128) hgrn2_scan_kernel(const Hgrn2Args a) {
     const int seg = blockIdx.z, h = blockIdx.y, v0 = blockIdx.x * COLS;
     const int HD = a.H * a.D;
     pdl_wait();
-    const int lo = a.cu[seg], hi = a.cu[seg + 1];
+    const int lo = a.seg[2 * seg], hi = a.seg[2 * seg + 1];
     if (lo >= hi) return;
     float S[RPT];
     float* st = a.state + (((size_t)a.seg_slot[seg] * a.H + h) * a.D + rg * RPT) * a.V + v0 + col;
@@ -142,7 +132,7 @@ static int launch_scan(const Hgrn2Args& a, cudaStream_t s) {
 }
 
 int hgrn2_scan(const Hgrn2Args& a, cudaStream_t s) {
-    DLP_REQUIRE(a.proj && a.fbias && a.lower && a.state && a.cu && a.seg_slot && a.pos && a.out, "hgrn2_scan: null argument");
+    DLP_REQUIRE(a.proj && a.fbias && a.lower && a.state && a.seg && a.seg_slot && a.pos && a.out, "hgrn2_scan: null argument");
     DLP_REQUIRE(a.H > 0 && a.D > 0 && a.V > 0 && a.n_seg > 0 && a.n_seg <= 65535, "hgrn2_scan: bad shape");
     if (a.D <= 64) return launch_scan<4, 16>(a, s);
     if (a.D <= 128) return launch_scan<4, 32>(a, s);

@@ -86,12 +86,22 @@ class TileTable:
 
 
 @dataclass
+class Segments:
+    """Row ranges of some of a batch's sequences."""
+    n: int
+    range: torch.Tensor         # [n, 2] first row, row behind the last
+    slot: torch.Tensor          # [n] sequence slot
+    chunk: torch.Tensor | None = None      # [chunks, 2] first row and length (long segments)
+    first: torch.Tensor | None = None      # [n + 1] first chunk of every segment
+
+
+@dataclass
 class Batch:
-    """Device-side description of one forward: T rows, grouped into segments (one per sequence)."""
+    """Device-side description of one forward: T rows, grouped into segments (one per sequence).  Recurrent mixers scan the short
+    segments token by token and take the long ones in chunks."""
     T: int
-    n_seg: int
-    cu: torch.Tensor            # [n_seg + 1] row range of every segment
-    seg_slot: torch.Tensor      # [n_seg] sequence slot
+    short: Segments | None
+    long: Segments | None
     tok_slot: torch.Tensor      # [T] sequence slot of every row
     pos: torch.Tensor           # [T]
     slot: torch.Tensor          # [T] cache row
@@ -141,6 +151,13 @@ class LayeredEngine(EngineCore):
         if lat:
             rows = self._split_ctas * 64
             self.latent_ws = (torch.zeros(rows * max(m.Rc for m in lat), dtype=f32, device=dev), torch.zeros(rows * 2, dtype=f32, device=dev))
+        # segments from this length on run the chunked recurrence (bf16 storage; the fp32 form always scans)
+        chunked = [m for m in mixers.values() if m.state is not None and m.chunked]
+        self.chunk_from = 2 * lops.HGRN2_CHUNK if chunked and self.dtype == torch.bfloat16 else 1 << 60
+        self.chunk_ws = None
+        if self.chunk_from < M:
+            n = M // lops.HGRN2_CHUNK + M // self.chunk_from + 1         # every long segment may end in a partial chunk
+            self.chunk_ws = tuple(torch.zeros(n * max(m.H * m.D * w(m) for m in chunked), dtype=f32, device=dev) for w in (lambda m: m.V, lambda m: 1))
         self._variant = 1                                            # key ranges per decode query
         self._decode_batches: dict[tuple, Batch] = {}
 
@@ -232,18 +249,26 @@ class LayeredEngine(EngineCore):
                 bm = lops.latent_tile_rows(H, B)
                 row0, rows = self._tile_lists(H, [1] * B, bm)
                 tiles[H] = TileTable(torch.tensor(row0, dtype=i32, device=dev), torch.tensor(rows, dtype=i32, device=dev), len(row0), bm, min(self._variant, max(1, self._split_ctas // len(row0))))
-            b = Batch(B, B, torch.arange(B + 1, dtype=i32, device=dev), self.active, self.active, self.pos, self.slot, tiles)
+            rng = torch.tensor([[i, i + 1] for i in range(B)], dtype=i32, device=dev)
+            b = Batch(B, Segments(B, rng, self.active), None, self.active, self.pos, self.slot, tiles)
             self._decode_batches[(B, self._variant)] = b
         return b
 
     def _mixed_batch(self, parts: list[tuple[int, list[int]]]) -> tuple[torch.Tensor, Batch]:
         """Grow every sequence by its tokens and upload the description in one copy."""
         lens = [len(t) for _, t in parts]
-        T, n = sum(lens), len(parts)
-        cols: list[torch.Tensor] = [torch.cat([torch.as_tensor(t, dtype=torch.int32) for _, t in parts])]
+        T = sum(lens)
         pos, slot = zip(*(self._advance_inputs(sid, len(t)) for sid, t in parts))
-        cols += [torch.cat(pos), torch.cat(slot), torch.cat([torch.full((len(t),), sid, dtype=torch.int32) for sid, t in parts]),
-                 torch.tensor([0] + torch.tensor(lens).cumsum(0).tolist(), dtype=torch.int32), torch.tensor([sid for sid, _ in parts], dtype=torch.int32)]
+        cols: list[torch.Tensor] = [torch.cat([torch.as_tensor(t, dtype=torch.int32) for _, t in parts]), torch.cat(pos), torch.cat(slot),
+                                    torch.cat([torch.full((len(t),), sid, dtype=torch.int32) for sid, t in parts])]
+        ends = torch.tensor(lens).cumsum(0).tolist()
+        segs = [(sid, hi - n, hi) for (sid, _), n, hi in zip(parts, lens, ends)]
+        groups = [[g for g in segs if (g[2] - g[1] >= self.chunk_from) == is_long] for is_long in (False, True)]
+        for is_long, grp in zip((False, True), groups):
+            lists = [[x for g in grp for x in g[1:]], [g[0] for g in grp]]
+            if is_long:
+                lists += lops.hgrn2_chunk_table([g[1:] for g in grp])
+            cols += [torch.tensor(x, dtype=torch.int32) for x in lists]
         shapes = []
         for H in self._latent_heads:
             bm = lops.latent_tile_rows(H, T)
@@ -251,10 +276,12 @@ class LayeredEngine(EngineCore):
             cols += [torch.tensor(row0, dtype=torch.int32), torch.tensor(rows, dtype=torch.int32)]
             shapes.append((H, bm, len(row0)))
         dev = iter(torch.cat(cols).to(self.device).split([c.numel() for c in cols]))
-        ids, pos_d, slot_d, tok_slot, cu, seg_slot = (next(dev) for _ in range(6))
+        ids, pos_d, slot_d, tok_slot = (next(dev) for _ in range(4))
+        short = Segments(len(groups[0]), next(dev), next(dev))
+        long = Segments(len(groups[1]), next(dev), next(dev), next(dev).view(-1, 2), next(dev))
         longest = max(self.seqs[sid].length + len(t) for sid, t in parts)
         tiles = {H: TileTable(next(dev), next(dev), nt, bm, self._n_splits(nt, longest)) for H, bm, nt in shapes}
-        return ids, Batch(T, n, cu, seg_slot, tok_slot, pos_d, slot_d, tiles)
+        return ids, Batch(T, short if short.n else None, long if long.n else None, tok_slot, pos_d, slot_d, tiles)
 
     def _run_mixed(self, parts: list[tuple[int, list[int]]]):
         """Forward over one mixed batch; updates the sequence lengths.  Returns the pending norm weight (see _forward)."""

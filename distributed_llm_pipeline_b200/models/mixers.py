@@ -71,6 +71,7 @@ class Hgrn2:
         if self.w_in.N != self.H * (2 * self.D + self.V) or self.w_out.K != self.H * self.V:
             raise ValueError("hgrn2: a projection does not fit heads, dim and vdim")
         self.state = (self.H, self.D, self.V)
+        self.chunked = self.D <= 128          # the chunk kernels keep a head's channels in one block
 
     def weights(self):
         return [self.w_in, self.w_out]
@@ -80,7 +81,11 @@ class Hgrn2:
 
     def mix(self, eng, il: int, proj: torch.Tensor, b) -> Rows:
         o = eng.buf("o", b.T, self.H * self.V)
-        lops.hgrn2(proj, self.fbias, self.lower, eng.rstate.layers[il], b.cu, b.seg_slot, b.n_seg, b.pos, o)
+        state = eng.rstate.layers[il]
+        for s in (b.short, b.long):
+            if s is not None:
+                chunks = (s.chunk, s.first, *eng.chunk_ws) if s is b.long and self.chunked else None
+                lops.hgrn2(proj, self.fbias, self.lower, state, s.range, s.slot, s.n, b.pos, o, chunks)
         return Rows(o, self.H * self.V, w2=self.norm, groups2=self.H)
 
 

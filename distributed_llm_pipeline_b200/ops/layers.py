@@ -13,6 +13,7 @@ from . import api
 from . import lib as _lib
 
 OUT_F32, OUT_GEGLU = 0, 1
+HGRN2_CHUNK = 64            # tokens per chunk of the chunked recurrence
 
 
 class RowStage(C.Structure):
@@ -23,9 +24,13 @@ class RowStage(C.Structure):
 
 
 class Hgrn2Args(C.Structure):
-    _fields_ = [("proj", C.c_void_p), ("ldp", C.c_int32), ("fbias", C.c_void_p), ("lower", C.c_void_p), ("state", C.c_void_p), ("cu", C.c_void_p),
+    _fields_ = [("proj", C.c_void_p), ("ldp", C.c_int32), ("fbias", C.c_void_p), ("lower", C.c_void_p), ("state", C.c_void_p), ("seg", C.c_void_p),
                 ("seg_slot", C.c_void_p), ("pos", C.c_void_p), ("out", C.c_void_p), ("ldo", C.c_int32), ("H", C.c_int32), ("D", C.c_int32), ("V", C.c_int32),
                 ("n_seg", C.c_int32)]
+
+
+class Hgrn2Chunks(C.Structure):
+    _fields_ = [("chunk", C.c_void_p), ("first", C.c_void_p), ("states", C.c_void_p), ("decay", C.c_void_p), ("n_chunks", C.c_int32), ("pad", C.c_int32)]
 
 
 class LatentArgs(C.Structure):
@@ -107,14 +112,33 @@ def latent_write(proj: torch.Tensor, w: torch.Tensor, eps: float, R: int, slot: 
     api._count()
 
 
-def hgrn2(proj: torch.Tensor, fbias, lower, state: torch.Tensor, cu, seg_slot, n_seg: int, pos, out: torch.Tensor, impl: int = 0):
-    """Gated linear recurrence of every segment; proj rows are q | f | v before their activations, state [slots, H, D, V]."""
+def hgrn2(proj: torch.Tensor, fbias, lower, state: torch.Tensor, seg, seg_slot, n_seg: int, pos, out: torch.Tensor, chunks=None):
+    """Gated linear recurrence of the listed segments; proj rows are q | f | v before their activations, state [slots, H, D, V], seg
+    [n_seg, 2] token ranges.  chunks = (chunk table [n, 2], first chunk of every segment [n_seg + 1], states workspace, decay workspace):
+    64-token chunks on the tensor cores (at most 128 channels per head) instead of the token scan."""
     _need_cuda(state, "hgrn2")
     _, H, D, V = state.shape
-    a = Hgrn2Args(_p(proj), proj.stride(0), _p(fbias), _p(lower), _p(state), _p(cu), _p(seg_slot), _p(pos), _p(out), out.stride(0), H, D, V, n_seg)
-    _lib.check(_lib.load().dlp_layers_hgrn2(C.byref(a), impl, api._stream()), "layers_hgrn2")
-    api._count()
+    a = Hgrn2Args(_p(proj), proj.stride(0), _p(fbias), _p(lower), _p(state), _p(seg), _p(seg_slot), _p(pos), _p(out), out.stride(0), H, D, V, n_seg)
+    c = None
+    if chunks is not None:
+        table, first, states, decay = chunks
+        n = table.shape[0]
+        if states.numel() < n * H * D * V or decay.numel() < n * H * D:
+            raise ValueError("hgrn2: workspace too small")
+        c = Hgrn2Chunks(_p(table), _p(first), _p(states), _p(decay), n, 0)
+    _lib.check(_lib.load().dlp_layers_hgrn2(C.byref(a), C.byref(c) if c is not None else None, api._stream()), "layers_hgrn2")
+    api._count(3 if c is not None else 1)
     return out
+
+
+def hgrn2_chunk_table(segs: list[tuple[int, int]]) -> tuple[list[int], list[int]]:
+    """(first token, length) of every chunk and the first chunk of every segment, for token ranges `segs`."""
+    table, first = [], [0]
+    for lo, hi in segs:
+        for t in range(lo, hi, HGRN2_CHUNK):
+            table += [t, min(HGRN2_CHUNK, hi - t)]
+        first.append(len(table) // 2)
+    return table, first
 
 
 def latent_tile_rows(H: int, T: int) -> int:

@@ -360,8 +360,9 @@ typedef struct {              /* how a row is formed in front of a matrix produc
 } dlp_row_stage;
 typedef struct {
     const float* proj; int32_t ldp; const float* fbias; const float* lower; float* state;
-    const int32_t* cu; const int32_t* seg_slot; const int32_t* pos; float* out; int32_t ldo, H, D, V, n_seg;
+    const int32_t* seg; const int32_t* seg_slot; const int32_t* pos; float* out; int32_t ldo, H, D, V, n_seg;
 } dlp_hgrn2_args;
+typedef struct { const int32_t* chunk; const int32_t* first; float* states; float* decay; int32_t n_chunks, pad; } dlp_hgrn2_chunks;
 typedef struct {
     const void* q; const void* cache; const int32_t* block_table; const int32_t* tok_slot; const int32_t* pos;
     const int32_t* tile_row0; const int32_t* tile_rows; void* out; float* part_o; float* part_ml;
@@ -376,7 +377,7 @@ int dlp_layers_head_matmul(const void* x, int x_f32, int ldx, int x_head, int kx
                            const float* gate, int ldg, int T, int f32, void* stream);
 int dlp_layers_embed(const void* table, int ld, const int32_t* ids, float* h, int E, int T, int vocab, int f32, void* stream);
 int dlp_layers_latent_write(const float* proj, int ldp, const float* w, float eps, int R, int Rc, const int32_t* slot, void* cache, int T, int f32, void* stream);
-int dlp_layers_hgrn2(const dlp_hgrn2_args* a, int impl, void* stream);   /* impl 0: token scan, 1: chunks on the tensor cores */
+int dlp_layers_hgrn2(const dlp_hgrn2_args* a, const dlp_hgrn2_chunks* chunks, void* stream);   /* chunks NULL: token scan; else 64-token chunks on the tensor cores */
 int dlp_layers_latent_attention(const dlp_latent_args* a, int f32, void* stream);
 
 #ifdef __cplusplus

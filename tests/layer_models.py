@@ -130,10 +130,10 @@ def install_host_ops(monkeypatch):
         rows = cache.view(-1, cache.shape[-1])
         rows[slot[:T].long(), :R] = (plain.rms(proj[:T, :R], eps) * w).to(cache.dtype)
 
-    def scan(proj, fbias, lower, state, cu, seg_slot, n_seg, pos, out, impl=0):
+    def scan(proj, fbias, lower, state, seg, seg_slot, n_seg, pos, out, chunks=None):
         _, H, D, V = state.shape
         for s in range(n_seg):
-            lo, hi, sl = int(cu[s]), int(cu[s + 1]), int(seg_slot[s])
+            (lo, hi), sl = seg.view(-1, 2)[s].tolist(), int(seg_slot[s])
             x = proj[lo:hi]
             q, f, v = x[:, :H * D], x[:, H * D:2 * H * D], x[:, 2 * H * D:]
             st = torch.zeros_like(state[sl]) if int(pos[lo]) == 0 else state[sl]
