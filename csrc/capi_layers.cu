@@ -24,8 +24,8 @@ int dlp_layers_linear(const void* x, int ldx, const void* w, int ldw, int N, int
     if (f32) return sgemm((const float*)x, ldx, (const float*)w, ldw, N, K, out, ldo, out_mode, T, (cudaStream_t)stream);
     if (out_mode == LO_GEGLU)       // rows 2i / 2i+1 of the interleaved matrix: two operands with twice the row stride
         return gemm_f16(w, (const uint8_t*)w + (size_t)ldw * 2, 2 * ldw, x, ldx, out, ldo, T, N / 2, K, 6, 1, 0, (cudaStream_t)stream, nullptr, nullptr, ws, ws_bytes);
-    DLP_REQUIRE(out_mode == LO_F32, "dlp_layers_linear: output mode %d", out_mode);
-    return gemm_f16(w, nullptr, ldw, x, ldx, out, ldo, T, N, K, 1, 1, 0, (cudaStream_t)stream, nullptr, nullptr, ws, ws_bytes);
+    DLP_REQUIRE(out_mode == LO_F32 || out_mode == LO_BF16, "dlp_layers_linear: output mode %d", out_mode);
+    return gemm_f16(w, nullptr, ldw, x, ldx, out, ldo, T, N, K, out_mode == LO_BF16 ? 4 : 1, 1, 0, (cudaStream_t)stream, nullptr, nullptr, ws, ws_bytes);
 }
 int dlp_layers_head_matmul(const void* x, int x_f32, int ldx, int x_head, int kx, const void* w, int Kp, int H, int N, int n_rows, void* out, int ldo, int out_head,
                            const float* gate, int ldg, int T, int f32, void* stream) {
@@ -46,5 +46,17 @@ int dlp_layers_latent_attention(const dlp_latent_args* a, int f32, void* stream)
     DLP_REQUIRE(a, "dlp_layers_latent_attention: null argument");
     return latent_attention(*reinterpret_cast<const LatentArgs*>(a), f32, (cudaStream_t)stream);
 }
+
+int dlp_layers_latent_gather(const void* cache, const int32_t* bt_row, int page, int Rc, void* out, int S, void* stream) {
+    return latent_gather(cache, bt_row, page, Rc, out, S, (cudaStream_t)stream);
+}
+int dlp_layers_head_rows(const float* x, int ldx, int D, int Dp, int H, void* out, int T, void* stream) {
+    return head_rows(x, ldx, D, Dp, H, out, T, (cudaStream_t)stream);
+}
+int dlp_layers_rows_attention(const void* q, const void* kv, int ldkv, int S, int T, int pos0, int H, int Dp, int Vp, int V, float scale, const float* gate, int ldg,
+                              void* out, int ldo, void* stream) {
+    return rows_attention(q, kv, ldkv, S, T, pos0, H, Dp, Vp, V, scale, gate, ldg, out, ldo, (cudaStream_t)stream);
+}
+int dlp_layers_rows_attention_error(int* flag) { return rows_attention_error(flag); }
 
 }  // extern "C"

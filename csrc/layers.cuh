@@ -28,7 +28,7 @@ struct RowStage {
     int Kp;
 };
 
-enum LinOut : int { LO_F32 = 0, LO_GEGLU = 1 };   // GEGLU: weight rows 2i / 2i+1 are gate_i / up_i, the output is gelu_tanh(gate) * up
+enum LinOut : int { LO_F32 = 0, LO_GEGLU = 1, LO_BF16 = 2 };   // GEGLU: weight rows 2i / 2i+1 are gate_i / up_i, the output is gelu_tanh(gate) * up
 
 int matvec(const RowStage& st, const void* w, int ldw, int N, void* out, int ldo, int out_mode, int T, int f32, cudaStream_t s);
 int stage_rows(const RowStage& st, void* xb, int ldxb, int T, int f32, cudaStream_t s);
@@ -91,5 +91,10 @@ struct LatentArgs {
     float scale;
 };
 int latent_attention(const LatentArgs& a, int f32, cudaStream_t s);
+int latent_gather(const void* cache, const int* bt, int page, int Rc, void* out, int S, cudaStream_t s);
+int head_rows(const float* x, int ldx, int D, int Dp, int H, void* out, int T, cudaStream_t s);
+int rows_attention(const void* q, const void* kv, int ldkv, int S, int T, int pos0, int H, int Dp, int Vp, int V, float scale, const float* gate, int ldg, void* out, int ldo,
+                   cudaStream_t s);
+int rows_attention_error(int* flag);
 
 }  // namespace dlp

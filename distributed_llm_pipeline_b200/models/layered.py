@@ -93,19 +93,21 @@ class Segments:
     slot: torch.Tensor          # [n] sequence slot
     chunk: torch.Tensor | None = None      # [chunks, 2] first row and length (long segments)
     first: torch.Tensor | None = None      # [n + 1] first chunk of every segment
+    host: tuple = ()            # long segments: (sequence slot, first row, row behind the last, cached tokens with them)
 
 
 @dataclass
 class Batch:
-    """Device-side description of one forward: T rows, grouped into segments (one per sequence).  Recurrent mixers scan the short
-    segments token by token and take the long ones in chunks."""
+    """Device-side description of one forward: T rows, grouped into segments (one per sequence), short segments first.  Recurrent mixers
+    scan the short ones token by token and take the long ones in chunks; latent attention expands keys and values for the long ones."""
     T: int
+    T_short: int
     short: Segments | None
     long: Segments | None
     tok_slot: torch.Tensor      # [T] sequence slot of every row
     pos: torch.Tensor           # [T]
     slot: torch.Tensor          # [T] cache row
-    tiles: dict[int, TileTable]
+    tiles: dict[tuple[int, bool], TileTable]      # by head count; True: tiles of the short segments only
 
 
 class LayeredEngine(EngineCore):
@@ -151,18 +153,26 @@ class LayeredEngine(EngineCore):
         if lat:
             rows = self._split_ctas * 64
             self.latent_ws = (torch.zeros(rows * max(m.Rc for m in lat), dtype=f32, device=dev), torch.zeros(rows * 2, dtype=f32, device=dev))
-        # segments from this length on run the chunked recurrence (bf16 storage; the fp32 form always scans)
+        # segments from this length on take the chunked recurrence and the expanded attention (bf16 storage; fp32 always takes the others)
+        self.long_from = 2 * lops.HGRN2_CHUNK if self.dtype == torch.bfloat16 else 1 << 60
+        self._expanding_heads = {m.H for m in lat if m.expand} - {m.H for m in lat if not m.expand}
         chunked = [m for m in mixers.values() if m.state is not None and m.chunked]
-        self.chunk_from = 2 * lops.HGRN2_CHUNK if chunked and self.dtype == torch.bfloat16 else 1 << 60
         self.chunk_ws = None
-        if self.chunk_from < M:
-            n = M // lops.HGRN2_CHUNK + M // self.chunk_from + 1         # every long segment may end in a partial chunk
+        if chunked and self.long_from <= M:
+            n = M // lops.HGRN2_CHUNK + M // self.long_from + 1         # every long segment may end in a partial chunk
             self.chunk_ws = tuple(torch.zeros(n * max(m.H * m.D * w(m) for m in chunked), dtype=f32, device=dev) for w in (lambda m: m.V, lambda m: 1))
         self._variant = 1                                            # key ranges per decode query
         self._decode_batches: dict[tuple, Batch] = {}
 
     def buf(self, name: str, rows: int, cols: int, dtype=None) -> torch.Tensor:
         return self._flat[name][:rows * cols].view(rows, cols)
+
+    def grow(self, name: str, rows: int, cols: int) -> torch.Tensor:
+        """A buffer in the storage type that grows with the longest context it was asked for (by half again, so that it settles)."""
+        n = rows * cols
+        if name not in self._flat or self._flat[name].numel() < n:
+            self._flat[name] = torch.zeros(n + n // 2, dtype=self.dtype, device=self.device)
+        return self.buf(name, rows, cols)
 
     # ---- matrix products -------------------------------------------------------------------------------
     def _product(self, r: Rows, w: Dense, out: torch.Tensor, T: int, geglu: bool = False) -> torch.Tensor:
@@ -248,14 +258,14 @@ class LayeredEngine(EngineCore):
             for H in self._latent_heads:
                 bm = lops.latent_tile_rows(H, B)
                 row0, rows = self._tile_lists(H, [1] * B, bm)
-                tiles[H] = TileTable(torch.tensor(row0, dtype=i32, device=dev), torch.tensor(rows, dtype=i32, device=dev), len(row0), bm, min(self._variant, max(1, self._split_ctas // len(row0))))
+                tiles[H, False] = TileTable(torch.tensor(row0, dtype=i32, device=dev), torch.tensor(rows, dtype=i32, device=dev), len(row0), bm, min(self._variant, max(1, self._split_ctas // len(row0))))
             rng = torch.tensor([[i, i + 1] for i in range(B)], dtype=i32, device=dev)
-            b = Batch(B, Segments(B, rng, self.active), None, self.active, self.pos, self.slot, tiles)
+            b = Batch(B, B, Segments(B, rng, self.active), None, self.active, self.pos, self.slot, tiles)
             self._decode_batches[(B, self._variant)] = b
         return b
 
     def _mixed_batch(self, parts: list[tuple[int, list[int]]]) -> tuple[torch.Tensor, Batch]:
-        """Grow every sequence by its tokens and upload the description in one copy."""
+        """Grow every sequence by its tokens (short parts first) and upload the description in one copy."""
         lens = [len(t) for _, t in parts]
         T = sum(lens)
         pos, slot = zip(*(self._advance_inputs(sid, len(t)) for sid, t in parts))
@@ -263,7 +273,9 @@ class LayeredEngine(EngineCore):
                                     torch.cat([torch.full((len(t),), sid, dtype=torch.int32) for sid, t in parts])]
         ends = torch.tensor(lens).cumsum(0).tolist()
         segs = [(sid, hi - n, hi) for (sid, _), n, hi in zip(parts, lens, ends)]
-        groups = [[g for g in segs if (g[2] - g[1] >= self.chunk_from) == is_long] for is_long in (False, True)]
+        groups = [[g for g in segs if (g[2] - g[1] >= self.long_from) == is_long] for is_long in (False, True)]
+        assert [g for grp in groups for g in grp] == segs
+        T_short = groups[0][-1][2] if groups[0] else 0
         for is_long, grp in zip((False, True), groups):
             lists = [[x for g in grp for x in g[1:]], [g[0] for g in grp]]
             if is_long:
@@ -271,17 +283,21 @@ class LayeredEngine(EngineCore):
             cols += [torch.tensor(x, dtype=torch.int32) for x in lists]
         shapes = []
         for H in self._latent_heads:
-            bm = lops.latent_tile_rows(H, T)
-            row0, rows = self._tile_lists(H, lens, bm)
-            cols += [torch.tensor(row0, dtype=torch.int32), torch.tensor(rows, dtype=torch.int32)]
-            shapes.append((H, bm, len(row0)))
+            for only_short, n in ((False, len(lens)), (True, len(groups[0]))):
+                if only_short and (not groups[1] or not n) or not only_short and groups[1] and H in self._expanding_heads:
+                    continue
+                bm = lops.latent_tile_rows(H, sum(lens[:n]))
+                row0, rows = self._tile_lists(H, lens[:n], bm)
+                cols += [torch.tensor(row0, dtype=torch.int32), torch.tensor(rows, dtype=torch.int32)]
+                shapes.append((H, only_short, bm, len(row0)))
         dev = iter(torch.cat(cols).to(self.device).split([c.numel() for c in cols]))
         ids, pos_d, slot_d, tok_slot = (next(dev) for _ in range(4))
         short = Segments(len(groups[0]), next(dev), next(dev))
-        long = Segments(len(groups[1]), next(dev), next(dev), next(dev).view(-1, 2), next(dev))
+        long = Segments(len(groups[1]), next(dev), next(dev), next(dev).view(-1, 2), next(dev),
+                        tuple((sid, lo, hi, self.seqs[sid].length + hi - lo) for sid, lo, hi in groups[1]))
         longest = max(self.seqs[sid].length + len(t) for sid, t in parts)
-        tiles = {H: TileTable(next(dev), next(dev), nt, bm, self._n_splits(nt, longest)) for H, bm, nt in shapes}
-        return ids, Batch(T, short if short.n else None, long if long.n else None, tok_slot, pos_d, slot_d, tiles)
+        tiles = {(H, only): TileTable(next(dev), next(dev), nt, bm, self._n_splits(nt, longest)) for H, only, bm, nt in shapes}
+        return ids, Batch(T, T_short, short if short.n else None, long if long.n else None, tok_slot, pos_d, slot_d, tiles)
 
     def _run_mixed(self, parts: list[tuple[int, list[int]]]):
         """Forward over one mixed batch; updates the sequence lengths.  Returns the pending norm weight (see _forward)."""
@@ -318,19 +334,22 @@ class LayeredEngine(EngineCore):
             offs.append(offs[-1] + len(w))
         done = [0] * len(entries)
         while any(d < len(t) for d, (_, t) in zip(done, entries)):
-            room, parts, rows, dst = self.max_tokens, [], [], []
-            for i, (sid, toks) in enumerate(entries):
+            room, cut = self.max_tokens, []
+            for i, (_, toks) in enumerate(entries):
                 n = min(room, len(toks) - done[i])
-                if n <= 0:
-                    continue
-                base = self.max_tokens - room
+                if n > 0:
+                    cut.append((i, n))
+                    room -= n
+            parts, rows, dst, base = [], [], [], 0
+            for i, n in sorted(cut, key=lambda c: c[1] >= self.long_from):      # short parts first
+                sid, toks = entries[i]
                 for j, p in enumerate(want[i]):
                     if done[i] <= p < done[i] + n:
                         rows.append(base + p - done[i])
                         dst.append(offs[i] + j)
                 parts.append((sid, toks[done[i]:done[i] + n]))
                 done[i] += n
-                room -= n
+                base += n
             pending = self._run_mixed(parts)
             if rows:
                 h = self._settle(sum(len(t) for _, t in parts), pending)
@@ -338,6 +357,8 @@ class LayeredEngine(EngineCore):
                     idx = torch.tensor(rows[k:k + self.max_rows], dtype=torch.long, device=self.device)
                     lg = self._head_rows(Rows(h[idx], self.E), len(idx), torch.empty(len(idx), self.cfg.vocab_size, dtype=torch.float32, device=self.device))
                     out[torch.tensor(dst[k:k + self.max_rows], dtype=torch.long, device=self.device)] = lg
+        if self.device.type == "cuda":
+            lops.check_waits()
         return out
 
     def _reserve(self, grow):

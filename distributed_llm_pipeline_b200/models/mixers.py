@@ -110,26 +110,44 @@ class LatentAttention:
         self.uk[:, :R, :D] = uk.transpose(1, 2)
         self.uv = torch.zeros(H, V, self.Rc, dtype=dtype, device=device)                  # per head [vdim, latent]
         self.uv[:, :, :R] = uv
+        # long prompt portions expand keys and values per head instead (tensor-core flash kernel; heads padded to 64 or 128)
+        self.expand = dtype == torch.bfloat16 and D <= 128 and V <= 128
+        self.Dp, self.Vp = pad_to(D, 64), pad_to(V, 64)
+        if self.expand:
+            ukv = torch.zeros(H * (self.Dp + self.Vp), self.Rc, dtype=dtype, device=device)
+            ukv[:H * self.Dp].view(H, self.Dp, self.Rc)[:, :D, :R] = uk
+            ukv[H * self.Dp:].view(H, self.Vp, self.Rc)[:, :V, :R] = uv
+            self.ukv = Dense(ukv, R)
 
     def weights(self):
-        return [self.w_in, self.w_out, Dense(self.uk.view(-1, self.uk.shape[2]), self.D), Dense(self.uv.view(-1, self.Rc), self.R)]
+        return [self.w_in, self.w_out, Dense(self.uk.view(-1, self.uk.shape[2]), self.D), Dense(self.uv.view(-1, self.Rc), self.R)] + ([self.ukv] if self.expand else [])
 
     def buffers(self, rows: int) -> dict[str, int]:
         return {"q": rows * self.H * self.Rc, "ctx": rows * self.H * self.Rc, "att": rows * self.w_out.Kp}
 
     def mix(self, eng, il: int, proj: torch.Tensor, b) -> Rows:
-        H, D, R, Rc, T = self.H, self.D, self.R, self.Rc, b.T
+        H, D, R, Rc, V = self.H, self.D, self.R, self.Rc, self.V
         cache = eng.kv.planes["c"][il]
-        lops.latent_write(proj[:, H * D:H * D + R], self.c_norm, eng.cfg.rms_eps, R, b.slot, cache, T)
-        q = eng.buf("q", T, H * Rc, eng.dtype)
-        lops.head_matmul(proj, D, D, self.uk, Rc, q, Rc, T)
-        ctx = eng.buf("ctx", T, H * Rc, eng.dtype)
-        t = b.tiles[H]
-        lops.latent_attention(q, cache, eng.kv.block_table, b.tok_slot, b.pos, t.row0, t.rows, t.n, t.bm, H, T, self.scale, ctx, n_splits=t.n_splits,
-                              workspace=eng.latent_ws)
-        att = eng.buf("att", T, self.w_out.Kp, eng.dtype)
-        lops.head_matmul(ctx, Rc, Rc, self.uv, self.V, att, self.V, T, gate=proj[:, H * D + R:])
-        return Rows(att, H * self.V)
+        lops.latent_write(proj[:, H * D:H * D + R], self.c_norm, eng.cfg.rms_eps, R, b.slot, cache, b.T)
+        gate = proj[:, H * D + R:]
+        att = eng.buf("att", b.T, self.w_out.Kp, eng.dtype)
+        long = b.long if self.expand else None
+        T = b.T_short if long is not None else b.T           # short segments come first
+        if T:
+            q = eng.buf("q", T, H * Rc, eng.dtype)
+            lops.head_matmul(proj, D, D, self.uk, Rc, q, Rc, T)
+            ctx = eng.buf("ctx", T, H * Rc, eng.dtype)
+            t = b.tiles[H, long is not None]
+            lops.latent_attention(q, cache, eng.kv.block_table, b.tok_slot, b.pos, t.row0, t.rows, t.n, t.bm, H, T, self.scale, ctx, n_splits=t.n_splits,
+                                  workspace=eng.latent_ws)
+            lops.head_matmul(ctx, Rc, Rc, self.uv, V, att, V, T, gate=gate)
+        for sid, lo, hi, S in (long.host if long is not None else ()):
+            c = eng.grow("c_rows", S, Rc)
+            lops.latent_gather(cache, eng.kv.block_table[sid], S, c)
+            kv = lops.linear(c, self.ukv.t, eng.grow("kv_rows", S, self.ukv.N))
+            q = lops.head_rows(proj[lo:hi], H, D, self.Dp, eng.grow("q_rows", hi - lo, H * self.Dp))
+            lops.rows_attention(q, kv, S, S - (hi - lo), H, self.Dp, self.Vp, V, self.scale, att[lo:hi], gate=gate[lo:hi])
+        return Rows(att, H * V)
 
 
 class GatedMlp:

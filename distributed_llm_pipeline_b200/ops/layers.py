@@ -12,7 +12,7 @@ import torch
 from . import api
 from . import lib as _lib
 
-OUT_F32, OUT_GEGLU = 0, 1
+OUT_F32, OUT_GEGLU, OUT_BF16 = 0, 1, 2
 HGRN2_CHUNK = 64            # tokens per chunk of the chunked recurrence
 
 
@@ -78,9 +78,10 @@ def linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, geglu: bool = Fa
     """x [T, K] (activation type, K = padded width) times w^T through the tcgen05 GEMM (bf16) or the fp32 kernel."""
     _need_cuda(x, "linear")
     f32 = w.dtype == torch.float32
+    mode = OUT_GEGLU if geglu else OUT_F32 if out.dtype == torch.float32 else OUT_BF16
     ws = None if f32 else api.gemm_workspace(x.device)
     _lib.check(_lib.load().dlp_layers_linear(_p(x), x.stride(0), _p(w), w.stride(0), w.shape[0], w.shape[1], _p(out), out.stride(0),
-                                             OUT_GEGLU if geglu else OUT_F32, x.shape[0], int(f32), _p(ws), 0 if ws is None else ws.numel(), api._stream()),
+                                             mode, x.shape[0], int(f32), _p(ws), 0 if ws is None else ws.numel(), api._stream()),
                "layers_linear")
     api._count()
     return out
@@ -155,3 +156,36 @@ def latent_attention(q, cache, block_table, tok_slot, pos, tile_row0, tile_rows,
     _lib.check(_lib.load().dlp_layers_latent_attention(C.byref(a), int(cache.dtype == torch.float32), api._stream()), "layers_latent_attention")
     api._count(2 if n_splits > 1 else 1)
     return out
+
+
+def latent_gather(cache, block_table_row, S: int, out):
+    """Latent rows 0 .. S-1 of one request out of its pages -> out [S, Rc] (bf16)."""
+    _need_cuda(cache, "latent_gather")
+    _lib.check(_lib.load().dlp_layers_latent_gather(_p(cache), _p(block_table_row), cache.shape[-2], cache.shape[-1], _p(out), S, api._stream()), "layers_latent_gather")
+    api._count()
+    return out
+
+
+def head_rows(x, H: int, D: int, Dp: int, out):
+    """fp32 columns [T, H * D] -> bf16 rows [T, H * Dp], heads padded with zeros."""
+    _need_cuda(x, "head_rows")
+    _lib.check(_lib.load().dlp_layers_head_rows(_p(x), x.stride(0), D, Dp, H, _p(out), x.shape[0], api._stream()), "layers_head_rows")
+    api._count()
+    return out
+
+
+def rows_attention(q, kv, S: int, pos0: int, H: int, Dp: int, Vp: int, V: int, scale: float, out, gate=None):
+    """Causal attention of q [T, H * Dp] at positions pos0 .. over kv [S, H * (Dp + Vp)]; out [T, H * V], each head times sigmoid(gate)."""
+    _need_cuda(q, "rows_attention")
+    _lib.check(_lib.load().dlp_layers_rows_attention(_p(q), _p(kv), kv.stride(0), S, q.shape[0], pos0, H, Dp, Vp, V, scale, _p(gate),
+                                                     gate.stride(0) if gate is not None else 0, _p(out), out.stride(0), api._stream()), "layers_rows_attention")
+    api._count()
+    return out
+
+
+def check_waits():
+    """Raise if a wait inside an attention kernel gave up since the last call (synchronises the device)."""
+    flag = C.c_int(0)
+    _lib.check(_lib.load().dlp_layers_rows_attention_error(C.byref(flag)), "rows_attention_error")
+    if flag.value:
+        raise _lib.DlpError("a wait inside the attention kernel ran into its limit")

@@ -82,6 +82,10 @@ def _declare(lib):
         "dlp_layers_latent_write": (i32, [vp, i32, vp, f32, i32, i32, vp, vp, i32, i32, vp]),
         "dlp_layers_hgrn2": (i32, [vp, vp, vp]),
         "dlp_layers_latent_attention": (i32, [vp, i32, vp]),
+        "dlp_layers_latent_gather": (i32, [vp, vp, i32, i32, vp, i32, vp]),
+        "dlp_layers_head_rows": (i32, [vp, i32, i32, i32, i32, vp, i32, vp]),
+        "dlp_layers_rows_attention": (i32, [vp, vp, i32, i32, i32, i32, i32, i32, i32, i32, f32, vp, i32, vp, i32, vp]),
+        "dlp_layers_rows_attention_error": (i32, [vp]),
         "dlp_gemv_moe": (i32, [W, W, vp, vp, f32, vp, i32, i32, vp, i32, vp, vp]),
     }
     for name, (res, args) in sigs.items():

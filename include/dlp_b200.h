@@ -368,7 +368,7 @@ typedef struct {
     const int32_t* tile_row0; const int32_t* tile_rows; void* out; float* part_o; float* part_ml;
     int32_t max_pages, page_size, H, Rc, T, n_tiles, bm, n_splits; float scale;
 } dlp_latent_args;
-/* decode product, 1..4 rows: out_mode 0 = fp32, 1 = GEGLU of interleaved (gate, up) rows -> activation type */
+/* decode product, 1..4 rows: out_mode 0 = fp32, 1 = GEGLU of interleaved (gate, up) rows -> activation type, 2 = bf16 (dlp_layers_linear) */
 int dlp_layers_matvec(const dlp_row_stage* st, const void* w, int ldw, int N, void* out, int ldo, int out_mode, int T, int f32, void* stream);
 int dlp_layers_stage_rows(const dlp_row_stage* st, void* xb, int ldxb, int T, int f32, void* stream);
 /* any number of rows: bf16 through the tcgen05 GEMM (ws: split-K workspace as for dlp_linear_ws), fp32 through an fp32 kernel */
@@ -379,6 +379,13 @@ int dlp_layers_embed(const void* table, int ld, const int32_t* ids, float* h, in
 int dlp_layers_latent_write(const float* proj, int ldp, const float* w, float eps, int R, int Rc, const int32_t* slot, void* cache, int T, int f32, void* stream);
 int dlp_layers_hgrn2(const dlp_hgrn2_args* a, const dlp_hgrn2_chunks* chunks, void* stream);   /* chunks NULL: token scan; else 64-token chunks on the tensor cores */
 int dlp_layers_latent_attention(const dlp_latent_args* a, int f32, void* stream);
+/* prompt portions with keys and values expanded per head (bf16): latent rows of one request out of its pages; query columns as padded rows;
+ * causal flash attention on plain rows kv [S, ldkv] (k in columns [0, H*Dp), v behind it), head sizes padded to 64 or 128 */
+int dlp_layers_latent_gather(const void* cache, const int32_t* bt_row, int page, int Rc, void* out, int S, void* stream);
+int dlp_layers_head_rows(const float* x, int ldx, int D, int Dp, int H, void* out, int T, void* stream);
+int dlp_layers_rows_attention(const void* q, const void* kv, int ldkv, int S, int T, int pos0, int H, int Dp, int Vp, int V, float scale, const float* gate, int ldg,
+                              void* out, int ldo, void* stream);
+int dlp_layers_rows_attention_error(int* flag);   /* *flag = 1: a wait inside the kernel gave up since the last call (synchronises) */
 
 #ifdef __cplusplus
 }

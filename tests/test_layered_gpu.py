@@ -199,6 +199,40 @@ def test_latent_attention(dt, H, R, page, splits):
     assert rel(out, torch.cat(want).reshape(T, -1)) < (6e-3 if dt == BF16 else 5e-6)
 
 
+@pytest.mark.parametrize("H,D,V,pos0,T", [(2, 64, 64, 0, 128), (3, 32, 48, 0, 300), (2, 128, 64, 77, 131), (1, 20, 128, 512, 130), (4, 128, 128, 1, 257)])
+def test_expanded_attention(H, D, V, pos0, T):
+    """The flash kernel on expanded rows: a key that stands out at tile edges, at the start, and at the query itself; later keys unseen."""
+    L, r = ops(), gen(T)
+    Dp, Vp, S, scale = (D + 63) // 64 * 64, (V + 63) // 64 * 64, pos0 + T, 0.17
+    k, v, q, gate = r(S, H, D).to(BF16), r(S, H, V).to(BF16), r(T, H, D, scale=D ** -0.5), r(T, H)
+    marks = [m for m in (0, 1, 63, 64, 127, 128, 255, 256, S - 1) if m < S]
+    for t in range(T):
+        for h in range(H):
+            j = marks[(t + h) % len(marks)]                  # also keys the query must not see
+            q[t, h] += k[j, h].float() * (12 / scale / D)
+    kv = torch.zeros(S, H * (Dp + Vp), dtype=BF16)
+    kv[:, :H * Dp].view(S, H, Dp)[:, :, :D] = k
+    kv[:, H * Dp:].view(S, H, Vp)[:, :, :V] = v
+    qp = torch.empty(T, H * Dp, dtype=BF16, device=DEV)
+    L.head_rows(q.reshape(T, H * D).to(DEV), H, D, Dp, qp)
+    out = torch.zeros(T, H * V + 3, dtype=BF16, device=DEV)
+    L.rows_attention(qp, kv.to(DEV), S, pos0, H, Dp, Vp, V, scale, out, gate=gate.to(DEV))
+    L.check_waits()
+    s = torch.einsum("thd,jhd->htj", q.to(BF16).to(F64), k.to(F64)) * scale
+    s = s.masked_fill(torch.arange(S)[None, None] > (pos0 + torch.arange(T))[None, :, None], -math.inf)
+    want = torch.einsum("htj,jhv->thv", torch.softmax(s, -1), v.to(F64)) / (1 + torch.exp(-gate.to(F64)))[:, :, None]
+    assert rel(out[:, :H * V], want.reshape(T, -1)) < 6e-3 and not out[:, H * V:].any()
+
+
+def test_latent_gather():
+    L = ops()
+    cache = torch.randn(9, 1, 16, 96, device=DEV).to(BF16)
+    bt = torch.tensor([7, 0, 3, 8], dtype=torch.int32, device=DEV)
+    out = torch.zeros(50, 96, dtype=BF16, device=DEV)
+    L.latent_gather(cache, bt, 50, out)
+    assert torch.equal(out, cache[[7, 0, 3, 8]].reshape(-1, 96)[:50])
+
+
 @pytest.mark.parametrize("dt", TYPES)
 def test_latent_write_and_embed(dt):
     L, r = ops(), gen(3)

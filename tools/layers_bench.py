@@ -270,9 +270,17 @@ def kernel_numbers(size: str, ctx: int = 2048, T: int = 2048):
     row0 = torch.arange(0, T * H, bm, device=DEV, dtype=i32)
     nr = torch.full_like(row0, bm)
     qa, ctxo = rnd(T, H * R), torch.zeros(T, H * R, device=DEV, dtype=bf)
+    at2 = torch.zeros(T, H * D, device=DEV, dtype=bf)
     row, z_t = bt1.view(1, -1), torch.zeros(T, device=DEV, dtype=i32)
     us = graph_us(lambda i: L.latent_attention(qa, cache, row, z_t, pos, row0, nr, row0.numel(), bm, H, T, D ** -0.5, ctxo), 1)
     add("talizen", f"attention prefill T={T} (absorbed)", "latent_attn_mma_kernel", us, T * H * D * 8, 2 * T * T * H * D)
+    ukv, cx, kvr, qx = rnd(2 * H * D, R), rnd(T, R), torch.zeros(T, 2 * H * D, device=DEV, dtype=bf), torch.zeros(T, H * D, device=DEV, dtype=bf)
+    us = graph_us(lambda i: L.latent_gather(cache, bt1, T, cx), 1)
+    add("talizen", f"latent gather T={T}", "latent_gather_kernel", us, T * R * 4, 0)
+    us = graph_us(lambda i: L.linear(cx, ukv, kvr), 1)
+    add("talizen", f"key / value expansion T={T}", "gemm_tcgen05_kernel", us, (T * R + 2 * T * H * D + 2 * H * D * R) * 2, 4 * T * H * D * R)
+    us = graph_us(lambda i: L.rows_attention(qx, kvr, T, 0, H, D, D, D, D ** -0.5, at2, gate=proj[:, :H]), 1)
+    add("talizen", f"attention prefill T={T} (expanded)", "attn_prefill_tc_kernel<FA_ROWS>", us, T * H * D * 8, 2 * T * T * H * D)
     return rows, src
 
 
