@@ -32,6 +32,7 @@ __global__ void __launch_bounds__(256, 1) latent_attn_mma_kernel(const LatentArg
     float* S = reinterpret_cast<float*>(cs + 2 * BN * LD);
     float* s_alpha = S + BM * LS;
     float* s_l = s_alpha + BM;
+    int* offs = reinterpret_cast<int*>(s_l + BM);         // [2][BN] cache row of every key of a tile (-1: outside the range)
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, mw = warp / NW, nw = warp % NW, g = lane >> 2, c = lane & 3;
     const int tile = blockIdx.x, split = blockIdx.y;
     pdl_wait();
@@ -41,18 +42,27 @@ __global__ void __launch_bounds__(256, 1) latent_attn_mma_kernel(const LatentArg
     const int* bt = a.block_table + (size_t)a.tok_slot[row0 / a.H] * a.max_pages;
     const __nv_bfloat16* cache = reinterpret_cast<const __nv_bfloat16*>(a.cache);
     const int chunks = Rc / 8;
-    auto load_tile = [&](int k0, int b) {
-        for (int i = tid; i < BN * chunks; i += 256) {
-            const int kk = i / chunks, ch = i - kk * chunks, key = k0 + kk;
-            const bool ok = key < kr.hi;
-            const int kc = ok ? key : 0;
-            const size_t src = ((size_t)bt[kc / a.page_size] * a.page_size + kc % a.page_size) * Rc + ch * 8;
-            cp_async16(cs + ((size_t)b * BN + kk) * LD + ch * 8, cache + src, ok);
+    auto find_rows = [&](int k0, int b) {
+        if (tid < BN) {
+            const int key = k0 + tid;
+            offs[b * BN + tid] = key < kr.hi ? bt[key / a.page_size] * a.page_size + key % a.page_size : -1;
+        }
+    };
+    auto load_tile = [&](int b) {           // eight threads per latent row
+#pragma unroll
+        for (int half = 0; half < 2; ++half) {
+            const int kk = half * 32 + (tid >> 3), row = offs[b * BN + kk];
+            const __nv_bfloat16* src = cache + (size_t)max(row, 0) * Rc;
+            __nv_bfloat16* dst = cs + ((size_t)b * BN + kk) * LD;
+            for (int ch = tid & 7; ch < chunks; ch += 8) cp_async16(dst + ch * 8, src + ch * 8, row >= 0);
         }
         cp_commit();
     };
     const int n_tiles = (kr.hi - kr.lo + BN - 1) / BN;
-    if (n_tiles > 0) load_tile(kr.lo, 0);
+    find_rows(kr.lo, 0);
+    find_rows(kr.lo + BN, 1);
+    __syncthreads();
+    if (n_tiles > 0) load_tile(0);
     {
         const uint4* q = reinterpret_cast<const uint4*>(reinterpret_cast<const __nv_bfloat16*>(a.q) + (size_t)row0 * Rc);
         for (int i = tid; i < BM * chunks; i += 256) {
@@ -67,26 +77,37 @@ __global__ void __launch_bounds__(256, 1) latent_attn_mma_kernel(const LatentArg
     float acc[NPAIR][2][4] = {};
     for (int it = 0; it < n_tiles; ++it) {
         const int k0 = kr.lo + it * BN, b = it & 1;
-        if (it + 1 < n_tiles) { load_tile(k0 + BN, b ^ 1); cp_wait<1>(); } else { cp_wait<0>(); }
+        if (it + 1 < n_tiles) { load_tile(b ^ 1); cp_wait<1>(); } else { cp_wait<0>(); }
         __syncthreads();
+        if (it + 2 < n_tiles) find_rows(k0 + 2 * BN, b);      // read behind the barriers of this iteration
         const __nv_bfloat16* ct = cs + (size_t)b * BN * LD;
         {   // scores: 16 rows x KPW keys per warp
-            float sacc[KPW / 8][4] = {};
-            for (int k = 0; k < Rc; k += 16) {
-                uint32_t af[4];
-                ldsm_x4(af, qs + (mw * 16 + (lane & 15)) * LD + k + (lane >> 4) * 8);
+            constexpr int NJ = KPW / 8, CH = NJ >= 4 ? 1 : NJ == 2 ? 2 : 4;      // independent accumulation chains
+            float sacc[CH][NJ][4] = {};
+#pragma unroll 2
+            for (int k = 0; k < Rc; k += 16 * CH) {
 #pragma unroll
-                for (int j = 0; j < KPW / 8; ++j) {
-                    uint32_t bf[2];
-                    ldsm_x2(bf, ct + (nw * KPW + j * 8 + (lane & 7)) * LD + k + ((lane >> 3) & 1) * 8);
-                    mma16816(sacc[j], af, bf[0], bf[1]);
+                for (int x = 0; x < CH; ++x) {
+                    if (CH > 2 && k + x * 16 >= Rc) break;           // Rc is a multiple of 32
+                    uint32_t af[4];
+                    ldsm_x4(af, qs + (mw * 16 + (lane & 15)) * LD + k + x * 16 + (lane >> 4) * 8);
+#pragma unroll
+                    for (int j = 0; j < NJ; ++j) {
+                        uint32_t bf[2];
+                        ldsm_x2(bf, ct + (nw * KPW + j * 8 + (lane & 7)) * LD + k + x * 16 + ((lane >> 3) & 1) * 8);
+                        mma16816(sacc[x][j], af, bf[0], bf[1]);
+                    }
                 }
             }
 #pragma unroll
-            for (int j = 0; j < KPW / 8; ++j)
+            for (int j = 0; j < NJ; ++j)
 #pragma unroll
-                for (int e = 0; e < 4; ++e)
-                    S[(mw * 16 + g + (e >> 1) * 8) * LS + nw * KPW + j * 8 + c * 2 + (e & 1)] = sacc[j][e] * a.scale;
+                for (int e = 0; e < 4; ++e) {
+                    float v = sacc[0][j][e];
+#pragma unroll
+                    for (int x = 1; x < CH; ++x) v += sacc[x][j][e];
+                    S[(mw * 16 + g + (e >> 1) * 8) * LS + nw * KPW + j * 8 + c * 2 + (e & 1)] = v * a.scale;
+                }
         }
         __syncthreads();
         {   // running softmax
@@ -240,23 +261,26 @@ __global__ void __launch_bounds__(128) latent_attn_kernel(const LatentArgs a) {
 
 template <typename WT>
 __global__ void __launch_bounds__(128) latent_combine_kernel(const LatentArgs a) {
+    __shared__ float w[32];                       // weight of every key range
     pdl_wait();
-    const int row = blockIdx.x;
+    const int row = blockIdx.x, lane = threadIdx.x & 31;
     const size_t stride = (size_t)a.T * a.H;
-    float m = -INFINITY, l = 0.f;
-    for (int s = 0; s < a.n_splits; ++s) m = fmaxf(m, a.part_ml[(s * stride + row) * 2]);
-    for (int s = 0; s < a.n_splits; ++s) {
-        const float ms = a.part_ml[(s * stride + row) * 2];
-        l += ms == -INFINITY ? 0.f : a.part_ml[(s * stride + row) * 2 + 1] * expf(ms - m);
+    if (threadIdx.x < 32) {
+        const bool ok = lane < a.n_splits;
+        const float ms = ok ? a.part_ml[(lane * stride + row) * 2] : -INFINITY, ls = ok ? a.part_ml[(lane * stride + row) * 2 + 1] : 0.f;
+        const float m = warp_max(ms), e = ms == -INFINITY ? 0.f : expf(ms - m);
+        const float l = warp_sum(e * ls);
+        w[lane] = l > 0.f ? e / l : 0.f;
     }
-    const float inv = l > 0.f ? 1.f / l : 0.f;
+    __syncthreads();
     for (int r = threadIdx.x; r < a.Rc; r += 128) {
         float v = 0.f;
+#pragma unroll 8
         for (int s = 0; s < a.n_splits; ++s) {
-            const float ms = a.part_ml[(s * stride + row) * 2];
-            if (ms != -INFINITY) v = fmaf(a.part_o[(s * stride + row) * a.Rc + r], expf(ms - m), v);
+            const float ws = w[s];
+            if (ws != 0.f) v = fmaf(a.part_o[(s * stride + row) * a.Rc + r], ws, v);
         }
-        reinterpret_cast<WT*>(a.out)[(size_t)row * a.Rc + r] = (WT)(v * inv);
+        reinterpret_cast<WT*>(a.out)[(size_t)row * a.Rc + r] = (WT)v;
     }
     pdl_launch_dependents();
 }
@@ -264,7 +288,7 @@ __global__ void __launch_bounds__(128) latent_combine_kernel(const LatentArgs a)
 template <int MW, int RMAX>
 static int launch_latent_mma(const LatentArgs& a, cudaStream_t s) {
     constexpr int BM = 16 * MW;
-    const size_t smem = (size_t)(BM + 128) * (a.Rc + 8) * 2 + (size_t)BM * 68 * 4 + BM * 8;
+    const size_t smem = (size_t)(BM + 128) * (a.Rc + 8) * 2 + (size_t)BM * 68 * 4 + BM * 8 + 512;
     DLP_REQUIRE(smem <= 227 * 1024, "latent_attention: %zu bytes of shared memory", smem);
     auto kern = latent_attn_mma_kernel<MW, RMAX>;
     if (first_use_on_device((const void*)kern)) DLP_CHECK_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024));
@@ -275,7 +299,7 @@ static int launch_latent_mma(const LatentArgs& a, cudaStream_t s) {
 int latent_attention(const LatentArgs& a, int f32, cudaStream_t s) {
     DLP_REQUIRE(a.q && a.cache && a.block_table && a.tok_slot && a.pos && a.out && a.tile_row0 && a.tile_rows, "latent_attention: null argument");
     DLP_REQUIRE(a.H > 0 && a.Rc > 0 && a.Rc % 32 == 0 && a.T > 0 && a.n_tiles > 0 && a.page_size > 0 && a.max_pages > 0, "latent_attention: bad shape");
-    DLP_REQUIRE(a.n_splits >= 1 && a.n_splits <= 64 && (a.n_splits == 1 || (a.part_o && a.part_ml)), "latent_attention: %d key ranges", a.n_splits);
+    DLP_REQUIRE(a.n_splits >= 1 && a.n_splits <= 32 && (a.n_splits == 1 || (a.part_o && a.part_ml)), "latent_attention: %d key ranges", a.n_splits);
     int rc = 0;
     if (!f32 && a.Rc <= 512) {
         DLP_REQUIRE(a.bm == 16 || a.bm == 32 || a.bm == 64, "latent_attention: tile of %d rows", a.bm);

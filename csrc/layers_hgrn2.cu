@@ -37,11 +37,27 @@ __device__ __forceinline__ void load_gates(const Hgrn2Args& a, const ChunkIn& c,
 }
 template <int VP, int NTH>
 __device__ __forceinline__ void load_values(const Hgrn2Args& a, const ChunkIn& c, int h, int v0, __nv_bfloat16* sv) {
-    constexpr int LDV = VP + 8;
+    constexpr int LDV = VP + 8, Q = HC * VP / 4 / NTH;      // four values a time
+    const float* base = a.proj + (size_t)c.t0 * a.ldp + 2 * a.H * a.D + h * a.V + v0;
+    if (v0 + VP <= a.V && a.ldp % 4 == 0 && (reinterpret_cast<uintptr_t>(base) & 15) == 0) {
+        float4 x[Q];
+#pragma unroll
+        for (int j = 0; j < Q; ++j) {
+            const int i = threadIdx.x + j * NTH, s = i / (VP / 4), v = i % (VP / 4);
+            x[j] = s < c.n ? *reinterpret_cast<const float4*>(base + (size_t)s * a.ldp + v * 4) : make_float4(0.f, 0.f, 0.f, 0.f);
+        }
+#pragma unroll
+        for (int j = 0; j < Q; ++j) {
+            const int i = threadIdx.x + j * NTH, s = i / (VP / 4), v = i % (VP / 4);
+            __nv_bfloat162* o = reinterpret_cast<__nv_bfloat162*>(sv + s * LDV + v * 4);
+            o[0] = __floats2bfloat162_rn(x[j].x, x[j].y);
+            o[1] = __floats2bfloat162_rn(x[j].z, x[j].w);
+        }
+        return;
+    }
     for (int i = threadIdx.x; i < HC * VP; i += NTH) {
         const int s = i / VP, v = i - s * VP;
-        const bool ok = s < c.n && v0 + v < a.V;
-        sv[s * LDV + v] = __float2bfloat16_rn(ok ? a.proj[(size_t)(c.t0 + s) * a.ldp + 2 * a.H * a.D + h * a.V + v0 + v] : 0.f);
+        sv[s * LDV + v] = __float2bfloat16_rn(s < c.n && v0 + v < a.V ? base[(size_t)s * a.ldp + v] : 0.f);
     }
 }
 __device__ __forceinline__ void split_one(float x, __nv_bfloat16& hi, __nv_bfloat16& lo) {
@@ -102,9 +118,15 @@ __global__ void __launch_bounds__(4 * DP) hgrn2_chunk_state_kernel(const Hgrn2Ar
 #pragma unroll
         for (int n = 0; n < 2; ++n)
 #pragma unroll
-            for (int e = 0; e < 4; ++e) {
-                const int dd = mt * 16 + (lane >> 2) + (e >> 1) * 8, v = v0 + (cg * NP + j) * 16 + n * 8 + (lane & 3) * 2 + (e & 1);
-                if (dd < a.D && v < a.V) u[(size_t)dd * a.V + v] = acc[j][n][e];
+            for (int e = 0; e < 4; e += 2) {
+                const int dd = mt * 16 + (lane >> 2) + (e >> 1) * 8, v = v0 + (cg * NP + j) * 16 + n * 8 + (lane & 3) * 2;
+                if (dd >= a.D) continue;
+                if (a.V % 2 == 0) {
+                    if (v < a.V) *reinterpret_cast<float2*>(u + (size_t)dd * a.V + v) = make_float2(acc[j][n][e], acc[j][n][e + 1]);
+                } else {
+                    if (v < a.V) u[(size_t)dd * a.V + v] = acc[j][n][e];
+                    if (v + 1 < a.V) u[(size_t)dd * a.V + v + 1] = acc[j][n][e + 1];
+                }
             }
     pdl_launch_dependents();
 }
@@ -225,12 +247,22 @@ __global__ void __launch_bounds__(4 * DP, 1) hgrn2_chunk_out_kernel(const Hgrn2A
 #pragma unroll
         for (int r = 0; r < 16; ++r) qt[r] *= pre;
     }
+    // the state the chunk starts from, requested now, used behind the chunk's own tokens
+    constexpr int SQ = DP * VP / 4 / NTH;
+    const float* S = cc.states + ((size_t)ch * a.H + h) * a.D * a.V;
+    const bool s_vec = a.V % 4 == 0;
+    float4 s4[SQ];
+#pragma unroll
+    for (int j = 0; j < SQ; ++j) {
+        const int i = tid + j * NTH, dd = i / (VP / 4), v = i % (VP / 4) * 4;
+        s4[j] = (s_vec && dd < a.D && v0 + v < a.V) ? *reinterpret_cast<const float4*>(S + (size_t)dd * a.V + v0 + v) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
     {   // diagonal blocks: thread (key token s, channel group) runs over the queries of the block
         const int s = tid / C::PARTS, part = tid % C::PARTS, b0 = s & ~15;
         float w[C::CPP];
 #pragma unroll
         for (int i = 0; i < C::CPP; ++i) w[i] = sk[s * LDF + diag_piece(part, i >> 2) + (i & 3)];
-#pragma unroll 1
+#pragma unroll 2
         for (int t = b0; t < b0 + 16; ++t) {
             float acc = 0.f;
             const bool later = t > s;
@@ -285,9 +317,17 @@ __global__ void __launch_bounds__(4 * DP, 1) hgrn2_chunk_out_kernel(const Hgrn2A
     // the block factors and the key rows are done with: state and decayed queries take their place
 #pragma unroll
     for (int r = 0; r < 16; ++r) split_one(qt[r], qhhi[(q * 16 + r) * LDK + d], qhlo[(q * 16 + r) * LDK + d]);
-    {
-        const float* S = cc.states + ((size_t)ch * a.H + h) * a.D * a.V;
-#pragma unroll 8
+    if (s_vec) {
+#pragma unroll
+        for (int j = 0; j < SQ; ++j) {
+            const int i = tid + j * NTH, o = i / (VP / 4) * LDV + i % (VP / 4) * 4;
+            uint32_t hi[2], lo[2];
+            split_bf16(s4[j].x, s4[j].y, hi[0], lo[0]);
+            split_bf16(s4[j].z, s4[j].w, hi[1], lo[1]);
+            *reinterpret_cast<uint2*>(shi + o) = make_uint2(hi[0], hi[1]);
+            *reinterpret_cast<uint2*>(slo + o) = make_uint2(lo[0], lo[1]);
+        }
+    } else {
         for (int i = tid; i < DP * VP; i += NTH) {
             const int dd = i / VP, v = i - dd * VP;
             split_one((dd < a.D && v0 + v < a.V) ? S[(size_t)dd * a.V + v0 + v] : 0.f, shi[dd * LDV + v], slo[dd * LDV + v]);

@@ -68,8 +68,90 @@ __device__ __forceinline__ float* stage_rms(int rows, int groups, int K, float e
     return rs;
 }
 
-template <typename XT, int NT, typename Put>
-__device__ __forceinline__ void stage_rows_dev(const RowStage& p, int t0, int rows, float* sums, bool store_h, Put put) {
+// Vector form: rows in slices of 128 values, one warp per slice and pass; groups are whole slices.
+__host__ __device__ inline bool stage_vec(const RowStage& p) {
+    return p.K % 128 == 0 && p.Kp == p.K && p.ldx % 8 == 0 && (!p.y || ((p.K / p.groups1) % 128 == 0 && p.ldy % 4 == 0 && p.ldh % 4 == 0)) &&
+           (!p.w2 || ((p.K / p.groups2) % 128 == 0 && p.w2_mod % 128 == 0));
+}
+template <typename F>
+__device__ __forceinline__ float* stage_rms_vec(int rows, int groups, int K, float eps, float* sums, F f) {
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5, spr = K >> 7, n = rows * spr;
+#pragma unroll 4
+    for (int i = warp; i < n; i += nw) {
+        const int t = i / spr;
+        const float4 v = f(t, (i - t * spr) * 128 + lane * 4);
+        const float a = warp_sum(fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, v.w * v.w))));
+        if (lane == 0) sums[i] = a;
+    }
+    __syncthreads();
+    float* rs = sums + n;
+    const int gs = K / groups, per = gs >> 7;
+    for (int i = threadIdx.x; i < rows * groups; i += blockDim.x) {
+        float a = 0.f;
+        for (int j = 0; j < per; ++j) a += sums[i * per + j];
+        rs[i] = 1.f / sqrtf(a / (float)gs + eps);
+    }
+    __syncthreads();
+    return rs;
+}
+template <typename XT>
+__device__ __forceinline__ float4 stage_x4(const RowStage& p, int t, int k) {
+    if (p.x_f32) return *reinterpret_cast<const float4*>(reinterpret_cast<const float*>(p.x) + (size_t)t * p.ldx + k);
+    if (sizeof(XT) == 4) return *reinterpret_cast<const float4*>(reinterpret_cast<const float*>(p.x) + (size_t)t * p.ldx + k);
+    const uint2 u = *reinterpret_cast<const uint2*>(reinterpret_cast<const __nv_bfloat16*>(p.x) + (size_t)t * p.ldx + k);
+    const float2 a = bf2_to_f2(u.x), b = bf2_to_f2(u.y);
+    return make_float4(a.x, a.y, b.x, b.y);
+}
+template <typename XT, typename Put4>
+__device__ __forceinline__ void stage_rows_vec(const RowStage& p, int t0, int rows, float* sums, bool store_h, Put4 put) {
+    const float* rs1 = nullptr;
+    const float* rs2 = nullptr;
+    const int gs1 = p.y ? p.K / p.groups1 : 1, gs2 = p.w2 ? p.K / p.groups2 : 1;
+    auto y4 = [&](int t, int k) { return *reinterpret_cast<const float4*>(p.y + (size_t)(t0 + t) * p.ldy + k); };
+    if (p.y) {
+        rs1 = stage_rms_vec(rows, p.groups1, p.K, p.eps, sums, y4);
+        sums += rows * (p.K / 128 + p.groups1);
+    }
+    auto base = [&](int t, int k) {
+        float4 v = stage_x4<XT>(p, t0 + t, k);
+        if (p.y) {
+            const float4 y = y4(t, k), w = *reinterpret_cast<const float4*>(p.w1 + k);
+            const float r = rs1[t * p.groups1 + k / gs1];
+            v.x = fmaf(y.x * r, w.x, v.x);
+            v.y = fmaf(y.y * r, w.y, v.y);
+            v.z = fmaf(y.z * r, w.z, v.z);
+            v.w = fmaf(y.w * r, w.w, v.w);
+        }
+        return v;
+    };
+    if (p.w2) rs2 = stage_rms_vec(rows, p.groups2, p.K, p.eps, sums, base);
+    const int q = p.K >> 2;
+#pragma unroll 2
+    for (int i = threadIdx.x; i < rows * q; i += blockDim.x) {
+        const int t = i / q, k = (i - t * q) * 4;
+        float4 v = base(t, k);
+        if (store_h && p.h_out) *reinterpret_cast<float4*>(p.h_out + (size_t)(t0 + t) * p.ldh + k) = v;
+        if (p.w2) {
+            const float r = rs2[t * p.groups2 + k / gs2];
+            const float4 w = *reinterpret_cast<const float4*>(p.w2 + k % p.w2_mod);
+            v = make_float4(v.x * r * w.x, v.y * r * w.y, v.z * r * w.z, v.w * r * w.w);
+        }
+        put(t, k, v);
+    }
+    __syncthreads();
+}
+__device__ __forceinline__ void put4(__nv_bfloat16* d, float4 v) {
+    __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
+    *reinterpret_cast<uint2*>(d) = make_uint2(*reinterpret_cast<uint32_t*>(&a), *reinterpret_cast<uint32_t*>(&b));
+}
+__device__ __forceinline__ void put4(float* d, float4 v) { *reinterpret_cast<float4*>(d) = v; }
+
+template <typename XT>
+__device__ __forceinline__ void stage_rows_dev(const RowStage& p, int t0, int rows, float* sums, bool store_h, XT* dst, int ldd) {
+    if (stage_vec(p)) {
+        stage_rows_vec<XT>(p, t0, rows, sums, store_h, [&](int t, int k, float4 v) { put4(dst + (size_t)t * ldd + k, v); });
+        return;
+    }
     const float* rs1 = nullptr;
     const float* rs2 = nullptr;
     const int gs1 = p.y ? p.K / p.groups1 : 1, gs2 = p.w2 ? p.K / p.groups2 : 1;
@@ -89,13 +171,17 @@ __device__ __forceinline__ void stage_rows_dev(const RowStage& p, int t0, int ro
                 if (store_h && p.h_out) p.h_out[(size_t)(t0 + t) * p.ldh + k] = v;
                 if (p.w2) v *= rs2[t * p.groups2 + k / gs2] * p.w2[k % p.w2_mod];
             }
-            put(t, k, v);
+            dst[(size_t)t * ldd + k] = Act<XT>::from_f(v);
         }
     }
     __syncthreads();
 }
 static size_t stage_bytes(const RowStage& p, int rows, int nwarps) {
-    return ((size_t)(p.y ? stage_scratch(rows, p.groups1, nwarps) : 0) + (p.w2 ? stage_scratch(rows, p.groups2, nwarps) : 0)) * 4 + 16;
+    auto need = [&](int groups) {
+        const int a = stage_scratch(rows, groups, nwarps), b = rows * (p.K / 128 + groups);
+        return (size_t)(a > b ? a : b);
+    };
+    return ((p.y ? need(p.groups1) : 0) + (p.w2 ? need(p.groups2) : 0)) * 4 + 16;
 }
 
 template <typename XT>
@@ -103,7 +189,7 @@ __global__ void __launch_bounds__(256) stage_rows_kernel(const RowStage p, XT* x
     extern __shared__ __align__(16) float st_sums[];
     pdl_wait();
     const int t0 = blockIdx.x;
-    stage_rows_dev<XT, 1>(p, t0, 1, st_sums, true, [&](int, int k, float v) { xb[(size_t)t0 * ldxb + k] = Act<XT>::from_f(v); });
+    stage_rows_dev<XT>(p, t0, 1, st_sums, true, xb + (size_t)t0 * ldxb, ldxb);
     pdl_launch_dependents();
 }
 
@@ -139,7 +225,7 @@ __global__ void __launch_bounds__(512, 1) matvec_kernel(const RowStage st, const
     int u = warp;
     if (u < units) issue(u, 0);
     pdl_wait();
-    stage_rows_dev<WT, NT>(st, 0, T, sums, blockIdx.x == 0, [&](int t, int k, float v) { xs[(size_t)t * K + k] = Act<WT>::from_f(v); });
+    stage_rows_dev<WT>(st, 0, T, sums, blockIdx.x == 0, xs, K);
     float* part = sums;      // [units][2][NT]: the staging scratch is free again
     auto reduce = [&](int u, int b) {
         const int pr = u / KC, c = u - pr * KC;
@@ -396,6 +482,76 @@ __global__ void __launch_bounds__(128) head_matmul_kernel(const void* x, int x_f
         }
 }
 
+// up to 16 tokens: a block takes 16 outputs of one head, its four warps share the inner dimension, so that every weight byte of the
+// block is requested at once
+__global__ void __launch_bounds__(128) head_matmul_small_kernel(const void* x, int x_f32, int ldx, int x_head, int kx, const __nv_bfloat16* __restrict__ w, int Kp, int N,
+                                                                int n_rows, __nv_bfloat16* out, int ldo, int out_head, const float* gate, int ldg, int T) {
+    extern __shared__ __align__(16) uint8_t hm_smem[];
+    __nv_bfloat16* xs = reinterpret_cast<__nv_bfloat16*>(hm_smem);      // [T][Kp + 8]
+    __shared__ float red[4][16][17];
+    const int ldxs = Kp + 8, h = blockIdx.y, n0 = blockIdx.x * 16;
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, g = lane >> 2, c = lane & 3;
+    const __nv_bfloat16* wr[2];
+    bool ok[2];
+#pragma unroll
+    for (int j = 0; j < 2; ++j) {
+        const int n = n0 + j * 8 + g;
+        ok[j] = n < n_rows;
+        wr[j] = w + ((size_t)h * n_rows + (ok[j] ? n : 0)) * Kp + c * 8;
+    }
+    constexpr int U = 4;                       // 32-wide inner blocks in flight
+    uint4 b[U][2];
+    auto load = [&](int k) {
+#pragma unroll
+        for (int u = 0; u < U; ++u)
+#pragma unroll
+            for (int j = 0; j < 2; ++j) b[u][j] = (ok[j] && k + u * 128 < Kp) ? ldg_nc_v4(wr[j] + k + u * 128) : make_uint4(0, 0, 0, 0);
+    };
+    load(warp * 32);                           // weights do not depend on the previous kernel
+    pdl_wait();
+    for (int t = 0; t < T; ++t)
+        for (int k = threadIdx.x; k < Kp; k += 128) {
+            float v = 0.f;
+            if (k < kx) {
+                const size_t o = (size_t)t * ldx + (size_t)h * x_head + k;
+                v = x_f32 ? reinterpret_cast<const float*>(x)[o] : __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(x)[o]);
+            }
+            xs[t * ldxs + k] = __float2bfloat16_rn(v);
+        }
+    __syncthreads();
+    float acc[2][4] = {};
+    for (int k0 = warp * 32; k0 < Kp; k0 += U * 128) {
+        if (k0 != warp * 32) load(k0);
+#pragma unroll
+        for (int u = 0; u < U; ++u) {
+            const int k = k0 + u * 128;
+            if (k < Kp) {
+                const uint4 zero = make_uint4(0, 0, 0, 0);
+                const uint4 lo = g < T ? *reinterpret_cast<const uint4*>(xs + g * ldxs + k + c * 8) : zero;
+                const uint4 hi = g + 8 < T ? *reinterpret_cast<const uint4*>(xs + (g + 8) * ldxs + k + c * 8) : zero;
+#pragma unroll
+                for (int j = 0; j < 2; ++j) {
+                    mma16816(acc[j], {lo.x, hi.x, lo.y, hi.y}, b[u][j].x, b[u][j].y);
+                    mma16816(acc[j], {lo.z, hi.z, lo.w, hi.w}, b[u][j].z, b[u][j].w);
+                }
+            }
+        }
+    }
+    pdl_launch_dependents();
+#pragma unroll
+    for (int j = 0; j < 2; ++j)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) red[warp][g + (e >> 1) * 8][j * 8 + c * 2 + (e & 1)] = acc[j][e];
+    __syncthreads();
+    for (int i = threadIdx.x; i < T * 16; i += 128) {
+        const int t = i >> 4, n = n0 + (i & 15);
+        if (n >= N) continue;
+        float v = red[0][t][i & 15] + red[1][t][i & 15] + red[2][t][i & 15] + red[3][t][i & 15];
+        if (gate) v *= 1.f / (1.f + expf(-gate[(size_t)t * ldg + h]));
+        out[(size_t)t * ldo + (size_t)h * out_head + n] = __float2bfloat16_rn(v);
+    }
+}
+
 __global__ void __launch_bounds__(128) head_matmul_f32_kernel(const float* x, int ldx, int x_head, int kx, const float* __restrict__ w, int Kp, int N, int n_rows,
                                                               float* out, int ldo, int out_head, const float* gate, int ldg) {
     extern __shared__ __align__(16) float hf_x[];
@@ -424,16 +580,22 @@ int head_matmul(const void* x, int x_f32, int ldx, int x_head, int kx, const voi
         }
         return 0;
     }
-    const int mt = T <= 16 ? 1 : 4;
-    const size_t smem = (size_t)16 * mt * (Kp + 8) * 2;
+    if (T <= 16) {
+        const size_t smem = (size_t)T * (Kp + 8) * 2;
+        DLP_REQUIRE(smem <= 200 * 1024, "head_matmul: inner size %d", Kp);
+        auto k1 = head_matmul_small_kernel;
+        if (first_use_on_device((const void*)k1)) DLP_CHECK_CUDA(cudaFuncSetAttribute(k1, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+        DLP_CHECK_CUDA(launch_pdl(k1, dim3((N + 15) / 16, H), dim3(128), smem, s, x, x_f32, ldx, x_head, kx, (const __nv_bfloat16*)w, Kp, N, n_rows, (__nv_bfloat16*)out, ldo,
+                                  out_head, gate, ldg, T));
+        return 0;
+    }
+    constexpr int MT = 4;
+    const size_t smem = (size_t)16 * MT * (Kp + 8) * 2;
     DLP_REQUIRE(smem <= 227 * 1024, "head_matmul: inner size %d", Kp);
-    dim3 grid((N + 63) / 64, H, (T + 16 * mt - 1) / (16 * mt));
-    auto k1 = head_matmul_kernel<1>;
-    auto k4 = head_matmul_kernel<4>;
-    if (first_use_on_device((const void*)k1)) DLP_CHECK_CUDA(cudaFuncSetAttribute(k1, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024));
+    dim3 grid((N + 63) / 64, H, (T + 16 * MT - 1) / (16 * MT));
+    auto k4 = head_matmul_kernel<MT>;
     if (first_use_on_device((const void*)k4)) DLP_CHECK_CUDA(cudaFuncSetAttribute(k4, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024));
-    DLP_CHECK_CUDA(launch_pdl(mt == 1 ? k1 : k4, grid, dim3(128), smem, s, x, x_f32, ldx, x_head, kx, (const __nv_bfloat16*)w, Kp, N, n_rows, (__nv_bfloat16*)out, ldo,
-                              out_head, gate, ldg, T));
+    DLP_CHECK_CUDA(launch_pdl(k4, grid, dim3(128), smem, s, x, x_f32, ldx, x_head, kx, (const __nv_bfloat16*)w, Kp, N, n_rows, (__nv_bfloat16*)out, ldo, out_head, gate, ldg, T));
     return 0;
 }
 

@@ -148,7 +148,7 @@ class LayeredEngine(EngineCore):
         self.logits = torch.zeros(max_seqs, cfg.vocab_size, dtype=f32, device=dev)
         lat = [m for m in mixers.values() if isinstance(m, LatentAttention)]
         self._latent_heads = sorted({m.H for m in lat})
-        self._split_ctas = 296                                       # two CTAs per SM: the key range is split until they are there
+        self._split_ctas = 148                                       # one CTA per SM: the key range is split until they are there
         self.latent_ws = None
         if lat:
             rows = self._split_ctas * 64
@@ -236,7 +236,7 @@ class LayeredEngine(EngineCore):
 
     # ---- batch descriptions ---------------------------------------------------------------------------------
     def _n_splits(self, n_tiles: int, max_len: int) -> int:
-        want, n = min(self._split_ctas // max(1, n_tiles), (max_len + 255) // 256, 32), 1
+        want, n = min(self._split_ctas // max(1, n_tiles), (max_len + 63) // 64, 32), 1
         while n * 2 <= want:
             n *= 2
         return n

@@ -197,7 +197,7 @@ def kernel_numbers(size: str, ctx: int = 2048, T: int = 2048):
         row0 = torch.tensor([b * H + i * bm for b in range(B) for i in range(per)], device=DEV, dtype=i32)
         nr = torch.tensor([min(bm, H - i * bm) for b in range(B) for i in range(per)], device=DEV, dtype=i32)
         ns = 1
-        while ns * 2 <= min(296 // (B * per), (ctx + 255) // 256, 32):
+        while ns * 2 <= min(148 // (B * per), (ctx + 63) // 64, 32):
             ns *= 2
         q, out = rnd(B, H * R), torch.zeros(B, H * R, device=DEV, dtype=bf)
         ws = (torch.zeros(ns * B * H * R, device=DEV), torch.zeros(ns * B * H * 2, device=DEV))
