@@ -21,7 +21,7 @@ for f in "${SRC[@]}"; do
   b="$(basename "$f" .cu)"
   objs+=("$OBJ/$b.o")
   MATH=(--use_fast_math)
-  case "$b" in layers_*) MATH=() ;; esac        # exact divisions, square roots and exponentials where a layer is specified in 32 bits
+  case "$b" in layers_attention_tc) ;; layers_*) MATH=() ;; esac        # exact divisions, square roots and exponentials where a layer is specified in 32 bits
   if [[ ! -f "$OBJ/$b.o" || "$f" -nt "$OBJ/$b.o" || -n "$(find "$HERE" -maxdepth 1 -name '*.cuh' -newer "$OBJ/$b.o" -print -quit)" || "$HERE/../include/dlp_b200.h" -nt "$OBJ/$b.o" ]]; then
     ( "$NVCC" "${FLAGS[@]}" ${MATH[@]+"${MATH[@]}"} -c "$f" -o "$OBJ/$b.o.tmp" > "$OBJ/$b.log" 2>&1 && mv "$OBJ/$b.o.tmp" "$OBJ/$b.o" || { cat "$OBJ/$b.log"; exit 1; } ) &
     pids+=($!)

@@ -273,13 +273,13 @@ __global__ void __launch_bounds__(128) latent_combine_kernel(const LatentArgs a)
         w[lane] = l > 0.f ? e / l : 0.f;
     }
     __syncthreads();
-    for (int r = threadIdx.x; r < a.Rc; r += 128) {
-        float v = 0.f;
-#pragma unroll 8
-        for (int s = 0; s < a.n_splits; ++s) {
-            const float ws = w[s];
-            if (ws != 0.f) v = fmaf(a.part_o[(s * stride + row) * a.Rc + r], ws, v);
-        }
+    const int r = blockIdx.y * 128 + threadIdx.x;
+    if (r < a.Rc) {
+        float x[32], v = 0.f;
+#pragma unroll
+        for (int s = 0; s < 32; ++s) x[s] = (s < a.n_splits && w[s] != 0.f) ? a.part_o[(s * stride + row) * a.Rc + r] : 0.f;
+#pragma unroll
+        for (int s = 0; s < 32; ++s) v = fmaf(x[s], w[s], v);
         reinterpret_cast<WT*>(a.out)[(size_t)row * a.Rc + r] = (WT)v;
     }
     pdl_launch_dependents();
@@ -313,8 +313,8 @@ int latent_attention(const LatentArgs& a, int f32, cudaStream_t s) {
     }
     if (rc) return rc;
     if (a.n_splits > 1) {
-        if (f32) DLP_CHECK_CUDA(launch_pdl(latent_combine_kernel<float>, dim3(a.T * a.H), dim3(128), 0, s, a));
-        else DLP_CHECK_CUDA(launch_pdl(latent_combine_kernel<__nv_bfloat16>, dim3(a.T * a.H), dim3(128), 0, s, a));
+        if (f32) DLP_CHECK_CUDA(launch_pdl(latent_combine_kernel<float>, dim3(a.T * a.H, (a.Rc + 127) / 128), dim3(128), 0, s, a));
+        else DLP_CHECK_CUDA(launch_pdl(latent_combine_kernel<__nv_bfloat16>, dim3(a.T * a.H, (a.Rc + 127) / 128), dim3(128), 0, s, a));
     }
     return 0;
 }

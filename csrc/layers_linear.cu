@@ -509,15 +509,20 @@ __global__ void __launch_bounds__(128) head_matmul_small_kernel(const void* x, i
     };
     load(warp * 32);                           // weights do not depend on the previous kernel
     pdl_wait();
-    for (int t = 0; t < T; ++t)
-        for (int k = threadIdx.x; k < Kp; k += 128) {
-            float v = 0.f;
-            if (k < kx) {
-                const size_t o = (size_t)t * ldx + (size_t)h * x_head + k;
-                v = x_f32 ? reinterpret_cast<const float*>(x)[o] : __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(x)[o]);
-            }
-            xs[t * ldxs + k] = __float2bfloat16_rn(v);
+    for (int i0 = threadIdx.x; i0 < T * Kp; i0 += 8 * 128) {      // eight loads in flight per thread
+        float v[8];
+#pragma unroll
+        for (int i = 0; i < 8; ++i) {
+            const int t = (i0 + i * 128) / Kp, k = (i0 + i * 128) - t * Kp;
+            const size_t o = (size_t)t * ldx + (size_t)h * x_head + k;
+            v[i] = (t < T && k < kx) ? (x_f32 ? reinterpret_cast<const float*>(x)[o] : __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(x)[o])) : 0.f;
         }
+#pragma unroll
+        for (int i = 0; i < 8; ++i) {
+            const int t = (i0 + i * 128) / Kp, k = (i0 + i * 128) - t * Kp;
+            if (t < T) xs[t * ldxs + k] = __float2bfloat16_rn(v[i]);
+        }
+    }
     __syncthreads();
     float acc[2][4] = {};
     for (int k0 = warp * 32; k0 < Kp; k0 += U * 128) {

@@ -316,7 +316,7 @@ class LayeredEngine(EngineCore):
         beside single tokens; want: for every entry the places among its tokens whose logits are returned (default: the last one).
         Returns fp32 logits [wanted, vocab] in the order of the entries.  A batch of single tokens is a decode step and runs as one
         (captured graph); more tokens than the engine's batch holds run as several forwards."""
-        entries = [(sid, [int(t) for t in toks]) for sid, toks in entries]
+        entries = [(sid, toks.tolist() if isinstance(toks, torch.Tensor) else list(toks)) for sid, toks in entries]
         if want is None:
             want = [[len(t) - 1] for _, t in entries]
         if len({sid for sid, _ in entries}) != len(entries) or any(not t for _, t in entries):
@@ -375,7 +375,7 @@ class LayeredEngine(EngineCore):
     @torch.no_grad()
     def prefill(self, sid: int, tokens, hidden_in=None, chunk: int | None = None, all_logits: bool = False):
         """Append `tokens` to one sequence; logits [vocab] of the last token, or [T, vocab] of all of them."""
-        toks = [int(t) for t in torch.as_tensor(tokens).tolist()]
+        toks = tokens.tolist() if isinstance(tokens, torch.Tensor) else list(tokens)
         chunk = min(chunk or len(toks), len(toks))
         outs = []
         for c0 in range(0, len(toks), chunk):

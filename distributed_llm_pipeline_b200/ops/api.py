@@ -28,7 +28,7 @@ launch_count = 0
 
 
 def _stream() -> int:
-    return torch.cuda.current_stream().cuda_stream
+    return torch._C._cuda_getCurrentRawStream(torch._C._cuda_getDevice())      # (the Stream object costs several times the launch wrapper)
 
 
 def _p(t: torch.Tensor | None) -> int:
