@@ -21,9 +21,11 @@ __device__ __forceinline__ KeyRange tile_keys(const LatentArgs& a, int row_last,
     return k;
 }
 
-template <int MW, int RMAX>
-__global__ void __launch_bounds__(256, 1) latent_attn_mma_kernel(const LatentArgs a) {
-    constexpr int BM = 16 * MW, BN = 64, NW = 8 / MW, KPW = BN / NW, LS = BN + 4;
+// MW: 16-row blocks of a tile; NWARP warps share a tile as MW x (NWARP / MW); BN keys per step.  (Four warps and 32-key steps, two blocks
+// to an SM, measured no faster for the 16- and 32-row decode tiles.)
+template <int MW, int NWARP, int BN, int RMAX>
+__global__ void __launch_bounds__(32 * NWARP, 1) latent_attn_mma_kernel(const LatentArgs a) {
+    constexpr int NTH = 32 * NWARP, BM = 16 * MW, NW = NWARP / MW, KPW = BN / NW, LS = BN + 4;
     constexpr int NPAIR = (RMAX / 16 + NW - 1) / NW;      // 16-column output blocks of a warp
     extern __shared__ __align__(16) uint8_t la_smem[];
     const int Rc = a.Rc, LD = Rc + 8;
@@ -50,8 +52,8 @@ __global__ void __launch_bounds__(256, 1) latent_attn_mma_kernel(const LatentArg
     };
     auto load_tile = [&](int b) {           // eight threads per latent row
 #pragma unroll
-        for (int half = 0; half < 2; ++half) {
-            const int kk = half * 32 + (tid >> 3), row = offs[b * BN + kk];
+        for (int part = 0; part < BN / (NTH / 8); ++part) {
+            const int kk = part * (NTH / 8) + (tid >> 3), row = offs[b * BN + kk];
             const __nv_bfloat16* src = cache + (size_t)max(row, 0) * Rc;
             __nv_bfloat16* dst = cs + ((size_t)b * BN + kk) * LD;
             for (int ch = tid & 7; ch < chunks; ch += 8) cp_async16(dst + ch * 8, src + ch * 8, row >= 0);
@@ -65,12 +67,12 @@ __global__ void __launch_bounds__(256, 1) latent_attn_mma_kernel(const LatentArg
     if (n_tiles > 0) load_tile(0);
     {
         const uint4* q = reinterpret_cast<const uint4*>(reinterpret_cast<const __nv_bfloat16*>(a.q) + (size_t)row0 * Rc);
-        for (int i = tid; i < BM * chunks; i += 256) {
+        for (int i = tid; i < BM * chunks; i += NTH) {
             const int r = i / chunks, ch = i - r * chunks;
             *reinterpret_cast<uint4*>(qs + r * LD + ch * 8) = r < rows ? q[(size_t)r * chunks + ch] : make_uint4(0, 0, 0, 0);
         }
     }
-    constexpr int TPR = 256 / BM;                          // softmax threads per row
+    constexpr int TPR = NTH / BM;                          // softmax threads per row
     const int sr = tid / TPR, sub = tid % TPR;
     const int my_pos = sr < rows ? a.pos[(row0 + sr) / a.H] : -1;
     float m_run = -INFINITY, l_run = 0.f;
@@ -285,15 +287,21 @@ __global__ void __launch_bounds__(128) latent_combine_kernel(const LatentArgs a)
     pdl_launch_dependents();
 }
 
-template <int MW, int RMAX>
+template <int MW, int NWARP, int BN, int RMAX>
 static int launch_latent_mma(const LatentArgs& a, cudaStream_t s) {
     constexpr int BM = 16 * MW;
-    const size_t smem = (size_t)(BM + 128) * (a.Rc + 8) * 2 + (size_t)BM * 68 * 4 + BM * 8 + 512;
+    const size_t smem = (size_t)(BM + 2 * BN) * (a.Rc + 8) * 2 + (size_t)BM * (BN + 4) * 4 + BM * 8 + 2 * BN * 4;
     DLP_REQUIRE(smem <= 227 * 1024, "latent_attention: %zu bytes of shared memory", smem);
-    auto kern = latent_attn_mma_kernel<MW, RMAX>;
+    auto kern = latent_attn_mma_kernel<MW, NWARP, BN, RMAX>;
     if (first_use_on_device((const void*)kern)) DLP_CHECK_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024));
-    DLP_CHECK_CUDA(launch_pdl(kern, dim3(a.n_tiles, a.n_splits), dim3(256), smem, s, a));
+    DLP_CHECK_CUDA(launch_pdl(kern, dim3(a.n_tiles, a.n_splits), dim3(32 * NWARP), smem, s, a));
     return 0;
+}
+template <int RMAX>
+static int launch_latent_tile(const LatentArgs& a, cudaStream_t s) {
+    if (a.bm == 16) return launch_latent_mma<1, 8, 64, RMAX>(a, s);
+    if (a.bm == 32) return launch_latent_mma<2, 8, 64, RMAX>(a, s);
+    return launch_latent_mma<4, 8, 64, RMAX>(a, s);
 }
 
 int latent_attention(const LatentArgs& a, int f32, cudaStream_t s) {
@@ -303,8 +311,7 @@ int latent_attention(const LatentArgs& a, int f32, cudaStream_t s) {
     int rc = 0;
     if (!f32 && a.Rc <= 512) {
         DLP_REQUIRE(a.bm == 16 || a.bm == 32 || a.bm == 64, "latent_attention: tile of %d rows", a.bm);
-        if (a.Rc <= 128) rc = a.bm == 16 ? launch_latent_mma<1, 128>(a, s) : a.bm == 32 ? launch_latent_mma<2, 128>(a, s) : launch_latent_mma<4, 128>(a, s);
-        else rc = a.bm == 16 ? launch_latent_mma<1, 512>(a, s) : a.bm == 32 ? launch_latent_mma<2, 512>(a, s) : launch_latent_mma<4, 512>(a, s);
+        rc = a.Rc <= 128 ? launch_latent_tile<128>(a, s) : launch_latent_tile<512>(a, s);
     } else {
         const size_t smem = (size_t)(2 * a.Rc + 64) * 4;
         DLP_REQUIRE(smem <= 48 * 1024, "latent_attention: latent of %d", a.Rc);

@@ -177,7 +177,7 @@ class LayeredEngine(EngineCore):
     # ---- matrix products -------------------------------------------------------------------------------
     def _product(self, r: Rows, w: Dense, out: torch.Tensor, T: int, geglu: bool = False) -> torch.Tensor:
         cfg = self.cfg
-        if T <= MATVEC_ROWS:
+        if T <= MATVEC_ROWS and lops.matvec_fits(T, w.t):
             st = lops.row_stage(r.x, r.K, w.Kp, cfg.rms_eps, r.y, r.w1, cfg.norm_groups, r.h_out, r.w2, r.groups2)
             return lops.matvec(st, w.t, out, T, geglu)
         x = r.x
@@ -191,7 +191,7 @@ class LayeredEngine(EngineCore):
         if pending is None:
             return Rows(self.hb[self.cur][:T], self.E)
         src = self.hb[self.cur][:T]
-        if T <= MATVEC_ROWS:        # every block of the mat-vec reads the old rows: the new ones go to the other buffer
+        if T <= MATVEC_ROWS:        # every block of a mat-vec reads the old rows: the new ones go to the other buffer
             self.cur ^= 1
         return Rows(src, self.E, y=self.y[:T], w1=pending, h_out=self.hb[self.cur][:T])
 

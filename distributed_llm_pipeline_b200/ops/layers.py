@@ -58,6 +58,11 @@ def row_stage(x: torch.Tensor, K: int, Kp: int, eps: float, y=None, w1=None, gro
                     h_out.stride(0) if h_out is not None else 0, _p(w2), groups2, w2.numel() if w2 is not None else 1, eps, K, Kp)
 
 
+def matvec_fits(T: int, w: torch.Tensor) -> bool:
+    """The staged rows and the partial sums fit the shared memory of one block (very wide fp32 rows do not)."""
+    return (T if T != 3 else 4) * w.shape[1] * w.element_size() <= 150 * 1024
+
+
 def matvec(st: RowStage, w: torch.Tensor, out: torch.Tensor, T: int, geglu: bool = False) -> torch.Tensor:
     """1..4 staged rows times w^T, w [N, ld] bf16 or fp32; out fp32 [T, N], or GEGLU of interleaved rows -> activation type [T, N/2]."""
     _need_cuda(w, "matvec")

@@ -297,7 +297,7 @@ def test_mixed_batches_and_reused_slots(models, name, dtype):
     """Eleven unequal requests through four slots and a pool that holds about two of the long ones, in random portions beside single tokens."""
     from distributed_llm_pipeline_b200.serving.trace_runner import TraceRunner
     cfg, w, path = models[name]
-    eng = engine(path, dtype, n_pages=40, max_batch_tokens=96)
+    eng = engine(path, dtype, n_pages=40, max_batch_tokens=200)
     run, g = TraceRunner(eng), torch.Generator().manual_seed(5)
     ids = {f"r{i}": lm.tokens(cfg, n, seed=i) for i, n in enumerate((200, 3, 120, 1, 64, 65, 180, 17, 16, 90, 31))}
     want = {k: plain.forward(cfg, w, v)[0] for k, v in ids.items()}
@@ -310,7 +310,7 @@ def test_mixed_batches_and_reused_slots(models, name, dtype):
             live.append(queue.pop(0))
         entries, rows = [], []
         for k in live:
-            n = [1, 1, 1, 2, 3, 16, 33, 70][int(torch.randint(0, 8, (1,), generator=g))]
+            n = [1, 1, 1, 2, 3, 16, 33, 70, 150][int(torch.randint(0, 9, (1,), generator=g))]
             n = min(n, len(ids[k]) - at[k])
             entries.append({"id": k, "tokens": ids[k][at[k]:at[k] + n], "want": list(range(n))})
             rows.append(want[k][at[k]:at[k] + n])
