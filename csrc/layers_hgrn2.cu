@@ -258,12 +258,14 @@ __global__ void __launch_bounds__(4 * DP, 1) hgrn2_chunk_out_kernel(const Hgrn2A
         s4[j] = (s_vec && dd < a.D && v0 + v < a.V) ? *reinterpret_cast<const float4*>(S + (size_t)dd * a.V + v0 + v) : make_float4(0.f, 0.f, 0.f, 0.f);
     }
     {   // diagonal blocks: thread (key token s, channel group) runs over the queries of the block
-        const int s = tid / C::PARTS, part = tid % C::PARTS, b0 = s & ~15;
+        // (a warp starts at its first key; the starts are spread evenly over the SM's four schedulers)
+        constexpr int JPW = 32 / C::PARTS, WPB = 16 / JPW;          // keys of a warp, warps of a block
+        const int b0 = warp / WPB * 16, s0 = b0 + (warp + warp / 4) % WPB * JPW, s = s0 + lane / C::PARTS, part = lane % C::PARTS;
         float w[C::CPP];
 #pragma unroll
         for (int i = 0; i < C::CPP; ++i) w[i] = sk[s * LDF + diag_piece(part, i >> 2) + (i & 3)];
 #pragma unroll 2
-        for (int t = b0; t < b0 + 16; ++t) {
+        for (int t = s0; t < b0 + 16; ++t) {
             float acc = 0.f;
             const bool later = t > s;
 #pragma unroll
@@ -334,7 +336,7 @@ __global__ void __launch_bounds__(4 * DP, 1) hgrn2_chunk_out_kernel(const Hgrn2A
         }
     }
     __syncthreads();
-    const int mt = warp & 3, cg = warp >> 2;
+    const int mt = (warp + (warp >> 2)) & 3, cg = warp >> 2;
     float acc[NP][2][4] = {};
 #pragma unroll 2
     for (int ks = 0; ks < DP / 16; ++ks) {

@@ -12,7 +12,6 @@ PP activation hand-off (see parallel/).
 """
 from __future__ import annotations
 
-import math
 import os
 
 import torch

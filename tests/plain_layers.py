@@ -5,10 +5,6 @@ complete sequence of one request and returns a value per token.
 """
 from __future__ import annotations
 
-import json
-import os
-import struct
-
 import torch
 
 F = torch.float64
