@@ -70,7 +70,7 @@ __host__ __device__ constexpr uint32_t make_idesc_f16_bmn(int m, int n, int fmt)
 
 struct FaParams {
     const int* bt_row;      // FA_PAGED: block-table row of the sequence
-    void* out;              // [T, ldo] fp16 (FA_PAGED) or bf16 (FA_ROWS)
+    void* out;              // [T, ldo] fp16 (FA_PAGED) or bf16
     int T, pos0, Hq, Hkv, page_size, max_pages;
     int ldo;
     // FA_ROWS
@@ -78,11 +78,21 @@ struct FaParams {
     int ldg, V;             // V: value size of a head (<= D2; the rest of the tile is padding)
     float scale;
     int* error;             // set when a wait ran into its limit
+    // FA_TILES
+    const int* tile_row0;   // [grid.x] first query row of a tile, and its rows (consecutive positions of one sequence)
+    const int* tile_rows;
+    const int* pos;         // [T]
+    const int* tok_slot;    // [T] block-table row
+    const int* block_table;
+    int q_head;             // columns from one query head to the next
+    int window, keep;       // position i sees key j <= i when i - j < window or j < keep
 };
 // FA_PAGED: fp16, K / V pages of a [pages][Hkv][page][D] cache, queries scaled in advance, fp16 softmax weights
 // FA_ROWS:  bf16, K / V as plain rows [keys][Hkv * D1 | D2], scores scaled in fp32, every softmax weight as two bf16 parts (value and
 //           remainder, two MMAs), optional output gate
-enum FaMode : int { FA_PAGED = 0, FA_ROWS = 1 };
+// FA_TILES: bf16 with the numerics of FA_ROWS, K / V pages of [pages][Hkv][page][<= D1 | <= D2] caches (tensor maps complete narrower heads
+//           with zeros), tiles of several sequences, sliding window with kept first keys: only key tiles that some row sees are read
+enum FaMode : int { FA_PAGED = 0, FA_ROWS = 1, FA_TILES = 2 };
 
 template <int D1, int D2, int MODE>
 struct FaCfg {
@@ -90,7 +100,7 @@ struct FaCfg {
     static constexpr int KB = D1 / 64, VB = D2 / 64;
     static constexpr int Q_BYTES = BM * D1 * 2;
     static constexpr int K_BYTES = BN * D1 * 2, V_BYTES = BN * D2 * 2;
-    static constexpr int P_PARTS = MODE == FA_ROWS ? 2 : 1;
+    static constexpr int P_PARTS = MODE == FA_PAGED ? 1 : 2;
     static constexpr int P_BYTES = BM * BN * 2;      // one part
     static constexpr int STAGES = 2;
     static constexpr int SMEM_BYTES = Q_BYTES + STAGES * (K_BYTES + V_BYTES) + P_PARTS * P_BYTES + 1024 + 256;
@@ -103,7 +113,8 @@ __global__ void __launch_bounds__(192, 1)
 attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_k,
                        const __grid_constant__ CUtensorMap tm_v, const FaParams p) {
     using Cfg = FaCfg<D1, D2, MODE>;
-    constexpr int BM = Cfg::BM, BN = Cfg::BN, KB = Cfg::KB, VB = Cfg::VB, FMT = MODE == FA_ROWS ? 1 : 0;
+    constexpr int BM = Cfg::BM, BN = Cfg::BN, KB = Cfg::KB, VB = Cfg::VB, FMT = MODE == FA_PAGED ? 0 : 1;
+    constexpr bool EXACT = MODE != FA_PAGED;                     // fp32 scores times scale, split softmax weights
     extern __shared__ uint8_t smem_raw[];
     uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
     uint8_t* sm_q = smem;                                        // [KB][128 rows][128 B]
@@ -123,12 +134,18 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_co
     uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 15);
 
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int qt = gridDim.x - 1 - blockIdx.x;        // heaviest (latest) query tiles first
-    const int t0 = qt * BM;
+    const int qt = gridDim.x - 1 - blockIdx.x;        // heaviest (latest) query tiles first (FA_TILES: in the order of the table)
+    const int t0 = MODE == FA_TILES ? p.tile_row0[blockIdx.x] : qt * BM;
+    const int rows = MODE == FA_TILES ? p.tile_rows[blockIdx.x] : min(BM, p.T - t0);
+    const int pos_t = MODE == FA_TILES ? p.pos[t0] : p.pos0 + t0;      // position of the first row
+    const int* bt_row = MODE == FA_TILES ? p.block_table + (size_t)p.tok_slot[t0] * p.max_pages : p.bt_row;
     const int hq = blockIdx.y;
     const int kvh = hq / (p.Hq / p.Hkv);
-    const int q_hi = p.pos0 + min(p.T, t0 + BM);      // keys visible to the last query of this tile
-    const int n_tiles = (q_hi + BN - 1) / BN;
+    const int q_hi = pos_t + rows;                    // keys visible to the last query of this tile
+    const int lo_tile = MODE == FA_TILES ? max(0, pos_t - p.window + 1) / BN : 0;            // first key tile the window shows
+    const int keep_tiles = MODE == FA_TILES ? min((p.keep + BN - 1) / BN, lo_tile) : 0;      // kept tiles in front of it
+    const int n_tiles = keep_tiles + (q_hi + BN - 1) / BN - lo_tile;
+    auto key_of = [&](int i) { return (MODE == FA_TILES && i >= keep_tiles ? lo_tile - keep_tiles + i : i) * BN; };
 
     if (warp == 0 && lane == 0) {
         tma_prefetch_desc(&tm_q);
@@ -160,16 +177,16 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_co
         // ===== producer =====
         if (lane == 0) {
             mbar_expect_tx(q_full, Cfg::Q_BYTES);
-            for (int kb = 0; kb < KB; ++kb) tma_load_2d(sm_q + kb * (BM * 128), &tm_q, q_full, hq * D1 + kb * 64, t0);
-            const int ps = MODE == FA_PAGED ? p.page_size : BN, chunks = BN / ps;
+            for (int kb = 0; kb < KB; ++kb) tma_load_2d(sm_q + kb * (BM * 128), &tm_q, q_full, hq * (MODE == FA_TILES ? p.q_head : D1) + kb * 64, t0);
+            const int ps = MODE == FA_ROWS ? BN : p.page_size, chunks = BN / ps;
             for (int i = 0; i < n_tiles; ++i) {
                 const int s = i & 1;
                 const uint32_t ph = (uint32_t)(i >> 1) & 1u;
-                const int n0 = i * BN;
+                const int n0 = key_of(i);
                 auto row_of = [&](int pc) {
                     if (MODE == FA_ROWS) return n0;
                     const int pi = min((n0 + pc * ps) / ps, p.max_pages - 1);
-                    return (p.bt_row[pi] * p.Hkv + kvh) * ps;
+                    return (bt_row[pi] * p.Hkv + kvh) * ps;
                 };
                 mbar_wait_g(&k_empty[s], ph ^ 1, p.error);
                 mbar_expect_tx(&k_full[s], Cfg::K_BYTES);
@@ -234,7 +251,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_co
         // ===== softmax / correction / epilogue: thread r <-> query row r =====
         const int q4 = warp & 3;                       // TMEM lane quarter this warp may access
         const int r = q4 * 32 + lane;
-        const int q_pos = p.pos0 + t0 + r;             // this query attends to keys 0 .. q_pos
+        const int q_pos = pos_t + r;                   // this query attends to keys 0 .. q_pos
         const uint32_t lane_addr = tmem_base + ((uint32_t)(q4 * 32) << 16);
         constexpr float LOG2E = 1.4426950408889634f;
         float m_run = -INFINITY, l_run = 0.f;
@@ -242,7 +259,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_co
         const int sw = r & 7;
         for (int i = 0; i < n_tiles; ++i) {
             const int s = i & 1;
-            const int n0 = i * BN;
+            const int n0 = key_of(i);
             mbar_wait_g(&s_full[s], (uint32_t)(i >> 1) & 1u, p.error);
             tc_fence_after();
             uint32_t sv[BN];
@@ -253,12 +270,12 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_co
             __syncwarp();
             if (lane == 0) mbar_arrive(&s_free[s]);    // the next-but-one score tile may overwrite this buffer
             float mx = m_run;
-            const bool diag = n0 + BN - 1 > p.pos0 + t0;          // some (query, key) pairs of this tile are masked
+            const bool diag = n0 + BN - 1 > pos_t || (MODE == FA_TILES && q_hi - 1 - n0 >= p.window && n0 + BN > p.keep);     // some (query, key) pairs of this tile are masked
 #pragma unroll
             for (int j = 0; j < BN; ++j) {
                 float v = __uint_as_float(sv[j]);
-                if (MODE == FA_ROWS) v *= p.scale;
-                if (diag && n0 + j > q_pos) v = -INFINITY;
+                if (EXACT) v *= p.scale;
+                if (diag && (n0 + j > q_pos || (MODE == FA_TILES && q_pos - (n0 + j) >= p.window && n0 + j >= p.keep))) v = -INFINITY;
                 sv[j] = __float_as_uint(v);
                 mx = fmaxf(mx, v);
             }
@@ -271,7 +288,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_co
             for (int j = 0; j < BN; j += 2) {
                 const float p0 = exp2f(__uint_as_float(sv[j]) * LOG2E - ms);
                 const float p1 = exp2f(__uint_as_float(sv[j + 1]) * LOG2E - ms);
-                if (MODE == FA_ROWS) {
+                if (EXACT) {
                     sum += p0 + p1;
                     sv[j] = __float_as_uint(p0);
                     sv[j + 1] = __float_as_uint(p1);
@@ -306,7 +323,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_co
 #pragma unroll
                 for (int c = 0; c < 8; ++c) {
                     uint8_t* dst = prow + b * (BM * 128) + ((c ^ sw) << 4);
-                    if (MODE == FA_ROWS) {
+                    if (EXACT) {
                         uint32_t hi[4], lo[4];
 #pragma unroll
                         for (int e = 0; e < 4; ++e) split_bf16(__uint_as_float(sv[b * 64 + c * 8 + 2 * e]), __uint_as_float(sv[b * 64 + c * 8 + 2 * e + 1]), hi[e], lo[e]);
@@ -332,11 +349,11 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_co
             uint32_t o[32];
             tmem_ld_32x32(lane_addr + Cfg::O_COL + c * 32, o);
             tc_wait_ld();
-            if (MODE == FA_ROWS) {
+            if (EXACT) {
                 __nv_bfloat16* orow = reinterpret_cast<__nv_bfloat16*>(p.out) + (size_t)t * p.ldo + (size_t)hq * p.V;
 #pragma unroll
                 for (int j = 0; j < 32; ++j)
-                    if (t < p.T && c * 32 + j < p.V) orow[c * 32 + j] = __float2bfloat16_rn(__uint_as_float(o[j]) * inv);
+                    if (r < rows && c * 32 + j < p.V) orow[c * 32 + j] = __float2bfloat16_rn(__uint_as_float(o[j]) * inv);
             } else if (t < p.T) {
                 __half* orow = reinterpret_cast<__half*>(p.out) + (size_t)t * p.ldo + (size_t)hq * D2;
 #pragma unroll

@@ -11,7 +11,7 @@ FLAGS=(-gencode arch=compute_100a,code=sm_100a -O3 -lineinfo -std=c++17 -Xcompil
 case "$PART" in
   all) OBJ="$HERE/build"; LIB="$OUT/libdlp_b200.so"; SRC=("$HERE"/*.cu) ;;
   layers) OBJ="$HERE/build/layers"; LIB="$OUT/libdlp_b200_layers.so"; FLAGS+=(-DDLP_LAYERS_ONLY)
-          SRC=("$HERE"/layers_*.cu "$HERE"/capi_layers.cu "$HERE"/capi_core.cu "$HERE"/elementwise.cu "$HERE"/gemm_tcgen05.cu) ;;
+          SRC=("$HERE"/layers_*.cu "$HERE"/capi_layers.cu "$HERE"/capi_core.cu "$HERE"/elementwise.cu "$HERE"/gemm_tcgen05.cu "$HERE"/moe.cu) ;;
   *) echo "build.sh: unknown part '$PART'" >&2; exit 2 ;;
 esac
 mkdir -p "$OBJ" "$OUT"
@@ -21,7 +21,7 @@ for f in "${SRC[@]}"; do
   b="$(basename "$f" .cu)"
   objs+=("$OBJ/$b.o")
   MATH=(--use_fast_math)
-  case "$b" in layers_attention_tc) ;; layers_*) MATH=() ;; esac        # exact divisions, square roots and exponentials where a layer is specified in 32 bits
+  case "$b" in layers_*_tc) ;; layers_*) MATH=() ;; esac        # exact divisions, square roots and exponentials where a layer is specified in 32 bits
   if [[ ! -f "$OBJ/$b.o" || "$f" -nt "$OBJ/$b.o" || -n "$(find "$HERE" -maxdepth 1 -name '*.cuh' -newer "$OBJ/$b.o" -print -quit)" || "$HERE/../include/dlp_b200.h" -nt "$OBJ/$b.o" ]]; then
     ( "$NVCC" "${FLAGS[@]}" ${MATH[@]+"${MATH[@]}"} -c "$f" -o "$OBJ/$b.o.tmp" > "$OBJ/$b.log" 2>&1 && mv "$OBJ/$b.o.tmp" "$OBJ/$b.o" || { cat "$OBJ/$b.log"; exit 1; } ) &
     pids+=($!)

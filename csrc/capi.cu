@@ -182,18 +182,9 @@ int dlp_moe_route_ex(const float* logits, int ld, int T, int n_expert, int top_k
     DLP_REQUIRE(logits && ids && weights && T > 0 && ld >= n_expert, "dlp_moe_route_ex: bad argument");
     return moe_route_ex(logits, ld, T, n_expert, top_k, renorm, ids, weights, (cudaStream_t)stream);
 }
-int dlp_moe_plan(const int32_t* ids, int n_assign, int n_expert, int token_tile, dlp_moe_plan_bufs* b, void* stream) {
-    DLP_REQUIRE(ids && b && b->pos && b->src && b->bounds && b->tile_expert && b->tile_row0 && b->tile_rows && b->n_tiles, "dlp_moe_plan: null argument");
-    return moe_plan(ids, n_assign, n_expert, token_tile, b->pos, b->src, b->bounds, b->tile_expert, b->tile_row0, b->tile_rows, b->n_tiles,
-                    (cudaStream_t)stream);
-}
-int dlp_moe_gather(const void* x, int ldx, const int32_t* src, int top_k, int n_assign, int K, void* xs, void* stream) {
-    DLP_REQUIRE(x && src && xs && n_assign > 0, "dlp_moe_gather: bad argument");
-    return moe_gather((const __half*)x, ldx, src, top_k, n_assign, K, (__half*)xs, (cudaStream_t)stream);
-}
 int dlp_moe_combine(const float* y, const int32_t* pos, const float* weights, int T, int top_k, int E, float* h, void* stream) {
     DLP_REQUIRE(y && pos && weights && h, "dlp_moe_combine: null argument");
-    return moe_combine(y, pos, weights, T, top_k, E, h, (cudaStream_t)stream);
+    return moe_combine(y, pos, weights, T, top_k, E, h, (cudaStream_t)stream, E, 1);
 }
 int dlp_linear_grouped(const dlp_weight* w0, const dlp_weight* w1, const void* xs, void* y, int ldy, int out_mode, int n_assign, int n_expert,
                        int rows_per_expert, int token_tile, const dlp_moe_plan_bufs* b, void* ws, size_t ws_bytes, void* stream) {

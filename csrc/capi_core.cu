@@ -1,5 +1,5 @@
 // The part of the C surface every build of the library has: error plumbing, device facts, step bookkeeping, sampling, the dense
-// tcgen05 GEMM (declarations: include/dlp_b200.h).
+// tcgen05 GEMM, the routing plan of expert layers (declarations: include/dlp_b200.h).
 #include <stdarg.h>
 #include <stdlib.h>
 #include <string.h>
@@ -93,5 +93,14 @@ int dlp_sample_dev(const float* logits, int R, int V, int ld, dlp_sample_params*
     DLP_REQUIRE(logits && out && params, "dlp_sample_dev: null argument");
     static_assert(sizeof(dlp_sample_params) == sizeof(SampleParams), "sampler record layout");
     return sample_dev(logits, R, V, ld, reinterpret_cast<SampleParams*>(params), row_slot, out, (cudaStream_t)stream);
+}
+int dlp_moe_plan(const int32_t* ids, int n_assign, int n_expert, int token_tile, dlp_moe_plan_bufs* b, void* stream) {
+    DLP_REQUIRE(ids && b && b->pos && b->src && b->bounds && b->tile_expert && b->tile_row0 && b->tile_rows && b->n_tiles, "dlp_moe_plan: null argument");
+    return moe_plan(ids, n_assign, n_expert, token_tile, b->pos, b->src, b->bounds, b->tile_expert, b->tile_row0, b->tile_rows, b->n_tiles,
+                    (cudaStream_t)stream);
+}
+int dlp_moe_gather(const void* x, int ldx, const int32_t* src, int top_k, int n_assign, int K, void* xs, void* stream) {
+    DLP_REQUIRE(x && src && xs && n_assign > 0, "dlp_moe_gather: bad argument");
+    return moe_gather((const __half*)x, ldx, src, top_k, n_assign, K, (__half*)xs, (cudaStream_t)stream);
 }
 }  // extern "C"

@@ -7,7 +7,8 @@
 
 using namespace dlp;
 
-static_assert(sizeof(dlp_row_stage) == sizeof(RowStage) && sizeof(dlp_hgrn2_args) == sizeof(Hgrn2Args) && sizeof(dlp_hgrn2_chunks) == sizeof(Hgrn2Chunks) && sizeof(dlp_latent_args) == sizeof(LatentArgs), "argument layout");
+static_assert(sizeof(dlp_row_stage) == sizeof(RowStage) && sizeof(dlp_hgrn2_args) == sizeof(Hgrn2Args) && sizeof(dlp_hgrn2_chunks) == sizeof(Hgrn2Chunks) && sizeof(dlp_latent_args) == sizeof(LatentArgs) &&
+              sizeof(dlp_expert_args) == sizeof(ExpertArgs) && sizeof(dlp_gqa_args) == sizeof(GqaArgs), "argument layout");
 
 extern "C" {
 
@@ -56,6 +57,42 @@ int dlp_layers_head_rows(const float* x, int ldx, int D, int Dp, int H, void* ou
 int dlp_layers_rows_attention(const void* q, const void* kv, int ldkv, int S, int T, int pos0, int H, int Dp, int Vp, int V, float scale, const float* gate, int ldg,
                               void* out, int ldo, void* stream) {
     return rows_attention(q, kv, ldkv, S, T, pos0, H, Dp, Vp, V, scale, gate, ldg, out, ldo, (cudaStream_t)stream);
+}
+int dlp_layers_route(const float* logits, int ld, const float* bias, int n_expert, int top, int32_t* ids, float* weights, int T, void* stream) {
+    return route(logits, ld, bias, n_expert, top, ids, weights, T, (cudaStream_t)stream);
+}
+int dlp_layers_expert_matvec(const dlp_row_stage* st, const dlp_expert_args* a, void* out, int ldo, int down, int T, int f32, void* stream) {
+    DLP_REQUIRE(st && a, "dlp_layers_expert_matvec: null argument");
+    return expert_matvec(*reinterpret_cast<const RowStage*>(st), *reinterpret_cast<const ExpertArgs*>(a), out, ldo, down, T, f32, (cudaStream_t)stream);
+}
+int dlp_layers_linear_grouped(const void* xs, int ldx, const void* w, int ldw, int rows_per_expert, int K, void* out, int ldo, int out_mode, int n_assign, int n_expert,
+                              int token_tile, const dlp_moe_plan_bufs* b, int f32, void* ws, size_t ws_bytes, void* stream) {
+    DLP_REQUIRE(xs && w && out && b && b->tile_expert && n_assign > 0 && n_expert > 0 && rows_per_expert > 0 && token_tile > 0, "dlp_layers_linear_grouped: bad argument");
+    DLP_REQUIRE(out_mode == LO_F32 || out_mode == LO_RELU2, "dlp_layers_linear_grouped: output mode %d", out_mode);
+    GemmGroup g;
+    g.tile_expert = b->tile_expert; g.tile_row0 = b->tile_row0; g.tile_rows = b->tile_rows; g.n_tiles = b->n_tiles;
+    g.rows_per_expert = rows_per_expert; g.n_expert = n_expert; g.bt = token_tile;
+    const int most = (n_assign + token_tile - 1) / token_tile + n_expert;      // every expert may end with one partial tile,
+    g.max_tiles = most < n_assign ? most : n_assign;                           // and a tile holds at least one row
+    if (f32) return sgemm((const float*)xs, ldx, (const float*)w, ldw, rows_per_expert, K, out, ldo, out_mode, n_assign, (cudaStream_t)stream, &g);
+    return gemm_f16(w, nullptr, ldw, xs, ldx, out, ldo, n_assign, rows_per_expert, K, out_mode == LO_RELU2 ? 7 : 1, 1, ws ? 0 : 1, (cudaStream_t)stream, nullptr, &g, ws,
+                    ws_bytes);
+}
+int dlp_layers_combine(const float* y, int ldy, const int32_t* pos, const float* weights, int T, int top, int E, float* out, void* stream) {
+    DLP_REQUIRE(y && pos && weights && out && top > 0, "dlp_layers_combine: bad argument");
+    return moe_combine(y, pos, weights, T, top, E, out, (cudaStream_t)stream, ldy, 0);
+}
+int dlp_layers_gqa_prepare(const dlp_gqa_args* a, int f32, void* stream) {
+    DLP_REQUIRE(a, "dlp_layers_gqa_prepare: null argument");
+    return gqa_prepare(*reinterpret_cast<const GqaArgs*>(a), f32, (cudaStream_t)stream);
+}
+int dlp_layers_gqa_attention(const dlp_gqa_args* a, int fused, int f32, void* stream) {
+    DLP_REQUIRE(a, "dlp_layers_gqa_attention: null argument");
+    return gqa_attention(*reinterpret_cast<const GqaArgs*>(a), fused, f32, (cudaStream_t)stream);
+}
+int dlp_layers_gqa_flash(const dlp_gqa_args* a, void* stream) {
+    DLP_REQUIRE(a, "dlp_layers_gqa_flash: null argument");
+    return gqa_flash(*reinterpret_cast<const GqaArgs*>(a), (cudaStream_t)stream);
 }
 int dlp_layers_rows_attention_error(int* flag) { return rows_attention_error(flag); }
 

@@ -7,6 +7,13 @@ namespace dlp {
 
 __device__ int g_rows_error;     // a wait of the flash kernel ran into its limit since the library was loaded
 
+int* flash_error_flag() {
+    int* p = nullptr;
+    const cudaError_t e = cudaGetSymbolAddress((void**)&p, g_rows_error);
+    if (e != cudaSuccess) set_error("flash_error_flag: %s", cudaGetErrorString(e));
+    return e == cudaSuccess ? p : nullptr;
+}
+
 // latent rows 0 .. S-1 of one request, out of its pages
 __global__ void __launch_bounds__(128) latent_gather_kernel(const uint4* cache, const int* bt, int page, int chunks, uint4* out) {
     pdl_wait();
@@ -60,7 +67,7 @@ int rows_attention(const void* q, const void* kv, int ldkv, int S, int T, int po
     FaParams p;
     memset(&p, 0, sizeof(p));
     p.out = out; p.T = T; p.pos0 = pos0; p.Hq = H; p.Hkv = H; p.page_size = 128; p.max_pages = 1; p.ldo = ldo; p.gate = gate; p.ldg = ldg; p.V = V; p.scale = scale;
-    DLP_CHECK_CUDA(cudaGetSymbolAddress((void**)&p.error, g_rows_error));
+    if ((p.error = flash_error_flag()) == nullptr) return -1;
     const void* v = (const uint8_t*)kv + (size_t)H * Dp * 2;
     if (Dp == 64 && Vp == 64) return launch_rows<64, 64>(q, kv, v, ldkv, S, p, s);
     if (Dp == 64 && Vp == 128) return launch_rows<64, 128>(q, kv, v, ldkv, S, p, s);
@@ -68,7 +75,7 @@ int rows_attention(const void* q, const void* kv, int ldkv, int S, int T, int po
     if (Dp == 128 && Vp == 128) return launch_rows<128, 128>(q, kv, v, ldkv, S, p, s);
     DLP_REQUIRE(false, "rows_attention: head sizes %d / %d", Dp, Vp);
 }
-// 0, or 1 when a wait of the kernel above gave up since the last call (synchronises)
+// 0, or 1 when a wait of a flash kernel gave up since the last call (synchronises)
 int rows_attention_error(int* flag) {
     DLP_CHECK_CUDA(cudaMemcpyFromSymbol(flag, g_rows_error, sizeof(int)));
     if (*flag) {

@@ -5,183 +5,13 @@
 //   stage_rows_kernel    the same row preparation as one launch, for the tcgen05 GEMM sizes.
 //   sgemm_kernel         fp32 storage, any number of rows (no reduced-precision product).
 //   head_matmul_kernel   one small matrix per head (latent attention's key absorption and value expansion), mma.sync m16n8k16.
-#include "layers.cuh"
+#include "layers_rows.cuh"
 #include "mma.cuh"
 
 namespace dlp {
 
-template <typename T> struct Act;
-template <> struct Act<__nv_bfloat16> {
-    static constexpr int VEC = 8;
-    static __device__ __forceinline__ float to_f(__nv_bfloat16 v) { return __bfloat162float(v); }
-    static __device__ __forceinline__ __nv_bfloat16 from_f(float v) { return __float2bfloat16_rn(v); }
-};
-template <> struct Act<float> {
-    static constexpr int VEC = 4;
-    static __device__ __forceinline__ float to_f(float v) { return v; }
-    static __device__ __forceinline__ float from_f(float v) { return v; }
-};
-
 __device__ __forceinline__ float gelu_tanh_f(float z) {
     return 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
-}
-
-// ---- row preparation ------------------------------------------------------------------------------------
-// NT rows starting at t0, all threads of the block.  `put(t, k, v)` receives every value of the padded row.  `sums` holds
-// stage_scratch(NT, groups) floats; ends with a barrier.
-__host__ __device__ inline int stage_parts(int rows, int groups, int nwarps) {
-    const int tg = rows * groups;
-    return tg >= nwarps ? 1 : (nwarps + tg - 1) / tg;
-}
-__host__ __device__ inline int stage_scratch(int rows, int groups, int nwarps) { return rows * groups * (stage_parts(rows, groups, nwarps) + 1); }
-
-template <typename XT>
-__device__ __forceinline__ float stage_x0(const RowStage& p, int t, int k) {
-    return p.x_f32 ? reinterpret_cast<const float*>(p.x)[(size_t)t * p.ldx + k] : Act<XT>::to_f(reinterpret_cast<const XT*>(p.x)[(size_t)t * p.ldx + k]);
-}
-
-// reciprocal root mean square of every (row, group) of f(t, k) -> sums[rows * groups * parts + t * groups + g]; returns that base
-template <typename F>
-__device__ __forceinline__ float* stage_rms(int rows, int groups, int K, float eps, float* sums, F f) {
-    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5;
-    const int parts = stage_parts(rows, groups, nw), gs = K / groups, per = ((gs + parts - 1) / parts + 31) / 32 * 32;
-    for (int i = warp; i < rows * groups * parts; i += nw) {
-        const int tg = i / parts, part = i - tg * parts, t = tg / groups, g = tg - t * groups;
-        const int lo = part * per, hi = min(gs, lo + per);
-        float a = 0.f;
-#pragma unroll 4
-        for (int k = lo + lane; k < hi; k += 32) {
-            const float v = f(t, g * gs + k);
-            a = fmaf(v, v, a);
-        }
-        a = warp_sum(a);
-        if (lane == 0) sums[i] = a;
-    }
-    __syncthreads();
-    float* rs = sums + rows * groups * parts;
-    for (int i = threadIdx.x; i < rows * groups; i += blockDim.x) {
-        float a = 0.f;
-        for (int j = 0; j < parts; ++j) a += sums[i * parts + j];
-        rs[i] = 1.f / sqrtf(a / (float)gs + eps);
-    }
-    __syncthreads();
-    return rs;
-}
-
-// Vector form: rows in slices of 128 values, one warp per slice and pass; groups are whole slices.
-__host__ __device__ inline bool stage_vec(const RowStage& p) {
-    return p.K % 128 == 0 && p.Kp == p.K && p.ldx % 8 == 0 && (!p.y || ((p.K / p.groups1) % 128 == 0 && p.ldy % 4 == 0 && p.ldh % 4 == 0)) &&
-           (!p.w2 || ((p.K / p.groups2) % 128 == 0 && p.w2_mod % 128 == 0));
-}
-template <typename F>
-__device__ __forceinline__ float* stage_rms_vec(int rows, int groups, int K, float eps, float* sums, F f) {
-    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5, spr = K >> 7, n = rows * spr;
-#pragma unroll 4
-    for (int i = warp; i < n; i += nw) {
-        const int t = i / spr;
-        const float4 v = f(t, (i - t * spr) * 128 + lane * 4);
-        const float a = warp_sum(fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, v.w * v.w))));
-        if (lane == 0) sums[i] = a;
-    }
-    __syncthreads();
-    float* rs = sums + n;
-    const int gs = K / groups, per = gs >> 7;
-    for (int i = threadIdx.x; i < rows * groups; i += blockDim.x) {
-        float a = 0.f;
-        for (int j = 0; j < per; ++j) a += sums[i * per + j];
-        rs[i] = 1.f / sqrtf(a / (float)gs + eps);
-    }
-    __syncthreads();
-    return rs;
-}
-template <typename XT>
-__device__ __forceinline__ float4 stage_x4(const RowStage& p, int t, int k) {
-    if (p.x_f32) return *reinterpret_cast<const float4*>(reinterpret_cast<const float*>(p.x) + (size_t)t * p.ldx + k);
-    if (sizeof(XT) == 4) return *reinterpret_cast<const float4*>(reinterpret_cast<const float*>(p.x) + (size_t)t * p.ldx + k);
-    const uint2 u = *reinterpret_cast<const uint2*>(reinterpret_cast<const __nv_bfloat16*>(p.x) + (size_t)t * p.ldx + k);
-    const float2 a = bf2_to_f2(u.x), b = bf2_to_f2(u.y);
-    return make_float4(a.x, a.y, b.x, b.y);
-}
-template <typename XT, typename Put4>
-__device__ __forceinline__ void stage_rows_vec(const RowStage& p, int t0, int rows, float* sums, bool store_h, Put4 put) {
-    const float* rs1 = nullptr;
-    const float* rs2 = nullptr;
-    const int gs1 = p.y ? p.K / p.groups1 : 1, gs2 = p.w2 ? p.K / p.groups2 : 1;
-    auto y4 = [&](int t, int k) { return *reinterpret_cast<const float4*>(p.y + (size_t)(t0 + t) * p.ldy + k); };
-    if (p.y) {
-        rs1 = stage_rms_vec(rows, p.groups1, p.K, p.eps, sums, y4);
-        sums += rows * (p.K / 128 + p.groups1);
-    }
-    auto base = [&](int t, int k) {
-        float4 v = stage_x4<XT>(p, t0 + t, k);
-        if (p.y) {
-            const float4 y = y4(t, k), w = *reinterpret_cast<const float4*>(p.w1 + k);
-            const float r = rs1[t * p.groups1 + k / gs1];
-            v.x = fmaf(y.x * r, w.x, v.x);
-            v.y = fmaf(y.y * r, w.y, v.y);
-            v.z = fmaf(y.z * r, w.z, v.z);
-            v.w = fmaf(y.w * r, w.w, v.w);
-        }
-        return v;
-    };
-    if (p.w2) rs2 = stage_rms_vec(rows, p.groups2, p.K, p.eps, sums, base);
-    const int q = p.K >> 2;
-#pragma unroll 2
-    for (int i = threadIdx.x; i < rows * q; i += blockDim.x) {
-        const int t = i / q, k = (i - t * q) * 4;
-        float4 v = base(t, k);
-        if (store_h && p.h_out) *reinterpret_cast<float4*>(p.h_out + (size_t)(t0 + t) * p.ldh + k) = v;
-        if (p.w2) {
-            const float r = rs2[t * p.groups2 + k / gs2];
-            const float4 w = *reinterpret_cast<const float4*>(p.w2 + k % p.w2_mod);
-            v = make_float4(v.x * r * w.x, v.y * r * w.y, v.z * r * w.z, v.w * r * w.w);
-        }
-        put(t, k, v);
-    }
-    __syncthreads();
-}
-__device__ __forceinline__ void put4(__nv_bfloat16* d, float4 v) {
-    __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
-    *reinterpret_cast<uint2*>(d) = make_uint2(*reinterpret_cast<uint32_t*>(&a), *reinterpret_cast<uint32_t*>(&b));
-}
-__device__ __forceinline__ void put4(float* d, float4 v) { *reinterpret_cast<float4*>(d) = v; }
-
-template <typename XT>
-__device__ __forceinline__ void stage_rows_dev(const RowStage& p, int t0, int rows, float* sums, bool store_h, XT* dst, int ldd) {
-    if (stage_vec(p)) {
-        stage_rows_vec<XT>(p, t0, rows, sums, store_h, [&](int t, int k, float4 v) { put4(dst + (size_t)t * ldd + k, v); });
-        return;
-    }
-    const float* rs1 = nullptr;
-    const float* rs2 = nullptr;
-    const int gs1 = p.y ? p.K / p.groups1 : 1, gs2 = p.w2 ? p.K / p.groups2 : 1;
-    if (p.y) rs1 = stage_rms(rows, p.groups1, p.K, p.eps, sums, [&](int t, int k) { return p.y[(size_t)(t0 + t) * p.ldy + k]; });
-    auto base = [&](int t, int k) {
-        float v = stage_x0<XT>(p, t0 + t, k);
-        if (p.y) v += p.y[(size_t)(t0 + t) * p.ldy + k] * rs1[t * p.groups1 + k / gs1] * p.w1[k];
-        return v;
-    };
-    if (p.w2) rs2 = stage_rms(rows, p.groups2, p.K, p.eps, sums + (p.y ? stage_scratch(rows, p.groups1, blockDim.x >> 5) : 0), base);
-    for (int t = 0; t < rows; ++t) {
-#pragma unroll 4
-        for (int k = threadIdx.x; k < p.Kp; k += blockDim.x) {
-            float v = 0.f;
-            if (k < p.K) {
-                v = base(t, k);
-                if (store_h && p.h_out) p.h_out[(size_t)(t0 + t) * p.ldh + k] = v;
-                if (p.w2) v *= rs2[t * p.groups2 + k / gs2] * p.w2[k % p.w2_mod];
-            }
-            dst[(size_t)t * ldd + k] = Act<XT>::from_f(v);
-        }
-    }
-    __syncthreads();
-}
-static size_t stage_bytes(const RowStage& p, int rows, int nwarps) {
-    auto need = [&](int groups) {
-        const int a = stage_scratch(rows, groups, nwarps), b = rows * (p.K / 128 + groups);
-        return (size_t)(a > b ? a : b);
-    };
-    return ((p.y ? need(p.groups1) : 0) + (p.w2 ? need(p.groups2) : 0)) * 4 + 16;
 }
 
 template <typename XT>
@@ -331,13 +161,6 @@ static int launch_matvec(const RowStage& st, const void* w, int ldw, int N, void
     return 0;
 }
 
-static int check_stage(const RowStage& st, const char* who) {
-    DLP_REQUIRE(st.x && st.K > 0 && st.Kp >= st.K, "%s: bad input row", who);
-    DLP_REQUIRE(!st.y || (st.w1 && st.groups1 > 0 && st.K % st.groups1 == 0), "%s: %d norm groups do not divide the width %d", who, st.groups1, st.K);
-    DLP_REQUIRE(!st.w2 || (st.w2_mod > 0 && st.groups2 > 0 && st.K % st.groups2 == 0), "%s: %d norm groups do not divide the width %d", who, st.groups2, st.K);
-    return 0;
-}
-
 int matvec(const RowStage& st, const void* w, int ldw, int N, void* out, int ldo, int out_mode, int T, int f32, cudaStream_t s) {
     int rc = check_stage(st, "matvec");
     if (rc) return rc;
@@ -367,11 +190,18 @@ int stage_rows(const RowStage& st, void* xb, int ldxb, int T, int f32, cudaStrea
 
 // ---- fp32 matrix product ---------------------------------------------------------------------------------
 __global__ void __launch_bounds__(256) sgemm_kernel(const float* __restrict__ x, int ldx, const float* __restrict__ w, int ldw, int N, int K, float* out, int ldo,
-                                                    int out_mode, int T) {
+                                                    int out_mode, int T, const GemmGroup grp) {
     __shared__ float xs[16][68], ws[16][68];
-    const int n0 = blockIdx.x * 64, t0 = blockIdx.y * 64, tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
+    const int n0 = blockIdx.x * 64, tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
+    int t0 = blockIdx.y * 64;
     float acc[4][4] = {};
     pdl_wait();
+    if (grp.tile_expert != nullptr) {        // rows sorted by expert: this tile's rows and its matrix in the stack
+        if ((int)blockIdx.y >= *grp.n_tiles) return;
+        t0 = grp.tile_row0[blockIdx.y];
+        T = t0 + grp.tile_rows[blockIdx.y];
+        w += (size_t)grp.tile_expert[blockIdx.y] * grp.rows_per_expert * ldw;
+    }
     for (int k0 = 0; k0 < K; k0 += 16) {
         for (int i = threadIdx.x; i < 64 * 16; i += 256) {
             const int r = i >> 4, k = i & 15;
@@ -405,15 +235,20 @@ __global__ void __launch_bounds__(256) sgemm_kernel(const float* __restrict__ x,
         } else {
 #pragma unroll
             for (int j = 0; j < 4; ++j)
-                if (n0 + tx * 4 + j < N) out[(size_t)t * ldo + n0 + tx * 4 + j] = acc[i][j];
+                if (n0 + tx * 4 + j < N) {
+                    const float u = fmaxf(acc[i][j], 0.f);
+                    out[(size_t)t * ldo + n0 + tx * 4 + j] = out_mode == LO_RELU2 ? u * u : acc[i][j];
+                }
         }
     }
 }
 
-int sgemm(const float* x, int ldx, const float* w, int ldw, int N, int K, void* out, int ldo, int out_mode, int T, cudaStream_t s) {
+int sgemm(const float* x, int ldx, const float* w, int ldw, int N, int K, void* out, int ldo, int out_mode, int T, cudaStream_t s, const GemmGroup* grp) {
     DLP_REQUIRE(x && w && out && N > 0 && K > 0 && T > 0, "sgemm: bad argument");
-    DLP_REQUIRE(out_mode == LO_F32 || (out_mode == LO_GEGLU && N % 2 == 0), "sgemm: output mode %d", out_mode);
-    DLP_CHECK_CUDA(launch_pdl(sgemm_kernel, dim3((N + 63) / 64, (T + 63) / 64), dim3(256), 0, s, x, ldx, w, ldw, N, K, (float*)out, ldo, out_mode, T));
+    DLP_REQUIRE(out_mode == LO_F32 || out_mode == LO_RELU2 || (out_mode == LO_GEGLU && N % 2 == 0), "sgemm: output mode %d", out_mode);
+    DLP_REQUIRE(!grp || (grp->bt == 64 && grp->max_tiles > 0 && grp->max_tiles <= 65535), "sgemm: grouped launches take 64-row tiles");
+    DLP_CHECK_CUDA(launch_pdl(sgemm_kernel, dim3((N + 63) / 64, grp ? grp->max_tiles : (T + 63) / 64), dim3(256), 0, s, x, ldx, w, ldw, N, K, (float*)out, ldo, out_mode, T,
+                              grp ? *grp : GemmGroup()));
     return 0;
 }
 

@@ -72,67 +72,75 @@ int moe_route_ex(const float* logits, int ld, int T, int n_expert, int top_k, in
     return 0;
 }
 
-// One CTA builds the whole plan.  Warp e' handles experts e', e'+nw, ...: it walks the assignment list in order (ballot + popc),
-// so rows of one expert keep the token order (stable, deterministic).
+// One CTA builds the whole plan.  Every warp takes one contiguous part of the assignment list, 32 at a time: it counts per expert
+// first, then - behind a scan over (expert, warp) - ranks its assignments among the equal ones of their 32 (match), so rows of one
+// expert keep the token order (stable, deterministic).
 __global__ void __launch_bounds__(1024) moe_plan_kernel(const int* __restrict__ ids, int n_assign, int n_expert, int bt, int* __restrict__ pos,
                                                         int* __restrict__ src, int* __restrict__ bounds, int* __restrict__ tile_expert,
                                                         int* __restrict__ tile_row0, int* __restrict__ tile_rows, int* __restrict__ n_tiles) {
-    __shared__ int cnt[MOE_MAX_EXPERTS + 1];
-    __shared__ int start[MOE_MAX_EXPERTS + 1];
-    __shared__ int tile0[MOE_MAX_EXPERTS + 1];
+    __shared__ int cnt[32][MOE_MAX_EXPERTS];              // assignments of a warp's part, then its first row
+    __shared__ int total[MOE_MAX_EXPERTS], start[MOE_MAX_EXPERTS + 1], tile0[MOE_MAX_EXPERTS + 1];
     pdl_wait();
     pdl_launch_dependents();
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5;
-    for (int e = warp; e < n_expert; e += nw) {           // pass 1: how many assignments per expert
-        int c = 0;
-        for (int i0 = 0; i0 < n_assign; i0 += 32) {
-            const int i = i0 + lane;
-            c += __popc(__ballot_sync(0xffffffffu, i < n_assign && ids[i] == e));
-        }
-        if (lane == 0) cnt[e] = c;
+    for (int i = threadIdx.x; i < nw * MOE_MAX_EXPERTS; i += blockDim.x) (&cnt[0][0])[i] = 0;
+    __syncthreads();
+    const int per = ((n_assign + nw - 1) / nw + 31) / 32 * 32, lo = warp * per, hi = min(n_assign, lo + per);
+    for (int i0 = lo; i0 < hi; i0 += 32) {
+        const int i = i0 + lane, e = i < hi ? ids[i] : -1;
+        const unsigned same = __match_any_sync(0xffffffffu, e);
+        if (e >= 0 && (same & ((1u << lane) - 1u)) == 0) cnt[warp][e] += __popc(same);      // the first of its equals adds for all
+        __syncwarp();
     }
     __syncthreads();
-    if (threadIdx.x == 0) {                               // exclusive scans: sorted-row bounds and first tile of each expert
+    for (int e = threadIdx.x; e < n_expert; e += blockDim.x) {
+        int acc = 0;
+        for (int w = 0; w < nw; ++w) { const int c = cnt[w][e]; cnt[w][e] = acc; acc += c; }
+        total[e] = acc;
+    }
+    __syncthreads();
+    if (warp == 0) {                                      // exclusive scans: sorted-row bounds and first tile of each expert
         int acc = 0, tacc = 0;
-        for (int e = 0; e < n_expert; ++e) {
-            start[e] = acc;
-            tile0[e] = tacc;
-            bounds[e] = acc;
-            acc += cnt[e];
-            tacc += (cnt[e] + bt - 1) / bt;
+        for (int e0 = 0; e0 < n_expert; e0 += 32) {
+            const int e = e0 + lane, c = e < n_expert ? total[e] : 0, t = (c + bt - 1) / bt;
+            int sc = c, st = t;
+#pragma unroll
+            for (int o = 1; o < 32; o <<= 1) {
+                const int a = __shfl_up_sync(0xffffffffu, sc, o), b = __shfl_up_sync(0xffffffffu, st, o);
+                if (lane >= o) { sc += a; st += b; }
+            }
+            if (e < n_expert) { start[e] = acc + sc - c; tile0[e] = tacc + st - t; bounds[e] = acc + sc - c; }
+            acc += __shfl_sync(0xffffffffu, sc, 31);
+            tacc += __shfl_sync(0xffffffffu, st, 31);
         }
-        start[n_expert] = acc;
-        bounds[n_expert] = acc;
-        tile0[n_expert] = tacc;
-        *n_tiles = tacc;
+        if (lane == 0) { bounds[n_expert] = start[n_expert] = acc; tile0[n_expert] = tacc; *n_tiles = tacc; }
     }
     __syncthreads();
-    for (int e = warp; e < n_expert; e += nw) {           // pass 2: sorted position of every assignment, in token order
-        int base = start[e];
-        for (int i0 = 0; i0 < n_assign; i0 += 32) {
-            const int i = i0 + lane;
-            const bool mine = i < n_assign && ids[i] == e;
-            const unsigned m = __ballot_sync(0xffffffffu, mine);
-            if (mine) {
-                const int r = base + __popc(m & ((1u << lane) - 1u));
-                pos[i] = r;
-                src[r] = i;
-            }
-            base += __popc(m);
+    for (int i0 = lo; i0 < hi; i0 += 32) {
+        const int i = i0 + lane, e = i < hi ? ids[i] : -1;
+        const unsigned same = __match_any_sync(0xffffffffu, e);
+        const int rank = __popc(same & ((1u << lane) - 1u));
+        const int base = e >= 0 ? start[e] + cnt[warp][e] : 0;
+        __syncwarp();
+        if (e >= 0) {
+            pos[i] = base + rank;
+            src[base + rank] = i;
+            if (rank == 0) cnt[warp][e] += __popc(same);
         }
-        const int nt = tile0[e + 1] - tile0[e];           // this expert's token tiles
-        for (int j = lane; j < nt; j += 32) {
+        __syncwarp();
+    }
+    for (int e = warp; e < n_expert; e += nw)             // token tiles
+        for (int j = lane; j < tile0[e + 1] - tile0[e]; j += 32) {
             tile_expert[tile0[e] + j] = e;
             tile_row0[tile0[e] + j] = start[e] + j * bt;
-            tile_rows[tile0[e] + j] = min(bt, cnt[e] - j * bt);
+            tile_rows[tile0[e] + j] = min(bt, total[e] - j * bt);
         }
-    }
 }
 
 int moe_plan(const int* ids, int n_assign, int n_expert, int bt, int* pos, int* src, int* bounds, int* tile_expert, int* tile_row0,
              int* tile_rows, int* n_tiles, cudaStream_t s) {
     DLP_REQUIRE(n_assign > 0 && n_expert >= 1 && n_expert <= MOE_MAX_EXPERTS && bt >= 16, "moe_plan: bad shape");
-    const int threads = n_expert >= 32 ? 1024 : 32 * n_expert;
+    const int threads = n_assign >= 1024 ? 1024 : (n_assign + 31) / 32 * 32;
     DLP_CHECK_CUDA(launch_pdl(moe_plan_kernel, dim3(1), dim3(threads), 0, s, ids, n_assign, n_expert, bt, pos, src, bounds, tile_expert,
                               tile_row0, tile_rows, n_tiles));
     return 0;
@@ -155,26 +163,35 @@ int moe_gather(const __half* x, int ldx, const int* src, int top_k, int n_assign
     return 0;
 }
 
-// h[t] += sum_j w[t,j] * y[pos[t*k+j]]   (one CTA per token; experts are added in slot order j = 0..k-1)
-__global__ void __launch_bounds__(256) moe_combine_kernel(const float* __restrict__ y, const int* __restrict__ pos, const float* __restrict__ w,
-                                                          int top_k, int E, float* __restrict__ h) {
+// h[t] (+)= sum_j w[t,j] * y[pos[t*k+j]]   (one CTA per token; experts are added in slot order j = 0..k-1)
+__global__ void __launch_bounds__(256) moe_combine_kernel(const float* __restrict__ y, int ldy, const int* __restrict__ pos, const float* __restrict__ w,
+                                                          int top_k, int E, float* __restrict__ h, int add) {
     pdl_wait();
     pdl_launch_dependents();
     const int t = blockIdx.x;
-    for (int k = threadIdx.x * 4; k < E; k += blockDim.x * 4) {
-        float4 acc = *reinterpret_cast<const float4*>(h + (size_t)t * E + k);
-        for (int j = 0; j < top_k; ++j) {
-            const float wj = w[t * top_k + j];
-            const float4 v = *reinterpret_cast<const float4*>(y + (size_t)pos[t * top_k + j] * E + k);
-            acc.x = fmaf(wj, v.x, acc.x); acc.y = fmaf(wj, v.y, acc.y); acc.z = fmaf(wj, v.z, acc.z); acc.w = fmaf(wj, v.w, acc.w);
+    if (E % 4 == 0) {
+        for (int k = threadIdx.x * 4; k < E; k += blockDim.x * 4) {
+            float4 acc = add ? *reinterpret_cast<const float4*>(h + (size_t)t * E + k) : make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 4
+            for (int j = 0; j < top_k; ++j) {
+                const float wj = w[t * top_k + j];
+                const float4 v = *reinterpret_cast<const float4*>(y + (size_t)pos[t * top_k + j] * ldy + k);
+                acc.x = fmaf(wj, v.x, acc.x); acc.y = fmaf(wj, v.y, acc.y); acc.z = fmaf(wj, v.z, acc.z); acc.w = fmaf(wj, v.w, acc.w);
+            }
+            *reinterpret_cast<float4*>(h + (size_t)t * E + k) = acc;
         }
-        *reinterpret_cast<float4*>(h + (size_t)t * E + k) = acc;
+        return;
+    }
+    for (int k = threadIdx.x; k < E; k += blockDim.x) {
+        float acc = add ? h[(size_t)t * E + k] : 0.f;
+        for (int j = 0; j < top_k; ++j) acc = fmaf(w[t * top_k + j], y[(size_t)pos[t * top_k + j] * ldy + k], acc);
+        h[(size_t)t * E + k] = acc;
     }
 }
 
-int moe_combine(const float* y, const int* pos, const float* w, int T, int top_k, int E, float* h, cudaStream_t s) {
-    DLP_REQUIRE(E % 4 == 0 && T > 0, "moe_combine: bad shape");
-    DLP_CHECK_CUDA(launch_pdl(moe_combine_kernel, dim3(T), dim3(256), 0, s, y, pos, w, top_k, E, h));
+int moe_combine(const float* y, const int* pos, const float* w, int T, int top_k, int E, float* h, cudaStream_t s, int ldy, int add) {
+    DLP_REQUIRE(E > 0 && T > 0 && ldy >= E && (E % 4 != 0 || ldy % 4 == 0), "moe_combine: bad shape");
+    DLP_CHECK_CUDA(launch_pdl(moe_combine_kernel, dim3(T), dim3(256), 0, s, y, ldy, pos, w, top_k, E, h, add));
     return 0;
 }
 

@@ -18,15 +18,25 @@ class LayerSpec:
     mixer: dict[str, Any]
     mlp: dict[str, Any] | None = None
 
-    def n_params(self, width: int) -> int:
+    def n_params(self, width: int, norm_parts: int = 1) -> int:
+        """norm_parts: vectors of one norm (2 with a bias)."""
         m = self.mixer
+        hd, hv = m["heads"] * m["dim"], m["heads"] * m["vdim"]
         if self.type == "hgrn2":
-            hd, hv = m["heads"] * m["dim"], m["heads"] * m["vdim"]
             n = width * (2 * hd + 2 * hv) + 2 * hd + m["vdim"]
+        elif self.type == "attention":
+            kd, kv = m["kv_heads"] * m["dim"], m["kv_heads"] * m["vdim"]
+            n = width * (hd + kd + kv + hv) + hd + kd
         else:       # latent_attention
-            hd, hv, r = m["heads"] * m["dim"], m["heads"] * m["vdim"], m["kv_rank"]
+            r = m["kv_rank"]
             n = width * (hd + r + m["heads"] + hv) + r * (hd + hv) + r
-        return n + width + (3 * width * self.mlp["ff"] + width if self.mlp else 0)
+        if self.mlp is None:
+            ff = 0
+        elif self.mlp["kind"] == "moe":
+            ff = self.mlp["router"]["experts"] * (2 * width * self.mlp["expert"]["ff"] + width + 1)
+        else:
+            ff = 3 * width * self.mlp["ff"]
+        return n + ff + (2 if self.mlp else 1) * norm_parts * width
 
 
 @dataclass(frozen=True)
@@ -96,6 +106,8 @@ class ModelConfig:
     qk_norm_full: bool = False
     # layer-list models (models/layered.py): every layer is described on its own; the head / feed-forward fields above do not apply
     layers: tuple[LayerSpec, ...] = ()
+    loop: tuple[int, int, int] = ()      # (start, stop, times): layers start .. stop-1 run `times` times in a row with the same weights; the
+                                         # embedding output joins the residual stream in front of every pass but the first
     norm_groups: int = 1           # the norm divides each of this many equal parts of the vector by its own root mean square
 
     @property
@@ -107,6 +119,15 @@ class ModelConfig:
     # smollm3: every `no_rope_step`-th layer attends without rotary position encoding (`llama.cpp/src/models/smollm3.cpp:26`)
     no_rope_step: int = 0
     learned_pos: bool = False      # gpt2, starcoder: h = tok_embd[id] + position_embd[pos], no rotary anywhere
+
+    def layer_runs(self) -> list[tuple[int, bool]]:
+        """Layer lists in the order of execution: (layer, whether the embedding output is added in front of it).  A run's place in this
+        list names its own cache and state."""
+        n = len(self.layers)
+        start, stop, times = self.loop or (0, n, 1)
+        order = [*range(start), *list(range(start, stop)) * times, *range(stop, n)]
+        width = stop - start
+        return [(il, start < i < start + times * width and (i - start) % width == 0) for i, il in enumerate(order)]
 
     @property
     def ffn_norm_name(self) -> str:
@@ -137,7 +158,8 @@ class ModelConfig:
 
     def n_params(self) -> int:
         if self.layers:
-            return 2 * self.vocab_size * self.n_embd + self.n_embd + sum(s.n_params(self.n_embd) for s in self.layers)
+            parts = 2 if self.norm_type == "layer" else 1
+            return 2 * self.vocab_size * self.n_embd + parts * self.n_embd + sum(s.n_params(self.n_embd, parts) for s in self.layers)
         attn = self.n_embd * (self.q_dim + 2 * self.kv_dim) + self.q_dim * self.n_embd
         ffn = 3 * self.n_embd * self.n_ff * max(1, self.n_expert) + (self.n_embd * self.n_expert if self.is_moe else 0)
         emb = self.vocab_size * self.n_embd * (1 if self.tie_embeddings else 2)

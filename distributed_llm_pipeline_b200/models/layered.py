@@ -1,8 +1,9 @@
-"""Step of layer-list models on the engine core: mixers of different kinds in one model, norms behind the sublayers.
+"""Step of layer-list models on the engine core: mixers of different kinds in one model, norms in front of or behind the sublayers.
 
 The residual stream is fp32.  A sublayer's output `y` is not added at once: it stays pending, and the next matrix product forms
-`h + norm(y)` while it prepares its input rows (in the mat-vec prologue for up to four rows, in one row kernel in front of the GEMM
-for more).  One forward takes any mix of prompt portions and single tokens of different sequences: projections run over all rows,
+`h + y` (or `h + norm(y)`), and the norm in front of it, while it prepares its input rows (in the mat-vec prologue for up to four rows, in
+one row kernel in front of the GEMM for more).  A range of layers may run several times: every run has its own cache and state, and the
+embedding output joins at the start of every pass but the first.  One forward takes any mix of prompt portions and single tokens of different sequences: projections run over all rows,
 mixers over the segments.
 """
 from __future__ import annotations
@@ -16,7 +17,7 @@ from ..ops import layers as lops
 from ..ops.weights import DeviceWeight
 from ..gguf.constants import GGMLType
 from .engine import EngineCore, PagedKVCache, RecurrentState
-from .mixers import MIXERS, MLPS, Dense, LatentAttention, Rows, pad_to
+from .mixers import MIXERS, MLPS, Attention, Dense, LatentAttention, RoutedExperts, Rows, pad_to
 from .modeldir import ModelDir, open_model_dir
 from .weights import ModelWeights
 
@@ -25,11 +26,27 @@ MATVEC_ROWS = 4
 
 
 @dataclass
+class Norm:
+    """Weight (fp32) of a norm; with a bias it is a layer norm."""
+    w: torch.Tensor
+    b: torch.Tensor | None = None
+
+
+@dataclass
+class Pending:
+    """What the next product adds to the residual stream first: the sublayer output in the engine's `y` (normalised with w1, or as it is),
+    and at the start of a loop pass the embedding output."""
+    w1: torch.Tensor | None = None
+    y: bool = True
+    emb: bool = False
+
+
+@dataclass
 class LayeredLayer:
     mixer: object
-    norm1: torch.Tensor
+    norm1: Norm
     mlp: object | None = None
-    norm2: torch.Tensor | None = None
+    norm2: Norm | None = None
 
     def weights(self):
         return self.mixer.weights() + (self.mlp.weights() if self.mlp is not None else [])
@@ -52,15 +69,20 @@ def load_layered_weights(src: str | ModelDir, device, dtype="bf16", progress=Non
         if t.shape != (n,):
             raise ValueError(f"{name} has the shape {tuple(t.shape)}, expected ({n},)")
         return t
+
+    def norm(name):
+        return Norm(f32(name, cfg.n_embd), f32(name + ".b", cfg.n_embd) if cfg.norm_type == "layer" else None)
     layers = {}
     for il, spec in enumerate(cfg.layers):
         if progress is not None and progress(il / cfg.n_layer) is False:
             raise LoadCancelled("load cancelled")
         p = f"l{il}."
-        lw = LayeredLayer(MIXERS[spec.type](spec.mixer, lambda n: f.tensor(p + "mix." + n), dev, dt), f32(p + "norm1", cfg.n_embd))
+        lw = LayeredLayer(MIXERS[spec.type](spec.mixer, lambda n: f.tensor(p + "mix." + n), dev, dt, cfg.rms_eps), norm(p + "norm1"))
+        if lw.mixer.w_in.K != cfg.n_embd or lw.mixer.w_out.N != cfg.n_embd:
+            raise ValueError(f"layer {il}: a mixer projection does not fit the width")
         if spec.mlp is not None:
-            lw.mlp = MLPS[spec.mlp["kind"]](spec.mlp, lambda n: f.tensor(p + "mlp." + n), dev, dt)
-            lw.norm2 = f32(p + "norm2", cfg.n_embd)
+            lw.mlp = MLPS[spec.mlp["kind"]](spec.mlp, lambda n: f.tensor(p + "mlp." + n), dev, dt, cfg.n_embd)
+            lw.norm2 = norm(p + "norm2")
         layers[il] = lw
 
     def table(name):
@@ -69,20 +91,24 @@ def load_layered_weights(src: str | ModelDir, device, dtype="bf16", progress=Non
             raise ValueError(f"{name} is [{w.N}, {w.K}], expected [{cfg.vocab_size}, {cfg.n_embd}]")
         return DeviceWeight(GGMLType.F32 if dt == torch.float32 else GGMLType.BF16, w.N, w.K, [w.t])
     emb, head = table("embed"), table("head")
-    out_norm = f32("final.norm", cfg.n_embd)
+    out_norm = norm("final.norm")
     if progress is not None and progress(1.0) is False:
         raise LoadCancelled("load cancelled")
-    return LayeredWeights(cfg, layers, range(cfg.n_layer), 0, 1, emb, out_norm, head, (0, cfg.vocab_size), None)
+    return LayeredWeights(cfg, layers, range(cfg.n_layer), 0, 1, emb, out_norm.w, head, (0, cfg.vocab_size), None, out_norm_b=out_norm.b)
 
 
 @dataclass
 class TileTable:
-    """(token, head) row tiles of one latent-attention shape."""
+    """Row tiles of one attention shape: (token, head) rows for latent attention, tokens for the others."""
     row0: torch.Tensor
     rows: torch.Tensor
     n: int
     bm: int
-    n_splits: int
+    n_splits: int = 1
+
+    @property
+    def table(self):
+        return self.row0, self.rows, self.n
 
 
 @dataclass
@@ -107,12 +133,31 @@ class Batch:
     tok_slot: torch.Tensor      # [T] sequence slot of every row
     pos: torch.Tensor           # [T]
     slot: torch.Tensor          # [T] cache row
-    tiles: dict[tuple[int, bool], TileTable]      # by head count; True: tiles of the short segments only
+    # latent attention: (head count, short only); windowed attention: ("tokens", query heads per key / value head, short only), "flash"
+    tiles: dict[object, TileTable]
+    decode: bool = False        # one token of every sequence
+    longest: int = 0            # tokens of the longest sequence, these included
+    ranges: dict[tuple, int] | None = None      # key ranges of the windowed attentions of a decode step (None: chosen by `longest`)
+
+    def key_ranges(self, m: Attention, t: TileTable) -> int:
+        return self.ranges[key_range_kind(m)] if self.ranges is not None else key_ranges(m, t.n, t.bm, self.longest)
+
+
+def key_range_kind(m: Attention) -> tuple:
+    return m.G, m.R, m.window, m.keep
+
+
+def key_ranges(m: Attention, n_tiles: int, bm: int, longest: int) -> int:
+    """Parts the visible keys are split into: about two blocks per SM, at least 64 keys each, at most a cluster of 16 blocks."""
+    want, n = min(2 * 148 // (n_tiles * lops.gqa_blocks(m.G, m.R, bm)), (m.visible(longest) + 63) // 64, 16), 1
+    while n * 2 <= want:
+        n *= 2
+    return n
 
 
 class LayeredEngine(EngineCore):
     mixed_batches = True
-    can_shift = False           # a recurrent state has no positions to slide
+    can_shift = False           # a recurrent state has no positions to slide, and cached keys are rotated
 
     def __init__(self, weights: LayeredWeights, n_ctx: int = 4096, max_seqs: int = 8, page_size: int = 64, max_batch_tokens: int = 2048,
                  n_pages: int | None = None, comm=None, first_stage: bool = True, last_stage: bool = True):
@@ -125,35 +170,44 @@ class LayeredEngine(EngineCore):
             lops.load_library()
         self.dtype = weights.tok_embd.planes[0].dtype
         self.E = cfg.n_embd
-        mixers = {il: lw.mixer for il, lw in weights.layers.items()}
+        self.runs = cfg.layer_runs()
+        mixers = {r: weights.layers[il].mixer for r, (il, _) in enumerate(self.runs)}      # by run: what a run keeps is its own
+        mlps = [lw.mlp for lw in weights.layers.values() if lw.mlp is not None]
         max_pages = (n_ctx + page_size - 1) // page_size
         planes: dict[str, dict] = {}
-        for il, m in mixers.items():
+        for r, m in mixers.items():
             for name, shape in m.planes.items():
-                planes.setdefault(name, {})[il] = shape
+                planes.setdefault(name, {})[r] = shape
         self.kv = PagedKVCache(planes, max_pages * max_seqs if n_pages is None else n_pages, page_size, max_seqs, max_pages, dev, dtype=self.dtype)
-        self.rstate = RecurrentState({il: m.state for il, m in mixers.items() if m.state is not None}, max_seqs, dev)
+        self.rstate = RecurrentState({r: m.state for r, m in mixers.items() if m.state is not None}, max_seqs, dev)
         M, f32 = self.max_rows, torch.float32
         self.hb = [torch.zeros(M, self.E, dtype=f32, device=dev) for _ in range(2)]      # residual stream; the mat-vec path alternates
         self.h = self.hb[0]
-        self.cur = 0
+        self.cur = 0                                                 # which of them holds it (-1: still the embedding output)
+        self.emb = torch.zeros(M, self.E, dtype=f32, device=dev) if any(again for _, again in self.runs) else None
         self.y = torch.zeros(M, self.E, dtype=f32, device=dev)
-        sizes = {"proj": M * max(m.w_in.N for m in mixers.values()), "xb": M * max([pad_to(self.E, 8)] + [w.Kp for lw in weights.layers.values() for w in lw.weights()]),
-                 "act": M * max([8] + [lw.mlp.w_down.Kp for lw in weights.layers.values() if lw.mlp is not None])}
-        for m in mixers.values():
-            for name, n in m.buffers(M).items():
+        sizes = {"proj": M * max(m.w_in.N for m in mixers.values()), "xb": M * max([pad_to(self.E, 8)] + [w.Kp for lw in weights.layers.values() for w in lw.weights()])}
+        for part in [*mixers.values(), *mlps]:
+            for name, n in part.buffers(M).items():
                 sizes[name] = max(sizes.get(name, 0), n)
-        types = {"proj": f32, "o": f32}
+        types = {"proj": f32, "o": f32, "router": f32, "gate_w": f32, "ey": f32, "ids": torch.int32}
         self._flat = {n: torch.zeros(sz, dtype=types.get(n, self.dtype), device=dev) for n, sz in sizes.items()}
+        experts = [m for m in mlps if isinstance(m, RoutedExperts)]
+        self.expert_plans = {n: ops.MoePlan(M * max(m.top for m in experts), n, dev) for n in {m.n for m in experts}}
         self.logits = torch.zeros(max_seqs, cfg.vocab_size, dtype=f32, device=dev)
         lat = [m for m in mixers.values() if isinstance(m, LatentAttention)]
         self._latent_heads = sorted({m.H for m in lat})
+        att = [m for m in mixers.values() if isinstance(m, Attention)]
+        self._att_kinds = {key_range_kind(m): m for m in att}
+        self._att_groups = sorted({m.R for m in att})
+        self._att_flash = any(m.flash for m in att)
+        self._att_all_flash = all(m.flash for m in att)
         self._split_ctas = 148                                       # one CTA per SM: the key range is split until they are there
         self.latent_ws = None
         if lat:
             rows = self._split_ctas * 64
             self.latent_ws = (torch.zeros(rows * max(m.Rc for m in lat), dtype=f32, device=dev), torch.zeros(rows * 2, dtype=f32, device=dev))
-        # segments from this length on take the chunked recurrence and the expanded attention (bf16 storage; fp32 always takes the others)
+        # segments from this length on take the chunked recurrence and the expanded / flash attention (bf16 storage; fp32 always takes the others)
         self.long_from = 2 * lops.HGRN2_CHUNK if self.dtype == torch.bfloat16 else 1 << 60
         self._expanding_heads = {m.H for m in lat if m.expand} - {m.H for m in lat if not m.expand}
         chunked = [m for m in mixers.values() if m.state is not None and m.chunked]
@@ -161,7 +215,7 @@ class LayeredEngine(EngineCore):
         if chunked and self.long_from <= M:
             n = M // lops.HGRN2_CHUNK + M // self.long_from + 1         # every long segment may end in a partial chunk
             self.chunk_ws = tuple(torch.zeros(n * max(m.H * m.D * w(m) for m in chunked), dtype=f32, device=dev) for w in (lambda m: m.V, lambda m: 1))
-        self._variant = 1                                            # key ranges per decode query
+        self._variant = (1, *(1 for _ in self._att_kinds))           # key ranges per decode query: latent attention, then every windowed kind
         self._decode_batches: dict[tuple, Batch] = {}
 
     def buf(self, name: str, rows: int, cols: int, dtype=None) -> torch.Tensor:
@@ -175,64 +229,77 @@ class LayeredEngine(EngineCore):
         return self.buf(name, rows, cols)
 
     # ---- matrix products -------------------------------------------------------------------------------
-    def _product(self, r: Rows, w: Dense, out: torch.Tensor, T: int, geglu: bool = False) -> torch.Tensor:
-        cfg = self.cfg
-        if T <= MATVEC_ROWS and lops.matvec_fits(T, w.t):
-            st = lops.row_stage(r.x, r.K, w.Kp, cfg.rms_eps, r.y, r.w1, cfg.norm_groups, r.h_out, r.w2, r.groups2)
-            return lops.matvec(st, w.t, out, T, geglu)
-        x = r.x
-        if r.y is not None or r.w2 is not None or x.dtype != self.dtype or x.shape[1] != w.Kp:
-            st = lops.row_stage(r.x, r.K, w.Kp, cfg.rms_eps, r.y, r.w1, cfg.norm_groups, r.h_out, r.w2, r.groups2)
-            x = lops.stage_rows(st, self.buf("xb", T, w.Kp), T)
-        return lops.linear(x[:T], w.t, out, geglu)
+    def stage(self, r: Rows, Kp: int):
+        """The row preparation of `r` as the kernels take it."""
+        return lops.row_stage(r.x, r.K, Kp, self.cfg.rms_eps, r.y, r.w1, self.cfg.norm_groups if r.w1 is not None else 1, r.h_out, r.w2, r.groups2, r.b2, r.e)
 
-    def _residual(self, T: int, pending) -> Rows:
-        """Rows of the residual stream with the pending sublayer output folded in on the way."""
-        if pending is None:
-            return Rows(self.hb[self.cur][:T], self.E)
-        src = self.hb[self.cur][:T]
-        if T <= MATVEC_ROWS:        # every block of a mat-vec reads the old rows: the new ones go to the other buffer
-            self.cur ^= 1
-        return Rows(src, self.E, y=self.y[:T], w1=pending, h_out=self.hb[self.cur][:T])
+    def staged(self, r: Rows, Kp: int, T: int) -> torch.Tensor:
+        """Rows of `r` in the storage type, prepared by one launch if they are not there as they are."""
+        if r.y is None and r.w2 is None and r.e is None and r.x.dtype == self.dtype and r.x.shape[1] == Kp:
+            return r.x[:T]
+        return lops.stage_rows(self.stage(r, Kp), self.buf("xb", T, Kp), T)
 
-    def _settle(self, T: int, pending):
-        """Fold the pending output into the residual stream now; returns the rows [T, E] fp32."""
+    def matvec_rows(self, T: int, w: Dense) -> bool:
+        return T <= MATVEC_ROWS and lops.matvec_fits(T, w.t)
+
+    def product(self, r: Rows, w: Dense, out: torch.Tensor, T: int, geglu: bool = False) -> torch.Tensor:
+        if self.matvec_rows(T, w):
+            return lops.matvec(self.stage(r, w.Kp), w.t, out, T, geglu)
+        return lops.linear(self.staged(r, w.Kp, T), w.t, out, geglu)
+
+    def _residual(self, T: int, pending: Pending | None, pre: Norm | None = None) -> Rows:
+        """Rows of the residual stream with what is pending folded in on the way, and the norm `pre` in front of a sublayer."""
+        src = (self.hb[self.cur] if self.cur >= 0 else self.emb)[:T]
+        r = Rows(src, self.E)
         if pending is not None:
+            # every block of a mat-vec reads the old rows: the new ones go to the other buffer (and the embedding output stays as it is)
+            self.cur = max(0, self.cur ^ 1 if T <= MATVEC_ROWS else self.cur)
+            r = Rows(src, self.E, y=self.y[:T] if pending.y else None, w1=pending.w1, h_out=self.hb[self.cur][:T], e=self.emb[:T] if pending.emb else None)
+        if pre is not None:
+            r.w2, r.b2 = pre.w, pre.b
+        return r
+
+    def _settle(self, T: int, pending: Pending | None):
+        """Fold what is pending into the residual stream now; returns the rows [T, E] fp32."""
+        if pending is not None:
+            src = (self.hb[self.cur] if self.cur >= 0 else self.emb)[:T]
+            self.cur = max(0, self.cur)
             h = self.hb[self.cur][:T]
-            st = lops.row_stage(h, self.E, self.E, self.cfg.rms_eps, self.y[:T], pending, self.cfg.norm_groups, h)
-            lops.stage_rows(st, self.buf("xb", T, self.E), T)
+            r = Rows(src, self.E, y=self.y[:T] if pending.y else None, w1=pending.w1, h_out=h, e=self.emb[:T] if pending.emb else None)
+            lops.stage_rows(self.stage(r, self.E), self.buf("xb", T, self.E), T)
         return self.hb[self.cur][:T]
 
     # ---- one forward over a batch ------------------------------------------------------------------------
-    def _forward(self, ids: torch.Tensor, b: Batch):
-        """Embedding and all layers; returns the norm weight of the output still pending in self.y (None: nothing pending)."""
-        T = b.T
-        self.cur = 0
-        lops.embed(self.w.tok_embd.planes[0], ids, self.hb[0], T)
+    def _forward(self, ids: torch.Tensor, b: Batch) -> Pending | None:
+        """Embedding and all layers; returns what is still to be added to the residual stream (None: nothing)."""
+        T, pre = b.T, self.cfg.pre_norm
+        self.cur = 0 if self.emb is None else -1
+        lops.embed(self.w.tok_embd.planes[0], ids, self.hb[0] if self.emb is None else self.emb, T)
         pending = None
-        for il, lw in self.w.layers.items():
+        for run, (il, again) in enumerate(self.runs):
+            lw = self.w.layers[il]
             m = lw.mixer
-            proj = self._product(self._residual(T, pending), m.w_in, self.buf("proj", T, m.w_in.N), T)
-            self._product(m.mix(self, il, proj, b), m.w_out, self.y[:T], T)
-            pending = lw.norm1
+            if again:
+                pending = Pending(pending.w1, True, True) if pending is not None else Pending(None, False, True)
+            proj = self.product(self._residual(T, pending, lw.norm1 if pre else None), m.w_in, self.buf("proj", T, m.w_in.N), T)
+            self.product(m.mix(self, run, proj, b), m.w_out, self.y[:T], T)
+            pending = Pending(None if pre else lw.norm1.w)
             if lw.mlp is not None:
-                g = lw.mlp
-                act = self._product(self._residual(T, pending), g.w_gu, self.buf("act", T, g.w_down.Kp), T, geglu=True)
-                self._product(Rows(act, g.w_down.K), g.w_down, self.y[:T], T)
-                pending = lw.norm2
+                lw.mlp.apply(self, self._residual(T, pending, lw.norm2 if pre else None), T)
+                pending = Pending(None if pre else lw.norm2.w)
             if self.eval_callback is not None or il in self.cvec:
                 h = self._settle(T, pending)
                 pending = None
                 if il in self.cvec:
                     h.add_(self.cvec[il])
                 if self.eval_callback is not None:
-                    self.eval_callback("l_out", il, h)
+                    self.eval_callback("l_out", run, h)
         return pending
 
     def _head_rows(self, r: Rows, n: int, out: torch.Tensor) -> torch.Tensor:
-        r.w2, r.groups2 = self.w.out_norm, self.cfg.norm_groups
+        r.w2, r.b2, r.groups2 = self.w.out_norm, self.w.out_norm_b, self.cfg.norm_groups
         head = self.w.lm_head
-        return self._product(r, Dense(head.planes[0], head.K), out, n)
+        return self.product(r, Dense(head.planes[0], head.K), out, n)
 
     # ---- batch descriptions ---------------------------------------------------------------------------------
     def _n_splits(self, n_tiles: int, max_len: int) -> int:
@@ -240,6 +307,12 @@ class LayeredEngine(EngineCore):
         while n * 2 <= want:
             n *= 2
         return n
+
+    @staticmethod
+    def _token_tiles(segs: list[tuple[int, int]], n: int) -> tuple[list[int], list[int]]:
+        """First row and length of every tile of up to n rows, for row ranges."""
+        tiles = [(t, min(n, hi - t)) for lo, hi in segs for t in range(lo, hi, n)]
+        return [t for t, _ in tiles], [c for _, c in tiles]
 
     def _tile_lists(self, H: int, lens: list[int], bm: int):
         row0, rows, base = [], [], 0
@@ -258,9 +331,12 @@ class LayeredEngine(EngineCore):
             for H in self._latent_heads:
                 bm = lops.latent_tile_rows(H, B)
                 row0, rows = self._tile_lists(H, [1] * B, bm)
-                tiles[H, False] = TileTable(torch.tensor(row0, dtype=i32, device=dev), torch.tensor(rows, dtype=i32, device=dev), len(row0), bm, min(self._variant, max(1, self._split_ctas // len(row0))))
+                tiles[H, False] = TileTable(torch.tensor(row0, dtype=i32, device=dev), torch.tensor(rows, dtype=i32, device=dev), len(row0), bm, min(self._variant[0], max(1, self._split_ctas // len(row0))))
             rng = torch.tensor([[i, i + 1] for i in range(B)], dtype=i32, device=dev)
-            b = Batch(B, B, Segments(B, rng, self.active), None, self.active, self.pos, self.slot, tiles)
+            rows = torch.arange(B, dtype=i32, device=dev), torch.ones(B, dtype=i32, device=dev)
+            tiles |= {("tokens", R, False): TileTable(*rows, B, lops.gqa_tile(R, 1)[0]) for R in self._att_groups}
+            b = Batch(B, B, Segments(B, rng, self.active), None, self.active, self.pos, self.slot, tiles, decode=True,
+                      ranges=dict(zip(self._att_kinds, self._variant[1:])))
             self._decode_batches[(B, self._variant)] = b
         return b
 
@@ -289,18 +365,32 @@ class LayeredEngine(EngineCore):
                 bm = lops.latent_tile_rows(H, sum(lens[:n]))
                 row0, rows = self._tile_lists(H, lens[:n], bm)
                 cols += [torch.tensor(row0, dtype=torch.int32), torch.tensor(rows, dtype=torch.int32)]
-                shapes.append((H, only_short, bm, len(row0)))
+                shapes.append(((H, only_short), bm, len(row0)))
+        for R in self._att_groups:
+            for only_short in (False, True):
+                part = groups[0] if only_short else segs
+                if only_short and (not groups[1] or not part) or not only_short and groups[1] and self._att_all_flash:
+                    continue
+                bm, n = lops.gqa_tile(R, max(g[2] - g[1] for g in part))
+                row0, rows = self._token_tiles([g[1:] for g in part], n)
+                cols += [torch.tensor(row0, dtype=torch.int32), torch.tensor(rows, dtype=torch.int32)]
+                shapes.append((("tokens", R, only_short), bm, len(row0)))
+        if groups[1] and self._att_flash:       # the tiles with the longest context first
+            order = sorted(((self.seqs[sid].length + t - lo, t, n) for sid, lo, hi in groups[1] for t, n in zip(*self._token_tiles([(lo, hi)], lops.FLASH_TILE))), reverse=True)
+            row0, rows = [t for _, t, _ in order], [n for _, _, n in order]
+            cols += [torch.tensor(row0, dtype=torch.int32), torch.tensor(rows, dtype=torch.int32)]
+            shapes.append(("flash", lops.FLASH_TILE, len(row0)))
         dev = iter(torch.cat(cols).to(self.device).split([c.numel() for c in cols]))
         ids, pos_d, slot_d, tok_slot = (next(dev) for _ in range(4))
         short = Segments(len(groups[0]), next(dev), next(dev))
         long = Segments(len(groups[1]), next(dev), next(dev), next(dev).view(-1, 2), next(dev),
                         tuple((sid, lo, hi, self.seqs[sid].length + hi - lo) for sid, lo, hi in groups[1]))
         longest = max(self.seqs[sid].length + len(t) for sid, t in parts)
-        tiles = {(H, only): TileTable(next(dev), next(dev), nt, bm, self._n_splits(nt, longest)) for H, only, bm, nt in shapes}
-        return ids, Batch(T, T_short, short if short.n else None, long if long.n else None, tok_slot, pos_d, slot_d, tiles)
+        tiles = {kind: TileTable(next(dev), next(dev), nt, bm, self._n_splits(nt, longest)) for kind, bm, nt in shapes}
+        return ids, Batch(T, T_short, short if short.n else None, long if long.n else None, tok_slot, pos_d, slot_d, tiles, longest=longest)
 
     def _run_mixed(self, parts: list[tuple[int, list[int]]]):
-        """Forward over one mixed batch; updates the sequence lengths.  Returns the pending norm weight (see _forward)."""
+        """Forward over one mixed batch; updates the sequence lengths.  Returns what is pending (see _forward)."""
         ids, b = self._mixed_batch(parts)
         pending = self._forward(ids, b)
         for sid, t in parts:
@@ -394,7 +484,7 @@ class LayeredEngine(EngineCore):
         sid = self.alloc_seq()
         try:
             h = self._settle(len(tokens), self._run_mixed([(sid, tokens)]))
-            st = lops.row_stage(h, self.E, self.E, self.cfg.rms_eps, w2=self.w.out_norm, groups2=self.cfg.norm_groups)
+            st = self.stage(Rows(h, self.E, w2=self.w.out_norm, groups2=self.cfg.norm_groups, b2=self.w.out_norm_b), self.E)
             xn = lops.stage_rows(st, self.buf("xb", len(tokens), self.E), len(tokens)).float()
         finally:
             self.free_seq(sid)
@@ -402,10 +492,12 @@ class LayeredEngine(EngineCore):
         return torch.nn.functional.normalize(e, dim=-1) if normalize else e.clone()
 
     def _choose_variant(self, B: int, max_len: int):
+        lat = 1
         if self._latent_heads:
             H = self._latent_heads[-1]
             bm = lops.latent_tile_rows(H, B)
-            self._variant = self._n_splits(B * ((H + bm - 1) // bm), max_len)
+            lat = self._n_splits(B * ((H + bm - 1) // bm), max_len)
+        self._variant = (lat, *(key_ranges(m, B, lops.gqa_tile(m.R, 1)[0], max_len) if m.mma else 1 for m in self._att_kinds.values()))
 
     def _decode_body(self, B: int, sample: bool):
         ops.advance(self.seq_len_dev, self.active, self.pos, self.slot, self.kv_len, self.kv.block_table, self.page_size, B)
@@ -427,6 +519,6 @@ class LayeredEngine(EngineCore):
                 self.cvec[il] = (v.float() * scale).to(self.device)
 
     def memory_breakdown(self) -> dict:
-        act = sum(t.numel() * t.element_size() for t in [*self.hb, self.y, self.logits, *self._flat.values(), *(self.latent_ws or ())])
+        act = sum(t.numel() * t.element_size() for t in [*self.hb, *([self.emb] if self.emb is not None else []), self.y, self.logits, *self._flat.values(), *(self.latent_ws or ())])
         return {"model": self.w.nbytes(), "kv_cache": self.kv.bytes(), "recurrent_state": self.rstate.bytes(), "compute": act, "graphs": len(self._graphs),
                 "device": str(self.device)}

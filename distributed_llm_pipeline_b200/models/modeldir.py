@@ -81,45 +81,72 @@ def write_safetensors(path: str, tensors: dict[str, torch.Tensor]) -> str:
 
 
 # ---- architectures -------------------------------------------------------------------------------------------------
+def _need(what: str, d, keys: tuple[str, ...]):
+    """Check that `d` has these keys, dotted ones inside nested objects: positive sizes, except where a rule below says otherwise."""
+    rules = {"scale": lambda v: isinstance(v, (int, float)), "base": lambda v: isinstance(v, (int, float)) and v > 0,
+             "keep_first": lambda v: isinstance(v, int) and v >= 0}
+    for path in keys:
+        v = d
+        for k in path.split("."):
+            if not isinstance(v, dict) or k not in v:
+                raise ValueError(f"{what}: {path} missing")
+            v = v[k]
+        if not rules.get(k, lambda v: isinstance(v, int) and v >= 1)(v):
+            raise ValueError(f"{what}: {path} = {v!r}")
+
+
 def _layer_list(cfg: dict, mixers: dict[str, tuple[str, ...]], mlps: dict[str, tuple[str, ...]]) -> tuple[LayerSpec, ...]:
     """Check every entry's type and sizes: `mixers` / `mlps` name the keys each kind must have."""
-    def need(what, d, keys):
-        missing = [k for k in keys if k not in d]
-        if missing:
-            raise ValueError(f"{what}: {', '.join(missing)} missing")
-        for k in keys:
-            v = d[k]
-            if k in ("scale",):
-                if not isinstance(v, (int, float)):
-                    raise ValueError(f"{what}: {k} = {v!r}")
-            elif not isinstance(v, int) or v < 1:
-                raise ValueError(f"{what}: {k} = {v!r} is not a positive size")
     out = []
     for i, e in enumerate(cfg["layers"]):
         if e["type"] not in mixers:
             raise ValueError(f"layer {i}: unknown mixer {e['type']!r}")
-        need(f"layer {i} ({e['type']})", e["mixer"], mixers[e["type"]])
+        _need(f"layer {i} ({e['type']})", e["mixer"], mixers[e["type"]])
         mlp = e.get("mlp")
         if mlp is not None:
             if mlp.get("kind") not in mlps:
                 raise ValueError(f"layer {i}: unknown feed-forward {mlp.get('kind')!r}")
-            need(f"layer {i} (feed-forward)", mlp, mlps[mlp["kind"]])
+            _need(f"layer {i} (feed-forward)", mlp, mlps[mlp["kind"]])
         out.append(LayerSpec(e["type"], dict(e["mixer"]), dict(mlp) if mlp is not None else None))
     return tuple(out)
+
+
+def _layered_config(name: str, cfg: dict, layers: tuple[LayerSpec, ...], **kw) -> ModelConfig:
+    return ModelConfig(name=name, arch=name, vocab_size=cfg["vocab"], n_embd=cfg["width"], n_layer=len(layers), n_head=0, n_head_kv=0, head_dim=0, n_ff=0,
+                       n_ctx_train=int(cfg.get("context", 1 << 20)), rms_eps=float(cfg["norm"]["eps"]), rope_dim=0, bos_id=-1, eos_id=-1, layers=layers, **kw)
 
 
 def talizen_config(cfg: dict) -> ModelConfig:
     """Talizen: HGRN2 and latent-attention layers in any order, tanh-gelu gated feed-forward or none, grouped norms behind the sublayers."""
     layers = _layer_list(cfg, {"hgrn2": ("heads", "dim", "vdim"), "latent_attention": ("heads", "dim", "vdim", "kv_rank", "scale")}, {"dense": ("ff",)})
-    norm = cfg["norm"]
-    if cfg["width"] % norm["groups"]:
-        raise ValueError(f"{norm['groups']} norm groups do not divide the width {cfg['width']}")
-    return ModelConfig(name="talizen", arch="talizen", vocab_size=cfg["vocab"], n_embd=cfg["width"], n_layer=len(layers), n_head=0, n_head_kv=0, head_dim=0,
-                       n_ff=max((s.mlp["ff"] for s in layers if s.mlp), default=0), n_ctx_train=int(cfg.get("context", 1 << 20)), rms_eps=float(norm["eps"]),
-                       rope_dim=0, bos_id=-1, eos_id=-1, layers=layers, norm_groups=norm["groups"])
+    groups = cfg["norm"]["groups"]
+    if cfg["width"] % groups:
+        raise ValueError(f"{groups} norm groups do not divide the width {cfg['width']}")
+    return _layered_config("talizen", cfg, layers, norm_groups=groups, pre_norm=False, post_norm=True)
 
 
-ARCHITECTURES = {"Talizen": talizen_config}
+def vozinex_config(cfg: dict) -> ModelConfig:
+    """Vozinex: windowed grouped-query attention with kept first tokens, routed experts or no feed-forward, layer norms in front of the
+    sublayers, a range of layers that runs several times."""
+    layers = _layer_list(cfg, {"attention": ("heads", "kv_heads", "dim", "vdim", "rot.dims", "rot.base", "scale", "mask.size", "mask.keep_first")},
+                         {"moe": ("expert.ff", "router.experts", "router.top")})
+    for i, s in enumerate(layers):
+        m = s.mixer
+        if m["heads"] % m["kv_heads"]:
+            raise ValueError(f"layer {i}: {m['kv_heads']} key / value heads do not divide {m['heads']} heads")
+        if m["rot"]["dims"] % 2 or m["rot"]["dims"] > m["dim"]:
+            raise ValueError(f"layer {i}: rotation of {m['rot']['dims']} of {m['dim']} dimensions")
+        if s.mlp and s.mlp["router"]["top"] > s.mlp["router"]["experts"]:
+            raise ValueError(f"layer {i}: {s.mlp['router']['top']} of {s.mlp['router']['experts']} experts")
+    loop = ()
+    if cfg.get("loop"):
+        loop = tuple(cfg["loop"].get(k) for k in ("start", "stop", "times"))
+        if not (all(isinstance(x, int) for x in loop) and 0 <= loop[0] < loop[1] <= len(layers) and loop[2] >= 1):
+            raise ValueError(f"loop {cfg['loop']!r} does not fit {len(layers)} layers")
+    return _layered_config("vozinex", cfg, layers, norm_type="layer", loop=loop)
+
+
+ARCHITECTURES = {"Talizen": talizen_config, "Vozinex": vozinex_config}
 
 
 @dataclass

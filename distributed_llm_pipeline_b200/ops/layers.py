@@ -1,4 +1,4 @@
-"""Ops of layer-list models (recurrent mixers, latent attention, norms behind the sublayers): thin wrappers over the C ABI.
+"""Ops of layer-list models (recurrent mixers, latent and windowed attention, routed experts, norms on either side): thin wrappers over the C ABI.
 
 There is no CPU form: the kernels are the only implementation.  Two storage types run through every op, bf16 and fp32 (`f32`); the
 residual stream, norms, recurrent states, attention scores and weights are fp32 in both.
@@ -12,15 +12,28 @@ import torch
 from . import api
 from . import lib as _lib
 
-OUT_F32, OUT_GEGLU, OUT_BF16 = 0, 1, 2
+OUT_F32, OUT_GEGLU, OUT_BF16, OUT_RELU2 = 0, 1, 2, 3
+MAX_EXPERTS, MAX_TOP = 256, 32
+GQA_MMA_DIM, GQA_FLASH_DIM = 256, 128      # widest heads of the tensor-core forms
+FLASH_TILE = 128            # tokens per tile of the tcgen05 flash kernel
 HGRN2_CHUNK = 64            # tokens per chunk of the chunked recurrence
 
 
 class RowStage(C.Structure):
-    """How a row is formed in front of a product: x (+ gnorm(y) * w1 -> h_out), then optionally gnorm(.) * w2."""
+    """How a row is formed in front of a product: x (+ y or gnorm(y) * w1) (+ e) (-> h_out), then optionally gnorm(.) * w2, or with b2 a layer norm."""
     _fields_ = [("x", C.c_void_p), ("x_f32", C.c_int32), ("ldx", C.c_int32), ("y", C.c_void_p), ("ldy", C.c_int32), ("w1", C.c_void_p),
                 ("groups1", C.c_int32), ("h_out", C.c_void_p), ("ldh", C.c_int32), ("w2", C.c_void_p), ("groups2", C.c_int32), ("w2_mod", C.c_int32),
-                ("eps", C.c_float), ("K", C.c_int32), ("Kp", C.c_int32)]
+                ("eps", C.c_float), ("K", C.c_int32), ("Kp", C.c_int32), ("b2", C.c_void_p), ("e", C.c_void_p), ("lde", C.c_int32)]
+
+
+class ExpertArgs(C.Structure):
+    _fields_ = [("logits", C.c_void_p), ("bias", C.c_void_p), ("w", C.c_void_p)] + [(n, C.c_int32) for n in ("ldl", "n_expert", "top", "rows", "ldw")]
+
+
+class GqaArgs(C.Structure):
+    _fields_ = [(n, C.c_void_p) for n in ("proj", "q_norm", "k_norm", "inv_freq", "q", "kc", "vc", "block_table", "tok_slot", "pos", "slot", "tile_row0", "tile_rows", "out")] + \
+               [(n, C.c_int32) for n in ("ldp", "ldo", "T", "H", "G", "D", "V", "Dc", "Vc", "rot", "max_pages", "page_size", "n_pages", "n_tiles", "bm", "n_splits", "window",
+                                         "keep")] + [("eps", C.c_float), ("scale", C.c_float)]
 
 
 class Hgrn2Args(C.Structure):
@@ -53,9 +66,10 @@ def _p(t):
     return None if t is None else t.data_ptr()
 
 
-def row_stage(x: torch.Tensor, K: int, Kp: int, eps: float, y=None, w1=None, groups1: int = 1, h_out=None, w2=None, groups2: int = 1) -> RowStage:
+def row_stage(x: torch.Tensor, K: int, Kp: int, eps: float, y=None, w1=None, groups1: int = 1, h_out=None, w2=None, groups2: int = 1,
+              b2=None, e=None) -> RowStage:
     return RowStage(_p(x), int(x.dtype == torch.float32), x.stride(0), _p(y), y.stride(0) if y is not None else 0, _p(w1), groups1, _p(h_out),
-                    h_out.stride(0) if h_out is not None else 0, _p(w2), groups2, w2.numel() if w2 is not None else 1, eps, K, Kp)
+                    h_out.stride(0) if h_out is not None else 0, _p(w2), groups2, w2.numel() if w2 is not None else 1, eps, K, Kp, _p(b2), _p(e), e.stride(0) if e is not None else 0)
 
 
 def matvec_fits(T: int, w: torch.Tensor) -> bool:
@@ -184,6 +198,119 @@ def rows_attention(q, kv, S: int, pos0: int, H: int, Dp: int, Vp: int, V: int, s
     _need_cuda(q, "rows_attention")
     _lib.check(_lib.load().dlp_layers_rows_attention(_p(q), _p(kv), kv.stride(0), S, q.shape[0], pos0, H, Dp, Vp, V, scale, _p(gate),
                                                      gate.stride(0) if gate is not None else 0, _p(out), out.stride(0), api._stream()), "layers_rows_attention")
+    api._count()
+    return out
+
+
+# ---- routed experts -------------------------------------------------------------------------------------------------------
+def route(logits: torch.Tensor, bias, n_expert: int, top: int, ids: torch.Tensor, weights: torch.Tensor, T: int):
+    """The `top` largest of logits + bias and the softmax over them -> ids, weights [T * top]."""
+    _need_cuda(logits, "route")
+    _lib.check(_lib.load().dlp_layers_route(_p(logits), logits.stride(0), _p(bias), n_expert, top, _p(ids), _p(weights), T, api._stream()), "layers_route")
+    api._count()
+
+
+def expert_matvec_fits(T: int, top: int, w: torch.Tensor) -> bool:
+    """The staged rows (one per token, or one per assignment in front of the down product) fit the shared memory of one block."""
+    return T * top * w.shape[1] * w.element_size() <= 150 * 1024
+
+
+def expert_matvec(st: RowStage, logits, bias, n_expert: int, top: int, w: torch.Tensor, rows: int, out: torch.Tensor, T: int, down: bool) -> torch.Tensor:
+    """1..4 staged rows times the matrices of their chosen experts, w [n_expert * rows, ld]: max(., 0)^2 -> out [T * top, ld] (activation type), or
+    (down; st: one row per assignment) the weighted sum over a token's experts -> out [T, ld] fp32."""
+    _need_cuda(w, "expert_matvec")
+    a = ExpertArgs(_p(logits), _p(bias), _p(w), logits.stride(0), n_expert, top, rows, w.stride(0))
+    _lib.check(_lib.load().dlp_layers_expert_matvec(C.byref(st), C.byref(a), _p(out), out.stride(0), int(down), T, int(w.dtype == torch.float32), api._stream()),
+               "layers_expert_matvec")
+    api._count()
+    return out
+
+
+def expert_plan(ids: torch.Tensor, n_expert: int, tile: int, plan):
+    """Expert-sorted order of the assignments and the row tiles of the grouped products (ops.api.MoePlan)."""
+    _need_cuda(ids, "expert_plan")
+    api.moe_plan(ids, n_expert, tile, plan)
+
+
+def expert_gather(x: torch.Tensor, plan, top: int, n: int, out: torch.Tensor) -> torch.Tensor:
+    """out[row] = x[token of the row]; rows are moved as 16-byte pieces, so fp32 rows count twice as many 2-byte elements."""
+    _need_cuda(x, "expert_gather")
+    api.moe_gather(x.view(torch.int16), plan, top, n, out.view(torch.int16))
+    return out
+
+
+def linear_grouped(xs: torch.Tensor, w: torch.Tensor, rows: int, n_expert: int, tile: int, plan, out: torch.Tensor, relu2: bool = False) -> torch.Tensor:
+    """out[row] = xs[row] . W_e^T for every expert-sorted row (e: the row's expert), one launch; relu2: max(., 0)^2 in the activation type."""
+    _need_cuda(xs, "linear_grouped")
+    f32 = w.dtype == torch.float32
+    ws = None if f32 else api.gemm_workspace(xs.device)
+    _lib.check(_lib.load().dlp_layers_linear_grouped(_p(xs), xs.stride(0), _p(w), w.stride(0), rows, w.shape[1], _p(out), out.stride(0), OUT_RELU2 if relu2 else OUT_F32,
+                                                     xs.shape[0], n_expert, tile, C.byref(plan.c), int(f32), _p(ws), 0 if ws is None else ws.numel(), api._stream()),
+               "layers_linear_grouped")
+    api._count()
+    return out
+
+
+def expert_combine(y: torch.Tensor, plan, weights: torch.Tensor, T: int, top: int, out: torch.Tensor) -> torch.Tensor:
+    """out[t] = sum of the weighted expert rows of token t, in the order of the choice."""
+    _need_cuda(y, "expert_combine")
+    _lib.check(_lib.load().dlp_layers_combine(_p(y), y.stride(0), _p(plan.pos), _p(weights), T, top, out.shape[1], _p(out), api._stream()), "layers_combine")
+    api._count()
+    return out
+
+
+# ---- windowed grouped-query attention ----------------------------------------------------------------------------------------
+def gqa_tile(R: int, longest: int) -> tuple[int, int]:
+    """Rows of a tile and the tokens it holds, for R query heads per key / value head and segments of up to `longest` tokens."""
+    bm = 16 if longest * R <= 16 or longest == 1 else 64
+    return bm, bm // min(R, bm)
+
+
+def gqa_blocks(G: int, R: int, bm: int) -> int:
+    """Blocks per tile and key range."""
+    return G * -(-R // min(R, bm))
+
+
+def gqa_args(shape, proj, kc, vc, block_table, tok_slot, pos, slot, out, T: int, q=None, tiles=None, bm: int = 16, n_splits: int = 1) -> GqaArgs:
+    """shape: models.mixers.Attention (heads, sizes, norms, rotation, window); tiles: (first rows, rows, count) of the launch."""
+    m = shape
+    row0, rows, n = tiles if tiles is not None else (None, None, 0)
+    return GqaArgs(_p(proj), _p(m.q_norm), _p(m.k_norm), _p(m.inv_freq), _p(q), _p(kc), _p(vc), _p(block_table), _p(tok_slot), _p(pos), _p(slot), _p(row0), _p(rows), _p(out),
+                   proj.stride(0) if proj is not None else 0, out.stride(0) if out is not None else 0, T, m.H, m.G, m.D, m.V, m.Dc, m.Vc, m.rot, block_table.shape[1],
+                   kc.shape[-2], kc.shape[0], n, bm, n_splits, m.window, m.keep, m.eps, m.scale)
+
+
+def gqa_prepare(m, proj, kc, vc, block_table, tok_slot, pos, slot, q, T: int):
+    """Projection rows -> normalised and rotated queries q [T, H * Dc]; keys and values into the pages."""
+    _need_cuda(kc, "gqa_prepare")
+    a = gqa_args(m, proj, kc, vc, block_table, tok_slot, pos, slot, None, T, q=q)
+    _lib.check(_lib.load().dlp_layers_gqa_prepare(C.byref(a), int(kc.dtype == torch.float32), api._stream()), "layers_gqa_prepare")
+    api._count()
+
+
+def gqa_attention(m, q, kc, vc, block_table, tok_slot, pos, tiles, bm: int, n_splits: int, out, T: int):
+    """Prepared queries over the cached keys their window shows, tiles of up to bm (token, head) rows of one key / value head."""
+    _need_cuda(kc, "gqa_attention")
+    a = gqa_args(m, None, kc, vc, block_table, tok_slot, pos, None, out, T, q=q, tiles=tiles, bm=bm, n_splits=n_splits)
+    _lib.check(_lib.load().dlp_layers_gqa_attention(C.byref(a), 0, int(kc.dtype == torch.float32), api._stream()), "layers_gqa_attention")
+    api._count()
+    return out
+
+
+def gqa_decode(m, proj, kc, vc, block_table, tok_slot, pos, tiles, n_splits: int, out, T: int):
+    """Single tokens straight from the projection: norm, rotation, cache write and attention in one launch (bf16)."""
+    _need_cuda(kc, "gqa_decode")
+    a = gqa_args(m, proj, kc, vc, block_table, tok_slot, pos, None, out, T, tiles=tiles, n_splits=n_splits)
+    _lib.check(_lib.load().dlp_layers_gqa_attention(C.byref(a), 1, 0, api._stream()), "layers_gqa_attention")
+    api._count()
+    return out
+
+
+def gqa_flash(m, q, kc, vc, block_table, tok_slot, pos, tiles, out, T: int):
+    """Prepared queries in tiles of 128 consecutive tokens (tcgen05 flash kernel, bf16)."""
+    _need_cuda(kc, "gqa_flash")
+    a = gqa_args(m, None, kc, vc, block_table, tok_slot, pos, None, out, T, q=q, tiles=tiles)
+    _lib.check(_lib.load().dlp_layers_gqa_flash(C.byref(a), api._stream()), "layers_gqa_flash")
     api._count()
     return out
 

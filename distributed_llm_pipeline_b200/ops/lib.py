@@ -85,6 +85,13 @@ def _declare(lib):
         "dlp_layers_latent_gather": (i32, [vp, vp, i32, i32, vp, i32, vp]),
         "dlp_layers_head_rows": (i32, [vp, i32, i32, i32, i32, vp, i32, vp]),
         "dlp_layers_rows_attention": (i32, [vp, vp, i32, i32, i32, i32, i32, i32, i32, i32, f32, vp, i32, vp, i32, vp]),
+        "dlp_layers_route": (i32, [vp, i32, vp, i32, i32, vp, vp, i32, vp]),
+        "dlp_layers_expert_matvec": (i32, [vp, vp, vp, i32, i32, i32, i32, vp]),
+        "dlp_layers_linear_grouped": (i32, [vp, i32, vp, i32, i32, i32, vp, i32, i32, i32, i32, i32, vp, i32, vp, sz, vp]),
+        "dlp_layers_combine": (i32, [vp, i32, vp, vp, i32, i32, i32, vp, vp]),
+        "dlp_layers_gqa_prepare": (i32, [vp, i32, vp]),
+        "dlp_layers_gqa_attention": (i32, [vp, i32, i32, vp]),
+        "dlp_layers_gqa_flash": (i32, [vp, vp]),
         "dlp_layers_rows_attention_error": (i32, [vp]),
         "dlp_gemv_moe": (i32, [W, W, vp, vp, f32, vp, i32, i32, vp, i32, vp, vp]),
     }

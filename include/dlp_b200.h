@@ -352,12 +352,21 @@ int dlp_memcpy_d2h(void* dst, const void* src, size_t bytes);
  * state, attention scores and weights are fp32 in both. */
 typedef struct {              /* how a row is formed in front of a matrix product (csrc/layers.cuh RowStage) */
     const void* x; int32_t x_f32, ldx;
-    const float* y; int32_t ldy;               /* x += gnorm(y; groups1) * w1 */
+    const float* y; int32_t ldy;               /* x += gnorm(y; groups1) * w1, or y as it is (w1 NULL) */
     const float* w1; int32_t groups1;
     float* h_out; int32_t ldh;
     const float* w2; int32_t groups2, w2_mod;  /* then gnorm(.; groups2) * w2[k % w2_mod] */
     float eps; int32_t K, Kp;
+    const float* b2;                           /* with b2: layer norm (centred) instead, . * w2 + b2 */
+    const float* e; int32_t lde;               /* a second addend of x */
 } dlp_row_stage;
+typedef struct { const float* logits; const float* bias; const void* w; int32_t ldl, n_expert, top, rows, ldw; } dlp_expert_args;
+typedef struct {              /* windowed grouped-query attention (csrc/layers.cuh GqaArgs) */
+    const float* proj; const float* q_norm; const float* k_norm; const float* inv_freq; void* q; void* kc; void* vc;
+    const int32_t* block_table; const int32_t* tok_slot; const int32_t* pos; const int32_t* slot; const int32_t* tile_row0; const int32_t* tile_rows; void* out;
+    int32_t ldp, ldo, T, H, G, D, V, Dc, Vc, rot, max_pages, page_size, n_pages, n_tiles, bm, n_splits, window, keep;
+    float eps, scale;
+} dlp_gqa_args;
 typedef struct {
     const float* proj; int32_t ldp; const float* fbias; const float* lower; float* state;
     const int32_t* seg; const int32_t* seg_slot; const int32_t* pos; float* out; int32_t ldo, H, D, V, n_seg;
@@ -369,6 +378,7 @@ typedef struct {
     int32_t max_pages, page_size, H, Rc, T, n_tiles, bm, n_splits; float scale;
 } dlp_latent_args;
 /* decode product, 1..4 rows: out_mode 0 = fp32, 1 = GEGLU of interleaved (gate, up) rows -> activation type, 2 = bf16 (dlp_layers_linear) */
+/* (out_mode 3, dlp_layers_linear_grouped: max(., 0)^2 in the activation type) */
 int dlp_layers_matvec(const dlp_row_stage* st, const void* w, int ldw, int N, void* out, int ldo, int out_mode, int T, int f32, void* stream);
 int dlp_layers_stage_rows(const dlp_row_stage* st, void* xb, int ldxb, int T, int f32, void* stream);
 /* any number of rows: bf16 through the tcgen05 GEMM (ws: split-K workspace as for dlp_linear_ws), fp32 through an fp32 kernel */
@@ -385,6 +395,18 @@ int dlp_layers_latent_gather(const void* cache, const int32_t* bt_row, int page,
 int dlp_layers_head_rows(const float* x, int ldx, int D, int Dp, int H, void* out, int T, void* stream);
 int dlp_layers_rows_attention(const void* q, const void* kv, int ldkv, int S, int T, int pos0, int H, int Dp, int Vp, int V, float scale, const float* gate, int ldg,
                               void* out, int ldo, void* stream);
+/* routed experts: router logits + bias -> the `top` largest and the softmax over them; decode products of the chosen experts (1..4 rows);
+ * any number of rows over expert-sorted rows (plan: dlp_moe_plan); out[t] = sum_j weights[t * top + j] * y[pos[t * top + j]] */
+int dlp_layers_route(const float* logits, int ld, const float* bias, int n_expert, int top, int32_t* ids, float* weights, int T, void* stream);
+int dlp_layers_expert_matvec(const dlp_row_stage* st, const dlp_expert_args* a, void* out, int ldo, int down, int T, int f32, void* stream);
+int dlp_layers_linear_grouped(const void* xs, int ldx, const void* w, int ldw, int rows_per_expert, int K, void* out, int ldo, int out_mode, int n_assign, int n_expert,
+                              int token_tile, const dlp_moe_plan_bufs* plan, int f32, void* ws, size_t ws_bytes, void* stream);
+int dlp_layers_combine(const float* y, int ldy, const int32_t* pos, const float* weights, int T, int top, int E, float* out, void* stream);
+/* windowed attention: projection rows -> queries and cache rows; tiles of (token, head) rows (fused: single tokens straight from the
+ * projection); tiles of 128 tokens (tcgen05, bf16) */
+int dlp_layers_gqa_prepare(const dlp_gqa_args* a, int f32, void* stream);
+int dlp_layers_gqa_attention(const dlp_gqa_args* a, int fused, int f32, void* stream);
+int dlp_layers_gqa_flash(const dlp_gqa_args* a, void* stream);
 int dlp_layers_rows_attention_error(int* flag);   /* *flag = 1: a wait inside the kernel gave up since the last call (synchronises) */
 
 #ifdef __cplusplus

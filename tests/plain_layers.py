@@ -1,4 +1,4 @@
-"""Plain, slow restatement of layer-list models (Talizen) for the tests: one function per mechanism, whole sequences, float64.
+"""Plain, slow restatement of layer-list models (Talizen, Vozinex) for the tests: one function per mechanism, whole sequences, float64.
 
 Nothing here is shared with the product path: no kernels, no cache, no batching, no code of the package.  Every function takes the
 complete sequence of one request and returns a value per token.
@@ -73,8 +73,69 @@ def gated_mlp(h: torch.Tensor, w: dict) -> torch.Tensor:
     return (gelu_tanh(h @ w["gate"].T) * (h @ w["up"].T)) @ w["down"].T
 
 
+def layer_norm(x: torch.Tensor, w: torch.Tensor, b: torch.Tensor, eps: float) -> torch.Tensor:
+    d = x - x.mean(-1, keepdim=True)
+    return d / torch.sqrt((d * d).mean(-1, keepdim=True) + eps) * w + b
+
+
+def rotate_half(x: torch.Tensor, dims: int, base: float, pos: torch.Tensor) -> torch.Tensor:
+    """x [T, H, d] at positions pos: dimension i < dims / 2 turns with dimension i + dims / 2, the rest stays."""
+    n = dims // 2
+    a = pos.to(x.dtype)[:, None] * base ** (-2 * torch.arange(n, dtype=x.dtype) / dims)
+    c, s = torch.cos(a)[:, None], torch.sin(a)[:, None]
+    u, v = x[..., :n], x[..., n:dims]
+    return torch.cat([u * c - v * s, v * c + u * s, x[..., dims:]], -1)
+
+
+def window_mask(T: int, size: int, keep_first: int) -> torch.Tensor:
+    """[query, key]: the last `size` keys up to the query itself, and the first `keep_first` of the sequence."""
+    i, j = torch.arange(T)[:, None], torch.arange(T)[None]
+    return (j <= i) & ((i - j < size) | (j < keep_first))
+
+
+def masked_softmax_attention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, scale: float, seen: torch.Tensor) -> torch.Tensor:
+    """q [T, H, d], k [T, G, d], v [T, G, dv]: consecutive groups of H / G query heads share a key / value head."""
+    T, H, G = q.shape[0], q.shape[1], k.shape[1]
+    out = torch.empty(T, H, v.shape[-1], dtype=q.dtype)
+    for h in range(H):
+        s = (q[:, h] @ k[:, h // (H // G)].T * scale).masked_fill(~seen, float("-inf"))
+        out[:, h] = torch.softmax(s, -1) @ v[:, h // (H // G)]
+    return out
+
+
+def attention_mixer(h: torch.Tensor, w: dict, m: dict, eps: float) -> torch.Tensor:
+    """Grouped-query attention: q and k are normalised over the whole projection, then rotated; sliding window with kept first tokens."""
+    T, H, G = h.shape[0], m["heads"], m["kv_heads"]
+    pos = torch.arange(T)
+    q = (rms(h @ w["q"].T, eps) * w["q.norm"]).reshape(T, H, m["dim"])
+    k = (rms(h @ w["k"].T, eps) * w["k.norm"]).reshape(T, G, m["dim"])
+    q, k = (rotate_half(x, m["rot"]["dims"], m["rot"]["base"], pos) for x in (q, k))
+    v = (h @ w["v"].T).reshape(T, G, m["vdim"])
+    o = masked_softmax_attention(q, k, v, m["scale"], window_mask(T, m["mask"]["size"], m["mask"]["keep_first"]))
+    return o.reshape(T, H * m["vdim"]) @ w["o"].T
+
+
+def route(h: torch.Tensor, w: torch.Tensor, b: torch.Tensor, top: int):
+    """Chosen experts [T, top] and their weights: softmax over the chosen logits only."""
+    z, ids = (h @ w.T + b).sort(dim=-1, descending=True, stable=True)
+    return ids[:, :top], torch.softmax(z[:, :top], -1)
+
+
+def expert(h: torch.Tensor, up: torch.Tensor, down: torch.Tensor) -> torch.Tensor:
+    return torch.clamp(h @ up.T, min=0) ** 2 @ down.T
+
+
+def moe_mlp(h: torch.Tensor, w: dict, top: int) -> torch.Tensor:
+    ids, p = route(h, w["router"], w["router.b"], top)
+    out = torch.zeros_like(h)
+    for t in range(h.shape[0]):
+        for e, x in zip(ids[t].tolist(), p[t]):
+            out[t] += x * expert(h[t], w[f"e{e}.up"], w[f"e{e}.down"])
+    return out
+
+
 def layer(x: torch.Tensor, spec: dict, w: dict, norm: dict) -> torch.Tensor:
-    """Both sublayers read x as it is; their outputs are normalised before they are added."""
+    """Talizen: both sublayers read x as it is; their outputs are normalised before they are added."""
     m = spec["mixer"]
     mix = {k[4:]: v for k, v in w.items() if k.startswith("mix.")}
     if spec["type"] == "hgrn2":
@@ -90,16 +151,41 @@ def layer(x: torch.Tensor, spec: dict, w: dict, norm: dict) -> torch.Tensor:
     return x
 
 
+def pre_norm_layer(x: torch.Tensor, spec: dict, w: dict, norm: dict) -> torch.Tensor:
+    """Vozinex: layer norms in front of the sublayers, whose outputs are added as they are."""
+    sub = {p: {k[4:]: v for k, v in w.items() if k.startswith(p + ".")} for p in ("mix", "mlp")}
+    x = x + attention_mixer(layer_norm(x, w["norm1"], w["norm1.b"], norm["eps"]), sub["mix"], spec["mixer"], norm["eps"])
+    if spec["mlp"] is not None:
+        x = x + moe_mlp(layer_norm(x, w["norm2"], w["norm2.b"], norm["eps"]), sub["mlp"], spec["mlp"]["router"]["top"])
+    return x
+
+
+def layer_runs(cfg: dict) -> list[tuple[int, bool]]:
+    """(layer, whether the embedding output is added in front of it) in the order of execution."""
+    n, lp = len(cfg["layers"]), cfg.get("loop")
+    if not lp:
+        return [(i, False) for i in range(n)]
+    inner = list(range(lp["start"], lp["stop"]))
+    passes = [(i, p > 0 and i == inner[0]) for p in range(lp["times"]) for i in inner]
+    return [(i, False) for i in range(lp["start"])] + passes + [(i, False) for i in range(lp["stop"], n)]
+
+
 def forward(cfg: dict, w: dict[str, torch.Tensor], tokens, dtype=F):
-    """Logits [T, vocab] and the residual stream after every layer [layers, T, width] of one whole sequence."""
+    """Logits [T, vocab] and the residual stream after every layer run [runs, T, width] of one whole sequence."""
     w = {k: v.to(dtype) for k, v in w.items()}
-    x = w["embed"][torch.as_tensor(list(tokens))]
+    pre = cfg["architecture"] == "Vozinex"
+    emb = x = w["embed"][torch.as_tensor(list(tokens))]
     after = []
-    for i, spec in enumerate(cfg["layers"]):
+    for i, again in layer_runs(cfg):
         p = f"l{i}."
-        x = layer(x, spec, {k[len(p):]: v for k, v in w.items() if k.startswith(p)}, cfg["norm"])
+        if again:
+            x = x + emb
+        x = (pre_norm_layer if pre else layer)(x, cfg["layers"][i], {k[len(p):]: v for k, v in w.items() if k.startswith(p)}, cfg["norm"])
         after.append(x)
-    x = grouped_norm(x, w["final.norm"], cfg["norm"]["groups"], cfg["norm"]["eps"])
+    if pre:
+        x = layer_norm(x, w["final.norm"], w["final.norm.b"], cfg["norm"]["eps"])
+    else:
+        x = grouped_norm(x, w["final.norm"], cfg["norm"]["groups"], cfg["norm"]["eps"])
     return x @ w["head"].T, torch.stack(after)
 
 

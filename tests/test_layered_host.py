@@ -62,6 +62,30 @@ def test_config_is_checked(tmp_path):
             open_model_dir(p)
 
 
+def test_windowed_config_is_checked(tmp_path):
+    cfg = lm.CONFIGS["experts"]
+    p = lm.write(str(tmp_path / "m"), cfg, lm.weights(cfg))
+    d = open_model_dir(p).cfg
+    assert (d.n_layer, d.norm_type, d.loop, d.rms_eps) == (4, "layer", (1, 3, 2), 3e-4)
+    assert d.layer_runs() == [(0, False), (1, False), (2, False), (1, True), (2, False), (3, False)] == plain.layer_runs(cfg)
+    assert d.n_params() == sum(t.numel() for t in lm.weights(cfg).values())
+    no_loop = {k: v for k, v in cfg.items() if k != "loop"}
+    for c, want in (({**cfg, "loop": {"start": 0, "stop": 4, "times": 3}}, [(i, r > 0 and i == 0) for r in range(3) for i in range(4)]), (no_loop, [(i, False) for i in range(4)]),
+                    ({**cfg, "loop": {"start": 3, "stop": 4, "times": 1}}, [(i, False) for i in range(4)])):
+        json.dump(c, open(os.path.join(p, "config.json"), "w"))
+        assert open_model_dir(p).cfg.layer_runs() == want == plain.layer_runs(c)
+    a = lm.attention
+    for bad in (a(6, 4, 8, 8, 0.3, 8, 4, 0), a(2, 2, 8, 8, 0.3, 10, 4, 0), a(2, 2, 8, 8, 0.3, 3, 4, 0), a(2, 2, 8, 8, 0.3, 8, 0, 0), a(2, 2, 8, 8, 0.3, 8, 4, -1), a(2, 2, 8, 8, "1", 8, 4, 0),
+                a(2, 2, 8, 8, 0.3, 8, 4, 0, 3, 4, 8), a(2, 2, 8, 8, 0.3, 8, 4, 0, 3, 2, 0)):
+        json.dump({**no_loop, "layers": [bad]}, open(os.path.join(p, "config.json"), "w"))
+        with pytest.raises(ValueError):
+            open_model_dir(p)
+    for loop in ((2, 2, 1), (0, 5, 2), (0, 2, 0), (-1, 2, 2), (0, 2, None)):
+        json.dump({**cfg, "loop": dict(zip(("start", "stop", "times"), loop))}, open(os.path.join(p, "config.json"), "w"))
+        with pytest.raises(ValueError):
+            open_model_dir(p)
+
+
 def test_loading_checks_shapes_and_can_be_cancelled(tmp_path):
     cfg = lm.CONFIGS["odd"]
     w = lm.weights(cfg)
@@ -73,6 +97,12 @@ def test_loading_checks_shapes_and_can_be_cancelled(tmp_path):
     lm.write(p, cfg, {**w, "l1.mix.lower": w["l1.mix.lower"][:-1]})
     with pytest.raises(ValueError):
         load_weights(p, "cpu")
+    cfg = lm.CONFIGS["experts"]
+    w = lm.weights(cfg)
+    for name in ("l0.mix.k", "l0.mix.q.norm", "l0.mix.o", "l0.norm1.b", "l2.mlp.e4.down", "l2.mlp.router", "l2.mlp.router.b", "final.norm.b"):
+        lm.write(p, cfg, {**w, name: w[name][:-1]})
+        with pytest.raises(ValueError):
+            load_weights(p, "cpu")
 
 
 @pytest.mark.parametrize("name", list(lm.CONFIGS))
@@ -90,8 +120,9 @@ def test_prompt_portions_and_single_tokens(model, name):
     assert len(eng.kv.free) == eng.kv.n_pages
 
 
-def test_batches_larger_than_the_buffers_and_reuse(model):
-    cfg, w, eng, _ = model("odd", max_batch_tokens=24, n_pages=12)
+@pytest.mark.parametrize("name", ["odd", "experts"])
+def test_batches_larger_than_the_buffers_and_reuse(model, name):
+    cfg, w, eng, _ = model(name, max_batch_tokens=24, n_pages=12)
     run = TraceRunner(eng)
     ids = {k: lm.tokens(cfg, n, seed=n) for k, n in dict(a=70, b=33, c=50, d=5, e=61).items()}
     want = {k: plain.forward(cfg, w, v)[0] for k, v in ids.items()}
@@ -141,8 +172,9 @@ def test_recurrent_state_is_kept_whole(model):
     assert lm.error(eng.prefill(a, ids, all_logits=True), want) < TOL
 
 
-def test_attention_only_models_can_roll_back(model):
-    cfg, w, eng, _ = model("attention")
+@pytest.mark.parametrize("name", ["attention", "experts"])
+def test_attention_only_models_can_roll_back(model, name):
+    cfg, w, eng, _ = model(name)
     ids = lm.tokens(cfg, 30)
     sid = eng.alloc_seq()
     eng.prefill(sid, ids[:12] + [0, 0, 0])
@@ -151,9 +183,10 @@ def test_attention_only_models_can_roll_back(model):
     assert lm.error(eng.prefill(sid, ids[12:], all_logits=True), plain.forward(cfg, w, ids)[0][12:]) < TOL
 
 
-def test_session_file(model, tmp_path):
+@pytest.mark.parametrize("name", ["odd", "experts"])
+def test_session_file(model, name, tmp_path):
     from distributed_llm_pipeline_b200.utils.session import load_sequence, save_sequence
-    cfg, w, eng, _ = model("odd")
+    cfg, w, eng, _ = model(name)
     ids = lm.tokens(cfg, 40)
     a = eng.alloc_seq()
     eng.prefill(a, ids[:37])
@@ -189,6 +222,24 @@ def test_hooks(model):
     assert torch.allclose(e.double(), plain.grouped_norm(after[-1], w["final.norm"].double(), 3, 3e-4), atol=1e-4)
 
 
+def test_hooks_between_looped_layers(model):
+    """The callback sees every run, and what it settles in front of a new pass does not lose the embedding output."""
+    cfg, w, eng, _ = model("experts")
+    ids = lm.tokens(cfg, 9)
+    want, after = plain.forward(cfg, w, ids)
+    for cut in ([9], [5, 1, 3]):
+        got, at, sid = {}, 0, eng.alloc_seq()
+        eng.eval_callback = lambda name, run, h: got.setdefault(run, []).append(h.clone())
+        for n in cut:
+            lg = eng.step([(sid, ids[at:at + n])])
+            at += n
+        assert sorted(got) == list(range(len(after))) and lm.error(lg, want[-1:]) < TOL
+        assert all((torch.cat(got[i]).double() - after[i]).abs().max() < 1e-4 for i in got)
+    eng.eval_callback = None
+    e = eng.embed(ids, "last", normalize=False)
+    assert torch.allclose(e.double(), plain.layer_norm(after[-1][-1], w["final.norm"].double(), w["final.norm.b"].double(), 3e-4), atol=1e-4)
+
+
 def check_greedy(cfg, w, prompt, out, min_gap):
     """Every generated token is the plain model's best one given what was generated before it (near ties aside)."""
     ids = list(prompt) + list(out)
@@ -198,7 +249,7 @@ def check_greedy(cfg, w, prompt, out, min_gap):
         assert row.max() - row[t] < min_gap, i
 
 
-@pytest.mark.parametrize("name", ["odd", "recurrent"])
+@pytest.mark.parametrize("name", ["odd", "recurrent", "experts"])
 def test_scheduler_mixes_prompts_and_decoding(model, name):
     cfg, w, eng, _ = model(name, n_seqs=3)
     sched = Scheduler(eng, IdTokenizer(cfg["vocab"]), n_batch=16, n_slots=3)
@@ -220,7 +271,7 @@ def test_scheduler_mixes_prompts_and_decoding(model, name):
     assert more.n_prompt_cached in (0, len(ids) - 1)
     check_greedy(cfg, w, ids + [3, 4], more.output_ids, 1e-3)
     edited = sched.generate(ids[:-3] + [5], n_predict=2, sampling=greedy)
-    assert edited.n_prompt_cached == 0
+    assert edited.n_prompt_cached == 0 or not eng.rstate
     check_greedy(cfg, w, ids[:-3] + [5], edited.output_ids, 1e-3)
 
 
