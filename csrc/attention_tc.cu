@@ -16,7 +16,7 @@ static int launch_fa(const __half* q, const __half* kc, const __half* vc, const 
     if (first_use_on_device((const void*)kern))
         DLP_CHECK_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, Cfg::SMEM_BYTES));
     dim3 grid((p.T + Cfg::BM - 1) / Cfg::BM, p.Hq);
-    kern<<<grid, 192, Cfg::SMEM_BYTES, s>>>(tq, tk, tv, p);
+    kern<<<grid, Cfg::THREADS, Cfg::SMEM_BYTES, s>>>(tq, tk, tv, p);
     DLP_LAUNCH_CHECK();
     return 0;
 }

@@ -5,7 +5,7 @@
 // mma.sync + cp.async with the accumulators in registers - which is also what attention.cu:attn_prefill_kernel is.  This kernel
 // is the sm_100a form of the same algorithm:
 //
-//   CTA = one tile of 128 queries of one query head.  192 threads:
+//   CTA = one tile of 128 queries of one query head.  192 threads (320 where four more softmax warps share a row):
 //     warp 0      producer   TMA: the Q tile once, then per 128-key tile the K and V rows page by page (the block table gives the
 //                            page ids; a page is a contiguous [page_size x D] block, box {64, page_size} of a 2-D map over the cache)
 //     warp 1      MMA        one thread issues  S = Q.K^T  (M = 128 queries, N = 128 keys, K = D) into one of two TMEM S buffers,
@@ -16,6 +16,8 @@
 //                            max / sum, P = exp2(..) written as fp16 into shared memory in the K-major swizzled layout the
 //                            second MMA reads as its A operand.  O is rescaled in TMEM only when a row maximum actually grew
 //                            (warp-uniform test), and normalised + stored as fp16 at the end.
+//                            (FA_ROWS / FA_TILES: warps 2-5 and 6-9 take 64 keys of every tile each, with a maximum, a sum and an O
+//                            accumulator of their own, and join them at the end.)
 //   QK^T of tile i+1 is issued before P.V of tile i, so the tensor pipe works on the next scores while the softmax warps are
 //   busy; K/V stages form a 2-deep ring.
 #pragma once
@@ -102,18 +104,20 @@ struct FaCfg {
     static constexpr int K_BYTES = BN * D1 * 2, V_BYTES = BN * D2 * 2;
     static constexpr int P_PARTS = MODE == FA_PAGED ? 1 : 2;
     static constexpr int P_BYTES = BM * BN * 2;      // one part
+    static constexpr int HALVES = MODE == FA_PAGED ? 1 : 2;      // groups of four softmax warps; each takes its part of a key tile into an O of its own
+    static constexpr int THREADS = 64 + 128 * HALVES;
     static constexpr int STAGES = 2;
     static constexpr int SMEM_BYTES = Q_BYTES + STAGES * (K_BYTES + V_BYTES) + P_PARTS * P_BYTES + 1024 + 256;
-    static constexpr int TMEM_COLS = 512;            // S0 [0,128)  S1 [128,256)  O [256, 256 + D2)
+    static constexpr int TMEM_COLS = 512;            // S0 [0,128)  S1 [128,256)  O [256, 256 + HALVES * D2)
     static constexpr int O_COL = 256;
 };
 
 template <int D1, int D2, int MODE>
-__global__ void __launch_bounds__(192, 1)
+__global__ void __launch_bounds__((FaCfg<D1, D2, MODE>::THREADS), 1)
 attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_k,
                        const __grid_constant__ CUtensorMap tm_v, const FaParams p) {
     using Cfg = FaCfg<D1, D2, MODE>;
-    constexpr int BM = Cfg::BM, BN = Cfg::BN, KB = Cfg::KB, VB = Cfg::VB, FMT = MODE == FA_PAGED ? 0 : 1;
+    constexpr int BM = Cfg::BM, BN = Cfg::BN, KB = Cfg::KB, VB = Cfg::VB, HALVES = Cfg::HALVES, FMT = MODE == FA_PAGED ? 0 : 1;
     constexpr bool EXACT = MODE != FA_PAGED;                     // fp32 scores times scale, split softmax weights
     extern __shared__ uint8_t smem_raw[];
     uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
@@ -129,9 +133,9 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_co
     uint64_t* v_empty = bars + 7;     // [2]
     uint64_t* s_full = bars + 9;      // [2]
     uint64_t* s_free = bars + 11;     // [2]
-    uint64_t* p_full = bars + 13;
-    uint64_t* pv_done = bars + 14;
-    uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 15);
+    uint64_t* p_full = bars + 13;     // [HALVES]
+    uint64_t* pv_done = bars + 15;    // [HALVES]
+    uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 17);
 
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int qt = gridDim.x - 1 - blockIdx.x;        // heaviest (latest) query tiles first (FA_TILES: in the order of the table)
@@ -158,10 +162,12 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_co
             mbar_init(&k_empty[s], 1);
             mbar_init(&v_empty[s], 1);
             mbar_init(&s_full[s], 1);
-            mbar_init(&s_free[s], 4);
+            mbar_init(&s_free[s], 4 * HALVES);
         }
-        mbar_init(p_full, 4);
-        mbar_init(pv_done, 1);
+        for (int h = 0; h < HALVES; ++h) {
+            mbar_init(&p_full[h], 4);
+            mbar_init(&pv_done[h], 1);
+        }
         mbar_fence_init();
     }
     if (warp == 1) {
@@ -211,20 +217,23 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_co
             constexpr uint32_t idesc_o = make_idesc_f16_bmn(BM, D2, FMT);
             auto issue_pv = [&](int j) {
                 const int s = j & 1;
-                mbar_wait_g(p_full, (uint32_t)j & 1u, p.error);
                 mbar_wait_g(&v_full[s], (uint32_t)(j >> 1) & 1u, p.error);
-                tc_fence_after();
 #pragma unroll
-                for (int kk = 0; kk < BN / 16; ++kk) {
-                    const uint64_t db = make_smem_desc_sw128_mn(smem_u32(sm_v + s * Cfg::V_BYTES + kk * 16 * 128), BN * 128);
+                for (int h = 0; h < HALVES; ++h) {
+                    mbar_wait_g(&p_full[h], (uint32_t)j & 1u, p.error);
+                    tc_fence_after();
 #pragma unroll
-                    for (int part = 0; part < Cfg::P_PARTS; ++part) {
-                        const uint64_t da = make_smem_desc_sw128(smem_u32(sm_p + part * Cfg::P_BYTES + (kk >> 2) * (BM * 128))) + (uint64_t)(2 * (kk & 3));
-                        tc_mma_f16(tmem_base + Cfg::O_COL, da, db, idesc_o, (j > 0 || kk > 0 || part > 0) ? 1u : 0u);
+                    for (int kk = h * (BN / 16 / HALVES); kk < (h + 1) * (BN / 16 / HALVES); ++kk) {
+                        const uint64_t db = make_smem_desc_sw128_mn(smem_u32(sm_v + s * Cfg::V_BYTES + kk * 16 * 128), BN * 128);
+#pragma unroll
+                        for (int part = 0; part < Cfg::P_PARTS; ++part) {
+                            const uint64_t da = make_smem_desc_sw128(smem_u32(sm_p + part * Cfg::P_BYTES + (kk >> 2) * (BM * 128))) + (uint64_t)(2 * (kk & 3));
+                            tc_mma_f16(tmem_base + Cfg::O_COL + h * D2, da, db, idesc_o, (j > 0 || kk > h * (BN / 16 / HALVES) || part > 0) ? 1u : 0u);
+                        }
                     }
+                    tc_commit(&pv_done[h]);
                 }
                 tc_commit(&v_empty[s]);
-                tc_commit(pv_done);
             };
             mbar_wait_g(q_full, 0, p.error);
             for (int i = 0; i < n_tiles; ++i) {
@@ -248,78 +257,86 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_co
             issue_pv(n_tiles - 1);
         }
     } else {
-        // ===== softmax / correction / epilogue: thread r <-> query row r =====
+        // ===== softmax / correction / epilogue: thread (half, r) <-> query row r, key columns [half * CW, + CW) of every tile =====
+        constexpr int CW = BN / HALVES;
         const int q4 = warp & 3;                       // TMEM lane quarter this warp may access
+        const int half = (warp - 2) >> 2;              // its own running maximum, sum and O accumulator
         const int r = q4 * 32 + lane;
         const int q_pos = pos_t + r;                   // this query attends to keys 0 .. q_pos
         const uint32_t lane_addr = tmem_base + ((uint32_t)(q4 * 32) << 16);
+        const uint32_t o_addr = lane_addr + Cfg::O_COL + half * D2;
         constexpr float LOG2E = 1.4426950408889634f;
+        const float c_in = EXACT ? p.scale * LOG2E : 1.f;         // EXACT: scores in units of log 2 from here on
+        constexpr float C_EXP = EXACT ? 1.f : LOG2E;
         float m_run = -INFINITY, l_run = 0.f;
-        uint8_t* prow = sm_p + r * 128;
+        uint8_t* prow = sm_p + half * (BM * 128) + r * 128;
         const int sw = r & 7;
         for (int i = 0; i < n_tiles; ++i) {
             const int s = i & 1;
-            const int n0 = key_of(i);
+            const int n0 = key_of(i) + half * CW;
             mbar_wait_g(&s_full[s], (uint32_t)(i >> 1) & 1u, p.error);
             tc_fence_after();
-            uint32_t sv[BN];
+            uint32_t sv[CW];
 #pragma unroll
-            for (int c = 0; c < BN / 32; ++c) tmem_ld_32x32(lane_addr + s * BN + c * 32, *reinterpret_cast<uint32_t(*)[32]>(&sv[c * 32]));
+            for (int c = 0; c < CW / 32; ++c) tmem_ld_32x32(lane_addr + s * BN + half * CW + c * 32, *reinterpret_cast<uint32_t(*)[32]>(&sv[c * 32]));
             tc_wait_ld();
             tc_fence_before();
             __syncwarp();
             if (lane == 0) mbar_arrive(&s_free[s]);    // the next-but-one score tile may overwrite this buffer
-            float mx = m_run;
-            const bool diag = n0 + BN - 1 > pos_t || (MODE == FA_TILES && q_hi - 1 - n0 >= p.window && n0 + BN > p.keep);     // some (query, key) pairs of this tile are masked
+            if (EXACT) {
 #pragma unroll
-            for (int j = 0; j < BN; ++j) {
-                float v = __uint_as_float(sv[j]);
-                if (EXACT) v *= p.scale;
-                if (diag && (n0 + j > q_pos || (MODE == FA_TILES && q_pos - (n0 + j) >= p.window && n0 + j >= p.keep))) v = -INFINITY;
-                sv[j] = __float_as_uint(v);
-                mx = fmaxf(mx, v);
+                for (int j = 0; j < CW; ++j) sv[j] = __float_as_uint(__uint_as_float(sv[j]) * c_in);
             }
-            const float m_new = mx;
-            const float ms = (m_new == -INFINITY) ? 0.f : m_new * LOG2E;
-            const float alpha = (m_run == -INFINITY) ? 0.f : exp2f(m_run * LOG2E - ms);
-            float sum = 0.f;
+            if (n0 + CW - 1 > pos_t || (MODE == FA_TILES && q_hi - 1 - n0 >= p.window && n0 + CW > p.keep)) {     // some (query, key) pairs are masked
+#pragma unroll
+                for (int j = 0; j < CW; ++j)
+                    if (n0 + j > q_pos || (MODE == FA_TILES && q_pos - (n0 + j) >= p.window && n0 + j >= p.keep)) sv[j] = __float_as_uint(-INFINITY);
+            }
+            float mx[4] = {m_run, -INFINITY, -INFINITY, -INFINITY};
+#pragma unroll
+            for (int j = 0; j < CW; ++j) mx[j & 3] = fmaxf(mx[j & 3], __uint_as_float(sv[j]));
+            const float m_new = fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3]));
+            const float ms = (m_new == -INFINITY) ? 0.f : m_new * C_EXP;
+            const float alpha = (m_run == -INFINITY) ? 0.f : exp2f(m_run * C_EXP - ms);
+            float sum[2] = {0.f, 0.f};
             // the weights replace the scores in registers: fp16 pairs in the lower half of sv (FA_PAGED), or fp32 until they are split
 #pragma unroll
-            for (int j = 0; j < BN; j += 2) {
-                const float p0 = exp2f(__uint_as_float(sv[j]) * LOG2E - ms);
-                const float p1 = exp2f(__uint_as_float(sv[j + 1]) * LOG2E - ms);
+            for (int j = 0; j < CW; j += 2) {
+                const float p0 = exp2f(__uint_as_float(sv[j]) * C_EXP - ms);
+                const float p1 = exp2f(__uint_as_float(sv[j + 1]) * C_EXP - ms);
                 if (EXACT) {
-                    sum += p0 + p1;
+                    sum[0] += p0;
+                    sum[1] += p1;
                     sv[j] = __float_as_uint(p0);
                     sv[j + 1] = __float_as_uint(p1);
                 } else {
                     const __half2 h = __floats2half2_rn(p0, p1);
                     const float2 hf = __half22float2(h);             // the sum uses the rounded values the tensor core will see
-                    sum += hf.x + hf.y;
+                    sum[0] += hf.x + hf.y;
                     sv[j / 2] = *reinterpret_cast<const uint32_t*>(&h);
                 }
             }
-            l_run = l_run * alpha + sum;
+            l_run = l_run * alpha + (sum[0] + sum[1]);
             m_run = m_new;
             if (i > 0) {
-                mbar_wait_g(pv_done, (uint32_t)(i - 1) & 1u, p.error);       // P.V of the previous tile has read P and updated O
+                mbar_wait_g(&pv_done[half], (uint32_t)(i - 1) & 1u, p.error);       // P.V of the previous tile has read P and updated O
                 tc_fence_after();
                 if (__any_sync(0xffffffffu, alpha != 1.f)) {      // a row maximum grew: rescale this warp's 32 rows of O
 #pragma unroll 1
                     for (int c = 0; c < D2 / 32; ++c) {
                         uint32_t o[32];
-                        tmem_ld_32x32(lane_addr + Cfg::O_COL + c * 32, o);
+                        tmem_ld_32x32(o_addr + c * 32, o);
                         tc_wait_ld();
 #pragma unroll
                         for (int j = 0; j < 32; ++j) o[j] = __float_as_uint(__uint_as_float(o[j]) * alpha);
-                        tmem_st_32x32(lane_addr + Cfg::O_COL + c * 32, o);
+                        tmem_st_32x32(o_addr + c * 32, o);
                     }
                     tc_wait_st();
                 }
             }
             // P row -> shared memory, K-major swizzled (16-byte chunk c of 64-key block b lands at chunk c ^ (r & 7))
 #pragma unroll
-            for (int b = 0; b < BN / 64; ++b)
+            for (int b = 0; b < CW / 64; ++b)
 #pragma unroll
                 for (int c = 0; c < 8; ++c) {
                     uint8_t* dst = prow + b * (BM * 128) + ((c ^ sw) << 4);
@@ -336,24 +353,61 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_co
             fence_proxy_async();
             tc_fence_before();
             __syncwarp();
-            if (lane == 0) mbar_arrive(p_full);
+            if (lane == 0) mbar_arrive(&p_full[half]);
         }
-        // epilogue: O / l -> fp16
-        mbar_wait_g(pv_done, (uint32_t)(n_tiles - 1) & 1u, p.error);
+        // epilogue: O / l in the output type; with two halves their accumulators are joined here
+        for (int h = 0; h < HALVES; ++h) mbar_wait_g(&pv_done[h], (uint32_t)(n_tiles - 1) & 1u, p.error);
         tc_fence_after();
+        float w0 = 1.f, w1 = 0.f;
+        if constexpr (HALVES == 2) {
+            float2* ml = reinterpret_cast<float2*>(sm_q);       // [half][128 rows]: every score product has read Q
+            ml[half * BM + r] = make_float2(m_run, l_run);
+            asm volatile("bar.sync 1, 256;" ::: "memory");      // the eight softmax warps
+            const float2 a = ml[r], b = ml[BM + r];
+            const float m = fmaxf(a.x, b.x);
+            w0 = a.x == -INFINITY ? 0.f : exp2f(a.x - m);
+            w1 = b.x == -INFINITY ? 0.f : exp2f(b.x - m);
+            l_run = a.y * w0 + b.y * w1;
+        }
         float inv = l_run > 0.f ? 1.f / l_run : 0.f;
         const int t = t0 + r;
         if (MODE == FA_ROWS && p.gate != nullptr && t < p.T) inv *= 1.f / (1.f + __expf(-p.gate[(size_t)t * p.ldg + hq]));
+        w0 *= inv;
+        w1 *= inv;
+        const bool wide = EXACT && ((p.V | p.ldo) & 7) == 0 && (reinterpret_cast<uintptr_t>(p.out) & 15) == 0;
 #pragma unroll 1
-        for (int c = 0; c < D2 / 32; ++c) {
+        for (int c = half * (D2 / 32 / HALVES); c < (half + 1) * (D2 / 32 / HALVES); ++c) {
             uint32_t o[32];
             tmem_ld_32x32(lane_addr + Cfg::O_COL + c * 32, o);
-            tc_wait_ld();
+            if constexpr (HALVES == 2) {
+                uint32_t o1[32];
+                tmem_ld_32x32(lane_addr + Cfg::O_COL + D2 + c * 32, o1);
+                tc_wait_ld();
+#pragma unroll
+                for (int j = 0; j < 32; ++j) o[j] = __float_as_uint(__uint_as_float(o[j]) * w0 + __uint_as_float(o1[j]) * w1);
+            } else {
+                tc_wait_ld();
+#pragma unroll
+                for (int j = 0; j < 32; ++j) o[j] = __float_as_uint(__uint_as_float(o[j]) * w0);
+            }
             if (EXACT) {
                 __nv_bfloat16* orow = reinterpret_cast<__nv_bfloat16*>(p.out) + (size_t)t * p.ldo + (size_t)hq * p.V;
+                if (wide) {
 #pragma unroll
-                for (int j = 0; j < 32; ++j)
-                    if (r < rows && c * 32 + j < p.V) orow[c * 32 + j] = __float2bfloat16_rn(__uint_as_float(o[j]) * inv);
+                    for (int j = 0; j < 32; j += 8) {
+                        uint32_t w[4];
+#pragma unroll
+                        for (int e = 0; e < 4; ++e) {
+                            const __nv_bfloat162 h = __floats2bfloat162_rn(__uint_as_float(o[j + 2 * e]), __uint_as_float(o[j + 2 * e + 1]));
+                            w[e] = *reinterpret_cast<const uint32_t*>(&h);
+                        }
+                        if (r < rows && c * 32 + j < p.V) *reinterpret_cast<uint4*>(orow + c * 32 + j) = make_uint4(w[0], w[1], w[2], w[3]);
+                    }
+                } else {
+#pragma unroll
+                    for (int j = 0; j < 32; ++j)
+                        if (r < rows && c * 32 + j < p.V) orow[c * 32 + j] = __float2bfloat16_rn(__uint_as_float(o[j]));
+                }
             } else if (t < p.T) {
                 __half* orow = reinterpret_cast<__half*>(p.out) + (size_t)t * p.ldo + (size_t)hq * D2;
 #pragma unroll
@@ -361,7 +415,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_co
                     uint32_t w[4];
 #pragma unroll
                     for (int e = 0; e < 4; ++e) {
-                        const __half2 h = __floats2half2_rn(__uint_as_float(o[j + 2 * e]) * inv, __uint_as_float(o[j + 2 * e + 1]) * inv);
+                        const __half2 h = __floats2half2_rn(__uint_as_float(o[j + 2 * e]), __uint_as_float(o[j + 2 * e + 1]));
                         w[e] = *reinterpret_cast<const uint32_t*>(&h);
                     }
                     *reinterpret_cast<uint4*>(orow + c * 32 + j) = make_uint4(w[0], w[1], w[2], w[3]);

@@ -55,7 +55,7 @@ static int launch_rows(const void* q, const void* k, const void* v, int ldkv, in
     if ((rc = make_tmap_2d(&tv, v, 1, (uint64_t)S, (uint64_t)p.Hkv * D2, (uint64_t)ldkv, Cfg::BN))) return rc;
     auto kern = attn_prefill_tc_kernel<D1, D2, FA_ROWS>;
     if (first_use_on_device((const void*)kern)) DLP_CHECK_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, Cfg::SMEM_BYTES));
-    kern<<<dim3((p.T + Cfg::BM - 1) / Cfg::BM, p.Hq), 192, Cfg::SMEM_BYTES, s>>>(tq, tk, tv, p);
+    kern<<<dim3((p.T + Cfg::BM - 1) / Cfg::BM, p.Hq), Cfg::THREADS, Cfg::SMEM_BYTES, s>>>(tq, tk, tv, p);
     DLP_LAUNCH_CHECK();
     return 0;
 }

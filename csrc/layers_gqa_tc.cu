@@ -16,7 +16,7 @@ static int launch_tiles(const GqaArgs& a, FaParams p, cudaStream_t s) {
     if ((rc = make_tmap_2d(&tv, a.vc, 1, rows, a.Vc, a.Vc, (uint32_t)a.page_size))) return rc;
     auto kern = attn_prefill_tc_kernel<D1, D2, FA_TILES>;
     if (first_use_on_device((const void*)kern)) DLP_CHECK_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, Cfg::SMEM_BYTES));
-    kern<<<dim3(a.n_tiles, a.H), 192, Cfg::SMEM_BYTES, s>>>(tq, tk, tv, p);
+    kern<<<dim3(a.n_tiles, a.H), Cfg::THREADS, Cfg::SMEM_BYTES, s>>>(tq, tk, tv, p);
     DLP_LAUNCH_CHECK();
     return 0;
 }

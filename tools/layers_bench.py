@@ -1,5 +1,6 @@
 #!/usr/bin/env python
-"""Throughput of layer-list models beside a Llama of equal size, and every kernel of both against its roofline (`bench.py --layers`).
+"""Throughput of layer-list models beside the closest GGUF model of equal size, and every kernel of both against its roofline
+(`bench.py --layers`): Talizen beside a Llama, Vozinex beside a Qwen3-MoE.
 
 Random weights at sizes of real models' layers.  Model numbers are device-timed with CUDA events around whole forwards (prefill) and
 blocks of graph replays (decode); a step streams weights larger than L2.  Kernel numbers: a captured graph of launches that rotate
@@ -24,6 +25,10 @@ SIZES = {   # name: (width, heads, head size, latent rank, ff, layers)
     "2048": (2048, 16, 128, 512, 5632, 8),
     "4096": (4096, 32, 128, 512, 14336, 4),
 }
+MOE_SIZES = {   # name: (width, heads, key / value heads, head size, experts, experts per token, ff of an expert, layers, window, kept first tokens)
+    "moe-2048": (2048, 32, 4, 128, 64, 8, 768, 4, 1984, 64),
+    "moe-4096": (4096, 32, 8, 128, 16, 2, 4096, 4, 1984, 64),
+}
 VOCAB = 32000
 
 
@@ -38,7 +43,7 @@ def peaks():
 def talizen(size: str):
     """Three recurrent layers to one of latent attention, a feed-forward in each, as weights in device memory."""
     from distributed_llm_pipeline_b200.gguf.constants import GGMLType
-    from distributed_llm_pipeline_b200.models.layered import LayeredLayer, LayeredWeights
+    from distributed_llm_pipeline_b200.models.layered import LayeredLayer, LayeredWeights, Norm
     from distributed_llm_pipeline_b200.models.mixers import MIXERS, MLPS
     from distributed_llm_pipeline_b200.models.modeldir import talizen_config
     from distributed_llm_pipeline_b200.ops.weights import DeviceWeight
@@ -59,11 +64,47 @@ def talizen(size: str):
             return {"f.b": torch.full((H * D,), 3.0), "lower": torch.rand(H * D) * 0.9, "norm": torch.ones(D), "dkv.norm": torch.ones(R)}[name]
         return g
     mlp_shapes = {"gate": (F, E), "up": (F, E), "down": (E, F)}
-    ones = torch.ones(E, device=DEV)
-    layers = {i: LayeredLayer(MIXERS[s.type](s.mixer, get(s.type), DEV, torch.bfloat16), ones, MLPS["dense"](s.mlp, lambda k: mat(*mlp_shapes[k]), DEV, torch.bfloat16), ones)
+    one = Norm(torch.ones(E, device=DEV))
+    layers = {i: LayeredLayer(MIXERS[s.type](s.mixer, get(s.type), DEV, torch.bfloat16, 1e-5), one, MLPS["dense"](s.mlp, lambda k: mat(*mlp_shapes[k]), DEV, torch.bfloat16, E), one)
               for i, s in enumerate(cfg.layers)}
     tab = [DeviceWeight(GGMLType.BF16, VOCAB, E, [mat(VOCAB, E)]) for _ in range(2)]
-    return LayeredWeights(cfg, layers, range(n), 0, 1, tab[0], ones, tab[1], (0, VOCAB), None)
+    return LayeredWeights(cfg, layers, range(n), 0, 1, tab[0], one.w, tab[1], (0, VOCAB), None)
+
+
+def vozinex(size: str):
+    """Windowed attention and routed experts in every layer, each layer once."""
+    from distributed_llm_pipeline_b200.gguf.constants import GGMLType
+    from distributed_llm_pipeline_b200.models.layered import LayeredLayer, LayeredWeights, Norm
+    from distributed_llm_pipeline_b200.models.mixers import MIXERS, MLPS
+    from distributed_llm_pipeline_b200.models.modeldir import vozinex_config
+    from distributed_llm_pipeline_b200.ops.weights import DeviceWeight
+    E, H, G, D, NE, k, F, n, window, keep = MOE_SIZES[size]
+    spec = {"type": "attention", "mixer": {"heads": H, "kv_heads": G, "dim": D, "vdim": D, "scale": D ** -0.5, "rot": {"dims": D, "base": 1e6}, "mask": {"size": window, "keep_first": keep}},
+            "mlp": {"kind": "moe", "expert": {"ff": F}, "router": {"experts": NE, "top": k}}}
+    cfg = vozinex_config({"width": E, "vocab": VOCAB, "norm": {"eps": 1e-5}, "layers": [spec] * n})
+
+    def mat(r, c):
+        return (torch.randn(r, c, device=DEV) * c ** -0.5).to(torch.bfloat16)
+    shapes = {"q": (H * D, E), "k": (G * D, E), "v": (G * D, E), "o": (E, H * D), "up": (F, E), "down": (E, F), "router": (NE, E)}
+    vecs = {"q.norm": H * D, "k.norm": G * D, "router.b": NE}
+
+    def get(name):
+        kind = name.split(".")[-1] if name.startswith("e") else name
+        return mat(*shapes[kind]) if kind in shapes else torch.ones(vecs[name])
+    norm = Norm(torch.ones(E, device=DEV), torch.zeros(E, device=DEV))
+    layers = {i: LayeredLayer(MIXERS[s.type](s.mixer, get, DEV, torch.bfloat16, 1e-5), norm, MLPS["moe"](s.mlp, get, DEV, torch.bfloat16, E), norm) for i, s in enumerate(cfg.layers)}
+    tab = [DeviceWeight(GGMLType.BF16, VOCAB, E, [mat(VOCAB, E)]) for _ in range(2)]
+    return LayeredWeights(cfg, layers, range(n), 0, 1, tab[0], norm.w, tab[1], (0, VOCAB), None, out_norm_b=norm.b)
+
+
+def qwen3moe(size: str):
+    from distributed_llm_pipeline_b200.gguf import write_synthetic_gguf
+    from distributed_llm_pipeline_b200.models.config import preset
+    from distributed_llm_pipeline_b200.models.weights import load_weights
+    E, H, G, D, NE, k, F, n, _, _ = MOE_SIZES[size]
+    cfg = preset("qwen3-30b-a3b", vocab_size=VOCAB, n_embd=E, n_layer=n, n_head=H, n_head_kv=G, head_dim=D, n_ff=F, rope_dim=D, n_expert=NE, n_expert_used=k)
+    with tempfile.TemporaryDirectory() as d:
+        return load_weights(write_synthetic_gguf(os.path.join(d, "m.gguf"), cfg, "F16", seed=0), DEV)
 
 
 def llama(size: str):
@@ -284,24 +325,196 @@ def kernel_numbers(size: str, ctx: int = 2048, T: int = 2048):
     return rows, src
 
 
+def moe_kernel_numbers(size: str, T: int = 2048):
+    """The same for windowed attention and routed experts beside Qwen3-MoE.  Decode attention reads what the window shows; expert weights
+    are streamed from other experts at every launch."""
+    from types import SimpleNamespace
+
+    from distributed_llm_pipeline_b200.gguf.constants import GGMLType
+    from distributed_llm_pipeline_b200.ops import api as ops
+    from distributed_llm_pipeline_b200.ops import layers as L
+    from distributed_llm_pipeline_b200.ops.weights import DeviceWeight
+    from distributed_llm_pipeline_b200.models.layered import key_ranges
+    L.load_library()
+    ops.need_full_library()
+    E, H, G, D, NE, k, F, _, window, keep = MOE_SIZES[size]
+    bf, f16, f32, i32 = torch.bfloat16, torch.float16, torch.float32, torch.int32
+    bw, fl, src = peaks()
+    rows = []
+
+    def rnd(*s, dt=bf):
+        return (torch.randn(*s, device=DEV) * 0.1).to(dt)
+
+    def add(model, kind, name, us, nbytes, flops):
+        roof = max(nbytes / bw, flops / fl) * 1e6
+        rows.append({"model": model, "kind": kind, "kernel": name, "us": round(us, 2), "roofline_us": round(roof, 2), "of_roofline": round(roof / us, 3)})
+    NI = (H + 2 * G) * D
+    ones, zero = torch.ones(E, device=DEV), torch.zeros(E, device=DEV)
+    for B in (1, 4):
+        for kind, N, K in (("matvec in", NI, E), ("matvec out", E, H * D), ("router", NE, E)):
+            nb, c = N * K * 2, copies(N * K * 2)
+            ws = [rnd(N, K) for _ in range(c)]
+            h, y, ho, x16, out = rnd(B, K, dt=f32), rnd(B, K, dt=f32), rnd(B, K, dt=f32), rnd(B, K), torch.zeros(B, N, device=DEV)
+            st = L.row_stage(x16, K, K, 1e-5) if kind == "matvec out" else L.row_stage(h, K, K, 1e-5, y, None, 1, ho, ones, 1, zero)
+            add("vozinex", f"{kind} B={B}", "matvec_kernel", graph_us(lambda i: L.matvec(st, ws[i], out, B), c), nb, 2 * B * N * K)
+            del ws
+            dw = [DeviceWeight(GGMLType.F16, N, K, [rnd(N, K, dt=f16)]) for _ in range(c)]
+            xh = rnd(B, K, dt=f16)
+            if kind == "matvec out":
+                us = graph_us(lambda i: ops.linear(dw[i], xh, "add", out=out), c)
+            elif kind == "matvec in":
+                us = graph_us(lambda i: ops.linear(dw[i], h, "f32", norm_w=ones, eps=1e-5, out=out), c)
+            else:
+                us = graph_us(lambda i: [ops.linear(dw[i], h[t:t + 1], "f32", norm_w=ones, eps=1e-5, out=out[t:t + 1]) for t in range(B)], c)
+            add("qwen3moe", f"{kind} B={B}", "gemv_dense_v3_kernel", us, nb, 2 * B * N * K)
+            del dw
+        # the chosen experts: k per token, other ones in every launch
+        A, sets = B * k, max(1, NE // (B * k))
+        stacks = copies(NE * F * E * 2)
+        n = sets * stacks
+        picks = [[(s * A + a) % NE for a in range(A)] for s in range(sets)]
+        hot = min(A, NE)
+        logits = []
+        for p in picks:
+            lg = torch.zeros(B, NE, device=DEV)
+            for a, e in enumerate(p):
+                lg[a // k, e] = 20.0 + a
+            logits.append(lg)
+        up, down = ([rnd(NE * F, E) for _ in range(stacks)], [rnd(NE * E, F) for _ in range(stacks)])
+        h, act, y = rnd(B, E, dt=f32), rnd(A, F), torch.zeros(B, E, device=DEV)
+        st, st2 = L.row_stage(h, E, E, 1e-5, w2=ones, b2=zero), L.row_stage(act, F, F, 1e-5)
+        us = graph_us(lambda i: L.expert_matvec(st, logits[i % sets], None, NE, k, up[i // sets], F, act, B, down=False), n)
+        add("vozinex", f"experts up B={B}", "expert_matvec_kernel", us, hot * F * E * 2, 2 * A * F * E)
+        us = graph_us(lambda i: L.expert_matvec(st2, logits[i % sets], None, NE, k, down[i // sets], E, y, B, down=True), n)
+        add("vozinex", f"experts down B={B}", "expert_matvec_kernel", us, hot * F * E * 2, 2 * A * F * E)
+        del up, down
+        gate, up, down = ([DeviceWeight(GGMLType.F16, NE * r, c, [rnd(NE * r, c, dt=f16)]) for _ in range(stacks)] for r, c in ((F, E), (F, E), (E, F)))
+        ids = [torch.tensor(p, device=DEV, dtype=i32) for p in picks]
+        acth, wt = rnd(A, F, dt=f16), torch.ones(A, device=DEV)
+        if NE <= 32:          # up to four rows: a mat-vec per (token, expert)
+            us = graph_us(lambda i: [ops.gemv_moe(gate[i // sets], h[a // k:a // k + 1], acth[a:a + 1], "swiglu", ids[i % sets][a:a + 1], F, w_up=up[i // sets], norm_w=ones, eps=1e-5)
+                                     for a in range(A)], n)
+            add("qwen3moe", f"experts up B={B}", "gemv (expert rows)", us, hot * 2 * F * E * 2, 4 * A * F * E)
+            us = graph_us(lambda i: [ops.gemv_moe(down[i // sets], acth[a:a + 1], y[a // k:a // k + 1], "add", ids[i % sets][a:a + 1], E, out_scale=wt[a:a + 1]) for a in range(A)], n)
+            add("qwen3moe", f"experts down B={B}", "gemv (expert rows)", us, hot * F * E * 2, 2 * A * F * E)
+        else:
+            plans = [ops.MoePlan(A, NE, DEV) for _ in ids]
+            for q, p in zip(ids, plans):
+                ops.moe_plan(q, NE, 16, p)
+            xs, yh = rnd(A, E, dt=f16), torch.zeros(A, E, device=DEV)
+            us = graph_us(lambda i: ops.linear_grouped(gate[i // sets], xs, acth, "swiglu", NE, F, 16, plans[i % sets], w_up=up[i // sets]), n)
+            add("qwen3moe", f"experts up B={B}", "gemm_tcgen05_kernel (grouped)", us, hot * 2 * F * E * 2, 4 * A * F * E)
+            us = graph_us(lambda i: ops.linear_grouped(down[i // sets], acth, yh, "f32", NE, E, 16, plans[i % sets]), n)
+            add("qwen3moe", f"experts down B={B}", "gemm_tcgen05_kernel (grouped)", us, hot * F * E * 2, 2 * A * F * E)
+        del gate, up, down
+    # decode attention: what the window shows of a long sequence, beside a plain cache of that many keys
+    m = SimpleNamespace(H=H, G=G, R=H // G, D=D, V=D, Dc=D, Vc=D, rot=D, window=window, keep=keep, eps=1e-5, scale=D ** -0.5, visible=lambda n: min(n, window + keep),
+                        q_norm=torch.ones(H * D, device=DEV), k_norm=torch.ones(G * D, device=DEV),
+                        inv_freq=(1e6 ** (-torch.arange(0, D, 2, dtype=torch.float64) / D)).float().to(DEV))
+    seen, ctx = window + keep, 8192
+    for B in (1, 4, 16):
+        c, mp = copies(B * seen * G * D * 4), ctx // 64
+        slot, pos = torch.arange(B, device=DEV, dtype=i32), torch.full((B,), ctx - 1, device=DEV, dtype=i32)
+        kc, vc = ([rnd(B * mp, G, 64, D) for _ in range(c)] for _ in range(2))
+        bt = torch.arange(B * mp, device=DEV, dtype=i32).view(B, mp)
+        proj, out = rnd(B, NI, dt=f32), torch.zeros(B, H * D, device=DEV, dtype=bf)
+        tiles = (slot, torch.ones_like(slot), B)
+        ns = key_ranges(m, B, L.gqa_tile(m.R, 1)[0], ctx)
+        us = graph_us(lambda i: L.gqa_decode(m, proj, kc[i], vc[i], bt, slot, pos, tiles, ns, out, B), c)
+        add("vozinex", f"attention decode B={B}", f"gqa_attn_mma_kernel (fused, {ns} key ranges)", us, B * seen * G * D * 4, 4 * B * H * seen * D)
+        del kc, vc
+        mp = (seen + 63) // 64
+        kc, vc = ([rnd(B * mp, G, 64, D, dt=f16) for _ in range(c)] for _ in range(2))
+        bt = torch.arange(B * mp, device=DEV, dtype=i32).view(B, mp)
+        kl, oh = torch.full((B,), seen, device=DEV, dtype=i32), torch.zeros(B, H * D, device=DEV, dtype=f16)
+        us = graph_us(lambda i: ops.attn_decode_rope(proj, m.inv_freq, kc[i], vc[i], bt, kl, H, G, D, bt_row=slot, n_splits=16, neox=True, out=oh), c)
+        add("qwen3moe", f"attention decode B={B}", "attn_decode_rope_kernel", us, B * seen * G * D * 4, 4 * B * H * seen * D)
+        qh = rnd(B, H * D, dt=f16)
+        ns = max(1, min(16, 2 * 148 // (B * G)))
+        wsl = (torch.zeros(B * H * ns * D, device=DEV), torch.zeros(B * H * ns * 2, device=DEV), torch.zeros(B * H, device=DEV, dtype=i32))
+        us = graph_us(lambda i: ops.attn_paged(qh, kc[i], vc[i], bt, kl, H, G, D, bt_row=slot, n_splits=ns, workspace=wsl, out=oh), c)
+        add("qwen3moe", f"attention decode B={B}", "attn_decode_kernel (without norm and rotation)", us, B * seen * G * D * 4, 4 * B * H * seen * D)
+        del kc, vc
+    # prompts
+    for kind, N, K in (("gemm in", NI, E), ("gemm out", E, H * D), ("router", NE, E)):
+        w, xi, out = rnd(N, K), rnd(T, K), torch.zeros(T, N, device=DEV)
+        add("vozinex", f"{kind} T={T}", "gemm_tcgen05_kernel", graph_us(lambda i: L.linear(xi, w, out), 1), (N * K + T * K + T * N * 2) * 2, 2 * T * N * K)
+        dw, xq = DeviceWeight(GGMLType.F16, N, K, [rnd(N, K, dt=f16)]), rnd(T, K, dt=f16)
+        o16 = torch.zeros(T, N, device=DEV, dtype=f16)
+        us = graph_us(lambda i: ops.linear(dw, xq, "f16", out=o16) if kind == "gemm in" else ops.linear(dw, xq, "add" if kind == "gemm out" else "f32", out=out), 1)
+        add("qwen3moe", f"{kind} T={T}", "gemm_tcgen05_kernel", us, (N * K + T * K + T * N * 2) * 2, 2 * T * N * K)
+    hs, y, xb, o16 = [rnd(T, E, dt=f32) for _ in range(4)], rnd(T, E, dt=f32), torch.zeros(T, E, device=DEV, dtype=bf), torch.zeros(T, E, device=DEV, dtype=f16)
+    us = graph_us(lambda i: L.stage_rows(L.row_stage(hs[i], E, E, 1e-5, y, None, 1, hs[i], ones, 1, zero), xb, T), 4)
+    add("vozinex", f"norm T={T}", "stage_rows_kernel", us, T * E * 14, 0)
+    add("qwen3moe", f"norm T={T}", "rmsnorm_kernel", graph_us(lambda i: ops.rmsnorm(hs[i], ones, 1e-5, delta=y, out=o16), 4), T * E * 14, 0)
+    A = T * k
+    logits = torch.randn(T, NE, device=DEV)
+    ids, w = torch.zeros(A, dtype=i32, device=DEV), torch.zeros(A, device=DEV)
+    add("vozinex", f"route T={T}", "route_kernel", graph_us(lambda i: L.route(logits, None, NE, k, ids, w, T), 1), T * NE * 4 + A * 8, 0)
+    add("qwen3moe", f"route T={T}", "moe_route_ex_kernel", graph_us(lambda i: ops.moe_route_ex(logits, NE, k, True, ids, w), 1), T * NE * 4 + A * 8, 0)
+    plan, per = ops.MoePlan(A, NE, DEV), A // NE
+    tile = 16 if per <= 16 else 32 if per <= 32 else 64 if per <= 96 else 128
+    add("both", f"plan T={T}", "moe_plan_kernel", graph_us(lambda i: ops.moe_plan(ids, NE, tile, plan), 1), A * 16, 0)
+    xs = rnd(A, E)
+    add("both", f"gather T={T}", "moe_gather_kernel", graph_us(lambda i: L.expert_gather(xb, plan, k, A, xs), 1), (T + A) * E * 2, 0)
+    up, down, act, ey = rnd(NE * F, E), rnd(NE * E, F), rnd(A, F), torch.zeros(A, E, device=DEV)
+    us = graph_us(lambda i: L.linear_grouped(xs, up, F, NE, tile, plan, act, relu2=True), 1)
+    add("vozinex", f"experts up T={T}", "gemm_tcgen05_kernel (grouped)", us, (NE * F * E + A * E + A * F) * 2, 2 * A * F * E)
+    us = graph_us(lambda i: L.linear_grouped(act, down, E, NE, tile, plan, ey), 1)
+    add("vozinex", f"experts down T={T}", "gemm_tcgen05_kernel (grouped)", us, (NE * F * E + A * F + A * E * 2) * 2, 2 * A * F * E)
+    us = graph_us(lambda i: L.expert_combine(ey, plan, w, T, k, y), 1)
+    add("vozinex", f"combine T={T}", "moe_combine_kernel", us, (A + T) * E * 4, 0)
+    add("qwen3moe", f"combine T={T}", "moe_combine_kernel", graph_us(lambda i: ops.moe_combine(ey, plan, w, T, k, y), 1), (A + 2 * T) * E * 4, 0)
+    del up, down
+    gate, up, down = (DeviceWeight(GGMLType.F16, NE * r, c, [rnd(NE * r, c, dt=f16)]) for r, c in ((F, E), (F, E), (E, F)))
+    xh, acth = rnd(A, E, dt=f16), rnd(A, F, dt=f16)
+    us = graph_us(lambda i: ops.linear_grouped(gate, xh, acth, "swiglu", NE, F, tile, plan, w_up=up), 1)
+    add("qwen3moe", f"experts up T={T}", "gemm_tcgen05_kernel (grouped)", us, (2 * NE * F * E + A * E + A * F) * 2, 4 * A * F * E)
+    us = graph_us(lambda i: ops.linear_grouped(down, acth, ey, "f32", NE, E, tile, plan), 1)
+    add("qwen3moe", f"experts down T={T}", "gemm_tcgen05_kernel (grouped)", us, (NE * F * E + A * F + A * E * 2) * 2, 2 * A * F * E)
+    proj, q = rnd(T, NI, dt=f32), torch.zeros(T, H * D, device=DEV, dtype=bf)
+    kc, vc = (rnd(4 * T // 64, G, 64, D) for _ in range(2))
+    bt = torch.arange(4 * T // 64, device=DEV, dtype=i32).view(1, -1)
+    slot0 = torch.zeros(T, device=DEV, dtype=i32)
+    out = torch.zeros(T, H * D, device=DEV, dtype=bf)
+    q16, k16, v16, o16 = rnd(T, H * D, dt=f16), rnd(4 * T // 64, G, 64, D, dt=f16), rnd(4 * T // 64, G, 64, D, dt=f16), torch.zeros(T, H * D, device=DEV, dtype=f16)
+    p16, ar = proj.to(f16), torch.arange(T, device=DEV, dtype=i32)
+    us = graph_us(lambda i: L.gqa_prepare(m, proj, kc, vc, bt, slot0, ar, ar, q, T), 1)
+    add("vozinex", f"norm, rotation, cache rows T={T}", "gqa_prepare_kernel", us, T * NI * 6, 0)
+    us = graph_us(lambda i: ops.rope_kv(p16, ar, ar, m.inv_freq, k16, v16, H, G, D, True), 1)
+    add("qwen3moe", f"norm, rotation, cache rows T={T}", "rope_kv_kernel", us, T * NI * 4, 0)
+    for p0 in (0, 3 * T):          # the whole prompt; a portion far behind the window
+        pos = torch.arange(p0, p0 + T, device=DEV, dtype=i32)
+        row0 = torch.arange(T - 128, -1, -128, device=DEV, dtype=i32)
+        tiles = (row0, torch.full_like(row0, 128), row0.numel())
+        mask = sum(min(p + 1, window + min(keep, max(0, p + 1 - window))) for p in range(p0, p0 + T))
+        us = graph_us(lambda i: L.gqa_flash(m, q, kc, vc, bt, slot0, pos, tiles, out, T), 1)
+        add("vozinex", f"attention prefill T={T} at {p0}", "attn_prefill_tc_kernel<FA_TILES>", us, (2 * H + 2 * G) * D * T * 2, 4 * mask * H * D)
+        us = graph_us(lambda i: ops.attn_prefill(q16, k16, v16, bt[0], p0, H, G, D, out=o16), 1)
+        add("qwen3moe", f"attention prefill T={T} at {p0}", "attn_prefill_tc_kernel", us, (2 * H + 2 * G) * D * T * 2, 4 * sum(range(p0 + 1, p0 + T + 1)) * H * D)
+    return rows, src
+
+
 def main(argv=None) -> dict:
     ap = argparse.ArgumentParser(description=__doc__.split("\n")[0])
-    ap.add_argument("--sizes", default=",".join(SIZES))
+    ap.add_argument("--sizes", default=",".join([*SIZES, *MOE_SIZES]))
     ap.add_argument("--no-models", action="store_true", help="kernels only")
     ap.add_argument("--no-kernels", action="store_true", help="whole models only")
     a = ap.parse_args(argv)
-    res = {"metric": "layers_bench", "unit": "tok/s", "data": "synthetic (random weights and token ids)", "dtype": "bf16 (talizen) / fp16 (llama)", "sizes": {}}
+    res = {"metric": "layers_bench", "unit": "tok/s", "data": "synthetic (random weights and token ids)", "dtype": "bf16 (talizen, vozinex) / fp16 (llama, qwen3moe)", "sizes": {}}
     for size in a.sizes.split(","):
-        E, H, D, R, F, n = SIZES[size]
-        r = {"config": {"width": E, "heads": H, "head_dim": D, "kv_rank": R, "ff": F, "layers": n, "vocab": VOCAB}}
+        moe = size in MOE_SIZES
+        names = ("width", "heads", "kv_heads", "head_dim", "experts", "experts_per_token", "ff", "layers", "window", "keep_first") if moe else \
+            ("width", "heads", "head_dim", "kv_rank", "ff", "layers")
+        r = {"config": {**dict(zip(names, MOE_SIZES[size] if moe else SIZES[size])), "vocab": VOCAB}}
         if not a.no_models:
-            for name, make in (("talizen", talizen), ("llama", llama)):
+            for name, make in (("vozinex", vozinex), ("qwen3moe", qwen3moe)) if moe else (("talizen", talizen), ("llama", llama)):
                 w = make(size)
                 r[name] = {"weights_gb": round(w.nbytes() / 1e9, 3), **model_numbers(w)}
                 del w
                 torch.cuda.empty_cache()
         if not a.no_kernels:
-            r["kernels"], res["peaks"] = kernel_numbers(size)
+            r["kernels"], res["peaks"] = (moe_kernel_numbers if moe else kernel_numbers)(size)
         res["sizes"][size] = r
     return res
 
