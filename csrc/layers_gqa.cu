@@ -48,6 +48,9 @@ __device__ __forceinline__ float gqa_sumsq(const float* x, int n) {      // this
     return s;
 }
 
+__device__ __forceinline__ void put2(__nv_bfloat16* d, float x, float y) { *reinterpret_cast<__nv_bfloat162*>(d) = __floats2bfloat162_rn(x, y); }
+__device__ __forceinline__ void put2(float* d, float x, float y) { *reinterpret_cast<float2*>(d) = make_float2(x, y); }
+
 template <typename WT>
 __global__ void __launch_bounds__(256) gqa_prepare_kernel(const GqaArgs a) {
     extern __shared__ __align__(16) uint8_t gq_smem[];
@@ -62,21 +65,23 @@ __global__ void __launch_bounds__(256) gqa_prepare_kernel(const GqaArgs a) {
     const float rq = a.q_norm ? 1.f / sqrtf(block_sum(gqa_sumsq(q, a.H * a.D), red) / (float)(a.H * a.D) + a.eps) : 1.f;
     const float rk = a.k_norm ? 1.f / sqrtf(block_sum(gqa_sumsq(k, a.G * a.D), red) / (float)(a.G * a.D) + a.eps) : 1.f;
     __syncthreads();
-    WT* qo = reinterpret_cast<WT*>(a.q) + (size_t)t * a.H * a.Dc;
-    for (int i = threadIdx.x; i < a.H * a.Dc; i += 256) {
-        const int h = i / a.Dc, d = i - h * a.Dc;
-        qo[i] = Act<WT>::from_f(d < a.D ? gqa_value(q + h * a.D, a.q_norm ? a.q_norm + h * a.D : nullptr, rq, cs, a.rot, d) : 0.f);
-    }
-    if (slot >= 0) {
-        const size_t page = slot / a.page_size, off = slot % a.page_size;
-        for (int i = threadIdx.x; i < a.G * a.Dc; i += 256) {
-            const int g = i / a.Dc, d = i - g * a.Dc;
-            reinterpret_cast<WT*>(a.kc)[((page * a.G + g) * a.page_size + off) * a.Dc + d] =
-                Act<WT>::from_f(d < a.D ? gqa_value(k + g * a.D, a.k_norm ? a.k_norm + g * a.D : nullptr, rk, cs, a.rot, d) : 0.f);
-        }
-        for (int i = threadIdx.x; i < a.G * a.Vc; i += 256) {
-            const int g = i / a.Vc, d = i - g * a.Vc;
-            reinterpret_cast<WT*>(a.vc)[((page * a.G + g) * a.page_size + off) * a.Vc + d] = Act<WT>::from_f(d < a.V ? v[g * a.V + d] : 0.f);
+    // a warp per head: query heads, then key heads, then value heads
+    const int lane = threadIdx.x & 31;
+    const size_t page = max(slot, 0) / a.page_size, off = max(slot, 0) % a.page_size;
+    for (int i = threadIdx.x >> 5; i < a.H + (slot >= 0 ? 2 * a.G : 0); i += 8) {
+        if (i < a.H + a.G) {
+            const bool is_q = i < a.H;
+            const int h = is_q ? i : i - a.H;
+            const float* x = (is_q ? q : k) + h * a.D;
+            const float* w = is_q ? a.q_norm : a.k_norm;
+            if (w) w += h * a.D;
+            WT* o = is_q ? reinterpret_cast<WT*>(a.q) + ((size_t)t * a.H + h) * a.Dc : reinterpret_cast<WT*>(a.kc) + ((page * a.G + h) * a.page_size + off) * a.Dc;
+            const float r = is_q ? rq : rk;
+            for (int d = lane * 2; d < a.Dc; d += 64) put2(o + d, d < a.D ? gqa_value(x, w, r, cs, a.rot, d) : 0.f, d + 1 < a.D ? gqa_value(x, w, r, cs, a.rot, d + 1) : 0.f);
+        } else {
+            const int g = i - a.H - a.G;
+            WT* o = reinterpret_cast<WT*>(a.vc) + ((page * a.G + g) * a.page_size + off) * a.Vc;
+            for (int d = lane * 2; d < a.Vc; d += 64) put2(o + d, d < a.V ? v[g * a.V + d] : 0.f, d + 1 < a.V ? v[g * a.V + d + 1] : 0.f);
         }
     }
     pdl_launch_dependents();

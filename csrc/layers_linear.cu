@@ -2,7 +2,7 @@
 //
 //   matvec_kernel        decode (1..4 rows): weights streamed once; the residual sum and the norms in front of a product run in the
 //                        prologue, GEGLU in the epilogue.  Any N, any K whose padded form is a multiple of 8.
-//   stage_rows_kernel    the same row preparation as one launch, for the tcgen05 GEMM sizes.
+//   stage_rows_kernel    the same row preparation as one launch, for the tcgen05 GEMM sizes (stage_ln_kernel: layer norm of wide rows).
 //   sgemm_kernel         fp32 storage, any number of rows (no reduced-precision product).
 //   head_matmul_kernel   one small matrix per head (latent attention's key absorption and value expansion), mma.sync m16n8k16.
 #include "layers_rows.cuh"
@@ -21,6 +21,61 @@ __global__ void __launch_bounds__(256) stage_rows_kernel(const RowStage p, XT* x
     const int t0 = blockIdx.x;
     stage_rows_dev<XT>(p, t0, 1, st_sums, true, xb + (size_t)t0 * ldxb, ldxb);
     pdl_launch_dependents();
+}
+
+// The pre-norm form (plain residual sum, layer norm) with the row in registers: everything is read once.  NV float4 per thread.
+template <typename XT, int NV>
+__global__ void __launch_bounds__(256) stage_ln_kernel(const RowStage p, XT* xb, int ldxb) {
+    __shared__ float red[32];
+    pdl_wait();
+    const int t = blockIdx.x, q = p.K >> 2;
+    float4 v[NV];
+    float a = 0.f;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+        const int k = (i * 256 + threadIdx.x) * 4;
+        v[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (k < p.K) {
+            v[i] = stage_x4<XT>(p, t, k);
+            if (p.y) {
+                const float4 y = *reinterpret_cast<const float4*>(p.y + (size_t)t * p.ldy + k);
+                v[i].x += y.x; v[i].y += y.y; v[i].z += y.z; v[i].w += y.w;
+            }
+            if (p.e) {
+                const float4 e = *reinterpret_cast<const float4*>(p.e + (size_t)t * p.lde + k);
+                v[i].x += e.x; v[i].y += e.y; v[i].z += e.z; v[i].w += e.w;
+            }
+            if (p.h_out) *reinterpret_cast<float4*>(p.h_out + (size_t)t * p.ldh + k) = v[i];
+        }
+        a += (v[i].x + v[i].y) + (v[i].z + v[i].w);
+    }
+    const float mean = block_sum(a, red) / (float)p.K;
+    a = 0.f;
+#pragma unroll
+    for (int i = 0; i < NV; ++i)
+        if (i * 256 + (int)threadIdx.x < q) {
+            v[i] = make_float4(v[i].x - mean, v[i].y - mean, v[i].z - mean, v[i].w - mean);
+            a = fmaf(v[i].x, v[i].x, fmaf(v[i].y, v[i].y, fmaf(v[i].z, v[i].z, fmaf(v[i].w, v[i].w, a))));
+        }
+    const float r = 1.f / sqrtf(block_sum(a, red) / (float)p.K + p.eps);
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+        const int k = (i * 256 + threadIdx.x) * 4;
+        if (k < p.K) {
+            const float4 w = *reinterpret_cast<const float4*>(p.w2 + k), b = *reinterpret_cast<const float4*>(p.b2 + k);
+            put4(xb + (size_t)t * ldxb + k, make_float4(fmaf(v[i].x * r, w.x, b.x), fmaf(v[i].y * r, w.y, b.y), fmaf(v[i].z * r, w.z, b.z), fmaf(v[i].w * r, w.w, b.w)));
+        }
+    }
+    pdl_launch_dependents();
+}
+template <typename XT>
+static cudaError_t launch_stage(const RowStage& st, XT* xb, int ldxb, int T, size_t smem, cudaStream_t s) {
+    if (st.b2 && !(st.y && st.w1) && stage_vec(st) && ldxb % 4 == 0 && st.K <= 8192) {
+        if (st.K <= 2048) return launch_pdl(stage_ln_kernel<XT, 2>, dim3(T), dim3(256), 0, s, st, xb, ldxb);
+        if (st.K <= 4096) return launch_pdl(stage_ln_kernel<XT, 4>, dim3(T), dim3(256), 0, s, st, xb, ldxb);
+        return launch_pdl(stage_ln_kernel<XT, 8>, dim3(T), dim3(256), 0, s, st, xb, ldxb);
+    }
+    return launch_pdl(stage_rows_kernel<XT>, dim3(T), dim3(256), smem, s, st, xb, ldxb);
 }
 
 // ---- decode mat-vec ------------------------------------------------------------------------------------------
@@ -183,8 +238,7 @@ int stage_rows(const RowStage& st, void* xb, int ldxb, int T, int f32, cudaStrea
     DLP_REQUIRE(xb && T > 0 && ldxb >= st.Kp, "stage_rows: bad argument");
     const size_t smem = stage_bytes(st, 1, 8);
     DLP_REQUIRE(smem <= 48 * 1024, "stage_rows: too many norm groups");
-    if (f32) DLP_CHECK_CUDA(launch_pdl(stage_rows_kernel<float>, dim3(T), dim3(256), smem, s, st, (float*)xb, ldxb));
-    else DLP_CHECK_CUDA(launch_pdl(stage_rows_kernel<__nv_bfloat16>, dim3(T), dim3(256), smem, s, st, (__nv_bfloat16*)xb, ldxb));
+    DLP_CHECK_CUDA(f32 ? launch_stage(st, (float*)xb, ldxb, T, smem, s) : launch_stage(st, (__nv_bfloat16*)xb, ldxb, T, smem, s));
     return 0;
 }
 

@@ -445,7 +445,7 @@ def moe_kernel_numbers(size: str, T: int = 2048):
         add("qwen3moe", f"{kind} T={T}", "gemm_tcgen05_kernel", us, (N * K + T * K + T * N * 2) * 2, 2 * T * N * K)
     hs, y, xb, o16 = [rnd(T, E, dt=f32) for _ in range(4)], rnd(T, E, dt=f32), torch.zeros(T, E, device=DEV, dtype=bf), torch.zeros(T, E, device=DEV, dtype=f16)
     us = graph_us(lambda i: L.stage_rows(L.row_stage(hs[i], E, E, 1e-5, y, None, 1, hs[i], ones, 1, zero), xb, T), 4)
-    add("vozinex", f"norm T={T}", "stage_rows_kernel", us, T * E * 14, 0)
+    add("vozinex", f"norm T={T}", "stage_ln_kernel", us, T * E * 14, 0)
     add("qwen3moe", f"norm T={T}", "rmsnorm_kernel", graph_us(lambda i: ops.rmsnorm(hs[i], ones, 1e-5, delta=y, out=o16), 4), T * E * 14, 0)
     A = T * k
     logits = torch.randn(T, NE, device=DEV)
