@@ -36,7 +36,7 @@ __global__ void __launch_bounds__(512, 1) expert_matvec_kernel(const RowStage st
         }
         __syncthreads();
     } else {
-        stage_rows_dev<WT>(st, 0, T, sums, false, xs, K);
+        stage_rows_dev<WT, true>(st, 0, T, sums, false, xs, K);
     }
     float* part = sums;                  // [units][2]
     uint4 buf[2][2][U];

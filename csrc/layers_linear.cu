@@ -14,12 +14,12 @@ __device__ __forceinline__ float gelu_tanh_f(float z) {
     return 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
 }
 
-template <typename XT>
+template <typename XT, bool FULL>
 __global__ void __launch_bounds__(256) stage_rows_kernel(const RowStage p, XT* xb, int ldxb) {
     extern __shared__ __align__(16) float st_sums[];
     pdl_wait();
     const int t0 = blockIdx.x;
-    stage_rows_dev<XT>(p, t0, 1, st_sums, true, xb + (size_t)t0 * ldxb, ldxb);
+    stage_rows_dev<XT, FULL>(p, t0, 1, st_sums, true, xb + (size_t)t0 * ldxb, ldxb);
     pdl_launch_dependents();
 }
 
@@ -75,14 +75,15 @@ static cudaError_t launch_stage(const RowStage& st, XT* xb, int ldxb, int T, siz
         if (st.K <= 4096) return launch_pdl(stage_ln_kernel<XT, 4>, dim3(T), dim3(256), 0, s, st, xb, ldxb);
         return launch_pdl(stage_ln_kernel<XT, 8>, dim3(T), dim3(256), 0, s, st, xb, ldxb);
     }
-    return launch_pdl(stage_rows_kernel<XT>, dim3(T), dim3(256), smem, s, st, xb, ldxb);
+    if (stage_full(st)) return launch_pdl(stage_rows_kernel<XT, true>, dim3(T), dim3(256), smem, s, st, xb, ldxb);
+    return launch_pdl(stage_rows_kernel<XT, false>, dim3(T), dim3(256), smem, s, st, xb, ldxb);
 }
 
 // ---- decode mat-vec ------------------------------------------------------------------------------------------
 // A unit is two weight rows x (32 * VEC * U) columns: U 16-byte loads per row and lane.  A block owns a contiguous range of row
 // pairs, its warps take the units in a fixed order and always hold the next unit's loads while they reduce the current one.  The
 // first unit is requested before the dependency wait: weights do not depend on the previous kernel.
-template <typename WT, int NT>
+template <typename WT, int NT, bool FULL>
 __global__ void __launch_bounds__(512, 1) matvec_kernel(const RowStage st, const WT* __restrict__ w, int ldw, int N, void* out, int ldo, int out_mode, int T) {
     constexpr int VEC = Act<WT>::VEC, U = 4, COLS = 32 * VEC * U;
     extern __shared__ __align__(16) uint8_t mv_smem[];
@@ -110,7 +111,7 @@ __global__ void __launch_bounds__(512, 1) matvec_kernel(const RowStage st, const
     int u = warp;
     if (u < units) issue(u, 0);
     pdl_wait();
-    stage_rows_dev<WT>(st, 0, T, sums, blockIdx.x == 0, xs, K);
+    stage_rows_dev<WT, FULL>(st, 0, T, sums, blockIdx.x == 0, xs, K);
     float* part = sums;      // [units][2][NT]: the staging scratch is free again
     auto reduce = [&](int u, int b) {
         const int pr = u / KC, c = u - pr * KC;
@@ -209,7 +210,7 @@ static int launch_matvec(const RowStage& st, const void* w, int ldw, int N, void
     const size_t part = (size_t)((pairs + grid - 1) / grid) * KC * 2 * NT * 4, stg = stage_bytes(st, T, 16);
     const size_t smem = xbytes + (part > stg ? part : stg);
     DLP_REQUIRE(smem <= 227 * 1024, "matvec: %d rows of width %d need %zu bytes of shared memory", T, st.Kp, smem);
-    auto kern = matvec_kernel<WT, NT>;
+    auto kern = stage_full(st) ? matvec_kernel<WT, NT, true> : matvec_kernel<WT, NT, false>;
     if (first_use_on_device((const void*)kern))
         DLP_CHECK_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024));
     DLP_CHECK_CUDA(launch_pdl(kern, dim3(grid), dim3(512), smem, s, st, (const WT*)w, ldw, N, out, ldo, out_mode, T));

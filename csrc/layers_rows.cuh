@@ -142,20 +142,22 @@ __device__ __forceinline__ float4 stage_x4(const RowStage& p, int t, int k) {
     const float2 a = bf2_to_f2(u.x), b = bf2_to_f2(u.y);
     return make_float4(a.x, a.y, b.x, b.y);
 }
-template <typename XT, typename Put4>
+// FULL = false leaves out what norms behind the sublayers do not need (y without w1, e, b2): fewer registers in the prologue.
+inline bool stage_full(const RowStage& p) { return p.e || p.b2 || (p.y && !p.w1); }
+template <typename XT, bool FULL, typename Put4>
 __device__ __forceinline__ void stage_rows_vec(const RowStage& p, int t0, int rows, float* sums, bool store_h, Put4 put) {
     const float* rs1 = nullptr;
     const float* rs2 = nullptr;
     const int gs1 = p.y ? p.K / p.groups1 : 1, gs2 = p.w2 ? p.K / p.groups2 : 1;
     auto y4 = [&](int t, int k) { return *reinterpret_cast<const float4*>(p.y + (size_t)(t0 + t) * p.ldy + k); };
-    if (p.y && p.w1) {
+    if (p.y && (!FULL || p.w1)) {
         rs1 = stage_rms_vec(rows, p.groups1, p.K, p.eps, sums, y4);
         sums += rows * (p.K / 128 + p.groups1);
     }
     auto add4 = [](float4& v, float4 a) { v.x += a.x; v.y += a.y; v.z += a.z; v.w += a.w; };
     auto base = [&](int t, int k) {
         float4 v = stage_x4<XT>(p, t0 + t, k);
-        if (p.y && !p.w1) {
+        if (FULL && p.y && !p.w1) {
             add4(v, y4(t, k));
         } else if (p.y) {
             const float4 y = y4(t, k), w = *reinterpret_cast<const float4*>(p.w1 + k);
@@ -165,17 +167,17 @@ __device__ __forceinline__ void stage_rows_vec(const RowStage& p, int t0, int ro
             v.z = fmaf(y.z * r, w.z, v.z);
             v.w = fmaf(y.w * r, w.w, v.w);
         }
-        if (p.e) add4(v, *reinterpret_cast<const float4*>(p.e + (size_t)(t0 + t) * p.lde + k));
+        if (FULL && p.e) add4(v, *reinterpret_cast<const float4*>(p.e + (size_t)(t0 + t) * p.lde + k));
         return v;
     };
-    if (p.w2) rs2 = p.b2 ? stage_moments_vec(rows, p.K, p.eps, sums, base) : stage_rms_vec(rows, p.groups2, p.K, p.eps, sums, base);
+    if (p.w2) rs2 = FULL && p.b2 ? stage_moments_vec(rows, p.K, p.eps, sums, base) : stage_rms_vec(rows, p.groups2, p.K, p.eps, sums, base);
     const int q = p.K >> 2;
 #pragma unroll 2
     for (int i = threadIdx.x; i < rows * q; i += blockDim.x) {
         const int t = i / q, k = (i - t * q) * 4;
         float4 v = base(t, k);
         if (store_h && p.h_out) *reinterpret_cast<float4*>(p.h_out + (size_t)(t0 + t) * p.ldh + k) = v;
-        if (p.w2 && p.b2) {
+        if (FULL && p.w2 && p.b2) {
             const float m = rs2[2 * t], r = rs2[2 * t + 1];
             const float4 w = *reinterpret_cast<const float4*>(p.w2 + k), b = *reinterpret_cast<const float4*>(p.b2 + k);
             v = make_float4(fmaf((v.x - m) * r, w.x, b.x), fmaf((v.y - m) * r, w.y, b.y), fmaf((v.z - m) * r, w.z, b.z), fmaf((v.w - m) * r, w.w, b.w));
@@ -194,24 +196,24 @@ __device__ __forceinline__ void put4(__nv_bfloat16* d, float4 v) {
 }
 __device__ __forceinline__ void put4(float* d, float4 v) { *reinterpret_cast<float4*>(d) = v; }
 
-template <typename XT>
+template <typename XT, bool FULL>
 __device__ __forceinline__ void stage_rows_dev(const RowStage& p, int t0, int rows, float* sums, bool store_h, XT* dst, int ldd) {
     if (stage_vec(p)) {
-        stage_rows_vec<XT>(p, t0, rows, sums, store_h, [&](int t, int k, float4 v) { put4(dst + (size_t)t * ldd + k, v); });
+        stage_rows_vec<XT, FULL>(p, t0, rows, sums, store_h, [&](int t, int k, float4 v) { put4(dst + (size_t)t * ldd + k, v); });
         return;
     }
     const float* rs1 = nullptr;
     const float* rs2 = nullptr;
     const int gs1 = p.y ? p.K / p.groups1 : 1, gs2 = p.w2 ? p.K / p.groups2 : 1;
-    if (p.y && p.w1) rs1 = stage_rms(rows, p.groups1, p.K, p.eps, sums, [&](int t, int k) { return p.y[(size_t)(t0 + t) * p.ldy + k]; });
+    if (p.y && (!FULL || p.w1)) rs1 = stage_rms(rows, p.groups1, p.K, p.eps, sums, [&](int t, int k) { return p.y[(size_t)(t0 + t) * p.ldy + k]; });
     auto base = [&](int t, int k) {
         float v = stage_x0<XT>(p, t0 + t, k);
-        if (p.y) v += p.w1 ? p.y[(size_t)(t0 + t) * p.ldy + k] * rs1[t * p.groups1 + k / gs1] * p.w1[k] : p.y[(size_t)(t0 + t) * p.ldy + k];
-        if (p.e) v += p.e[(size_t)(t0 + t) * p.lde + k];
+        if (p.y) v += !FULL || p.w1 ? p.y[(size_t)(t0 + t) * p.ldy + k] * rs1[t * p.groups1 + k / gs1] * p.w1[k] : p.y[(size_t)(t0 + t) * p.ldy + k];
+        if (FULL && p.e) v += p.e[(size_t)(t0 + t) * p.lde + k];
         return v;
     };
-    if (p.y && p.w1) sums += stage_scratch(rows, p.groups1, blockDim.x >> 5);
-    if (p.w2) rs2 = p.b2 ? stage_moments(rows, p.K, p.eps, sums, base) : stage_rms(rows, p.groups2, p.K, p.eps, sums, base);
+    if (p.y && (!FULL || p.w1)) sums += stage_scratch(rows, p.groups1, blockDim.x >> 5);
+    if (p.w2) rs2 = FULL && p.b2 ? stage_moments(rows, p.K, p.eps, sums, base) : stage_rms(rows, p.groups2, p.K, p.eps, sums, base);
     for (int t = 0; t < rows; ++t) {
 #pragma unroll 4
         for (int k = threadIdx.x; k < p.Kp; k += blockDim.x) {
@@ -219,7 +221,7 @@ __device__ __forceinline__ void stage_rows_dev(const RowStage& p, int t0, int ro
             if (k < p.K) {
                 v = base(t, k);
                 if (store_h && p.h_out) p.h_out[(size_t)(t0 + t) * p.ldh + k] = v;
-                if (p.w2) v = p.b2 ? fmaf((v - rs2[2 * t]) * rs2[2 * t + 1], p.w2[k], p.b2[k]) : v * (rs2[t * p.groups2 + k / gs2] * p.w2[k % p.w2_mod]);
+                if (p.w2) v = FULL && p.b2 ? fmaf((v - rs2[2 * t]) * rs2[2 * t + 1], p.w2[k], p.b2[k]) : v * (rs2[t * p.groups2 + k / gs2] * p.w2[k % p.w2_mod]);
             }
             dst[(size_t)t * ldd + k] = Act<XT>::from_f(v);
         }
