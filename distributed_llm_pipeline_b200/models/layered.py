@@ -3,8 +3,8 @@
 The residual stream is fp32.  A sublayer's output `y` is not added at once: it stays pending, and the next matrix product forms
 `h + y` (or `h + norm(y)`), and the norm in front of it, while it prepares its input rows (in the mat-vec prologue for up to four rows, in
 one row kernel in front of the GEMM for more).  A range of layers may run several times: every run has its own cache and state, and the
-embedding output joins at the start of every pass but the first.  One forward takes any mix of prompt portions and single tokens of different sequences: projections run over all rows,
-mixers over the segments.
+embedding output joins at the start of every pass but the first.  One forward takes any mix of prompt portions and single tokens of
+different sequences: projections run over all rows, mixers over the segments.
 """
 from __future__ import annotations
 
