@@ -80,6 +80,7 @@ struct FaParams {
     int ldg, V;             // V: value size of a head (<= D2; the rest of the tile is padding)
     float scale;
     int* error;             // set when a wait ran into its limit
+    int window, keep, chunk;       // (FA_PAGED: none) position i sees key j <= i when i - j < window and (chunk > 0) both are in one chunk, or when j < keep
     // FA_TILES
     const int* tile_row0;   // [grid.x] first query row of a tile, and its rows (consecutive positions of one sequence)
     const int* tile_rows;
@@ -87,7 +88,6 @@ struct FaParams {
     const int* tok_slot;    // [T] block-table row
     const int* block_table;
     int q_head;             // columns from one query head to the next
-    int window, keep, chunk;       // position i sees key j <= i when i - j < window and (chunk > 0) both are in one chunk, or when j < keep
     int maps, out_f32;      // maps: query heads take turns over that many key heads of a key / value head;  out is fp32
 };
 // FA_PAGED: fp16, K / V pages of a [pages][Hkv][page][D] cache, queries scaled in advance, fp16 softmax weights
@@ -99,7 +99,7 @@ enum FaMode : int { FA_PAGED = 0, FA_ROWS = 1, FA_TILES = 2 };
 
 template <int D1, int D2, int MODE>
 struct FaCfg {
-    static constexpr int BM = 128, BN = 128;
+    static constexpr int BM = 128, BN = D1 > 128 ? 64 : 128;      // (wider keys: shorter key tiles)
     static constexpr int KB = D1 / 64, VB = D2 / 64;
     static constexpr int Q_BYTES = BM * D1 * 2;
     static constexpr int K_BYTES = BN * D1 * 2, V_BYTES = BN * D2 * 2;
@@ -148,10 +148,10 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_co
     const int kvh = hq / (p.Hq / p.Hkv);
     const int q_hi = pos_t + rows;                    // keys visible to the last query of this tile
     auto first_key = [&](int pos) { return max(max(0, pos - p.window + 1), p.chunk > 0 ? pos / p.chunk * p.chunk : 0); };
-    const int lo_tile = MODE == FA_TILES ? first_key(pos_t) / BN : 0;            // first key tile the window shows
-    const int keep_tiles = MODE == FA_TILES ? min((p.keep + BN - 1) / BN, lo_tile) : 0;      // kept tiles in front of it
+    const int lo_tile = EXACT ? first_key(pos_t) / BN : 0;                       // first key tile the window shows
+    const int keep_tiles = EXACT ? min((p.keep + BN - 1) / BN, lo_tile) : 0;      // kept tiles in front of it
     const int n_tiles = keep_tiles + (q_hi + BN - 1) / BN - lo_tile;
-    auto key_of = [&](int i) { return (MODE == FA_TILES && i >= keep_tiles ? lo_tile - keep_tiles + i : i) * BN; };
+    auto key_of = [&](int i) { return (EXACT && i >= keep_tiles ? lo_tile - keep_tiles + i : i) * BN; };
 
     if (warp == 0 && lane == 0) {
         tma_prefetch_desc(&tm_q);
@@ -265,14 +265,13 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_co
         const int half = (warp - 2) >> 2;              // its own running maximum, sum and O accumulator
         const int r = q4 * 32 + lane;
         const int q_pos = pos_t + r;                   // this query attends to keys 0 .. q_pos
-        const int q_first = MODE == FA_TILES ? first_key(q_pos) : 0, q_first_hi = MODE == FA_TILES ? first_key(q_hi - 1) : 0;      // (FA_TILES: from its first key on, and the kept ones)
+        const int q_first = EXACT ? first_key(q_pos) : 0, q_first_hi = EXACT ? first_key(q_hi - 1) : 0;      // (from its first key on, and the kept ones)
         const uint32_t lane_addr = tmem_base + ((uint32_t)(q4 * 32) << 16);
         const uint32_t o_addr = lane_addr + Cfg::O_COL + half * D2;
         constexpr float LOG2E = 1.4426950408889634f;
         const float c_in = EXACT ? p.scale * LOG2E : 1.f;         // EXACT: scores in units of log 2 from here on
         constexpr float C_EXP = EXACT ? 1.f : LOG2E;
         float m_run = -INFINITY, l_run = 0.f;
-        uint8_t* prow = sm_p + half * (BM * 128) + r * 128;
         const int sw = r & 7;
         for (int i = 0; i < n_tiles; ++i) {
             const int s = i & 1;
@@ -290,10 +289,10 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_co
 #pragma unroll
                 for (int j = 0; j < CW; ++j) sv[j] = __float_as_uint(__uint_as_float(sv[j]) * c_in);
             }
-            if (n0 + CW - 1 > pos_t || (MODE == FA_TILES && q_first_hi > n0 && n0 + CW > p.keep)) {     // some (query, key) pairs are masked
+            if (n0 + CW - 1 > pos_t || (EXACT && q_first_hi > n0 && n0 + CW > p.keep)) {     // some (query, key) pairs are masked
 #pragma unroll
                 for (int j = 0; j < CW; ++j)
-                    if (n0 + j > q_pos || (MODE == FA_TILES && n0 + j < q_first && n0 + j >= p.keep)) sv[j] = __float_as_uint(-INFINITY);
+                    if (n0 + j > q_pos || (EXACT && n0 + j < q_first && n0 + j >= p.keep)) sv[j] = __float_as_uint(-INFINITY);
             }
             float mx[4] = {m_run, -INFINITY, -INFINITY, -INFINITY};
 #pragma unroll
@@ -339,10 +338,11 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_co
             }
             // P row -> shared memory, K-major swizzled (16-byte chunk c of 64-key block b lands at chunk c ^ (r & 7))
 #pragma unroll
-            for (int b = 0; b < CW / 64; ++b)
+            for (int b = 0; b < (CW + 63) / 64; ++b)
 #pragma unroll
-                for (int c = 0; c < 8; ++c) {
-                    uint8_t* dst = prow + b * (BM * 128) + ((c ^ sw) << 4);
+                for (int c = 0; c < (CW < 64 ? CW : 64) / 8; ++c) {
+                    const int col = half * CW + b * 64 + c * 8;
+                    uint8_t* dst = sm_p + (col >> 6) * (BM * 128) + r * 128 + ((((col & 63) >> 3) ^ sw) << 4);
                     if (EXACT) {
                         uint32_t hi[4], lo[4];
 #pragma unroll

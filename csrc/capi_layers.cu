@@ -9,25 +9,30 @@ using namespace dlp;
 
 static_assert(sizeof(dlp_row_stage) == sizeof(RowStage) && sizeof(dlp_hgrn2_args) == sizeof(Hgrn2Args) && sizeof(dlp_scan_chunks) == sizeof(ScanChunks) && sizeof(dlp_latent_args) == sizeof(LatentArgs) &&
               sizeof(dlp_expert_args) == sizeof(ExpertArgs) && sizeof(dlp_route_rule) == sizeof(RouteRule) && sizeof(dlp_ssd_args) == sizeof(SsdArgs) &&
-              sizeof(dlp_conv_args) == sizeof(ConvArgs) && sizeof(dlp_gqa_args) == sizeof(GqaArgs), "argument layout");
+              sizeof(dlp_conv_args) == sizeof(ConvArgs) && sizeof(dlp_gqa_args) == sizeof(GqaArgs) && sizeof(dlp_out_tail) == sizeof(OutTail) &&
+              sizeof(dlp_latent_rows) == sizeof(LatentRows) && sizeof(dlp_delta_args) == sizeof(DeltaArgs) && sizeof(dlp_delta_chunks) == sizeof(DeltaChunks), "argument layout");
 
 extern "C" {
 
-int dlp_layers_matvec(const dlp_row_stage* st, const void* w, int ldw, int N, void* out, int ldo, int out_mode, int T, int f32, void* stream) {
+int dlp_layers_matvec(const dlp_row_stage* st, const void* w, int ldw, int N, void* out, int ldo, int out_mode, const dlp_out_tail* tail, int T, int f32, void* stream) {
     DLP_REQUIRE(st, "dlp_layers_matvec: null argument");
-    return matvec(*reinterpret_cast<const RowStage*>(st), w, ldw, N, out, ldo, out_mode, T, f32, (cudaStream_t)stream);
+    return matvec(*reinterpret_cast<const RowStage*>(st), w, ldw, N, out, ldo, out_mode, T, f32, (cudaStream_t)stream, reinterpret_cast<const OutTail*>(tail));
 }
 int dlp_layers_stage_rows(const dlp_row_stage* st, void* xb, int ldxb, int T, int f32, void* stream) {
     DLP_REQUIRE(st, "dlp_layers_stage_rows: null argument");
     return stage_rows(*reinterpret_cast<const RowStage*>(st), xb, ldxb, T, f32, (cudaStream_t)stream);
 }
-int dlp_layers_linear(const void* x, int ldx, const void* w, int ldw, int N, int K, void* out, int ldo, int out_mode, int T, int f32, void* ws, size_t ws_bytes, void* stream) {
+int dlp_layers_linear(const void* x, int ldx, const void* w, int ldw, int N, int K, void* out, int ldo, int out_mode, const dlp_out_tail* tail, int T, int f32, void* ws, size_t ws_bytes,
+                      void* stream) {
+    const OutTail* tl = reinterpret_cast<const OutTail*>(tail);
     DLP_REQUIRE(x && w && out && N > 0 && T > 0, "dlp_layers_linear: bad argument");
-    if (f32) return sgemm((const float*)x, ldx, (const float*)w, ldw, N, K, out, ldo, out_mode, T, (cudaStream_t)stream);
+    if (f32) return sgemm((const float*)x, ldx, (const float*)w, ldw, N, K, out, ldo, out_mode, T, (cudaStream_t)stream, nullptr, tl);
+    DLP_REQUIRE(!tl || (out_mode == LO_F32 && tl->n2 >= 0 && (tl->n2 >= N || (tl->out2 && tl->ldo2 >= N - tl->n2))), "dlp_layers_linear: what follows the sums");
     if (out_mode == LO_GEGLU || out_mode == LO_SWIGLU)       // rows 2i / 2i+1 of the interleaved matrix: two operands with twice the row stride
         return gemm_f16(w, (const uint8_t*)w + (size_t)ldw * 2, 2 * ldw, x, ldx, out, ldo, T, N / 2, K, out_mode == LO_GEGLU ? 6 : 8, 1, 0, (cudaStream_t)stream, nullptr, nullptr, ws, ws_bytes);
     DLP_REQUIRE(out_mode == LO_F32 || out_mode == LO_BF16 || out_mode == LO_RELU2, "dlp_layers_linear: output mode %d", out_mode);
-    return gemm_f16(w, nullptr, ldw, x, ldx, out, ldo, T, N, K, out_mode == LO_BF16 ? 4 : out_mode == LO_RELU2 ? 7 : 1, 1, 0, (cudaStream_t)stream, nullptr, nullptr, ws, ws_bytes);
+    return gemm_f16(w, nullptr, ldw, x, ldx, out, ldo, T, N, K, tl ? 9 : out_mode == LO_BF16 ? 4 : out_mode == LO_RELU2 ? 7 : 1, 1, 0, (cudaStream_t)stream, nullptr, nullptr, ws, ws_bytes,
+                    tl);
 }
 int dlp_layers_head_matmul(const void* x, int x_f32, int ldx, int x_head, int kx, const void* w, int Kp, int H, int N, int n_rows, void* out, int ldo, int out_head,
                            const float* gate, int ldg, int T, int f32, void* stream) {
@@ -36,8 +41,15 @@ int dlp_layers_head_matmul(const void* x, int x_f32, int ldx, int x_head, int kx
 int dlp_layers_embed(const void* table, int ld, const int32_t* ids, float* h, int E, int T, int vocab, float scale, int f32, void* stream) {
     return embed_rows(table, ld, ids, h, E, T, vocab, scale, f32, (cudaStream_t)stream);
 }
-int dlp_layers_latent_write(const float* proj, int ldp, const float* w, float eps, int R, int Rc, const int32_t* slot, void* cache, int T, int f32, void* stream) {
-    return latent_write(proj, ldp, w, eps, R, Rc, slot, cache, T, f32, (cudaStream_t)stream);
+int dlp_layers_latent_write(const dlp_latent_rows* a, int T, int f32, void* stream) {
+    DLP_REQUIRE(a, "dlp_layers_latent_write: null argument");
+    return latent_write(*reinterpret_cast<const LatentRows*>(a), T, f32, (cudaStream_t)stream);
+}
+int dlp_layers_delta(const dlp_delta_args* a, const dlp_delta_chunks* chunks, const dlp_conv_args* conv, int mode, void* stream) {
+    DLP_REQUIRE(a && mode >= 0 && mode <= 2 && (mode != 1 || chunks), "dlp_layers_delta: bad argument");
+    const DeltaArgs& d = *reinterpret_cast<const DeltaArgs*>(a);
+    if (mode == 1) return delta_chunked(d, *reinterpret_cast<const DeltaChunks*>(chunks), (cudaStream_t)stream);
+    return mode == 2 ? delta_decode(d, reinterpret_cast<const ConvArgs*>(conv), (cudaStream_t)stream) : delta_scan(d, (cudaStream_t)stream);
 }
 int dlp_layers_hgrn2(const dlp_hgrn2_args* a, const dlp_scan_chunks* chunks, void* stream) {
     DLP_REQUIRE(a, "dlp_layers_hgrn2: null argument");
@@ -65,9 +77,9 @@ int dlp_layers_latent_gather(const void* cache, const int32_t* bt_row, int page,
 int dlp_layers_head_rows(const float* x, int ldx, int D, int Dp, int H, void* out, int T, void* stream) {
     return head_rows(x, ldx, D, Dp, H, out, T, (cudaStream_t)stream);
 }
-int dlp_layers_rows_attention(const void* q, const void* kv, int ldkv, int S, int T, int pos0, int H, int Dp, int Vp, int V, float scale, const float* gate, int ldg,
-                              void* out, int ldo, void* stream) {
-    return rows_attention(q, kv, ldkv, S, T, pos0, H, Dp, Vp, V, scale, gate, ldg, out, ldo, (cudaStream_t)stream);
+int dlp_layers_rows_attention(const void* q, const void* kv, int ldkv, int S, int T, int pos0, int H, int Dp, int Vp, int V, int window, float scale, const float* gate,
+                              int ldg, void* out, int ldo, void* stream) {
+    return rows_attention(q, kv, ldkv, S, T, pos0, H, Dp, Vp, V, window, scale, gate, ldg, out, ldo, (cudaStream_t)stream);
 }
 int dlp_layers_route(const float* logits, int ld, const dlp_route_rule* rule, int32_t* ids, float* weights, int T, void* stream) {
     DLP_REQUIRE(rule, "dlp_layers_route: null argument");

@@ -39,7 +39,7 @@ int make_tmap_2d(CUtensorMap* out, const void* base, int is_bf16, uint64_t rows,
 // Y[T,N] (op)= X[T,K] . W0[N,K]^T  (and W1 for SwiGLU).  X/W are fp16 (is_bf16=0) or bf16 (is_bf16=1).
 int gemm_f16(const void* w0, const void* w1, int ldw, const void* x, int ldx, void* y, int ldy, int T, int N, int K,
              int epilogue, int is_bf16, int split_k, cudaStream_t stream, const GemmCollective* coll, const GemmGroup* grp, void* ws,
-             size_t ws_bytes) {
+             size_t ws_bytes, const OutTail* tail) {
     // grouped: N = output features of ONE expert, w0/w1 = stacks of all experts (rows_total = what the tensor map must cover)
     DLP_REQUIRE(T > 0 && N > 0 && K > 0, "gemm: empty problem T=%d N=%d K=%d", T, N, K);
     DLP_REQUIRE(grp == nullptr || (grp->tile_expert && grp->tile_row0 && grp->tile_rows && grp->n_tiles && grp->max_tiles > 0 && split_k <= 1 &&
@@ -48,7 +48,7 @@ int gemm_f16(const void* w0, const void* w1, int ldw, const void* x, int ldx, vo
     DLP_REQUIRE(K % 8 == 0, "gemm: K=%d must be a multiple of 8", K);
     const int na = epi_is_gated(epilogue) ? 2 : 1;
     DLP_REQUIRE(na == 1 || w1 != nullptr, "gemm: a gated epilogue needs the up-projection weight");
-    DLP_REQUIRE((epilogue != EPI_GEGLU_BF16 && epilogue != EPI_SWIGLU_BF16 && epilogue != EPI_RELU2_BF16) || is_bf16, "gemm: the bf16 epilogues are built for bf16 operands");
+    DLP_REQUIRE((epilogue != EPI_GEGLU_BF16 && epilogue != EPI_SWIGLU_BF16 && epilogue != EPI_RELU2_BF16 && epilogue != EPI_TAIL_BF16) || is_bf16, "gemm: the bf16 epilogues are built for bf16 operands");
     const int total_kb = (K + GEMM_BK - 1) / GEMM_BK;
     int splits = split_k;
     if (splits <= 0) {  // auto: fill the machine when the epilogue can reduce across CTAs
@@ -65,6 +65,8 @@ int gemm_f16(const void* w0, const void* w1, int ldw, const void* x, int ldx, vo
     GemmParams p;
     memset(&p, 0, sizeof(p));
     if (coll) p.coll = *coll;
+    DLP_REQUIRE((epilogue == EPI_TAIL_BF16) == (tail != nullptr) && (!tail || grp == nullptr), "gemm: what follows the sums and the epilogue do not fit");
+    if (tail) p.tail = *tail;
     DLP_REQUIRE(epilogue != EPI_RS_PUSH_F32 || (coll && coll->rs_rows > 0 && coll->rs_done && coll->rs_tp >= 1 && coll->rs_tp <= 8 && splits == 1),
                 "gemm: the reduce-scatter epilogue needs a collective descriptor and no atomic split-K");
     p.y = y; p.T = T; p.N = N; p.K = K; p.ldy = ldy; p.epilogue = epilogue;

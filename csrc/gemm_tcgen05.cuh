@@ -20,7 +20,8 @@ constexpr int GEMM_BM = 128;  // output features per CTA (UMMA M)
 constexpr int GEMM_BK = 64;   // K elements per pipeline stage (= 128 B of fp16: one swizzle atom)
 
 enum GemmEpilogue : int { EPI_STORE_F16 = 0, EPI_STORE_F32 = 1, EPI_ATOMIC_ADD_F32 = 2, EPI_SWIGLU_F16 = 3,
-                          EPI_STORE_BF16 = 4, EPI_RS_PUSH_F32 = 5, EPI_GEGLU_BF16 = 6, EPI_RELU2_BF16 = 7, EPI_SWIGLU_BF16 = 8 };
+                          EPI_STORE_BF16 = 4, EPI_RS_PUSH_F32 = 5, EPI_GEGLU_BF16 = 6, EPI_RELU2_BF16 = 7, EPI_SWIGLU_BF16 = 8,
+                          EPI_TAIL_BF16 = 9 /* OutTail: fp32, the second part as bf16 */ };
 constexpr bool epi_is_gated(int e) { return e == EPI_SWIGLU_F16 || e == EPI_GEGLU_BF16 || e == EPI_SWIGLU_BF16; }   // two accumulators: gate and up
 
 struct GemmParams {
@@ -35,6 +36,7 @@ struct GemmParams {
     // arrives last at the tile's counter adds the partials in split order and runs the epilogue.  nullptr: not used.
     float* ws;
     unsigned* ws_counters;
+    OutTail tail;          // EPI_TAIL_BF16
 };
 
 template <int BT, int NA>
@@ -124,6 +126,21 @@ __device__ __forceinline__ void epi_loop(const GemmParams& p, const uint32_t (&r
                 ++owner;
                 if (owner < p.coll.rs_tp) dst = p.coll.rs_peer_buf[owner] + (size_t)p.coll.rs_rank * p.coll.rs_rows * p.N + n;
             }
+        }
+        return;
+    }
+    if (MODE == EPI_TAIL_BF16) {
+        const float bias = p.tail.bias != nullptr ? p.tail.bias[n] : 0.f;
+        if (n < p.tail.n2) {
+            float* dst = reinterpret_cast<float*>(p.y) + (size_t)tb * p.ldy + n;
+#pragma unroll
+            for (int j = 0; j < CH; ++j, dst += p.ldy)
+                if (tb + j < t_end) *dst = __uint_as_float(r0[j]) + bias;
+        } else {
+            __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(p.tail.out2) + (size_t)tb * p.tail.ldo2 + (n - p.tail.n2);
+#pragma unroll
+            for (int j = 0; j < CH; ++j, dst += p.tail.ldo2)
+                if (tb + j < t_end) *dst = __float2bfloat16_rn(xielu(__uint_as_float(r0[j]) + bias, p.tail.pos, p.tail.neg));
         }
         return;
     }
@@ -317,6 +334,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tm_w0, const __grid_cons
                     case EPI_GEGLU_BF16: if (NA == 2 && AB_FMT == 1) epi_loop<EPI_GEGLU_BF16, CH>(p, r0, r1, tb, n, t_end); break;
                     case EPI_SWIGLU_BF16: if (NA == 2 && AB_FMT == 1) epi_loop<EPI_SWIGLU_BF16, CH>(p, r0, r1, tb, n, t_end); break;
                     case EPI_RELU2_BF16: if (NA == 1 && AB_FMT == 1) epi_loop<EPI_RELU2_BF16, CH>(p, r0, r1, tb, n, t_end); break;
+                    case EPI_TAIL_BF16: if (NA == 1 && AB_FMT == 1) epi_loop<EPI_TAIL_BF16, CH>(p, r0, r1, tb, n, t_end); break;
                     case EPI_RS_PUSH_F32: epi_loop<EPI_RS_PUSH_F32, CH>(p, r0, r1, tb, n, t_end); break;
                 }
             }

@@ -132,10 +132,20 @@ struct GemmGroup {
     int bt = 0;                         // token-tile size the table was built for
 };
 
+// What a product of the layer-list models does behind its sums besides storing them: a bias, and output features from n2 on (those of a second
+// matrix stacked under the first) behind xIELU in the activation type, to a place of their own.
+//   xIELU(z) = z / 2 + (z > 0 ? pos z^2 : neg (exp(z) - 1 - z))
+struct OutTail {
+    const float* bias = nullptr;        // [N] (nullptr: none)
+    void* out2 = nullptr;               // [T, ldo2]
+    int n2 = 0x7fffffff, ldo2 = 0;
+    float pos = 0.f, neg = 0.f;
+};
+
 int gemv(const GemvParams& p, int wtype, cudaStream_t stream);
 int gemm_f16(const void* w0, const void* w1, int ldw, const void* x, int ldx, void* y, int ldy, int T, int N, int K,
              int epilogue, int is_bf16, int split_k, cudaStream_t stream, const GemmCollective* coll = nullptr,
-             const GemmGroup* grp = nullptr, void* ws = nullptr, size_t ws_bytes = 0);
+             const GemmGroup* grp = nullptr, void* ws = nullptr, size_t ws_bytes = 0, const OutTail* tail = nullptr);
 int gemm_quant(const QWeight& w0, const QWeight* w1, int wtype, const void* x, int ldx, void* y, int ldy, int T, int epilogue,
                int split_k, cudaStream_t stream, const GemmCollective* coll = nullptr, const GemmGroup* grp = nullptr, void* ws = nullptr,
                size_t ws_bytes = 0);

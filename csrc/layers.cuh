@@ -15,7 +15,8 @@ namespace dlp {
 //   v = v + e                                   when e: a second addend (the embedding output at the start of a loop pass; -> h_out)
 //   v = gnorm(v; groups2) * w2[k % w2_mod]      when w2 without b2: final norm, or the per-head norm of a recurrent mixer
 //   v = (v - mean) / sqrt(var + eps) * w2 + b2  when w2 and b2: layer norm over the row (groups2 = 1)
-//   v = v * sigmoid(g)                          when gate == 1
+//   v = v * sigmoid(g)                          when gate == 1;  v * silu(g) when gate == 3
+// and behind the row's Kp values, `tail` values in the activation type as they are (the other half of a stacked product's input; mat-vec only).
 // (pair and gate come with mixer outputs, y and e with the residual stream: never both)
 // gnorm splits the row into equal consecutive groups and divides each by its own sqrt(mean square + eps).
 struct RowStage {
@@ -41,8 +42,10 @@ struct RowStage {
     int ldg;
     int gate;             // GATE_*
     float lam;
+    const void* tail;     // [T, ld_tail]
+    int ld_tail, K_tail;
 };
-enum RowGate : int { GATE_NONE = 0, GATE_SIGMOID_AFTER = 1, GATE_SILU_BEFORE = 2 };
+enum RowGate : int { GATE_NONE = 0, GATE_SIGMOID_AFTER = 1, GATE_SILU_BEFORE = 2, GATE_SILU_AFTER = 3 };
 
 // GEGLU, SWIGLU: weight rows 2i / 2i+1 are gate_i / up_i, the output is gelu_tanh(gate) * up or silu(gate) * up.  RELU2: max(., 0)^2.
 // All three in the activation type.
@@ -71,16 +74,30 @@ struct ExpertArgs {
     int ldw_s, ldx_s, ld_act_s;
 };
 
-int matvec(const RowStage& st, const void* w, int ldw, int N, void* out, int ldo, int out_mode, int T, int f32, cudaStream_t s);
+int matvec(const RowStage& st, const void* w, int ldw, int N, void* out, int ldo, int out_mode, int T, int f32, cudaStream_t s, const OutTail* tail = nullptr);
 int stage_rows(const RowStage& st, void* xb, int ldxb, int T, int f32, cudaStream_t s);
-int sgemm(const float* x, int ldx, const float* w, int ldw, int N, int K, void* out, int ldo, int out_mode, int T, cudaStream_t s, const GemmGroup* grp = nullptr);
+int sgemm(const float* x, int ldx, const float* w, int ldw, int N, int K, void* out, int ldo, int out_mode, int T, cudaStream_t s, const GemmGroup* grp = nullptr,
+          const OutTail* tail = nullptr);
 // 1..4 rows: down = 0: act(W_e h) of every chosen expert -> act [T * top, ldo]; down = 1: sum of the weighted W_e act rows -> fp32 [T, ldo]
 int expert_matvec(const RowStage& st, const ExpertArgs& a, void* out, int ldo, int down, int T, int f32, cudaStream_t s);
 int route(const float* logits, int ld, const RouteRule& rule, int* ids, float* w, int T, cudaStream_t s);
 int head_matmul(const void* x, int x_f32, int ldx, int x_head, int kx, const void* w, int Kp, int H, int N, int n_rows, void* out, int ldo, int out_head,
                 const float* gate, int ldg, int T, int f32, cudaStream_t s);
 int embed_rows(const void* table, int ld, const int* ids, float* h, int E, int T, int vocab, float scale, int f32, cudaStream_t s);
-int latent_write(const float* proj, int ldp, const float* w, float eps, int R, int Rc, const int* slot, void* cache, int T, int f32, cudaStream_t s);
+// Cache rows of latent attention: the first R columns behind their RMS norm, then `rot` columns turned by their position; with q also the last
+// `rot` of every head's Dq query columns, in place.  Pairs are neighbours when `adjacent`, else half-split.
+struct LatentRows {
+    const float* proj;        // [T, ldp]
+    const float* w;           // [R]
+    const int* slot;          // [T] (below zero: not cached)
+    void* cache;              // rows of Rc
+    const int* pos;           // [T]
+    const float* inv_freq;    // [rot / 2]
+    float* q;                 // [T, ldq] (nullptr: none)
+    int ldp, R, Rc, rot, adjacent, ldq, H, Dq;
+    float eps, rot_scale;     // rot_scale: factor on cosine and sine
+};
+int latent_write(const LatentRows& a, int T, int f32, cudaStream_t s);
 
 struct Hgrn2Args {
     const float* proj;    // [T, ldp]: q_raw [H*D] | f_raw [H*D] | v [H*V]
@@ -130,7 +147,7 @@ struct SsdArgs {
 struct ConvArgs {
     const float* x;       // [T, ldx]
     const float* w;       // [taps, channels], the last row is the current token's
-    const float* b;       // [channels]
+    const float* b;       // [channels] (nullptr: none)
     float* ring;          // [slots, taps, channels]
     int ldx, taps, channels;
 };
@@ -139,6 +156,38 @@ constexpr int SSD_CHUNK = 128;
 int ssd_chunked(const SsdArgs& a, const ScanChunks& c, cudaStream_t s);                 // chunks of SSD_CHUNK tokens; c.decay: [n_chunks, H]
 int ssd_decode(const SsdArgs& a, const ConvArgs* conv, cudaStream_t s);                 // one token per segment; conv: q, k, v point into conv->x
 int conv_rows(const ConvArgs& c, const int* seg, const int* seg_slot, const int* pos, int n_seg, int longest, void* out, int ldo, int f32, cudaStream_t s);
+
+// Gated delta rule (layers_delta.cu): S <- f S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q.  q and k are made unit vectors per head
+// (x / sqrt(sum x^2 + unit_eps)), q is scaled by q_scale;  f = exp(log_decay[h] softplus(a + dt_bias[h])), beta = sigmoid(b).
+struct DeltaArgs {
+    const void* q;            // rows of T tokens behind convolution and activation: first column of the first head; fp32 or (rows_f32 = 0) bf16
+    const void* k;
+    const void* v;
+    const float* a;           // [T, lda]
+    const float* b;           // [T, ldb]
+    const float* log_decay;   // [H]
+    const float* dt_bias;     // [H]
+    float* state;             // [slots, H, D, V]
+    const int* seg;           // [n_seg][2]
+    const int* seg_slot;
+    const int* pos;           // [T]
+    float* out;               // [T, ldo]
+    int ldq, ldk, ldv, rows_f32, hpg, lda, ldb, ldo, H, D, V, n_seg;      // hpg consecutive heads share q and k
+    float unit_eps, q_scale;
+};
+constexpr int DELTA_CHUNK = 64;
+struct DeltaChunks {
+    const int* chunk;         // [n_chunks][2], as in ScanChunks
+    const int* first;         // [n_seg + 1]
+    void* states;             // [n_chunks, H, 2, D, V] bf16: the state a chunk starts from, value and remainder
+    void* solve;              // [n_chunks, H, 2, 64, 64] bf16: the chunk's triangular inverse, value and remainder
+    void* u;                  // [2, T, H * V] bf16: what every token writes, value and remainder
+    float* gates;             // [n_chunks, H, 64, 4]: cumulative log2 decay, 1 / |k|, beta
+    int n_chunks, T;
+};
+int delta_scan(const DeltaArgs& a, cudaStream_t s);
+int delta_decode(const DeltaArgs& a, const ConvArgs* conv, cudaStream_t s);        // one token per segment; conv: q, k, v point into conv->x
+int delta_chunked(const DeltaArgs& a, const DeltaChunks& c, cudaStream_t s);
 
 #ifdef __CUDACC__
 template <typename T> struct Act;
@@ -293,17 +342,17 @@ struct LatentArgs {
     const int* pos;           // [T]
     const int* tile_row0;     // [n_tiles] first (token * H + head) row of a tile; a tile never spans two requests
     const int* tile_rows;     // [n_tiles]
-    void* out;                // [T, H, Rc]
-    float* part_o;            // [n_splits][T * H][Rc]  (n_splits > 1)
+    void* out;                // [T, H, Vc]
+    float* part_o;            // [n_splits][T * H][Vc]  (n_splits > 1)
     float* part_ml;           // [n_splits][T * H][2]
-    int max_pages, page_size, H, Rc, T, n_tiles, bm, n_splits;
+    int max_pages, page_size, H, Rc, Vc, T, n_tiles, bm, n_splits, window;      // Vc: leading columns of a cached row that are values; position i sees i - window + 1 .. i
     float scale;
 };
 int latent_attention(const LatentArgs& a, int f32, cudaStream_t s);
 int latent_gather(const void* cache, const int* bt, int page, int Rc, void* out, int S, cudaStream_t s);
 int head_rows(const float* x, int ldx, int D, int Dp, int H, void* out, int T, cudaStream_t s);
-int rows_attention(const void* q, const void* kv, int ldkv, int S, int T, int pos0, int H, int Dp, int Vp, int V, float scale, const float* gate, int ldg, void* out, int ldo,
-                   cudaStream_t s);
+int rows_attention(const void* q, const void* kv, int ldkv, int S, int T, int pos0, int H, int Dp, int Vp, int V, int window, float scale, const float* gate, int ldg, void* out,
+                   int ldo, cudaStream_t s);
 int rows_attention_error(int* flag);
 int* flash_error_flag();      // device flag a bounded wait raises (nullptr: error set)
 
@@ -330,6 +379,10 @@ struct GqaArgs {
     void* out;                // [T, ldo] (maps > 1: fp32)
     int ldp, ldo, T, H, G, D, V, Dc, Vc, rot, max_pages, page_size, n_pages, n_tiles, bm, n_splits, window, keep, chunk, maps, adjacent;
     float eps, scale;
+    float rot_scale;          // factor on cosine and sine
+    float* v_first;           // [T, G * V] values that several layers share a part of: written (v_mix 1), or mixed in (v_mix 2): (1 - v_lam) v + v_lam v_first
+    int v_mix;
+    float v_lam;
 };
 int gqa_prepare(const GqaArgs& a, int f32, cudaStream_t s);                   // proj -> q rows and cache rows
 int gqa_attention(const GqaArgs& a, int fused, int f32, cudaStream_t s);      // tiles of (token, head) rows; fused: single tokens straight from proj

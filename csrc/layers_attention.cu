@@ -3,6 +3,8 @@
 // latent row they read.  Scores and softmax weights stay in fp32: for the tensor cores a weight is split into two bf16 parts (the
 // rounded value and the rest), whose products with the latent rows are summed.
 //
+// The values may be the leading columns only (behind them: a key part with positions that the heads share); a sliding window may hide early keys.
+//
 //   latent_attn_mma_kernel   bf16 latents up to 512 wide: mma.sync m16n8k16, latent tiles double-buffered with cp.async
 //   latent_attn_kernel       any width, bf16 or fp32 storage
 //   latent_combine_kernel    joins the key ranges of a split launch
@@ -11,13 +13,13 @@
 
 namespace dlp {
 
-struct KeyRange { int len, lo, hi; };      // keys visible to the tile's last row; the part of them this split reads
-__device__ __forceinline__ KeyRange tile_keys(const LatentArgs& a, int row_last, int split, int step) {
+struct KeyRange { int lo, hi; };           // the part that this split reads of the keys some row of the tile sees
+__device__ __forceinline__ KeyRange tile_keys(const LatentArgs& a, int row_first, int row_last, int split, int step) {
+    const int len = min(a.pos[row_last / a.H] + 1, a.max_pages * a.page_size), first = min(len, max(0, a.pos[row_first / a.H] - a.window + 1));
+    const int per = ((len - first + a.n_splits - 1) / a.n_splits + step - 1) / step * step;
     KeyRange k;
-    k.len = min(a.pos[row_last / a.H] + 1, a.max_pages * a.page_size);
-    const int per = ((k.len + a.n_splits - 1) / a.n_splits + step - 1) / step * step;
-    k.lo = min(k.len, split * per);
-    k.hi = min(k.len, k.lo + per);
+    k.lo = min(len, first + split * per);
+    k.hi = min(len, k.lo + per);
     return k;
 }
 
@@ -28,7 +30,7 @@ __global__ void __launch_bounds__(32 * NWARP, 1) latent_attn_mma_kernel(const La
     constexpr int NTH = 32 * NWARP, BM = 16 * MW, NW = NWARP / MW, KPW = BN / NW, LS = BN + 4;
     constexpr int NPAIR = (RMAX / 16 + NW - 1) / NW;      // 16-column output blocks of a warp
     extern __shared__ __align__(16) uint8_t la_smem[];
-    const int Rc = a.Rc, LD = Rc + 8;
+    const int Rc = a.Rc, Vc = a.Vc, LD = Rc + 8;
     __nv_bfloat16* qs = reinterpret_cast<__nv_bfloat16*>(la_smem);
     __nv_bfloat16* cs = qs + BM * LD;                     // [2][BN][LD]
     float* S = reinterpret_cast<float*>(cs + 2 * BN * LD);
@@ -40,7 +42,7 @@ __global__ void __launch_bounds__(32 * NWARP, 1) latent_attn_mma_kernel(const La
     pdl_wait();
     const int row0 = a.tile_row0[tile], rows = a.tile_rows[tile];
     if (rows <= 0) return;
-    const KeyRange kr = tile_keys(a, row0 + rows - 1, split, BN);
+    const KeyRange kr = tile_keys(a, row0, row0 + rows - 1, split, BN);
     const int* bt = a.block_table + (size_t)a.tok_slot[row0 / a.H] * a.max_pages;
     const __nv_bfloat16* cache = reinterpret_cast<const __nv_bfloat16*>(a.cache);
     const int chunks = Rc / 8;
@@ -118,7 +120,7 @@ __global__ void __launch_bounds__(32 * NWARP, 1) latent_attn_mma_kernel(const La
 #pragma unroll
             for (int i = 0; i < BN / TPR; ++i) {
                 const int kk = i * TPR + sub, key = k0 + kk;
-                v[i] = (key <= my_pos && key < kr.hi) ? row[kk] : -INFINITY;
+                v[i] = (key <= my_pos && key > my_pos - a.window && key < kr.hi) ? row[kk] : -INFINITY;
                 mx = fmaxf(mx, v[i]);
             }
 #pragma unroll
@@ -157,7 +159,7 @@ __global__ void __launch_bounds__(32 * NWARP, 1) latent_attn_mma_kernel(const La
 #pragma unroll
                 for (int j = 0; j < NPAIR; ++j) {
                     const int col = (j * NW + nw) * 16;
-                    if (col < Rc) {
+                    if (col < Vc) {
                         uint32_t bf[4];
                         ldsm_x4_t(bf, ct + (kk * 16 + (lane & 15)) * LD + col + (lane >> 4) * 8);
                         mma16816(acc[j][0], hi, bf[0], bf[1]);
@@ -191,12 +193,12 @@ __global__ void __launch_bounds__(32 * NWARP, 1) latent_attn_mma_kernel(const La
 #pragma unroll
             for (int n = 0; n < 2; ++n) {
                 const int col = (j * NW + nw) * 16 + n * 8 + c * 2;
-                if (col >= Rc) continue;
+                if (col >= Vc) continue;
                 const float x = acc[j][n][half * 2], y = acc[j][n][half * 2 + 1];
                 if (a.n_splits > 1)
-                    *reinterpret_cast<float2*>(a.part_o + ((size_t)split * a.T * a.H + row) * Rc + col) = make_float2(x, y);
+                    *reinterpret_cast<float2*>(a.part_o + ((size_t)split * a.T * a.H + row) * Vc + col) = make_float2(x, y);
                 else
-                    *reinterpret_cast<__nv_bfloat162*>(reinterpret_cast<__nv_bfloat16*>(a.out) + row * Rc + col) = __floats2bfloat162_rn(x * inv, y * inv);
+                    *reinterpret_cast<__nv_bfloat162*>(reinterpret_cast<__nv_bfloat16*>(a.out) + row * Vc + col) = __floats2bfloat162_rn(x * inv, y * inv);
             }
     }
 }
@@ -206,17 +208,17 @@ template <typename WT>
 __global__ void __launch_bounds__(128) latent_attn_kernel(const LatentArgs a) {
     extern __shared__ __align__(16) uint8_t la_smem[];
     float* q = reinterpret_cast<float*>(la_smem);         // [Rc]
-    float* acc = q + a.Rc;                                // [Rc]
-    float* s = acc + a.Rc;                                // [64]
+    float* acc = q + a.Rc;                                // [Vc]
+    float* s = acc + a.Vc;                                // [64]
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-    const int row = blockIdx.x, t = row / a.H, split = blockIdx.y, Rc = a.Rc;
+    const int row = blockIdx.x, t = row / a.H, split = blockIdx.y, Rc = a.Rc, Vc = a.Vc;
     pdl_wait();
-    const KeyRange kr = tile_keys(a, row, split, 64);
+    const KeyRange kr = tile_keys(a, row, row, split, 64);
     const int* bt = a.block_table + (size_t)a.tok_slot[t] * a.max_pages;
     const WT* cache = reinterpret_cast<const WT*>(a.cache);
     for (int r = tid; r < Rc; r += 128) {
         q[r] = (float)reinterpret_cast<const WT*>(a.q)[(size_t)row * Rc + r];
-        acc[r] = 0.f;
+        if (r < Vc) acc[r] = 0.f;
     }
     float m = -INFINITY, l = 0.f;
     for (int k0 = kr.lo; k0 < kr.hi; k0 += 64) {
@@ -241,7 +243,7 @@ __global__ void __launch_bounds__(128) latent_attn_kernel(const LatentArgs a) {
         __syncthreads();
         if (warp == 0) { s[lane] = p0; s[lane + 32] = p1; }
         __syncthreads();
-        for (int r = tid; r < Rc; r += 128) {
+        for (int r = tid; r < Vc; r += 128) {
             float v = acc[r] * alpha;
             for (int kk = 0; kk < n; ++kk) {
                 const int key = k0 + kk;
@@ -253,11 +255,11 @@ __global__ void __launch_bounds__(128) latent_attn_kernel(const LatentArgs a) {
     pdl_launch_dependents();
     if (a.n_splits > 1) {
         const size_t o = (size_t)split * a.T * a.H + row;
-        for (int r = tid; r < Rc; r += 128) a.part_o[o * Rc + r] = acc[r];
+        for (int r = tid; r < Vc; r += 128) a.part_o[o * Vc + r] = acc[r];
         if (tid == 0) { a.part_ml[o * 2] = m; a.part_ml[o * 2 + 1] = l; }
     } else {
         const float inv = l > 0.f ? 1.f / l : 0.f;
-        for (int r = tid; r < Rc; r += 128) reinterpret_cast<WT*>(a.out)[(size_t)row * Rc + r] = (WT)(acc[r] * inv);
+        for (int r = tid; r < Vc; r += 128) reinterpret_cast<WT*>(a.out)[(size_t)row * Vc + r] = (WT)(acc[r] * inv);
     }
 }
 
@@ -276,13 +278,13 @@ __global__ void __launch_bounds__(128) latent_combine_kernel(const LatentArgs a)
     }
     __syncthreads();
     const int r = blockIdx.y * 128 + threadIdx.x;
-    if (r < a.Rc) {
+    if (r < a.Vc) {
         float x[32], v = 0.f;
 #pragma unroll
-        for (int s = 0; s < 32; ++s) x[s] = (s < a.n_splits && w[s] != 0.f) ? a.part_o[(s * stride + row) * a.Rc + r] : 0.f;
+        for (int s = 0; s < 32; ++s) x[s] = (s < a.n_splits && w[s] != 0.f) ? a.part_o[(s * stride + row) * a.Vc + r] : 0.f;
 #pragma unroll
         for (int s = 0; s < 32; ++s) v = fmaf(x[s], w[s], v);
-        reinterpret_cast<WT*>(a.out)[(size_t)row * a.Rc + r] = (WT)v;
+        reinterpret_cast<WT*>(a.out)[(size_t)row * a.Vc + r] = (WT)v;
     }
     pdl_launch_dependents();
 }
@@ -307,21 +309,22 @@ static int launch_latent_tile(const LatentArgs& a, cudaStream_t s) {
 int latent_attention(const LatentArgs& a, int f32, cudaStream_t s) {
     DLP_REQUIRE(a.q && a.cache && a.block_table && a.tok_slot && a.pos && a.out && a.tile_row0 && a.tile_rows, "latent_attention: null argument");
     DLP_REQUIRE(a.H > 0 && a.Rc > 0 && a.Rc % 32 == 0 && a.T > 0 && a.n_tiles > 0 && a.page_size > 0 && a.max_pages > 0, "latent_attention: bad shape");
+    DLP_REQUIRE(a.Vc > 0 && a.Vc % 32 == 0 && a.Vc <= a.Rc && a.window >= 1, "latent_attention: values of %d of %d columns, window of %d", a.Vc, a.Rc, a.window);
     DLP_REQUIRE(a.n_splits >= 1 && a.n_splits <= 32 && (a.n_splits == 1 || (a.part_o && a.part_ml)), "latent_attention: %d key ranges", a.n_splits);
     int rc = 0;
-    if (!f32 && a.Rc <= 512) {
+    if (!f32 && a.Vc <= 512 && a.Rc <= 640) {
         DLP_REQUIRE(a.bm == 16 || a.bm == 32 || a.bm == 64, "latent_attention: tile of %d rows", a.bm);
-        rc = a.Rc <= 128 ? launch_latent_tile<128>(a, s) : launch_latent_tile<512>(a, s);
+        rc = a.Vc <= 128 ? launch_latent_tile<128>(a, s) : launch_latent_tile<512>(a, s);
     } else {
-        const size_t smem = (size_t)(2 * a.Rc + 64) * 4;
+        const size_t smem = (size_t)(a.Rc + a.Vc + 64) * 4;
         DLP_REQUIRE(smem <= 48 * 1024, "latent_attention: latent of %d", a.Rc);
         DLP_CHECK_CUDA(f32 ? launch_pdl(latent_attn_kernel<float>, dim3(a.T * a.H, a.n_splits), dim3(128), smem, s, a)
                            : launch_pdl(latent_attn_kernel<__nv_bfloat16>, dim3(a.T * a.H, a.n_splits), dim3(128), smem, s, a));
     }
     if (rc) return rc;
     if (a.n_splits > 1) {
-        if (f32) DLP_CHECK_CUDA(launch_pdl(latent_combine_kernel<float>, dim3(a.T * a.H, (a.Rc + 127) / 128), dim3(128), 0, s, a));
-        else DLP_CHECK_CUDA(launch_pdl(latent_combine_kernel<__nv_bfloat16>, dim3(a.T * a.H, (a.Rc + 127) / 128), dim3(128), 0, s, a));
+        if (f32) DLP_CHECK_CUDA(launch_pdl(latent_combine_kernel<float>, dim3(a.T * a.H, (a.Vc + 127) / 128), dim3(128), 0, s, a));
+        else DLP_CHECK_CUDA(launch_pdl(latent_combine_kernel<__nv_bfloat16>, dim3(a.T * a.H, (a.Vc + 127) / 128), dim3(128), 0, s, a));
     }
     return 0;
 }

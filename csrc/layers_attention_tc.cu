@@ -60,19 +60,21 @@ static int launch_rows(const void* q, const void* k, const void* v, int ldkv, in
     return 0;
 }
 
-// q [T, H * Dp], kv rows [S, ldkv]: k at column 0 (H * Dp), v at column H * Dp (H * Vp); queries are positions pos0 .. pos0 + T - 1
-int rows_attention(const void* q, const void* kv, int ldkv, int S, int T, int pos0, int H, int Dp, int Vp, int V, float scale, const float* gate, int ldg, void* out, int ldo,
-                   cudaStream_t s) {
-    DLP_REQUIRE(q && kv && out && T > 0 && pos0 >= 0 && S >= pos0 + T && H > 0 && V <= Vp, "rows_attention: bad argument");
+// q [T, H * Dp], kv rows [S, ldkv]: k at column 0 (H * Dp), v at column H * Dp (H * Vp); queries are rows pos0 .. pos0 + T - 1 of them and see the `window` rows up to their own
+int rows_attention(const void* q, const void* kv, int ldkv, int S, int T, int pos0, int H, int Dp, int Vp, int V, int window, float scale, const float* gate, int ldg, void* out,
+                   int ldo, cudaStream_t s) {
+    DLP_REQUIRE(q && kv && out && T > 0 && pos0 >= 0 && S >= pos0 + T && H > 0 && V <= Vp && window >= 1, "rows_attention: bad argument");
     FaParams p;
     memset(&p, 0, sizeof(p));
-    p.out = out; p.T = T; p.pos0 = pos0; p.Hq = H; p.Hkv = H; p.page_size = 128; p.max_pages = 1; p.ldo = ldo; p.gate = gate; p.ldg = ldg; p.V = V; p.scale = scale;
+    p.out = out; p.T = T; p.pos0 = pos0; p.Hq = H; p.Hkv = H; p.page_size = 128; p.max_pages = 1; p.ldo = ldo; p.gate = gate; p.ldg = ldg; p.V = V; p.scale = scale; p.window = window;
     if ((p.error = flash_error_flag()) == nullptr) return -1;
     const void* v = (const uint8_t*)kv + (size_t)H * Dp * 2;
     if (Dp == 64 && Vp == 64) return launch_rows<64, 64>(q, kv, v, ldkv, S, p, s);
     if (Dp == 64 && Vp == 128) return launch_rows<64, 128>(q, kv, v, ldkv, S, p, s);
     if (Dp == 128 && Vp == 64) return launch_rows<128, 64>(q, kv, v, ldkv, S, p, s);
     if (Dp == 128 && Vp == 128) return launch_rows<128, 128>(q, kv, v, ldkv, S, p, s);
+    if (Dp == 192 && Vp == 64) return launch_rows<192, 64>(q, kv, v, ldkv, S, p, s);
+    if (Dp == 192 && Vp == 128) return launch_rows<192, 128>(q, kv, v, ldkv, S, p, s);
     DLP_REQUIRE(false, "rows_attention: head sizes %d / %d", Dp, Vp);
 }
 // 0, or 1 when a wait of a flash kernel gave up since the last call (synchronises)

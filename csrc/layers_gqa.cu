@@ -40,8 +40,16 @@ __device__ __forceinline__ void gqa_angles(const GqaArgs& a, int pos, float2* cs
     for (int i = threadIdx.x; i < a.rot / 2; i += blockDim.x) {
         float s, c;
         sincosf((float)pos * a.inv_freq[i], &s, &c);
-        cs[i] = make_float2(c, s);
+        cs[i] = make_float2(c * a.rot_scale, s * a.rot_scale);
     }
+}
+// value i of the projection, mixed with the first mixing layer's; `keep`: this is that layer, and the caller stores its values
+__device__ __forceinline__ float gqa_mixed(const GqaArgs& a, int t, const float* v, int i, bool keep) {
+    if (a.v_mix == 0) return v[i];
+    float* first = a.v_first + (size_t)t * a.G * a.V + i;
+    if (a.v_mix == 2) return fmaf(a.v_lam, *first, (1.f - a.v_lam) * v[i]);
+    if (keep) *first = v[i];
+    return v[i];
 }
 __device__ __forceinline__ float gqa_sumsq(const float* x, int n) {      // this thread's share
     float s = 0.f;
@@ -92,7 +100,7 @@ __global__ void __launch_bounds__(256) gqa_prepare_kernel(const GqaArgs a) {
         } else {
             const int g = i - a.H - kh;
             WT* o = reinterpret_cast<WT*>(a.vc) + ((page * a.G + g) * a.page_size + off) * a.Vc;
-            for (int d = lane * 2; d < a.Vc; d += 64) put2(o + d, d < a.V ? v[g * a.V + d] : 0.f, d + 1 < a.V ? v[g * a.V + d + 1] : 0.f);
+            for (int d = lane * 2; d < a.Vc; d += 64) put2(o + d, d < a.V ? gqa_mixed(a, t, v, g * a.V + d, true) : 0.f, d + 1 < a.V ? gqa_mixed(a, t, v, g * a.V + d + 1, true) : 0.f);
         }
     }
     pdl_launch_dependents();
@@ -209,7 +217,7 @@ __global__ void __launch_bounds__(32 * NWARP) gqa_attn_mma_kernel(const GqaArgs 
         }
         if (owns_new) {                     // the new token's key and value: into the pages and, below, into this block's last tile
             const int kd = a.G * MAPS * a.D;
-            const float* vp = kp + kd + g * a.V;
+            const float* vp = kp + kd;
             const float rk = a.k_norm ? 1.f / sqrtf(block_sum(gqa_sumsq(kp, kd), red) / (float)kd + a.eps) : 1.f;
             const size_t row = cache_row(q_hi);
             const size_t krow = MAPS * row - (MAPS - 1) * (row % a.page_size);
@@ -220,7 +228,7 @@ __global__ void __launch_bounds__(32 * NWARP) gqa_attn_mma_kernel(const GqaArgs 
                 if (hg == 0) reinterpret_cast<__nv_bfloat16*>(a.kc)[(krow + (size_t)m * a.page_size) * a.Dc + d] = x;
             }
             for (int d = tid; d < a.Vc; d += NTH) {
-                const __nv_bfloat16 x = __float2bfloat16_rn(d < a.V ? vp[d] : 0.f);
+                const __nv_bfloat16 x = __float2bfloat16_rn(d < a.V ? gqa_mixed(a, t0, vp, g * a.V + d, hg == 0) : 0.f);
                 v_new[d] = x;
                 if (hg == 0) reinterpret_cast<__nv_bfloat16*>(a.vc)[row * a.Vc + d] = x;
             }
@@ -457,6 +465,7 @@ static int check_gqa(const GqaArgs& a, const char* who) {
                 a.H, a.G, a.D, a.V);
     DLP_REQUIRE(a.rot >= 0 && a.rot % 2 == 0 && a.rot <= a.D && (a.rot == 0 || a.inv_freq), "%s: rotation of %d dimensions", who, a.rot);
     DLP_REQUIRE(a.T > 0 && a.page_size > 0 && a.max_pages > 0 && a.window >= 1 && a.keep >= 0 && a.chunk >= 0, "%s: bad shape", who);
+    DLP_REQUIRE(a.v_mix >= 0 && a.v_mix <= 2 && (a.v_mix == 0 || a.v_first), "%s: value mixing %d", who, a.v_mix);
     DLP_REQUIRE((a.maps == 1 || a.maps == 2) && (a.H / a.G) % a.maps == 0, "%s: %d maps", who, a.maps);
     return 0;
 }

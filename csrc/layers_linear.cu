@@ -84,16 +84,27 @@ static cudaError_t launch_stage(const RowStage& st, XT* xb, int ldxb, int T, siz
     return launch_pdl(kern, dim3(T), dim3(256), smem, s, st, xb, ldxb);
 }
 
+template <typename WT>
+__device__ __forceinline__ void store_tail(const OutTail& tl, void* out, int ldo, int t, int n, float v) {
+    if (tl.bias != nullptr) v += tl.bias[n];
+    if (n < tl.n2) reinterpret_cast<float*>(out)[(size_t)t * ldo + n] = v;
+    else reinterpret_cast<WT*>(tl.out2)[(size_t)t * tl.ldo2 + n - tl.n2] = Act<WT>::from_f(xielu(v, tl.pos, tl.neg));
+}
+static int check_tail(const OutTail* tl, int N, int out_mode, const char* who) {
+    DLP_REQUIRE(!tl || (out_mode == LO_F32 && tl->n2 >= 0 && (tl->n2 >= N || (tl->out2 && tl->ldo2 >= N - tl->n2))), "%s: what follows the sums", who);
+    return 0;
+}
+
 // ---- decode mat-vec ------------------------------------------------------------------------------------------
 // A unit is two weight rows x (32 * VEC * U) columns: U 16-byte loads per row and lane.  A block owns a contiguous range of row
 // pairs, its warps take the units in a fixed order and always hold the next unit's loads while they reduce the current one.  The
 // first unit is requested before the dependency wait: weights do not depend on the previous kernel.
 template <typename WT, int NT, int FORM>
-__global__ void __launch_bounds__(512, 1) matvec_kernel(const RowStage st, const WT* __restrict__ w, int ldw, int N, void* out, int ldo, int out_mode, int T) {
+__global__ void __launch_bounds__(512, 1) matvec_kernel(const RowStage st, const WT* __restrict__ w, int ldw, int N, void* out, int ldo, int out_mode, int T, const OutTail tl) {
     constexpr int VEC = Act<WT>::VEC, U = 4, COLS = 32 * VEC * U;
     extern __shared__ __align__(16) uint8_t mv_smem[];
     WT* xs = reinterpret_cast<WT*>(mv_smem);
-    const int K = st.Kp;
+    const int K = st.Kp + st.K_tail;
     size_t off = ((size_t)NT * K * sizeof(WT) + 15) & ~size_t(15);
     float* sums = reinterpret_cast<float*>(mv_smem + off);
     const int KC = (K + COLS - 1) / COLS;
@@ -116,6 +127,7 @@ __global__ void __launch_bounds__(512, 1) matvec_kernel(const RowStage st, const
     int u = warp;
     if (u < units) issue(u, 0);
     pdl_wait();
+    if (st.K_tail > 0) stage_tails<WT>(st, T, xs, K);
     stage_rows_dev<WT, FORM>(st, 0, T, sums, blockIdx.x == 0, xs, K);
     float* part = sums;      // [units][2][NT]: the staging scratch is free again
     auto reduce = [&](int u, int b) {
@@ -205,50 +217,51 @@ __global__ void __launch_bounds__(512, 1) matvec_kernel(const RowStage st, const
             o[0] = Act<WT>::from_f(a0 * a0);
             if (row + 1 < N) o[1] = Act<WT>::from_f(a1 * a1);
         } else {
-            float* o = reinterpret_cast<float*>(out) + (size_t)t * ldo + row;
-            o[0] = a0;
-            if (row + 1 < N) o[1] = a1;
+            store_tail<WT>(tl, out, ldo, t, row, a0);
+            if (row + 1 < N) store_tail<WT>(tl, out, ldo, t, row + 1, a1);
         }
     }
 }
 
 template <typename WT, int NT>
-static int launch_matvec(const RowStage& st, const void* w, int ldw, int N, void* out, int ldo, int out_mode, int T, cudaStream_t s) {
+static int launch_matvec(const RowStage& st, const void* w, int ldw, int N, void* out, int ldo, int out_mode, int T, cudaStream_t s, const OutTail& tl) {
     constexpr int COLS = 32 * Act<WT>::VEC * 4;
-    const int pairs = (N + 1) / 2, KC = (st.Kp + COLS - 1) / COLS;
+    const int K = st.Kp + st.K_tail, pairs = (N + 1) / 2, KC = (K + COLS - 1) / COLS;
     const int grid = pairs < sm_count() ? pairs : sm_count();
-    const size_t xbytes = ((size_t)NT * st.Kp * sizeof(WT) + 15) & ~size_t(15);
+    const size_t xbytes = ((size_t)NT * K * sizeof(WT) + 15) & ~size_t(15);
     const size_t part = (size_t)((pairs + grid - 1) / grid) * KC * 2 * NT * 4, stg = stage_bytes(st, T, 16);
     const size_t smem = xbytes + (part > stg ? part : stg);
-    DLP_REQUIRE(smem <= 227 * 1024, "matvec: %d rows of width %d need %zu bytes of shared memory", T, st.Kp, smem);
+    DLP_REQUIRE(smem <= 227 * 1024, "matvec: %d rows of width %d need %zu bytes of shared memory", T, K, smem);
     const int form = stage_form(st);
     auto kern = form == ST_MIXER ? matvec_kernel<WT, NT, ST_MIXER> : form == ST_SUM ? matvec_kernel<WT, NT, ST_SUM> : matvec_kernel<WT, NT, ST_NORMED>;
     if (first_use_on_device((const void*)kern))
         DLP_CHECK_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024));
-    DLP_CHECK_CUDA(launch_pdl(kern, dim3(grid), dim3(512), smem, s, st, (const WT*)w, ldw, N, out, ldo, out_mode, T));
+    DLP_CHECK_CUDA(launch_pdl(kern, dim3(grid), dim3(512), smem, s, st, (const WT*)w, ldw, N, out, ldo, out_mode, T, tl));
     return 0;
 }
 
-int matvec(const RowStage& st, const void* w, int ldw, int N, void* out, int ldo, int out_mode, int T, int f32, cudaStream_t s) {
+int matvec(const RowStage& st, const void* w, int ldw, int N, void* out, int ldo, int out_mode, int T, int f32, cudaStream_t s, const OutTail* tail) {
     int rc = check_stage(st, "matvec");
+    if (!rc) rc = check_tail(tail, N, out_mode, "matvec");
     if (rc) return rc;
+    const OutTail tl = tail ? *tail : OutTail();
     DLP_REQUIRE(w && out && N > 0 && T >= 1 && T <= 4, "matvec: bad argument (T=%d N=%d)", T, N);
-    DLP_REQUIRE(st.Kp % 8 == 0 && ldw % 8 == 0 && ldw >= st.Kp, "matvec: row length %d / stride %d must be multiples of 8", st.Kp, ldw);
+    DLP_REQUIRE(st.Kp % 8 == 0 && ldw % 8 == 0 && ldw >= st.Kp + st.K_tail, "matvec: row length %d / stride %d must be multiples of 8", st.Kp, ldw);
     DLP_REQUIRE(out_mode == LO_F32 || out_mode == LO_RELU2 || ((out_mode == LO_GEGLU || out_mode == LO_SWIGLU) && N % 2 == 0), "matvec: output mode %d", out_mode);
     if (f32) {
-        if (T == 1) return launch_matvec<float, 1>(st, w, ldw, N, out, ldo, out_mode, T, s);
-        if (T == 2) return launch_matvec<float, 2>(st, w, ldw, N, out, ldo, out_mode, T, s);
-        return launch_matvec<float, 4>(st, w, ldw, N, out, ldo, out_mode, T, s);
+        if (T == 1) return launch_matvec<float, 1>(st, w, ldw, N, out, ldo, out_mode, T, s, tl);
+        if (T == 2) return launch_matvec<float, 2>(st, w, ldw, N, out, ldo, out_mode, T, s, tl);
+        return launch_matvec<float, 4>(st, w, ldw, N, out, ldo, out_mode, T, s, tl);
     }
-    if (T == 1) return launch_matvec<__nv_bfloat16, 1>(st, w, ldw, N, out, ldo, out_mode, T, s);
-    if (T == 2) return launch_matvec<__nv_bfloat16, 2>(st, w, ldw, N, out, ldo, out_mode, T, s);
-    return launch_matvec<__nv_bfloat16, 4>(st, w, ldw, N, out, ldo, out_mode, T, s);
+    if (T == 1) return launch_matvec<__nv_bfloat16, 1>(st, w, ldw, N, out, ldo, out_mode, T, s, tl);
+    if (T == 2) return launch_matvec<__nv_bfloat16, 2>(st, w, ldw, N, out, ldo, out_mode, T, s, tl);
+    return launch_matvec<__nv_bfloat16, 4>(st, w, ldw, N, out, ldo, out_mode, T, s, tl);
 }
 
 int stage_rows(const RowStage& st, void* xb, int ldxb, int T, int f32, cudaStream_t s) {
     int rc = check_stage(st, "stage_rows");
     if (rc) return rc;
-    DLP_REQUIRE(xb && T > 0 && ldxb >= st.Kp, "stage_rows: bad argument");
+    DLP_REQUIRE(xb && T > 0 && ldxb >= st.Kp && st.K_tail == 0, "stage_rows: bad argument");
     const size_t smem = stage_bytes(st, 1, 8);
     DLP_REQUIRE(smem <= 48 * 1024, "stage_rows: too many norm groups");
     DLP_CHECK_CUDA(f32 ? launch_stage(st, (float*)xb, ldxb, T, smem, s) : launch_stage(st, (__nv_bfloat16*)xb, ldxb, T, smem, s));
@@ -257,7 +270,7 @@ int stage_rows(const RowStage& st, void* xb, int ldxb, int T, int f32, cudaStrea
 
 // ---- fp32 matrix product ---------------------------------------------------------------------------------
 __global__ void __launch_bounds__(256) sgemm_kernel(const float* __restrict__ x, int ldx, const float* __restrict__ w, int ldw, int N, int K, float* out, int ldo,
-                                                    int out_mode, int T, const GemmGroup grp) {
+                                                    int out_mode, int T, const GemmGroup grp, const OutTail tl) {
     __shared__ float xs[16][68], ws[16][68];
     const int n0 = blockIdx.x * 64, tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
     int t0 = blockIdx.y * 64;
@@ -304,18 +317,22 @@ __global__ void __launch_bounds__(256) sgemm_kernel(const float* __restrict__ x,
             for (int j = 0; j < 4; ++j)
                 if (n0 + tx * 4 + j < N) {
                     const float u = fmaxf(acc[i][j], 0.f);
-                    out[(size_t)t * ldo + n0 + tx * 4 + j] = out_mode == LO_RELU2 ? u * u : acc[i][j];
+                    if (out_mode == LO_RELU2) out[(size_t)t * ldo + n0 + tx * 4 + j] = u * u;
+                    else store_tail<float>(tl, out, ldo, t, n0 + tx * 4 + j, acc[i][j]);
                 }
         }
     }
 }
 
-int sgemm(const float* x, int ldx, const float* w, int ldw, int N, int K, void* out, int ldo, int out_mode, int T, cudaStream_t s, const GemmGroup* grp) {
+int sgemm(const float* x, int ldx, const float* w, int ldw, int N, int K, void* out, int ldo, int out_mode, int T, cudaStream_t s, const GemmGroup* grp,
+          const OutTail* tail) {
     DLP_REQUIRE(x && w && out && N > 0 && K > 0 && T > 0, "sgemm: bad argument");
+    const int rc = check_tail(tail, N, out_mode, "sgemm");
+    if (rc) return rc;
     DLP_REQUIRE(out_mode == LO_F32 || out_mode == LO_RELU2 || ((out_mode == LO_GEGLU || out_mode == LO_SWIGLU) && N % 2 == 0), "sgemm: output mode %d", out_mode);
     DLP_REQUIRE(!grp || (grp->bt == 64 && grp->max_tiles > 0 && grp->max_tiles <= 65535), "sgemm: grouped launches take 64-row tiles");
     DLP_CHECK_CUDA(launch_pdl(sgemm_kernel, dim3((N + 63) / 64, grp ? grp->max_tiles : (T + 63) / 64), dim3(256), 0, s, x, ldx, w, ldw, N, K, (float*)out, ldo, out_mode, T,
-                              grp ? *grp : GemmGroup()));
+                              grp ? *grp : GemmGroup(), tail ? *tail : OutTail()));
     return 0;
 }
 

@@ -1,7 +1,7 @@
 // Token mixers with a state of their own, and the small row kernels around them.
 //
 //   embed_rows           token rows of the embedding table -> fp32 residual stream
-//   latent_write         latent of latent attention: RMS norm, then the paged latent cache
+//   latent_write         latent of latent attention: RMS norm, then the paged latent cache; rotation of the key part behind it and of the queries
 //   hgrn2_scan           gated linear recurrence over the tokens of every segment (layers_scan.cuh)
 #include "layers_scan.cuh"
 
@@ -24,24 +24,59 @@ int embed_rows(const void* table, int ld, const int* ids, float* h, int E, int T
     return 0;
 }
 
+// x (u, v of pair i) turned by the pair's angle
+__device__ __forceinline__ float2 turned(const float* x, int i, int rot, int adjacent, float2 cs, int& u, int& v) {
+    u = adjacent ? 2 * i : i;
+    v = adjacent ? 2 * i + 1 : i + rot / 2;
+    return make_float2(x[u] * cs.x - x[v] * cs.y, x[v] * cs.x + x[u] * cs.y);
+}
 template <typename WT>
-__global__ void __launch_bounds__(128) latent_write_kernel(const float* proj, int ldp, const float* w, float eps, int R, int Rc, const int* slot, WT* cache) {
+__global__ void __launch_bounds__(128) latent_write_kernel(const LatentRows a) {
+    extern __shared__ __align__(16) uint8_t lw_smem[];
+    float2* cs = reinterpret_cast<float2*>(lw_smem);       // [rot / 2]
     __shared__ float red[32];
     pdl_wait();
-    const int t = blockIdx.x;
-    const float* x = proj + (size_t)t * ldp;
-    float a = 0.f;
-    for (int k = threadIdx.x; k < R; k += 128) a = fmaf(x[k], x[k], a);
-    const float rs = 1.f / sqrtf(block_sum(a, red) / (float)R + eps);
-    const int sl = slot[t];
-    if (sl >= 0)
-        for (int k = threadIdx.x; k < Rc; k += 128) cache[(size_t)sl * Rc + k] = (WT)(k < R ? x[k] * rs * w[k] : 0.f);
+    const int t = blockIdx.x, np = a.rot / 2;
+    const float* x = a.proj + (size_t)t * a.ldp;
+    for (int i = threadIdx.x; i < np; i += 128) {
+        float s, c;
+        sincosf((float)a.pos[t] * a.inv_freq[i], &s, &c);
+        cs[i] = make_float2(c * a.rot_scale, s * a.rot_scale);
+    }
+    float ss = 0.f;
+    for (int k = threadIdx.x; k < a.R; k += 128) ss = fmaf(x[k], x[k], ss);
+    const float rs = 1.f / sqrtf(block_sum(ss, red) / (float)a.R + a.eps);
+    __syncthreads();
+    const int sl = a.slot[t];
+    if (sl >= 0) {
+        WT* row = reinterpret_cast<WT*>(a.cache) + (size_t)sl * a.Rc;
+        for (int k = threadIdx.x; k < a.Rc; k += 128)
+            if (k < a.R || k >= a.R + a.rot) row[k] = (WT)(k < a.R ? x[k] * rs * a.w[k] : 0.f);
+        for (int i = threadIdx.x; i < np; i += 128) {
+            int u, v;
+            const float2 y = turned(x + a.R, i, a.rot, a.adjacent, cs[i], u, v);
+            row[a.R + u] = (WT)y.x;
+            row[a.R + v] = (WT)y.y;
+        }
+    }
+    if (a.q != nullptr) {
+        float* q = a.q + (size_t)t * a.ldq + a.Dq - a.rot;
+        for (int j = threadIdx.x; j < a.H * np; j += 128) {
+            const int h = j / np, i = j - h * np;
+            float* p = q + (size_t)h * a.Dq;
+            int u, v;
+            const float2 y = turned(p, i, a.rot, a.adjacent, cs[i], u, v);
+            p[u] = y.x;
+            p[v] = y.y;
+        }
+    }
     pdl_launch_dependents();
 }
-int latent_write(const float* proj, int ldp, const float* w, float eps, int R, int Rc, const int* slot, void* cache, int T, int f32, cudaStream_t s) {
-    DLP_REQUIRE(proj && w && slot && cache && R > 0 && Rc >= R && T > 0, "latent_write: bad argument");
-    if (f32) DLP_CHECK_CUDA(launch_pdl(latent_write_kernel<float>, dim3(T), dim3(128), 0, s, proj, ldp, w, eps, R, Rc, slot, (float*)cache));
-    else DLP_CHECK_CUDA(launch_pdl(latent_write_kernel<__nv_bfloat16>, dim3(T), dim3(128), 0, s, proj, ldp, w, eps, R, Rc, slot, (__nv_bfloat16*)cache));
+int latent_write(const LatentRows& a, int T, int f32, cudaStream_t s) {
+    DLP_REQUIRE(a.proj && a.w && a.slot && a.cache && a.R > 0 && a.rot >= 0 && a.rot % 2 == 0 && a.Rc >= a.R + a.rot && T > 0, "latent_write: bad argument");
+    DLP_REQUIRE(a.rot == 0 || (a.pos && a.inv_freq && a.rot <= 8192 && (!a.q || (a.H > 0 && a.Dq >= a.rot && a.ldq >= a.H * a.Dq))), "latent_write: rotation of %d columns", a.rot);
+    const size_t smem = (size_t)(a.rot / 2) * 8;
+    DLP_CHECK_CUDA(f32 ? launch_pdl(latent_write_kernel<float>, dim3(T), dim3(128), smem, s, a) : launch_pdl(latent_write_kernel<__nv_bfloat16>, dim3(T), dim3(128), smem, s, a));
     return 0;
 }
 

@@ -150,6 +150,7 @@ inline int stage_form(const RowStage& p) { return p.g || p.pair ? ST_MIXER : p.e
 // gates: a row that is staged in bf16 takes the hardware exponential
 template <typename XT> __device__ __forceinline__ float row_silu(float z) { return sizeof(XT) == 2 ? silu_fast(z) : silu_exact(z); }
 template <typename XT> __device__ __forceinline__ float row_sigmoid(float z) { return sizeof(XT) == 2 ? __fdividef(1.f, 1.f + __expf(-z)) : sigmoid_exact(z); }
+__device__ __forceinline__ bool gate_after(const RowStage& p) { return p.gate == GATE_SIGMOID_AFTER || p.gate == GATE_SILU_AFTER; }
 // place in an x row of value k of the first map (the second one lies `pair` values on)
 __device__ __forceinline__ int stage_pair(const RowStage& p, int k) { return k + k / p.pair * p.pair; }
 template <typename XT>
@@ -172,6 +173,7 @@ __device__ __forceinline__ float4 stage_mixer4(const RowStage& p, int t, int k) 
 template <typename XT>
 __device__ __forceinline__ float4 stage_gate4(const RowStage& p, int t, int k, float4 v) {
     const float4 g = *reinterpret_cast<const float4*>(p.g + (size_t)t * p.ldg + k);
+    if (p.gate == GATE_SILU_AFTER) return make_float4(v.x * row_silu<XT>(g.x), v.y * row_silu<XT>(g.y), v.z * row_silu<XT>(g.z), v.w * row_silu<XT>(g.w));
     return make_float4(v.x * row_sigmoid<XT>(g.x), v.y * row_sigmoid<XT>(g.y), v.z * row_sigmoid<XT>(g.z), v.w * row_sigmoid<XT>(g.w));
 }
 template <typename XT>
@@ -226,7 +228,7 @@ __device__ __forceinline__ void stage_mixer_held(const RowStage& p, int t0, int 
                 const float4 w = *reinterpret_cast<const float4*>(p.w2 + k % p.w2_mod);
                 v[j] = make_float4(v[j].x * r * w.x, v[j].y * r * w.y, v[j].z * r * w.z, v[j].w * r * w.w);
             }
-            if (p.gate == GATE_SIGMOID_AFTER) v[j] = stage_gate4<XT>(p, t0 + t, k, v[j]);
+            if (gate_after(p)) v[j] = stage_gate4<XT>(p, t0 + t, k, v[j]);
             put(t, k, v[j]);
         }
     }
@@ -280,7 +282,7 @@ __device__ __forceinline__ void stage_rows_vec(const RowStage& p, int t0, int ro
             const float4 w = *reinterpret_cast<const float4*>(p.w2 + k % p.w2_mod);
             v = make_float4(v.x * r * w.x, v.y * r * w.y, v.z * r * w.z, v.w * r * w.w);
         }
-        if (FORM == ST_MIXER && p.gate == GATE_SIGMOID_AFTER) v = stage_gate4<XT>(p, t0 + t, k, v);
+        if (FORM == ST_MIXER && gate_after(p)) v = stage_gate4<XT>(p, t0 + t, k, v);
         put(t, k, v);
     }
     __syncthreads();
@@ -319,12 +321,25 @@ __device__ __forceinline__ void stage_rows_dev(const RowStage& p, int t0, int ro
                 v = base(t, k);
                 if (store_h && p.h_out) p.h_out[(size_t)(t0 + t) * p.ldh + k] = v;
                 if (p.w2) v = FULL && p.b2 ? fmaf((v - rs2[2 * t]) * rs2[2 * t + 1], p.w2[k], p.b2[k]) : v * (rs2[t * p.groups2 + k / gs2] * p.w2[k % p.w2_mod]);
-                if (FORM == ST_MIXER && p.gate == GATE_SIGMOID_AFTER) v *= row_sigmoid<XT>(p.g[(size_t)(t0 + t) * p.ldg + k]);
+                if (FORM == ST_MIXER && gate_after(p)) {
+                    const float g = p.g[(size_t)(t0 + t) * p.ldg + k];
+                    v *= p.gate == GATE_SILU_AFTER ? row_silu<XT>(g) : row_sigmoid<XT>(g);
+                }
             }
             dst[(size_t)t * ldd + k] = Act<XT>::from_f(v);
         }
     }
     __syncthreads();
+}
+// the rows' tails behind their Kp values (no barrier: the rows themselves are staged next)
+template <typename XT>
+__device__ __forceinline__ void stage_tails(const RowStage& p, int rows, XT* dst, int ldd) {
+    constexpr int VEC = Act<XT>::VEC;
+    const int n = p.K_tail / VEC;
+    for (int i = threadIdx.x; i < rows * n; i += blockDim.x) {
+        const int t = i / n, k = (i - t * n) * VEC;
+        *reinterpret_cast<uint4*>(dst + (size_t)t * ldd + p.Kp + k) = *reinterpret_cast<const uint4*>(reinterpret_cast<const XT*>(p.tail) + (size_t)t * p.ld_tail + k);
+    }
 }
 inline size_t stage_bytes(const RowStage& p, int rows, int nwarps) {
     auto need = [&](int groups) {
@@ -338,6 +353,8 @@ inline int check_stage(const RowStage& st, const char* who) {
     DLP_REQUIRE(st.x && st.K > 0 && st.Kp >= st.K, "%s: bad input row", who);
     DLP_REQUIRE(!(st.pair || st.g) || (!st.y && !st.e && !st.b2 && !st.h_out && st.pair >= 0 && (!st.pair || st.K % st.pair == 0) && (st.gate == GATE_NONE || st.g)), "%s: pairs of %d, gate %d",
                 who, st.pair, st.gate);
+    DLP_REQUIRE(st.K_tail == 0 || (st.K_tail > 0 && st.K_tail % 8 == 0 && st.Kp % 8 == 0 && st.tail && st.ld_tail % 8 == 0 && (reinterpret_cast<uintptr_t>(st.tail) & 15) == 0),
+                "%s: tail of %d values", who, st.K_tail);
     DLP_REQUIRE(!st.y || (st.groups1 > 0 && st.K % st.groups1 == 0), "%s: %d norm groups do not divide the width %d", who, st.groups1, st.K);
     DLP_REQUIRE(!st.b2 || (st.w2 && st.groups2 == 1 && st.w2_mod == st.K), "%s: a layer norm spans the whole row", who);
     DLP_REQUIRE(!st.w2 || (st.w2_mod > 0 && st.groups2 > 0 && st.K % st.groups2 == 0), "%s: %d norm groups do not divide the width %d", who, st.groups2, st.K);

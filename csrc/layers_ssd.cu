@@ -13,27 +13,22 @@
 //   U = sum_s exp(L_end - L_s) dt_s k_s v_s^T          o_t = exp(L_t) S_start^T q_t + sum_{s <= t} exp(L_t - L_s) dt_s (q_t . k_s) v_s
 // Exponents are never positive.  q, k and v (projections behind their activation) are bf16 operands; decays, step sizes, token weights and
 // states are fp32 and enter the tensor cores as two bf16 parts (value and remainder).
+#include "layers_chunks.cuh"
 #include "layers_scan.cuh"
-#include "mma.cuh"
 
 namespace dlp {
 
-__device__ __forceinline__ float softplus_exact(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
 __device__ __forceinline__ float ssd_step(const SsdArgs& a, int t, int h) { return a.dt ? softplus_exact(a.dt[(size_t)t * a.lddt + h] + a.dt_bias[h]) : 1.f; }
 
 // ---- token by token ------------------------------------------------------------------------------------------------------------------
-__device__ __forceinline__ float ssd_row(const void* rows, int f32, int act, size_t i) {
-    const float x = f32 ? reinterpret_cast<const float*>(rows)[i] : __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(rows)[i]);
-    return act ? silu_exact(x) : x;
-}
 __device__ __forceinline__ void scan_channel(const SsdArgs& a, int t, int h, int d, float& q, float& f, float& k) {
     const int g = h / a.hpg;
     const float dt = ssd_step(a, t, h);
-    q = ssd_row(a.q, a.rows_f32, a.act, (size_t)t * a.ldq + g * a.D + d);
-    k = ssd_row(a.k, a.rows_f32, a.act, (size_t)t * a.ldk + g * a.D + d) * dt;
+    q = mix_row(a.q, a.rows_f32, a.act, (size_t)t * a.ldq + g * a.D + d);
+    k = mix_row(a.k, a.rows_f32, a.act, (size_t)t * a.ldk + g * a.D + d) * dt;
     f = a.dt ? expf(a.log_decay[h] * dt) : a.decay[h];
 }
-__device__ __forceinline__ float scan_value(const SsdArgs& a, int t, int h, int c) { return ssd_row(a.v, a.rows_f32, a.act, (size_t)t * a.ldv + h * a.V + c); }
+__device__ __forceinline__ float scan_value(const SsdArgs& a, int t, int h, int c) { return mix_row(a.v, a.rows_f32, a.act, (size_t)t * a.ldv + h * a.V + c); }
 __device__ __forceinline__ float scan_out(const SsdArgs& a, int h, float o, float v) { return a.skip ? fmaf(a.skip[h], v, o) : o; }
 
 static int check_ssd(const SsdArgs& a, const char* who) {
@@ -80,14 +75,14 @@ __global__ void __launch_bounds__(256) ssd_decode_kernel(const SsdArgs a, const 
                 const int c = (int)(row - (cv.x + (size_t)t * cv.ldx));
                 float* ring = cv.ring + (size_t)slot * cv.taps * cv.channels + c;
                 const float now = *row;
-                x = fmaf(cv.w[(size_t)(cv.taps - 1) * cv.channels + c], now, cv.b[c]);
+                x = fmaf(cv.w[(size_t)(cv.taps - 1) * cv.channels + c], now, cv.b ? cv.b[c] : 0.f);
                 for (int lag = 1; lag < cv.taps; ++lag)
                     if (pos >= lag) x = fmaf(cv.w[(size_t)(cv.taps - 1 - lag) * cv.channels + c], ring[(size_t)((pos - lag) % cv.taps) * cv.channels], x);
                 x = silu_exact(x);
                 if (part == 2 || first_block) ring[(size_t)(pos % cv.taps) * cv.channels] = now;
             } else {
-                x = part == 0 ? ssd_row(a.q, a.rows_f32, a.act, (size_t)t * a.ldq + col) : part == 1 ? ssd_row(a.k, a.rows_f32, a.act, (size_t)t * a.ldk + col)
-                                                                                                      : ssd_row(a.v, a.rows_f32, a.act, (size_t)t * a.ldv + col);
+                x = part == 0 ? mix_row(a.q, a.rows_f32, a.act, (size_t)t * a.ldq + col) : part == 1 ? mix_row(a.k, a.rows_f32, a.act, (size_t)t * a.ldk + col)
+                                                                                                      : mix_row(a.v, a.rows_f32, a.act, (size_t)t * a.ldv + col);
             }
         }
         sd_smem[i] = part == 1 ? x * dt : x;
@@ -140,7 +135,7 @@ int ssd_decode(const SsdArgs& a, const ConvArgs* cv, cudaStream_t s) {
     const int rc = check_ssd(a, "ssd_decode");
     if (rc) return rc;
     DLP_REQUIRE(a.D <= 256 && a.V % 4 == 0 && (reinterpret_cast<uintptr_t>(a.state) & 15) == 0, "ssd_decode: state of %d x %d", a.D, a.V);
-    DLP_REQUIRE(!cv || (cv->x && cv->w && cv->b && cv->ring && cv->taps >= 1 && a.rows_f32 && a.ldq == cv->ldx && a.ldk == cv->ldx && a.ldv == cv->ldx), "ssd_decode: convolution");
+    DLP_REQUIRE(!cv || (cv->x && cv->w && cv->ring && cv->taps >= 1 && a.rows_f32 && a.ldq == cv->ldx && a.ldk == cv->ldx && a.ldv == cv->ldx), "ssd_decode: convolution");
     if (a.D <= 64) return launch_decode<2>(a, cv, s);
     if (a.D <= 128) return launch_decode<4>(a, cv, s);
     return launch_decode<8>(a, cv, s);
@@ -164,7 +159,7 @@ __global__ void __launch_bounds__(128) conv_rows_kernel(const ConvArgs cv, const
             const int p = p0 + t - lo;
             return p >= 0 ? ring[(size_t)(p % taps) * cv.channels] : 0.f;
         };
-        const float b = cv.b[c];
+        const float b = cv.b ? cv.b[c] : 0.f;
         if (TAPS > 0) {
             float w[TAPS > 0 ? TAPS : 1], win[TAPS > 0 ? TAPS : 1];
 #pragma unroll
@@ -201,7 +196,7 @@ static int launch_conv(const ConvArgs& c, const int* seg, const int* seg_slot, c
     return 0;
 }
 int conv_rows(const ConvArgs& c, const int* seg, const int* seg_slot, const int* pos, int n_seg, int longest, void* out, int ldo, int f32, cudaStream_t s) {
-    DLP_REQUIRE(c.x && c.w && c.b && c.ring && seg && seg_slot && pos && out && n_seg > 0 && n_seg <= 65535 && longest > 0 && longest <= 65535 * CONV_TILE, "conv_rows: bad argument");
+    DLP_REQUIRE(c.x && c.w && c.ring && seg && seg_slot && pos && out && n_seg > 0 && n_seg <= 65535 && longest > 0 && longest <= 65535 * CONV_TILE, "conv_rows: bad argument");
     DLP_REQUIRE(c.taps >= 1 && c.taps <= CONV_TILE && c.channels > 0 && c.ldx >= c.channels && ldo >= c.channels, "conv_rows: %d taps (at most %d) of %d channels", c.taps, CONV_TILE,
                 c.channels);
     return f32 ? launch_conv(c, seg, seg_slot, pos, n_seg, longest, (float*)out, ldo, s) : launch_conv(c, seg, seg_slot, pos, n_seg, longest, (__nv_bfloat16*)out, ldo, s);
@@ -210,70 +205,6 @@ int conv_rows(const ConvArgs& c, const int* seg, const int* seg_slot, const int*
 // ---- chunks --------------------------------------------------------------------------------------------------------------------------------
 constexpr int SC = SSD_CHUNK, SSD_NTH = 256, SSD_VP = 64, SSD_LDV = SSD_VP + 8;
 
-// R rows of W columns (columns past ncols and rows past n are zero), four values a time: put(row, column, values)
-template <typename RT, int R, int W, typename Put>
-__device__ __forceinline__ void ssd_rows(const RT* base, int ld, int n, int ncols, int act, Put put) {
-    constexpr int QN = R * W / 4 / SSD_NTH, QB = QN < 8 ? QN : 8;
-    const bool vec = ld % 4 == 0 && ncols % 4 == 0 && (reinterpret_cast<uintptr_t>(base) & (4 * sizeof(RT) - 1)) == 0;
-#pragma unroll 1
-    for (int b = 0; b < QN; b += QB) {
-        float4 x[QB];
-#pragma unroll
-        for (int j = 0; j < QB; ++j) {
-            const int i = threadIdx.x + (b + j) * SSD_NTH, s = i / (W / 4), c = i % (W / 4) * 4;
-            const RT* p = base + (size_t)s * ld + c;
-            x[j] = make_float4(0.f, 0.f, 0.f, 0.f);
-            if (s < n && c < ncols) {
-                if (vec) {
-                    if (sizeof(RT) == 4) {
-                        x[j] = *reinterpret_cast<const float4*>(p);
-                    } else {
-                        const uint2 u = *reinterpret_cast<const uint2*>(p);
-                        const float2 lo = bf2_to_f2(u.x), hi = bf2_to_f2(u.y);
-                        x[j] = make_float4(lo.x, lo.y, hi.x, hi.y);
-                    }
-                } else {
-                    x[j].x = Act<RT>::to_f(p[0]);
-                    if (c + 1 < ncols) x[j].y = Act<RT>::to_f(p[1]);
-                    if (c + 2 < ncols) x[j].z = Act<RT>::to_f(p[2]);
-                    if (c + 3 < ncols) x[j].w = Act<RT>::to_f(p[3]);
-                }
-            }
-        }
-#pragma unroll
-        for (int j = 0; j < QB; ++j) {
-            const int i = threadIdx.x + (b + j) * SSD_NTH;
-            if (act) x[j] = make_float4(silu_fast(x[j].x), silu_fast(x[j].y), silu_fast(x[j].z), silu_fast(x[j].w));
-            put(i / (W / 4), i % (W / 4) * 4, x[j]);
-        }
-    }
-}
-__device__ __forceinline__ void put_bf16(__nv_bfloat16* d, float4 v) {
-    const __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
-    *reinterpret_cast<uint2*>(d) = make_uint2(*reinterpret_cast<const uint32_t*>(&a), *reinterpret_cast<const uint32_t*>(&b));
-}
-__device__ __forceinline__ void put_split(__nv_bfloat16* hi, __nv_bfloat16* lo, float4 v) {
-    uint2 h, l;
-    split_bf16(v.x, v.y, h.x, l.x);
-    split_bf16(v.z, v.w, h.y, l.y);
-    *reinterpret_cast<uint2*>(hi) = h;
-    *reinterpret_cast<uint2*>(lo) = l;
-}
-// the chunk's rows as bf16 in shared memory [SC][W + 8]; bf16 rows arrive with cp.async (the caller waits)
-template <typename RT, int W>
-__device__ __forceinline__ void ssd_tile(const void* rows, int ld, size_t col0, int t0, int n, int ncols, int act, __nv_bfloat16* dst) {
-    const RT* base = reinterpret_cast<const RT*>(rows) + (size_t)t0 * ld + col0;
-    if (sizeof(RT) == 2 && !act && ld % 8 == 0 && ncols % 8 == 0 && (reinterpret_cast<uintptr_t>(base) & 15) == 0) {
-#pragma unroll 4
-        for (int i = threadIdx.x; i < SC * W / 8; i += SSD_NTH) {
-            const int s = i / (W / 8), c = i % (W / 8) * 8;
-            const bool ok = s < n && c < ncols;
-            cp_async16(dst + s * (W + 8) + c, ok ? base + (size_t)s * ld + c : base, ok);
-        }
-        return;
-    }
-    ssd_rows<RT, SC, W>(base, ld, n, ncols, act, [&](int s, int c, float4 x) { put_bf16(dst + s * (W + 8) + c, x); });
-}
 // step sizes and cumulative log2 decays of a chunk (tokens past its end: no step, no decay); ends with a barrier
 __device__ __forceinline__ void ssd_decays(const SsdArgs& a, int t0, int n, int h, float* sdt, float* sL, float* carry) {
     static_assert(SC == 128, "one warp per 32 tokens");
@@ -315,11 +246,11 @@ __global__ void __launch_bounds__(SSD_NTH) ssd_chunk_state_kernel(const SsdArgs 
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, ch = blockIdx.x, h = blockIdx.y, v0 = blockIdx.z * SSD_VP;
     pdl_wait();
     const int t0 = cc.chunk[2 * ch], n = cc.chunk[2 * ch + 1];
-    ssd_tile<RT, DP>(a.k, a.ldk, (size_t)(h / a.hpg) * a.D, t0, n, a.D, a.act, sk);
+    chunk_tile<RT, SC, DP, SSD_NTH>(a.k, a.ldk, (size_t)(h / a.hpg) * a.D, t0, n, a.D, a.act, sk);
     cp_commit();
     ssd_decays(a, t0, n, h, sdt, sL, carry);
     const float end = sL[SC - 1];
-    ssd_rows<RT, SC, SSD_VP>(reinterpret_cast<const RT*>(a.v) + (size_t)t0 * a.ldv + h * a.V + v0, a.ldv, n, min(SSD_VP, a.V - v0), a.act, [&](int s, int c, float4 x) {
+    chunk_rows<RT, SC, SSD_VP, SSD_NTH>(reinterpret_cast<const RT*>(a.v) + (size_t)t0 * a.ldv + h * a.V + v0, a.ldv, n, min(SSD_VP, a.V - v0), a.act, [&](int s, int c, float4 x) {
         const float w = exp2f(end - sL[s]) * sdt[s];
         put_split(vhi + s * LDV + c, vlo + s * LDV + c, make_float4(x.x * w, x.y * w, x.z * w, x.w * w));
     });
@@ -390,9 +321,9 @@ __global__ void __launch_bounds__(SSD_NTH, DP == 256 ? 1 : 2) ssd_chunk_out_kern
     pdl_wait();
     const int t0 = cc.chunk[2 * ch], n = cc.chunk[2 * ch + 1], ncol = min(SSD_VP, a.V - v0);
     const size_t qk0 = (size_t)(h / a.hpg) * a.D;
-    ssd_tile<RT, DP>(a.q, a.ldq, qk0, t0, n, a.D, a.act, sq);
-    ssd_tile<RT, DP>(a.k, a.ldk, qk0, t0, n, a.D, a.act, sk);
-    ssd_tile<RT, SSD_VP>(a.v, a.ldv, (size_t)h * a.V + v0, t0, n, ncol, a.act, sv);
+    chunk_tile<RT, SC, DP, SSD_NTH>(a.q, a.ldq, qk0, t0, n, a.D, a.act, sq);
+    chunk_tile<RT, SC, DP, SSD_NTH>(a.k, a.ldk, qk0, t0, n, a.D, a.act, sk);
+    chunk_tile<RT, SC, SSD_VP, SSD_NTH>(a.v, a.ldv, (size_t)h * a.V + v0, t0, n, ncol, a.act, sv);
     cp_commit();
     const float* S = cc.states + ((size_t)ch * a.H + h) * a.D * a.V + v0;
     const bool s_vec = a.V % 4 == 0;

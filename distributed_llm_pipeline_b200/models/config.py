@@ -18,8 +18,8 @@ class LayerSpec:
     mixer: dict[str, Any]
     mlp: dict[str, Any] | None = None
 
-    def n_params(self, width: int, norm_parts: int = 1) -> int:
-        """norm_parts: vectors of one norm (2 with a bias)."""
+    def n_params(self, width: int, norm_parts: int = 1, one_norm: bool = False) -> int:
+        """norm_parts: vectors of one norm (2 with a bias); one_norm: mixer and feed-forward share theirs."""
         m = self.mixer
         hd, hv = m["heads"] * m.get("dim", 0), m["heads"] * m["vdim"]
         if self.type == "hgrn2":
@@ -32,9 +32,14 @@ class LayerSpec:
         elif self.type == "attention":
             kd, kv, maps = m["kv_heads"] * m["dim"], m["kv_heads"] * m["vdim"], 2 if "diff" in m else 1
             n = width * (maps * (hd + kd) + kv + hv) + (hd + kd if m.get("qk_norm") else 0) + (4 * m["dim"] if maps == 2 else 0)
+            n += (hd + kd + kv if m.get("bias") else 0) + (1 if m.get("v_mix") else 0)
+        elif self.type == "delta":
+            ch = 2 * m["kv_heads"] * m["dim"] + hv
+            n = width * (ch + 2 * hv + 2 * m["heads"]) + ch * m["conv"] + 2 * m["heads"] + m["vdim"]
         else:       # latent_attention
-            r = m["kv_rank"]
-            n = width * (hd + r + m["heads"] + hv) + r * (hd + hv) + r
+            r, p, qr = m["kv_rank"], m.get("rot_dim", 0), m.get("q_rank", 0)
+            q = hd + m["heads"] * p
+            n = (width * qr + qr + qr * q if qr else width * q) + width * (r + p + hv + (m["heads"] if m.get("gate") else 0)) + r * (hd + hv) + r
         if self.mlp is None:
             ff = 0
         elif self.mlp["kind"] == "moe":
@@ -42,11 +47,11 @@ class LayerSpec:
             ff = self.mlp["router"]["experts"] * ((3 if ex.get("gated") else 2) * width * ex["ff"] + width + 1)
             if self.mlp.get("shared"):
                 ff += 3 * width * self.mlp["shared"]["ff"] + width
-        elif self.mlp["kind"] == "relu2":
-            ff = 2 * width * self.mlp["ff"]
+        elif self.mlp["kind"] in ("relu2", "xielu"):
+            ff = 2 * width * self.mlp["ff"] + (2 if self.mlp["kind"] == "xielu" else 0)
         else:
             ff = 3 * width * self.mlp["ff"]
-        return n + ff + (2 if self.mlp else 1) * norm_parts * width
+        return n + ff + (2 if self.mlp and not one_norm else 1) * norm_parts * width
 
 
 @dataclass(frozen=True)
@@ -170,7 +175,7 @@ class ModelConfig:
     def n_params(self) -> int:
         if self.layers:
             parts = 2 if self.norm_type == "layer" else 1
-            return 2 * self.vocab_size * self.n_embd + parts * self.n_embd + sum(s.n_params(self.n_embd, parts) for s in self.layers)
+            return 2 * self.vocab_size * self.n_embd + parts * self.n_embd + sum(s.n_params(self.n_embd, parts, self.parallel_residual) for s in self.layers)
         attn = self.n_embd * (self.q_dim + 2 * self.kv_dim) + self.q_dim * self.n_embd
         ffn = 3 * self.n_embd * self.n_ff * max(1, self.n_expert) + (self.n_embd * self.n_expert if self.is_moe else 0)
         emb = self.vocab_size * self.n_embd * (1 if self.tie_embeddings else 2)

@@ -2,7 +2,7 @@
 
 The residual stream is fp32.  A sublayer's output `y` is not added at once: it stays pending, and the next matrix product forms
 `h + y` (or `h + norm(y)`), and the norm in front of it, while it prepares its input rows (in the mat-vec prologue for up to four rows, in
-one row kernel in front of the GEMM for more).  A range of layers may run several times: every run has its own cache and state, and the
+one row kernel in front of the GEMM for more).  A mixer and a feed-forward that read the same norm share their products (mixers.Joined).  A range of layers may run several times: every run has its own cache and state, and the
 embedding output may join at the start of every pass but the first.  One forward takes any mix of prompt portions and single tokens of
 different sequences: projections run over all rows, mixers over the segments.
 """
@@ -17,7 +17,7 @@ from ..ops import layers as lops
 from ..ops.weights import DeviceWeight
 from ..gguf.constants import GGMLType
 from .engine import EngineCore, PagedKVCache, RecurrentState
-from .mixers import MIXERS, MLPS, Attention, Dense, LatentAttention, RoutedExperts, Rows, pad_to
+from .mixers import MIXERS, MLPS, Attention, Dense, Joined, LatentAttention, RoutedExperts, Rows, XieluMlp, pad_to
 from .modeldir import ModelDir, open_model_dir
 from .weights import ModelWeights
 
@@ -47,6 +47,17 @@ class LayeredLayer:
     norm1: Norm
     mlp: object | None = None
     norm2: Norm | None = None
+    joined: Joined | None = None        # mixer and feed-forward on the same norm (mlp and norm2 are None)
+
+    @property
+    def proj_cols(self) -> int:
+        return self.mixer.w_in.N if self.joined is None else self.joined.n
+
+    def join(self):
+        """Run mixer and feed-forward side by side, behind norm1."""
+        if not isinstance(self.mlp, XieluMlp):
+            raise NotImplementedError(f"parallel sublayers with a feed-forward of {type(self.mlp).__name__}")
+        self.joined, self.mlp = Joined(self.mixer, self.mlp), None
 
     def weights(self):
         return self.mixer.weights() + (self.mlp.weights() if self.mlp is not None else [])
@@ -82,7 +93,10 @@ def load_layered_weights(src: str | ModelDir, device, dtype="bf16", progress=Non
             raise ValueError(f"layer {il}: a mixer projection does not fit the width")
         if spec.mlp is not None:
             lw.mlp = MLPS[spec.mlp["kind"]](spec.mlp, lambda n: f.tensor(p + "mlp." + n), dev, dt, cfg.n_embd)
-            lw.norm2 = norm(p + "norm2")
+            if cfg.parallel_residual:
+                lw.join()
+            else:
+                lw.norm2 = norm(p + "norm2")
         layers[il] = lw
 
     def table(name):
@@ -133,7 +147,7 @@ class Batch:
     tok_slot: torch.Tensor      # [T] sequence slot of every row
     pos: torch.Tensor           # [T]
     slot: torch.Tensor          # [T] cache row
-    # latent attention: (head count, short only); windowed attention: ("tokens", query heads per key / value head, short only), "flash"
+    # latent attention: (its kind, short only); windowed attention: ("tokens", query heads per key / value head, short only), "flash"
     tiles: dict[object, TileTable]
     decode: bool = False        # one token of every sequence
     longest: int = 0            # tokens of the longest sequence, these included
@@ -191,17 +205,18 @@ class LayeredEngine(EngineCore):
         self.cur = 0                                                 # which of them holds it (-1: still the embedding output)
         self.emb = torch.zeros(M, self.E, dtype=f32, device=dev) if any(again for _, again in self.runs) else None
         self.y = torch.zeros(M, self.E, dtype=f32, device=dev)
-        sizes = {"proj": M * max(m.w_in.N for m in mixers.values()), "xb": M * max([pad_to(self.E, 8)] + [w.Kp for lw in weights.layers.values() for w in lw.weights()])}
-        for part in [*mixers.values(), *mlps]:
+        joined = [lw.joined for lw in weights.layers.values() if lw.joined is not None]
+        sizes = {"proj": M * max(lw.proj_cols for lw in weights.layers.values()), "xb": M * max([pad_to(self.E, 8)] + [w.Kp for lw in weights.layers.values() for w in lw.weights()])}
+        for part in [*mixers.values(), *mlps, *joined]:
             for name, n in part.buffers(M).items():
                 sizes[name] = max(sizes.get(name, 0), n)
-        types = {"proj": f32, "o": f32, "router": f32, "gate_w": f32, "ey": f32, "ys": f32, "ids": torch.int32}
+        types = {"proj": f32, "o": f32, "router": f32, "gate_w": f32, "ey": f32, "ys": f32, "q_up": f32, "v_first": f32, "delta_g": f32, "ids": torch.int32}
         self._flat = {n: torch.zeros(sz, dtype=types.get(n, self.dtype), device=dev) for n, sz in sizes.items()}
         experts = [m for m in mlps if isinstance(m, RoutedExperts)]
         self.expert_plans = {n: ops.MoePlan(M * max(m.top for m in experts), n, dev) for n in {m.n for m in experts}}
         self.logits = torch.zeros(max_seqs, cfg.vocab_size, dtype=f32, device=dev)
         lat = [m for m in mixers.values() if isinstance(m, LatentAttention)]
-        self._latent_heads = sorted({m.H for m in lat})
+        self._latent_kinds = sorted({m.kind for m in lat})
         att = [m for m in mixers.values() if isinstance(m, Attention)]
         self._att_kinds = {key_range_kind(m): m for m in att}
         self._att_groups = sorted({m.R for m in att})
@@ -211,21 +226,24 @@ class LayeredEngine(EngineCore):
         self.latent_ws = None
         if lat:
             rows = self._split_ctas * 64
-            self.latent_ws = (torch.zeros(rows * max(m.Rc for m in lat), dtype=f32, device=dev), torch.zeros(rows * 2, dtype=f32, device=dev))
+            self.latent_ws = (torch.zeros(rows * max(m.Vc for m in lat), dtype=f32, device=dev), torch.zeros(rows * 2, dtype=f32, device=dev))
         # segments from this length on take the chunked recurrence and the expanded / flash attention (bf16 storage; fp32 always takes the others)
-        self.long_from = 128 if self.dtype == torch.bfloat16 else 1 << 60
-        self._expanding_heads = {m.H for m in lat if m.expand} - {m.H for m in lat if not m.expand}
+        self.long_from = lops.LONG_FROM if self.dtype == torch.bfloat16 else 1 << 60
+        self._expanding_kinds = {m.kind for m in lat if m.expand} - {m.kind for m in lat if not m.expand}
         chunked = [m for m in mixers.values() if m.states and m.chunk]
         self._chunk_sizes = sorted({m.chunk for m in chunked})
         self.chunk_ws = None
         if chunked and self.long_from <= M:
-            n = M // self._chunk_sizes[0] + M // self.long_from + 1         # every long segment may end in a partial chunk
+            n = lops.most_chunks(M, self._chunk_sizes[0])
             self.chunk_ws = tuple(torch.zeros(n * max(m.H * m.D * w(m) for m in chunked), dtype=f32, device=dev) for w in (lambda m: m.V, lambda m: 1))
-        self._variant = (1, *(1 for _ in self._att_kinds))           # key ranges per decode query: latent attention, then every windowed kind
+        self._variant = (1,) * (len(self._latent_kinds) + len(self._att_kinds))      # key ranges per decode query: every kind of latent, then of windowed attention
         self._decode_batches: dict[tuple, Batch] = {}
 
     def buf(self, name: str, rows: int, cols: int, dtype=None) -> torch.Tensor:
         return self._flat[name][:rows * cols].view(rows, cols)
+
+    def flat(self, name: str) -> torch.Tensor:
+        return self._flat[name]
 
     def grow(self, name: str, rows: int, cols: int) -> torch.Tensor:
         """A buffer in the storage type that grows with the longest context it was asked for (by half again, so that it settles)."""
@@ -237,7 +255,8 @@ class LayeredEngine(EngineCore):
     # ---- matrix products -------------------------------------------------------------------------------
     def stage(self, r: Rows, Kp: int):
         """The row preparation of `r` as the kernels take it."""
-        return lops.row_stage(r.x, r.K, Kp, self.cfg.rms_eps, r.y, r.w1, self.cfg.norm_groups if r.w1 is not None else 1, r.h_out, r.w2, r.groups2, r.b2, r.e, r.pair, r.lam, r.g, r.gate)
+        return lops.row_stage(r.x, r.K, Kp, self.cfg.rms_eps, r.y, r.w1, self.cfg.norm_groups if r.w1 is not None else 1, r.h_out, r.w2, r.groups2, r.b2, r.e, r.pair, r.lam, r.g, r.gate,
+                              r.tail)
 
     def staged(self, r: Rows, Kp: int, T: int) -> torch.Tensor:
         """Rows of `r` in the storage type, prepared by one launch if they are not there as they are."""
@@ -248,10 +267,11 @@ class LayeredEngine(EngineCore):
     def matvec_rows(self, T: int, w: Dense) -> bool:
         return T <= MATVEC_ROWS and lops.matvec_fits(T, w.t)
 
-    def product(self, r: Rows, w: Dense, out: torch.Tensor, T: int, act: int = lops.OUT_F32) -> torch.Tensor:
+    def product(self, r: Rows, w: Dense, out: torch.Tensor, T: int, act: int = lops.OUT_F32, tail=None) -> torch.Tensor:
+        """tail: what follows the sums (ops.layers.out_tail)."""
         if self.matvec_rows(T, w):
-            return lops.matvec(self.stage(r, w.Kp), w.t, out, T, act)
-        return lops.linear(self.staged(r, w.Kp, T), w.t, out, act)
+            return lops.matvec(self.stage(r, w.Kp - (r.tail.shape[1] if r.tail is not None else 0)), w.t, out, T, act, tail)
+        return lops.linear(self.staged(r, w.Kp, T), w.t, out, act, tail)
 
     def _residual(self, T: int, pending: Pending | None, pre: Norm | None = None) -> Rows:
         """Rows of the residual stream with what is pending folded in on the way, and the norm `pre` in front of a sublayer."""
@@ -287,8 +307,12 @@ class LayeredEngine(EngineCore):
             m = lw.mixer
             if again:
                 pending = Pending(pending.w1, True, True) if pending is not None else Pending(None, False, True)
-            proj = self.product(self._residual(T, pending, lw.norm1 if pre else None), m.w_in, self.buf("proj", T, m.w_in.N), T)
-            self.product(m.mix(self, run, proj, b), m.w_out, self.y[:T], T)
+            rows = self._residual(T, pending, lw.norm1 if pre else None)
+            if lw.joined is not None:
+                lw.joined.apply(self, run, rows, b)
+            else:
+                proj = self.product(rows, m.w_in, self.buf("proj", T, m.w_in.N), T, tail=lops.out_tail(m.bias) if m.bias is not None else None)
+                self.product(m.mix(self, run, proj, b), m.w_out, self.y[:T], T)
             pending = Pending(None if pre else lw.norm1.w)
             if lw.mlp is not None:
                 lw.mlp.apply(self, self._residual(T, pending, lw.norm2 if pre else None), T)
@@ -334,15 +358,16 @@ class LayeredEngine(EngineCore):
         if b is None:
             dev, i32 = self.device, torch.int32
             tiles = {}
-            for H in self._latent_heads:
-                bm = lops.latent_tile_rows(H, B)
+            for kind, splits in zip(self._latent_kinds, self._variant):
+                H, _, Rc = kind
+                bm = lops.latent_tile_rows(H, B, Rc)
                 row0, rows = self._tile_lists(H, [1] * B, bm)
-                tiles[H, False] = TileTable(torch.tensor(row0, dtype=i32, device=dev), torch.tensor(rows, dtype=i32, device=dev), len(row0), bm, min(self._variant[0], max(1, self._split_ctas // len(row0))))
+                tiles[kind, False] = TileTable(torch.tensor(row0, dtype=i32, device=dev), torch.tensor(rows, dtype=i32, device=dev), len(row0), bm, min(splits, max(1, self._split_ctas // len(row0))))
             rng = torch.tensor([[i, i + 1] for i in range(B)], dtype=i32, device=dev)
             rows = torch.arange(B, dtype=i32, device=dev), torch.ones(B, dtype=i32, device=dev)
             tiles |= {("tokens", R, False): TileTable(*rows, B, lops.gqa_tile(R, 1)[0]) for R in self._att_groups}
             b = Batch(B, B, Segments(B, rng, self.active), None, self.active, self.pos, self.slot, tiles, decode=True,
-                      ranges=dict(zip(self._att_kinds, self._variant[1:])))
+                      ranges=dict(zip(self._att_kinds, self._variant[len(self._latent_kinds):])))
             self._decode_batches[(B, self._variant)] = b
         return b
 
@@ -364,14 +389,15 @@ class LayeredEngine(EngineCore):
                 lists += lops.scan_chunk_table([g[1:] for g in grp], size)
             cols += [torch.tensor(x, dtype=torch.int32) for x in lists]
         shapes = []
-        for H in self._latent_heads:
+        for kind in self._latent_kinds:
+            H, _, Rc = kind
             for only_short, n in ((False, len(lens)), (True, len(groups[0]))):
-                if only_short and (not groups[1] or not n) or not only_short and groups[1] and H in self._expanding_heads:
+                if only_short and (not groups[1] or not n) or not only_short and groups[1] and kind in self._expanding_kinds:
                     continue
-                bm = lops.latent_tile_rows(H, sum(lens[:n]))
+                bm = lops.latent_tile_rows(H, sum(lens[:n]), Rc)
                 row0, rows = self._tile_lists(H, lens[:n], bm)
                 cols += [torch.tensor(row0, dtype=torch.int32), torch.tensor(rows, dtype=torch.int32)]
-                shapes.append(((H, only_short), bm, len(row0)))
+                shapes.append(((kind, only_short), bm, len(row0)))
         for R in self._att_groups:
             for only_short in (False, True):
                 part = groups[0] if only_short else segs
@@ -393,7 +419,8 @@ class LayeredEngine(EngineCore):
         long = Segments(len(groups[1]), next(dev), next(dev), most[1], {size: (next(dev).view(-1, 2), next(dev)) for size in self._chunk_sizes},
                         tuple((sid, lo, hi, self.seqs[sid].length + hi - lo) for sid, lo, hi in groups[1]))
         longest = max(self.seqs[sid].length + len(t) for sid, t in parts)
-        tiles = {kind: TileTable(next(dev), next(dev), nt, bm, self._n_splits(nt, longest)) for kind, bm, nt in shapes}
+        # (latent attention: a tile sees its rows' windows)
+        tiles = {key: TileTable(next(dev), next(dev), nt, bm, self._n_splits(nt, min(longest, key[0][1] + bm)) if key[0] in self._latent_kinds else 1) for key, bm, nt in shapes}
         return ids, Batch(T, T_short, short if short.n else None, long if long.n else None, tok_slot, pos_d, slot_d, tiles, longest=longest)
 
     def _run_mixed(self, parts: list[tuple[int, list[int]]]):
@@ -499,12 +526,11 @@ class LayeredEngine(EngineCore):
         return torch.nn.functional.normalize(e, dim=-1) if normalize else e.clone()
 
     def _choose_variant(self, B: int, max_len: int):
-        lat = 1
-        if self._latent_heads:
-            H = self._latent_heads[-1]
-            bm = lops.latent_tile_rows(H, B)
-            lat = self._n_splits(B * ((H + bm - 1) // bm), max_len)
-        self._variant = (lat, *(key_ranges(m, B, lops.gqa_tile(m.R, 1)[0], max_len) if m.mma else 1 for m in self._att_kinds.values()))
+        lat = []
+        for H, window, Rc in self._latent_kinds:
+            bm = lops.latent_tile_rows(H, B, Rc)
+            lat.append(self._n_splits(B * ((H + bm - 1) // bm), min(max_len, window)))
+        self._variant = (*lat, *(key_ranges(m, B, lops.gqa_tile(m.R, 1)[0], max_len) if m.mma else 1 for m in self._att_kinds.values()))
 
     def _decode_body(self, B: int, sample: bool):
         ops.advance(self.seq_len_dev, self.active, self.pos, self.slot, self.kv_len, self.kv.block_table, self.page_size, B)

@@ -85,7 +85,7 @@ def _need(what: str, d, keys: tuple[str, ...]):
     """Check that `d` has these keys, dotted ones inside nested objects: positive sizes, except where a rule below says otherwise."""
     number = lambda v: isinstance(v, (int, float)) and not isinstance(v, bool)
     positive = lambda v: number(v) and v > 0
-    rules = {"scale": number, "diff": number, "base": positive, "factor": positive, "low": positive, "high": positive, "original": positive,
+    rules = {"scale": number, "diff": number, "base": positive, "factor": positive, "low": positive, "high": positive, "original": positive, "fast": positive, "slow": positive,
              "logit_scale": number, "keep_first": lambda v: isinstance(v, int) and v >= 0, "decay": lambda v: isinstance(v, list) and all(number(x) and 0 <= x <= 1 for x in v)}
     for path in keys:
         v = d
@@ -121,6 +121,9 @@ def _layered_config(name: str, cfg: dict, layers: tuple[LayerSpec, ...], **kw) -
 def talizen_config(cfg: dict) -> ModelConfig:
     """Talizen: HGRN2 and latent-attention layers in any order, tanh-gelu gated feed-forward or none, grouped norms behind the sublayers."""
     layers = _layer_list(cfg, {"hgrn2": ("heads", "dim", "vdim"), "latent_attention": ("heads", "dim", "vdim", "kv_rank", "scale")}, {"dense": ("ff",)})
+    for s in layers:
+        if s.type == "latent_attention":
+            s.mixer["gate"] = True
     groups = cfg["norm"]["groups"]
     if cfg["width"] % groups:
         raise ValueError(f"{groups} norm groups do not divide the width {cfg['width']}")
@@ -200,7 +203,44 @@ def nifalorn_config(cfg: dict) -> ModelConfig:
                            logit_scale=1.0 / float(cfg["logit_scale"]))
 
 
-ARCHITECTURES = {"Talizen": talizen_config, "Vozinex": vozinex_config, "Nifalorn": nifalorn_config}
+def rigalorn_config(cfg: dict) -> ModelConfig:
+    """Rigalorn: windowed attention with biases, YaRN rotation and values mixed across layers, the gated delta rule, and latent attention with
+    low-rank queries and a windowed rotated part, in any order; mixer and xIELU feed-forward (or none) side by side behind one RMS norm."""
+    layers = _layer_list(cfg, {"attention": ("heads", "kv_heads", "dim", "vdim", "rot.dims", "rot.base", "scale"), "delta": ("heads", "kv_heads", "dim", "vdim", "conv"),
+                               "latent_attention": ("heads", "dim", "vdim", "q_rank", "kv_rank", "rot_dim", "rot.dims", "rot.base", "scale")}, {"dense": ("ff",)})
+    out, values = [], None
+    for i, s in enumerate(layers):
+        m, what = dict(s.mixer), f"layer {i}"
+        if s.type == "delta":
+            if m["heads"] % m["kv_heads"]:
+                raise ValueError(f"{what}: {m['kv_heads']} query / key heads do not divide {m['heads']} heads")
+            if m["conv"] > 32:
+                raise ValueError(f"{what}: a convolution over {m['conv']} tokens (at most 32)")
+        else:
+            if m.get("mask"):
+                _need(what, m, ("mask.size",))
+            scaling = m["rot"].get("scaling")
+            if scaling is not None:
+                _need(what, scaling, ("factor", "fast", "slow", "original"))
+                if m["rot"]["base"] == 1:
+                    raise ValueError(f"{what}: scaled rotation of base 1")
+        if s.type == "attention":
+            _check_attention(what, m)
+            m["bias"] = True
+            if m.get("v_mix"):
+                size = m["kv_heads"], m["vdim"]
+                if values not in (None, size):
+                    raise ValueError(f"{what}: mixes values of {values[0]} heads of {values[1]} into {size[0]} of {size[1]}")
+                m["v_mix"], values = "first" if values is None else "later", size
+        if s.type == "latent_attention" and (m["rot"]["dims"] != m["rot_dim"] or m["rot_dim"] % 2):
+            raise ValueError(f"{what}: rotation of {m['rot']['dims']} of {m['rot_dim']} dimensions")
+        out.append(LayerSpec(s.type, m, {**s.mlp, "kind": "xielu"} if s.mlp is not None else None))
+    cfg = {"embedding": {"scale": 1.0}, **cfg}
+    _need("config", cfg, ("embedding.scale",))
+    return _layered_config("rigalorn", cfg, tuple(out), embedding_scale=float(cfg["embedding"]["scale"]), parallel_residual=True)
+
+
+ARCHITECTURES = {"Talizen": talizen_config, "Vozinex": vozinex_config, "Nifalorn": nifalorn_config, "Rigalorn": rigalorn_config}
 
 
 @dataclass

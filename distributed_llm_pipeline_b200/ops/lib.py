@@ -74,19 +74,20 @@ def _declare(lib):
         "dlp_sample": (i32, [vp, i32, i32, i32, i32, f32, f32, f32, u32, vp, vp, vp]),
         "dlp_f32_to_f16": (i32, [vp, vp, sz, vp]),
         "dlp_moe_route": (i32, [vp, i32, i32, i32, vp, vp, vp]),
-        "dlp_layers_matvec": (i32, [vp, vp, i32, i32, vp, i32, i32, i32, i32, vp]),
+        "dlp_layers_matvec": (i32, [vp, vp, i32, i32, vp, i32, i32, vp, i32, i32, vp]),
         "dlp_layers_stage_rows": (i32, [vp, vp, i32, i32, i32, vp]),
-        "dlp_layers_linear": (i32, [vp, i32, vp, i32, i32, i32, vp, i32, i32, i32, i32, vp, sz, vp]),
+        "dlp_layers_linear": (i32, [vp, i32, vp, i32, i32, i32, vp, i32, i32, vp, i32, i32, vp, sz, vp]),
         "dlp_layers_head_matmul": (i32, [vp, i32, i32, i32, i32, vp, i32, i32, i32, i32, vp, i32, i32, vp, i32, i32, i32, vp]),
         "dlp_layers_embed": (i32, [vp, i32, vp, vp, i32, i32, i32, f32, i32, vp]),
-        "dlp_layers_latent_write": (i32, [vp, i32, vp, f32, i32, i32, vp, vp, i32, i32, vp]),
+        "dlp_layers_latent_write": (i32, [vp, i32, i32, vp]),
+        "dlp_layers_delta": (i32, [vp, vp, vp, i32, vp]),
         "dlp_layers_hgrn2": (i32, [vp, vp, vp]),
         "dlp_layers_ssd": (i32, [vp, vp, vp, i32, vp]),
         "dlp_layers_conv_rows": (i32, [vp, vp, vp, vp, i32, i32, vp, i32, i32, vp]),
         "dlp_layers_latent_attention": (i32, [vp, i32, vp]),
         "dlp_layers_latent_gather": (i32, [vp, vp, i32, i32, vp, i32, vp]),
         "dlp_layers_head_rows": (i32, [vp, i32, i32, i32, i32, vp, i32, vp]),
-        "dlp_layers_rows_attention": (i32, [vp, vp, i32, i32, i32, i32, i32, i32, i32, i32, f32, vp, i32, vp, i32, vp]),
+        "dlp_layers_rows_attention": (i32, [vp, vp, i32, i32, i32, i32, i32, i32, i32, i32, i32, f32, vp, i32, vp, i32, vp]),
         "dlp_layers_route": (i32, [vp, i32, vp, vp, vp, i32, vp]),
         "dlp_layers_expert_matvec": (i32, [vp, vp, vp, i32, i32, i32, i32, vp]),
         "dlp_layers_linear_grouped": (i32, [vp, i32, vp, i32, i32, i32, vp, i32, i32, i32, i32, i32, vp, i32, vp, sz, vp]),

@@ -360,9 +360,13 @@ typedef struct {              /* how a row is formed in front of a matrix produc
     const float* b2;                           /* with b2: layer norm (centred) instead, . * w2 + b2 */
     const float* e; int32_t lde;               /* a second addend of x */
     int32_t pair;                              /* x rows hold two vectors of `pair` values per head: x1 - lam * x2 */
-    const float* g; int32_t ldg; int32_t gate; /* 1: the row times sigmoid(g) at the end; 2: x times silu(g) in front of the norm */
+    const float* g; int32_t ldg; int32_t gate; /* 1: the row times sigmoid(g) at the end; 2: x times silu(g) in front of the norm; 3: the row times silu(g) at the end */
     float lam;
+    const void* tail; int32_t ld_tail, K_tail; /* mat-vec: values behind the row's Kp as they are */
 } dlp_row_stage;
+typedef struct {              /* behind a product's sums (csrc/kernels.cuh OutTail): bias [N]; outputs from n2 on behind xIELU in the activation type -> out2 [T, ldo2] */
+    const float* bias; void* out2; int32_t n2, ldo2; float pos, neg;
+} dlp_out_tail;
 typedef struct { const float* bias; int32_t n_expert, top, sigmoid, groups, keep; float scale; } dlp_route_rule;      /* csrc/layers.cuh RouteRule */
 typedef struct {              /* csrc/layers.cuh ExpertArgs */
     const float* logits; dlp_route_rule rule; const void* w; int32_t ldl, rows, ldw, act;
@@ -372,7 +376,7 @@ typedef struct {              /* windowed grouped-query attention (csrc/layers.c
     const float* proj; const float* q_norm; const float* k_norm; const float* inv_freq; void* q; void* kc; void* vc;
     const int32_t* block_table; const int32_t* tok_slot; const int32_t* pos; const int32_t* slot; const int32_t* tile_row0; const int32_t* tile_rows; void* out;
     int32_t ldp, ldo, T, H, G, D, V, Dc, Vc, rot, max_pages, page_size, n_pages, n_tiles, bm, n_splits, window, keep, chunk, maps, adjacent;
-    float eps, scale;
+    float eps, scale, rot_scale; float* v_first; int32_t v_mix; float v_lam;
 } dlp_gqa_args;
 typedef struct {
     const float* proj; int32_t ldp; const float* fbias; const float* lower; float* state;
@@ -388,18 +392,31 @@ typedef struct { const int32_t* chunk; const int32_t* first; float* states; floa
 typedef struct {
     const void* q; const void* cache; const int32_t* block_table; const int32_t* tok_slot; const int32_t* pos;
     const int32_t* tile_row0; const int32_t* tile_rows; void* out; float* part_o; float* part_ml;
-    int32_t max_pages, page_size, H, Rc, T, n_tiles, bm, n_splits; float scale;
+    int32_t max_pages, page_size, H, Rc, Vc, T, n_tiles, bm, n_splits, window; float scale;
 } dlp_latent_args;
+typedef struct {              /* cache rows of latent attention (csrc/layers.cuh LatentRows) */
+    const float* proj; const float* w; const int32_t* slot; void* cache; const int32_t* pos; const float* inv_freq; float* q;
+    int32_t ldp, R, Rc, rot, adjacent, ldq, H, Dq; float eps, rot_scale;
+} dlp_latent_rows;
+typedef struct {              /* gated delta rule (csrc/layers.cuh DeltaArgs) */
+    const void* q; const void* k; const void* v; const float* a; const float* b; const float* log_decay; const float* dt_bias; float* state;
+    const int32_t* seg; const int32_t* seg_slot; const int32_t* pos; float* out;
+    int32_t ldq, ldk, ldv, rows_f32, hpg, lda, ldb, ldo, H, D, V, n_seg; float unit_eps, q_scale;
+} dlp_delta_args;
+typedef struct { const int32_t* chunk; const int32_t* first; void* states; void* solve; void* u; float* gates; int32_t n_chunks, T; } dlp_delta_chunks;      /* csrc/layers.cuh DeltaChunks */
 /* decode product, 1..4 rows: out_mode 0 = fp32, 2 = bf16 (dlp_layers_linear); in the activation type: 1 = GEGLU of interleaved (gate, up) rows,
  * 3 = max(., 0)^2, 4 = SwiGLU of interleaved rows */
-int dlp_layers_matvec(const dlp_row_stage* st, const void* w, int ldw, int N, void* out, int ldo, int out_mode, int T, int f32, void* stream);
+int dlp_layers_matvec(const dlp_row_stage* st, const void* w, int ldw, int N, void* out, int ldo, int out_mode, const dlp_out_tail* tail, int T, int f32, void* stream);
 int dlp_layers_stage_rows(const dlp_row_stage* st, void* xb, int ldxb, int T, int f32, void* stream);
 /* any number of rows: bf16 through the tcgen05 GEMM (ws: split-K workspace as for dlp_linear_ws), fp32 through an fp32 kernel */
-int dlp_layers_linear(const void* x, int ldx, const void* w, int ldw, int N, int K, void* out, int ldo, int out_mode, int T, int f32, void* ws, size_t ws_bytes, void* stream);
+int dlp_layers_linear(const void* x, int ldx, const void* w, int ldw, int N, int K, void* out, int ldo, int out_mode, const dlp_out_tail* tail, int T, int f32, void* ws, size_t ws_bytes,
+                      void* stream);
 int dlp_layers_head_matmul(const void* x, int x_f32, int ldx, int x_head, int kx, const void* w, int Kp, int H, int N, int n_rows, void* out, int ldo, int out_head,
                            const float* gate, int ldg, int T, int f32, void* stream);
 int dlp_layers_embed(const void* table, int ld, const int32_t* ids, float* h, int E, int T, int vocab, float scale, int f32, void* stream);
-int dlp_layers_latent_write(const float* proj, int ldp, const float* w, float eps, int R, int Rc, const int32_t* slot, void* cache, int T, int f32, void* stream);
+int dlp_layers_latent_write(const dlp_latent_rows* a, int T, int f32, void* stream);
+/* gated delta rule: mode 0 = token scan, 1 = 64-token chunks on the tensor cores (bf16 rows), 2 = one token per segment, with conv as in dlp_layers_ssd */
+int dlp_layers_delta(const dlp_delta_args* a, const dlp_delta_chunks* chunks, const dlp_conv_args* conv, int mode, void* stream);
 int dlp_layers_hgrn2(const dlp_hgrn2_args* a, const dlp_scan_chunks* chunks, void* stream);   /* chunks NULL: token scan; else 64-token chunks on the tensor cores */
 /* scalar-decay recurrences: mode 0 = token scan, 1 = 128-token chunks (chunks->decay: [n_chunks, H]), 2 = one token per segment, with conv: q, k
  * and v are the raw columns in conv->x; convolution and silu of whole portions (longest: tokens of the longest segment) */
@@ -407,11 +424,12 @@ int dlp_layers_ssd(const dlp_ssd_args* a, const dlp_scan_chunks* chunks, const d
 int dlp_layers_conv_rows(const dlp_conv_args* c, const int32_t* seg, const int32_t* seg_slot, const int32_t* pos, int n_seg, int longest, void* out, int ldo, int f32, void* stream);
 int dlp_layers_latent_attention(const dlp_latent_args* a, int f32, void* stream);
 /* prompt portions with keys and values expanded per head (bf16): latent rows of one request out of its pages; query columns as padded rows;
- * causal flash attention on plain rows kv [S, ldkv] (k in columns [0, H*Dp), v behind it), head sizes padded to 64 or 128 */
+ * causal flash attention on plain rows kv [S, ldkv] (k in columns [0, H*Dp), v behind it) over the last `window` of them, head sizes padded to 64
+ * or 128 (keys: or 192) */
 int dlp_layers_latent_gather(const void* cache, const int32_t* bt_row, int page, int Rc, void* out, int S, void* stream);
 int dlp_layers_head_rows(const float* x, int ldx, int D, int Dp, int H, void* out, int T, void* stream);
-int dlp_layers_rows_attention(const void* q, const void* kv, int ldkv, int S, int T, int pos0, int H, int Dp, int Vp, int V, float scale, const float* gate, int ldg,
-                              void* out, int ldo, void* stream);
+int dlp_layers_rows_attention(const void* q, const void* kv, int ldkv, int S, int T, int pos0, int H, int Dp, int Vp, int V, int window, float scale, const float* gate,
+                              int ldg, void* out, int ldo, void* stream);
 /* routed experts: chosen experts and weights from router logits; decode products of the chosen experts (1..4 rows); any number of rows over
  * expert-sorted rows (plan: dlp_moe_plan; gated output modes: rows_per_expert counts both interleaved rows);
  * out[t] = sum_j weights[t * top + j] * y[pos[t * top + j]] (+ sigmoid(gs[t]) * ys[t]) */

@@ -39,6 +39,25 @@ def differential(heads, kv_heads, dim, vdim, scale, rot, size, diff, mlp=None, b
                                            "rot": {"dims": rot, "base": base, "scaling": dict(zip(("factor", "low", "high", "original"), scaling))}}, "mlp": mlp}
 
 
+def delta(heads, kv_heads, dim, vdim, conv, ff=None):
+    return {"type": "delta", "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "conv": conv}, "mlp": None if ff is None else dense(ff)}
+
+
+def biased_attention(heads, kv_heads, dim, vdim, scale, rot, size, v_mix=True, ff=None, base=10000.0, yarn=(8.0, 64, 32.0, 1.0)):
+    r = {"dims": rot, "base": base, **({"scaling": dict(zip(("factor", "original", "fast", "slow"), yarn))} if yarn else {})}
+    return {"type": "attention", "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": scale, "rot": r, "mask": {"size": size}, "v_mix": v_mix},
+            "mlp": None if ff is None else dense(ff)}
+
+
+def low_rank_latent(heads, dim, rot, vdim, q_rank, rank, scale, size, ff=None, base=10000.0):
+    return {"type": "latent_attention", "mixer": {"heads": heads, "dim": dim, "rot_dim": rot, "vdim": vdim, "q_rank": q_rank, "kv_rank": rank, "scale": scale, "mask": {"size": size},
+                                                  "rot": {"dims": rot, "base": base}}, "mlp": None if ff is None else dense(ff)}
+
+
+def rigalorn(width, vocab, layers, eps=1e-5, emb=1.0):
+    return {"architecture": "Rigalorn", "width": width, "vocab": vocab, "norm": {"eps": eps}, "layers": layers, "embedding": {"scale": emb}}
+
+
 def dense(ff):
     return {"kind": "dense", "ff": ff}
 
@@ -97,6 +116,18 @@ CONFIGS = {
                                 differential(2, 1, 96, 64, 0.1, 96, 1000, 0.0)], loop=(0, 1, 2), emb=11.0),
     # states of every register-resident size and beyond
     "states": nifalorn(96, 64, [lightning(2, 128, 128, mlp=dense(96)), lightning(1, 160, 72), mamba2(2, 64, 256, 1, 4, 2), mamba2(2, 20, 300, 2, 3, 1), mamba2(4, 32, 128, 2, 4, 1)], emb=0.5),
+    # every mixer of Rigalorn, with and without a feed-forward, at sizes that are no multiple of a vector load; windows below a page; the first layer
+    # that mixes values is not the first attention
+    "parallel": rigalorn(72, 101, [biased_attention(6, 2, 20, 12, 0.4, 12, 24, v_mix=False, ff=52), low_rank_latent(5, 12, 6, 20, 28, 40, 0.35, 19, ff=36), delta(6, 2, 20, 12, 3, ff=52),
+                                   biased_attention(4, 2, 16, 24, 0.3, 16, 9, yarn=None), delta(3, 3, 12, 10, 1), biased_attention(2, 2, 24, 24, 0.35, 8, 33, ff=20, base=500.0),
+                                   low_rank_latent(3, 8, 2, 12, 17, 25, 0.5, 40)], eps=3e-4, emb=3.0),
+    # delta rules only: one head, one group, long and short convolutions, states of every register-resident size and beyond
+    "deltas": rigalorn(64, 60, [delta(4, 1, 64, 48, 4, ff=40), delta(2, 2, 128, 128, 2, ff=64), delta(1, 1, 160, 40, 6), delta(2, 1, 300, 12, 3), delta(5, 5, 8, 7, 32, ff=24)], eps=1e-6),
+    # heads and latents for every form of the attentions: expanded keys of 64, 128 and 192, beyond them, latents above 512, more heads than a tile;
+    # windows above a page and a key tile, one token, more than the sequence
+    "windows": rigalorn(256, 320, [low_rank_latent(4, 48, 16, 64, 96, 96, 0.14, 70, ff=96), biased_attention(8, 2, 128, 64, 0.12, 64, 150, ff=128, yarn=(4.0, 40, 8.0, 0.5)),
+                                   low_rank_latent(2, 128, 64, 128, 160, 512, 0.1, 131, ff=72), biased_attention(6, 2, 64, 64, 0.15, 64, 1), low_rank_latent(20, 40, 24, 24, 64, 160, 0.15, 1000),
+                                   low_rank_latent(1, 200, 8, 40, 32, 544, 0.1, 33, ff=8)], emb=11.0),
     "attention": config(80, 64, 5, [latent(4, 16, 24, 32, 0.4, 40), latent(49, 8, 4, 64, 0.4)]),
 }
 
@@ -147,6 +178,38 @@ def nifalorn_weights(cfg: dict, g, rnd, mat) -> dict[str, torch.Tensor]:
     return w
 
 
+def rigalorn_weights(cfg: dict, g, rnd, mat) -> dict[str, torch.Tensor]:
+    E, V = cfg["width"], cfg["vocab"]
+    w = {"embed": rnd(V, E, scale=1 / cfg["embedding"]["scale"]), "head": mat(V, E, 2.0), "final.norm": rnd(E, scale=0.2, mean=1.0)}
+    for i, s in enumerate(cfg["layers"]):
+        p, m, mix = f"l{i}.", s["mixer"], f"l{i}.mix."
+        w[p + "norm1"] = rnd(E, scale=0.2, mean=1.0)
+        H, D, Vd = m["heads"], m["dim"], m["vdim"]
+        if s["type"] == "delta":
+            G, taps = m["kv_heads"], m["conv"]
+            for n, rows in (("q", G * D), ("k", G * D), ("v", H * Vd)):
+                w.update({mix + n: mat(rows, E, 1.5), mix + n + ".conv": rnd(rows, taps, scale=taps ** -0.5, mean=0.3)})
+            w.update({mix + "g": mat(H * Vd, E, 1.5), mix + "b": mat(H, E, 1.5), mix + "a": mat(H, E, 1.5), mix + "dt_bias": rnd(H, scale=1.5, mean=-3.0), mix + "A_log": rnd(H, scale=1.0),
+                      mix + "norm": rnd(Vd, scale=0.2, mean=1.0)})
+        elif s["type"] == "attention":
+            G = m["kv_heads"]
+            sharp = (2.5 / (m["scale"] * D ** 0.5)) ** 0.5          # scores of a few units, so that single keys count
+            for n, rows, gain in (("q", H * D, sharp), ("k", G * D, sharp), ("v", G * Vd, 1.5)):
+                w.update({mix + n: mat(rows, E, gain), mix + n + ".b": rnd(rows, scale=0.4)})
+            if m["v_mix"]:
+                w[mix + "vmix"] = rnd(1, scale=0.2, mean=0.5)[0]
+        else:
+            R, P, Q = m["kv_rank"], m["rot_dim"], m["q_rank"]
+            sharp = 2.5 / (m["scale"] * (D + P) ** 0.5)
+            w.update({mix + "dq": mat(Q, E), mix + "dq.norm": rnd(Q, scale=0.3, mean=1.0), mix + "uq": mat(H * (D + P), Q, sharp), mix + "dkv": mat(R + P, E), mix + "dkv.norm": rnd(R, scale=0.3, mean=1.0),
+                      mix + "uk": mat(H * D, R), mix + "uv": mat(H * Vd, R)})
+        w[mix + "o"] = mat(E, H * Vd)
+        if s["mlp"] is not None:
+            ff = s["mlp"]["ff"]
+            w.update({p + "mlp.up": mat(ff, E), p + "mlp.down": mat(E, ff, 0.7), p + "mlp.act": rnd(2)})
+    return w
+
+
 def weights(cfg: dict, seed: int = 0) -> dict[str, torch.Tensor]:
     g = torch.Generator().manual_seed(seed)
 
@@ -157,6 +220,8 @@ def weights(cfg: dict, seed: int = 0) -> dict[str, torch.Tensor]:
         return rnd(n, k, scale=gain / k ** 0.5)
     if cfg["architecture"] == "Nifalorn":
         return nifalorn_weights(cfg, g, rnd, mat)
+    if cfg["architecture"] == "Rigalorn":
+        return rigalorn_weights(cfg, g, rnd, mat)
     E, V = cfg["width"], cfg["vocab"]
     w = {"embed": rnd(V, E), "head": mat(V, E, 2.0), "final.norm": rnd(E, scale=0.2, mean=1.0)}
     if cfg["architecture"] == "Vozinex":
@@ -231,8 +296,8 @@ def install_host_ops(monkeypatch):
     """Replace the kernel launches of ops.layers by plain fp32 code, so that engine, cache, state slots and scheduler run on the host."""
     from distributed_llm_pipeline_b200.ops import layers as L
 
-    def row_stage(x, K, Kp, eps, y=None, w1=None, groups1=1, h_out=None, w2=None, groups2=1, b2=None, e=None, pair=0, lam=0.0, g=None, gate=0):
-        return dict(x=x, K=K, Kp=Kp, eps=eps, y=y, w1=w1, groups1=groups1, h_out=h_out, w2=w2, groups2=groups2, b2=b2, e=e, pair=pair, lam=lam, g=g, gate=gate)
+    def row_stage(x, K, Kp, eps, y=None, w1=None, groups1=1, h_out=None, w2=None, groups2=1, b2=None, e=None, pair=0, lam=0.0, g=None, gate=0, tail=None):
+        return dict(x=x, K=K, Kp=Kp, eps=eps, y=y, w1=w1, groups1=groups1, h_out=h_out, w2=w2, groups2=groups2, b2=b2, e=e, pair=pair, lam=lam, g=g, gate=gate, tail=tail)
 
     def staged(st, T):
         if st["pair"]:
@@ -252,17 +317,28 @@ def install_host_ops(monkeypatch):
             v = plain.layer_norm(v, st["w2"], st["b2"], st["eps"])
         elif st["w2"] is not None:
             v = plain.grouped_norm(v, st["w2"].repeat(st["K"] // st["w2"].numel()), st["groups2"], st["eps"])
-        if st["gate"] == 1:
-            v = v * plain.sigmoid(st["g"][:T, :st["K"]])
-        return torch.nn.functional.pad(v, (0, st["Kp"] - st["K"]))
+        if st["gate"] in (1, 3):
+            v = v * (plain.sigmoid if st["gate"] == 1 else plain.silu)(st["g"][:T, :st["K"]])
+        v = torch.nn.functional.pad(v, (0, st["Kp"] - st["K"]))
+        return v if st["tail"] is None else torch.cat([v, st["tail"][:T].to(v.dtype)], 1)
 
     def behind(r, act):
         if act in (L.OUT_GEGLU, L.OUT_SWIGLU):
             return (plain.gelu_tanh if act == L.OUT_GEGLU else plain.silu)(r[..., 0::2]) * r[..., 1::2]
         return torch.clamp(r, min=0) ** 2 if act == L.OUT_RELU2 else r
 
-    def product(x, w, out, act):
+    def out_tail(bias=None, n2=1 << 30, out2=None, act=(0.0, 0.0)):
+        return bias, n2, out2, act
+
+    def product(x, w, out, act, tail=None):
         r = behind(x.float() @ w.float().T, act)
+        if tail is not None:
+            bias, n2, out2, (pos, neg) = tail
+            r = r if bias is None else r + bias
+            if n2 < r.shape[1]:
+                z = r[:, n2:]
+                out2[:r.shape[0], :z.shape[1]] = (z / 2 + torch.where(z > 0, pos * z * z, neg * (torch.expm1(z) - z))).to(out2.dtype)
+                r = r[:, :n2]
         out[:r.shape[0], :r.shape[1]] = r.to(out.dtype)
         return out
 
@@ -281,9 +357,16 @@ def install_host_ops(monkeypatch):
     def embed(table, ids, h, T, scale=1.0):
         h[:T] = table[ids[:T].long(), :h.shape[1]].float() * scale
 
-    def latent_write(proj, w, eps, R, slot, cache, T):
+    def latent_write(proj, w, eps, R, slot, cache, T, rot=None, q=None, heads=0):
         rows = cache.view(-1, cache.shape[-1])
         rows[slot[:T].long(), :R] = (plain.rms(proj[:T, :R], eps) * w).to(cache.dtype)
+        if rot is not None:
+            pos, f, amp = rot
+            P = 2 * len(f)
+            rows[slot[:T].long(), R:R + P] = (amp * plain.rotate_pairs(proj[:T, None, R:R + P], f, pos[:T]))[:, 0].to(cache.dtype)
+            for h in range(heads):
+                part = q[:T, (h + 1) * q.shape[1] // heads - P:(h + 1) * q.shape[1] // heads]
+                part.copy_(amp * plain.rotate_pairs(part[:, None], f, pos[:T])[:, 0])
 
     def scan(proj, fbias, lower, state, seg, seg_slot, n_seg, pos, out, chunks=None):
         _, H, D, V = state.shape
@@ -301,8 +384,7 @@ def install_host_ops(monkeypatch):
         _, H, D, V = state.shape
         if conv is not None:
             x, w, b, ring = conv
-            y = torch.empty_like(x)
-            conv_rows(x, w, b, ring, seg, seg_slot, n_seg, 1, pos, y)
+            y = conv_rows(x, w, b, ring, seg, seg_slot, n_seg, 1, pos, torch.empty_like(x))
             n = D * H // hpg
             rows = y[:, -n:], y[:, -2 * n:-n], y[:, :H * V]
         for s in range(n_seg):
@@ -320,6 +402,23 @@ def install_host_ops(monkeypatch):
             out[lo:hi] = (o + (skip[:, None] * v if skip is not None else 0)).reshape(hi - lo, -1)
         return out
 
+    def delta(rows, hpg, state, a, b, log_decay, dt_bias, seg, seg_slot, n_seg, pos, out, unit_eps, chunks=None, conv=None, single=False):
+        _, H, D, V = state.shape
+        n = D * H // hpg
+        assert unit_eps == 1e-6
+        if conv is not None:
+            y = conv_rows(*conv, seg, seg_slot, n_seg, 1, pos, torch.empty_like(conv[0]))
+            rows = y, y[:, n:], y[:, 2 * n:]
+        for s in range(n_seg):
+            (lo, hi), sl = seg.view(-1, 2)[s].tolist(), int(seg_slot[s])
+            assert not single or hi - lo == 1
+            q, k, v = (r[lo:hi, :m].float().reshape(hi - lo, -1, w) for r, m, w in zip(rows, (n, n, H * V), (D, D, V)))
+            q, k = (plain.unit(x).repeat_interleave(hpg, 1) for x in (q, k))
+            f = torch.exp(log_decay * plain.softplus(a[lo:hi, :H] + dt_bias))
+            o, state[sl] = plain.delta_scan(q * D ** -0.5, k, v, f, plain.sigmoid(b[lo:hi, :H]), torch.zeros_like(state[sl]) if int(pos[lo]) == 0 else state[sl])
+            out[lo:hi, :H * V] = o.reshape(hi - lo, -1)
+        return out
+
     def conv_rows(x, w, b, ring, seg, seg_slot, n_seg, longest, pos, out):
         taps, ch = w.shape
         for s in range(n_seg):
@@ -327,12 +426,12 @@ def install_host_ops(monkeypatch):
             assert hi - lo <= longest
             p0 = int(pos[lo])
             before = torch.stack([ring[sl, p % taps] if p >= 0 else torch.zeros(ch) for p in range(p0 - taps + 1, p0)]) if taps > 1 else torch.zeros(0, ch)
-            out[lo:hi, :ch] = plain.silu(plain.causal_conv(x[lo:hi, :ch], w.T, b, before))
+            out[lo:hi, :ch] = plain.silu(plain.causal_conv(x[lo:hi, :ch], w.T, torch.zeros(ch) if b is None else b, before))
             for t in range(max(lo, hi - taps), hi):
                 ring[sl, (p0 + t - lo) % taps] = x[t, :ch]
         return out
 
-    def attention(q, cache, block_table, tok_slot, pos, tile_row0, tile_rows, n_tiles, bm, H, T, scale, out, n_splits=1, workspace=None):
+    def attention(q, cache, block_table, tok_slot, pos, tile_row0, tile_rows, n_tiles, bm, H, T, scale, out, n_splits=1, workspace=None, window=1 << 30):
         page, Rc = cache.shape[-2], cache.shape[-1]
         rows = cache.view(-1, Rc)
         seen = torch.zeros(T * H, dtype=torch.bool)
@@ -342,10 +441,10 @@ def install_host_ops(monkeypatch):
             seen[r0:r0 + n] = True
         assert seen.all()
         for t in range(T):
-            k = torch.arange(int(pos[t]) + 1)
+            k = torch.arange(max(0, int(pos[t]) + 1 - window), int(pos[t]) + 1)
             c = rows[block_table[int(tok_slot[t]), k // page].long() * page + k % page].float()
             p = torch.softmax(q[t].view(H, Rc).float() @ c.T * scale, -1)
-            out[t] = (p @ c).reshape(-1).to(out.dtype)
+            out[t] = (p @ c)[:, :out.shape[1] // H].reshape(-1).to(out.dtype)
         return out
 
     def choose(logits, r):
@@ -398,19 +497,30 @@ def install_host_ops(monkeypatch):
         if shared is not None:
             out[:T] += plain.sigmoid(shared[1][:T, :1]) * shared[0][:T]
 
-    def gqa_prepare(m, proj, kc, vc, block_table, tok_slot, pos, slot, q, T):
+    def gqa_prepare(m, proj, kc, vc, block_table, tok_slot, pos, slot, q, T, mix=None):
         HD, GD, ps = m.H * m.D, m.G * m.maps * m.D, kc.shape[-2]
         q.zero_()
 
         def turn(x, p):
-            return plain.rotate_pairs(x, m.inv_freq, p) if m.adjacent else plain.rotate_half(x, m.rot, m.base, p)
+            if m.adjacent:
+                return plain.rotate_pairs(x, m.inv_freq, p)
+            a = p.float()[:, None, None] * m.inv_freq
+            n, c, s = m.rot // 2, m.rot_scale * torch.cos(a), m.rot_scale * torch.sin(a)
+            return torch.cat([x[..., :n] * c - x[..., n:2 * n] * s, x[..., n:2 * n] * c + x[..., :n] * s, x[..., 2 * n:]], -1)
+        values = proj[:T, HD + GD:HD + GD + m.G * m.V]
+        if mix is not None:
+            first, lam = mix
+            if lam is None:
+                first.copy_(values)
+            else:
+                values = (1 - lam) * values + lam * first
         for t in range(T):
             a, b = (turn((plain.rms(x, m.eps) * n if n is not None else x).view(1, -1, m.D), pos[t:t + 1])
                     for x, n in ((proj[t, :HD], m.q_norm), (proj[t, HD:HD + GD], m.k_norm)))
             q[t].view(m.H, m.Dc)[:, :m.D] = a[0]
             page, off = int(slot[t]) // ps, int(slot[t]) % ps
             kc[page, :, off, :m.D] = b[0]
-            vc[page, :, off, :m.V] = proj[t, HD + GD:].view(m.G, m.V)
+            vc[page, :, off, :m.V] = values[t].view(m.G, m.V)
 
     def gqa_attention(m, q, kc, vc, block_table, tok_slot, pos, tiles, bm, n_splits, out, T):
         row0, rows, n = tiles
@@ -431,9 +541,9 @@ def install_host_ops(monkeypatch):
         assert len(seen) == len(set(seen))
         return out
     for name, fn in dict(route=route, expert_matvec=expert_matvec, expert_plan=expert_plan, expert_gather=expert_gather, linear_grouped=linear_grouped,
-                         expert_combine=expert_combine, ssd=ssd, conv_rows=conv_rows, conv_args=lambda *a: a, gqa_prepare=gqa_prepare, gqa_attention=gqa_attention).items():
+                         expert_combine=expert_combine, ssd=ssd, delta=delta, out_tail=out_tail, conv_rows=conv_rows, conv_args=lambda *a: a, gqa_prepare=gqa_prepare, gqa_attention=gqa_attention).items():
         monkeypatch.setattr(L, name, fn)
     for name, fn in dict(row_stage=row_stage, stage_rows=stage_rows, head_matmul=head_matmul, embed=embed, latent_write=latent_write, hgrn2=scan,
-                         latent_attention=attention, matvec=lambda st, w, out, T, act=0: product(staged(st, T), w, out, act),
-                         linear=lambda x, w, out, act=0: product(x, w, out, act)).items():
+                         latent_attention=attention, matvec=lambda st, w, out, T, act=0, tail=None: product(staged(st, T), w, out, act, tail),
+                         linear=lambda x, w, out, act=0, tail=None: product(x, w, out, act, tail)).items():
         monkeypatch.setattr(L, name, fn)

@@ -1,10 +1,11 @@
-"""Plain, slow restatement of layer-list models (Talizen, Vozinex, Nifalorn) for the tests: one function per mechanism, whole sequences, float64.
+"""Plain, slow restatement of layer-list models (Talizen, Vozinex, Nifalorn, Rigalorn) for the tests: one function per mechanism, whole sequences, float64.
 
 Nothing here is shared with the product path: no kernels, no cache, no batching, no code of the package.  Every function takes the
 complete sequence of one request and returns a value per token.
 """
 from __future__ import annotations
 
+import functools
 import math
 
 import torch
@@ -283,6 +284,118 @@ def nifalorn_layer(x: torch.Tensor, spec: dict, w: dict, norm: dict) -> torch.Te
     return x
 
 
+def yarn_rotation(rot: dict) -> tuple[torch.Tensor, float]:
+    """Rotation frequencies and the factor on both cosine and sine.  With YaRN scaling, pairs that turn more than `fast` times within the
+    original context keep their frequency, those below `slow` turns are slowed down by `factor`, with a linear ramp over the pair number between."""
+    n, base = rot["dims"], rot["base"]
+    f = [base ** (-2 * i / n) for i in range(n // 2)]
+    s = rot.get("scaling")
+    if not s:
+        return torch.tensor(f, dtype=F), 1.0
+
+    def pair_of(turns):
+        return n * math.log(s["original"] / (2 * math.pi * turns)) / (2 * math.log(base))
+    lo, hi = max(math.floor(pair_of(s["fast"])), 0), min(math.ceil(pair_of(s["slow"])), n - 1)
+    out = []
+    for i, x in enumerate(f):
+        ramp = min(max((i - lo) / max(hi - lo, 0.001), 0.0), 1.0)
+        out.append(x / s["factor"] * ramp + x * (1 - ramp))
+    return torch.tensor(out, dtype=F), 0.1 * math.log(s["factor"]) + 1
+
+
+def turn_half(x: torch.Tensor, rot: dict, pos: torch.Tensor) -> torch.Tensor:
+    """x [T, H, d]: dimension i turns with dimension i + dims / 2 at the (scaled) frequencies of `rot`."""
+    f, amp = yarn_rotation(rot)
+    n = len(f)
+    a = pos.to(x.dtype)[:, None] * f.to(x.dtype)
+    c, s = amp * torch.cos(a)[:, None], amp * torch.sin(a)[:, None]
+    u, v = x[..., :n], x[..., n:2 * n]
+    return torch.cat([u * c - v * s, v * c + u * s, x[..., 2 * n:]], -1)
+
+
+def mix_values(v: torch.Tensor, first: torch.Tensor | None, lam: torch.Tensor) -> torch.Tensor:
+    """The first mixing layer keeps its values; the later ones blend them in."""
+    return v if first is None else (1 - lam) * v + lam * first
+
+
+def biased_attention_mixer(h: torch.Tensor, w: dict, m: dict, first: torch.Tensor | None = None):
+    """Grouped-query attention with biases on q, k and v, a sliding window, and values mixed with those of the first mixing layer.  Returns
+    the output and the layer's own values (before mixing)."""
+    T, H, G = h.shape[0], m["heads"], m["kv_heads"]
+    pos = torch.arange(T)
+    q, k, v = (h @ w[n].T + w[n + ".b"] for n in ("q", "k", "v"))
+    q, k = turn_half(q.reshape(T, H, m["dim"]), m["rot"], pos), turn_half(k.reshape(T, G, m["dim"]), m["rot"], pos)
+    mixed = mix_values(v, first, w["vmix"]) if m.get("v_mix") else v
+    o = masked_softmax_attention(q, k, mixed.reshape(T, G, m["vdim"]), m["scale"], window_mask(T, m["mask"]["size"], 0))
+    return o.reshape(T, H * m["vdim"]) @ w["o"].T, v
+
+
+def unit(x: torch.Tensor) -> torch.Tensor:
+    return x / torch.sqrt((x * x).sum(-1, keepdim=True) + 1e-6)
+
+
+def softplus(z: torch.Tensor) -> torch.Tensor:
+    return torch.log1p(torch.exp(-z.abs())) + torch.clamp(z, min=0)
+
+
+def delta_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, g: torch.Tensor, beta: torch.Tensor, state: torch.Tensor | None = None):
+    """q, k [T, H, d], v [T, H, dv], decay g and write strength beta [T, H] -> o [T, H, dv] and the last state [H, d, dv].  What the decayed
+    state already answers to k is taken off v before it is written."""
+    T, H, d = q.shape
+    S = torch.zeros(H, d, v.shape[-1], dtype=q.dtype) if state is None else state.clone()
+    out = []
+    for t in range(T):
+        S = g[t][:, None, None] * S
+        u = beta[t][:, None] * (v[t] - (S * k[t][:, :, None]).sum(1))
+        S = S + k[t][:, :, None] * u[:, None, :]
+        out.append((S * q[t][:, :, None]).sum(1))
+    return torch.stack(out), S
+
+
+def delta_mixer(h: torch.Tensor, w: dict, m: dict, eps: float) -> torch.Tensor:
+    T, H, G, D = h.shape[0], m["heads"], m["kv_heads"], m["dim"]
+    q, k, v = (silu(causal_conv(h @ w[n].T, w[n + ".conv"], torch.zeros(w[n].shape[0], dtype=h.dtype))) for n in ("q", "k", "v"))
+    q, k = (unit(x.reshape(T, G, D)).repeat_interleave(H // G, 1) for x in (q, k))
+    g = torch.exp(-torch.exp(w["A_log"]) * softplus(h @ w["a"].T + w["dt_bias"]))
+    o, _ = delta_scan(q * D ** -0.5, k, v.reshape(T, H, m["vdim"]), g, sigmoid(h @ w["b"].T))
+    return (rms(o, eps) * w["norm"]).reshape(T, -1) * silu(h @ w["g"].T) @ w["o"].T
+
+
+def low_rank_latent_mixer(h: torch.Tensor, w: dict, m: dict, eps: float) -> torch.Tensor:
+    """Latent attention whose queries pass a latent too; every head has a part with positions (neighbouring pairs), its key shared by all heads."""
+    T, H, D, V, R, P = h.shape[0], m["heads"], m["dim"], m["vdim"], m["kv_rank"], m["rot_dim"]
+    pos, (f, amp) = torch.arange(T), yarn_rotation(m["rot"])
+    q = ((rms(h @ w["dq"].T, eps) * w["dq.norm"]) @ w["uq"].T).reshape(T, H, D + P)
+    kv = h @ w["dkv"].T
+    c, kr = rms(kv[:, :R], eps) * w["dkv.norm"], amp * rotate_pairs(kv[:, None, R:], f, pos)
+    q = torch.cat([q[..., :D], amp * rotate_pairs(q[..., D:], f, pos)], -1)
+    k = torch.cat([(c @ w["uk"].T).reshape(T, H, D), kr.expand(T, H, P)], -1)
+    o = masked_softmax_attention(q, k, (c @ w["uv"].T).reshape(T, H, V), m["scale"], window_mask(T, m["mask"]["size"], 0))
+    return o.reshape(T, H * V) @ w["o"].T
+
+
+def xielu(z: torch.Tensor, p: torch.Tensor, q: torch.Tensor) -> torch.Tensor:
+    return z / 2 + torch.where(z > 0, softplus(p) * z * z, (0.5 + softplus(q)) * (torch.expm1(torch.clamp(z, max=0)) - z))
+
+
+def xielu_mlp(h: torch.Tensor, w: dict) -> torch.Tensor:
+    return xielu(h @ w["up"].T, w["act"][0], w["act"][1]) @ w["down"].T
+
+
+def rigalorn_layer(x: torch.Tensor, spec: dict, w: dict, norm: dict, kept: dict) -> torch.Tensor:
+    """One norm; mixer and feed-forward both read its output.  `kept`: values of the first layer that mixes them."""
+    sub = {p: {k[4:]: v for k, v in w.items() if k.startswith(p + ".")} for p in ("mix", "mlp")}
+    m = spec["mixer"]
+    h = rms(x, norm["eps"]) * w["norm1"]
+    if spec["type"] == "attention":
+        y, v = biased_attention_mixer(h, sub["mix"], m, kept.get("v"))
+        if m.get("v_mix"):
+            kept.setdefault("v", v)
+    else:
+        y = {"delta": delta_mixer, "latent_attention": low_rank_latent_mixer}[spec["type"]](h, sub["mix"], m, norm["eps"])
+    return x + (y + xielu_mlp(h, sub["mlp"]) if spec["mlp"] is not None else y)
+
+
 def layer(x: torch.Tensor, spec: dict, w: dict, norm: dict) -> torch.Tensor:
     """Talizen: both sublayers read x as it is; their outputs are normalised before they are added."""
     m = spec["mixer"]
@@ -326,13 +439,16 @@ def final_rows(cfg: dict, w: dict, x: torch.Tensor) -> torch.Tensor:
         return layer_norm(x, w["final.norm"], w["final.norm.b"], eps)
     if cfg["architecture"] == "Nifalorn":
         return rms(x, eps) * (1 + w["final.norm"])
+    if cfg["architecture"] == "Rigalorn":
+        return rms(x, eps) * w["final.norm"]
     return grouped_norm(x, w["final.norm"], cfg["norm"]["groups"], eps)
 
 
 def forward(cfg: dict, w: dict[str, torch.Tensor], tokens, dtype=F):
     """Logits [T, vocab] and the residual stream after every layer run [runs, T, width] of one whole sequence."""
     w = {k: v.to(dtype) for k, v in w.items()}
-    run = {"Talizen": layer, "Vozinex": pre_norm_layer, "Nifalorn": nifalorn_layer}[cfg["architecture"]]
+    kept = {}
+    run = {"Talizen": layer, "Vozinex": pre_norm_layer, "Nifalorn": nifalorn_layer, "Rigalorn": functools.partial(rigalorn_layer, kept=kept)}[cfg["architecture"]]
     emb = x = w["embed"][torch.as_tensor(list(tokens))] * cfg.get("embedding", {}).get("scale", 1.0)
     after = []
     for i, again in layer_runs(cfg):

@@ -462,7 +462,7 @@ def attention_case(H, G, D, V, window, keep, page, spans, dt, seed, rot=None, q_
     perm = torch.randperm(max_pages * len(spans) + 3, generator=torch.Generator().manual_seed(seed))
     bt = perm[:max_pages * len(spans)].view(len(spans), max_pages).to(torch.int32)
     Dc, Vc = (D + 15) // 16 * 16, (V + 15) // 16 * 16
-    m = SimpleNamespace(H=H, G=G, R=H // G, D=D, V=V, Dc=Dc, Vc=Vc, rot=rot, base=1000.0, window=window, keep=keep, chunk=chunk, maps=maps, adjacent=adjacent, eps=1e-4, scale=0.3,
+    m = SimpleNamespace(H=H, G=G, R=H // G, D=D, V=V, Dc=Dc, Vc=Vc, rot=rot, base=1000.0, window=window, keep=keep, chunk=chunk, maps=maps, adjacent=adjacent, rot_scale=1.0, eps=1e-4, scale=0.3,
                         q_norm=(r(H * D, scale=0.2) + 1).to(DEV) if q_norm else None, k_norm=(r(G * maps * D, scale=0.2) + 1).to(DEV) if q_norm else None,
                         inv_freq=(1000.0 ** (-2.0 * torch.arange(rot // 2, dtype=F64) / rot)).float().to(DEV) if rot else None)
     kc, vc = torch.full((len(perm), G * maps, page, Dc), 30.0), torch.full((len(perm), G, page, Vc), 1e4)      # rows nobody wrote

@@ -410,7 +410,7 @@ def moe_kernel_numbers(size: str, T: int = 2048):
             add("qwen3moe", f"experts down B={B}", "gemm_tcgen05_kernel (grouped)", us, hot * F * E * 2, 2 * A * F * E)
         del gate, up, down
     # decode attention: what the window shows of a long sequence, beside a plain cache of that many keys
-    m = SimpleNamespace(H=H, G=G, R=H // G, D=D, V=D, Dc=D, Vc=D, rot=D, window=window, keep=keep, chunk=0, maps=1, adjacent=False, eps=1e-5, scale=D ** -0.5, visible=lambda n: min(n, window + keep),
+    m = SimpleNamespace(H=H, G=G, R=H // G, D=D, V=D, Dc=D, Vc=D, rot=D, window=window, keep=keep, chunk=0, maps=1, adjacent=False, rot_scale=1.0, eps=1e-5, scale=D ** -0.5, visible=lambda n: min(n, window + keep),
                         q_norm=torch.ones(H * D, device=DEV), k_norm=torch.ones(G * D, device=DEV),
                         inv_freq=(1e6 ** (-torch.arange(0, D, 2, dtype=torch.float64) / D)).float().to(DEV))
     seen, ctx = window + keep, 8192

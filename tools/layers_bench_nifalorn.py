@@ -174,9 +174,9 @@ def kernel_numbers(size: str, graph_us, copies, peaks, T: int = 2048):
         add("nifalorn", f"recurrence decode, mamba2 B={B}", "ssd_decode_kernel (with the convolution)", us, nb, 6 * B * M * N * 64)
     # decode attention over one chunk
     rot = (5e5 ** (-torch.arange(0, 64, 2, dtype=torch.float64) / 64)).float().to(DEV)
-    two = SimpleNamespace(H=2 * A, G=G, R=2 * A // G, D=64, V=D, Dc=64, Vc=D, rot=64, window=1 << 30, keep=0, chunk=chunk, maps=2, adjacent=True, eps=1e-5, scale=0.125, q_norm=None, k_norm=None,
+    two = SimpleNamespace(H=2 * A, G=G, R=2 * A // G, D=64, V=D, Dc=64, Vc=D, rot=64, window=1 << 30, keep=0, chunk=chunk, maps=2, adjacent=True, rot_scale=1.0, eps=1e-5, scale=0.125, q_norm=None, k_norm=None,
                           inv_freq=rot, visible=lambda n: min(n, chunk))
-    one = SimpleNamespace(H=A, G=G, R=A // G, D=D, V=D, Dc=D, Vc=D, rot=D, window=chunk, keep=0, chunk=0, maps=1, adjacent=False, eps=1e-5, scale=D ** -0.5, visible=lambda n: min(n, chunk),
+    one = SimpleNamespace(H=A, G=G, R=A // G, D=D, V=D, Dc=D, Vc=D, rot=D, window=chunk, keep=0, chunk=0, maps=1, adjacent=False, rot_scale=1.0, eps=1e-5, scale=D ** -0.5, visible=lambda n: min(n, chunk),
                           q_norm=torch.ones(AD, device=DEV), k_norm=torch.ones(G * D, device=DEV), inv_freq=(1e6 ** (-torch.arange(0, D, 2, dtype=torch.float64) / D)).float().to(DEV))
     NI, ctx = AD + 2 * G * D, 4 * chunk
     for B in (1, 4, 16):
