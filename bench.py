@@ -356,7 +356,7 @@ def main():
     ap.add_argument("--emulate-tp", type=int, default=0, help="1 GPU only: time rank 0 of an N-way tensor-parallel step (profiling aid)")
     ap.add_argument("--no-tp-check", action="store_true", help="skip the fused-vs-NCCL greedy token comparison")
     ap.add_argument("--tp-impl", default=os.environ.get("DLP_TP_IMPL", "fused"), choices=["fused", "nccl"])
-    ap.add_argument("--layers", nargs="?", const="2048,4096,moe-2048,moe-4096,hybrid-2048,hybrid-4096", default=None, metavar="SIZES",
+    ap.add_argument("--layers", nargs="?", const="2048,4096,moe-2048,moe-4096,hybrid-2048,hybrid-4096,parallel-2048,parallel-4096", default=None, metavar="SIZES",
                     help="instead of the headline workload: layer-list models beside the closest other model of equal size, and each kernel against its roofline (tools/layers_bench.py)")
     args = ap.parse_args()
     if args.layers:

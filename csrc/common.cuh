@@ -86,6 +86,11 @@ __device__ __forceinline__ float warp_max(float v) {
 // block-wide sum; `red` must hold >= 32 floats of shared memory. All threads get the result.
 // see OutTail (kernels.cuh); expm1f keeps the digits of exp(z) - 1 next to zero
 __device__ __forceinline__ float xielu(float z, float pos, float neg) { return fmaf(0.5f, z, z > 0.f ? pos * z * z : neg * (expm1f(z) - z)); }
+// where the result is rounded to bf16: exp(z) - 1 - z as its series next to zero
+__device__ __forceinline__ float xielu_fast(float z, float pos, float neg) {
+    const float zz = z * z, near = zz * fmaf(z, fmaf(z, 1.f / 24.f, 1.f / 6.f), 0.5f), far = __expf(z) - 1.f - z;
+    return fmaf(0.5f, z, z > 0.f ? pos * zz : neg * (z > -0.0625f ? near : far));
+}
 __device__ __forceinline__ float block_sum(float v, float* red) {
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = (blockDim.x + 31) >> 5;
     v = warp_sum(v);

@@ -110,7 +110,7 @@ __device__ __forceinline__ void prefetch_row_slice(const QWeight& w, int row, in
 }
 
 template <int MODE, int CH>
-__device__ __forceinline__ void epi_loop(const GemmParams& p, const uint32_t (&r0)[CH], const uint32_t (&r1)[CH], int tb, int n, int t_end) {
+__device__ __forceinline__ void epi_loop(const GemmParams& p, const uint32_t (&r0)[CH], const uint32_t (&r1)[CH], int tb, int n, int t_end, float bias = 0.f) {
     if (MODE == EPI_RS_PUSH_F32) {
         // GEMM -> reduce-scatter: token t is owned by rank t / rs_rows; our partial for it goes straight into that rank's
         // reduce buffer, slot [our rank][t % rs_rows][n] (NVLink store).  Owner / local row advance incrementally.
@@ -130,17 +130,17 @@ __device__ __forceinline__ void epi_loop(const GemmParams& p, const uint32_t (&r
         return;
     }
     if (MODE == EPI_TAIL_BF16) {
-        const float bias = p.tail.bias != nullptr ? p.tail.bias[n] : 0.f;
         if (n < p.tail.n2) {
             float* dst = reinterpret_cast<float*>(p.y) + (size_t)tb * p.ldy + n;
 #pragma unroll
             for (int j = 0; j < CH; ++j, dst += p.ldy)
                 if (tb + j < t_end) *dst = __uint_as_float(r0[j]) + bias;
         } else {
+            const float pos = p.tail.pos, neg = p.tail.neg;
             __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(p.tail.out2) + (size_t)tb * p.tail.ldo2 + (n - p.tail.n2);
 #pragma unroll
             for (int j = 0; j < CH; ++j, dst += p.tail.ldo2)
-                if (tb + j < t_end) *dst = __float2bfloat16_rn(xielu(__uint_as_float(r0[j]) + bias, p.tail.pos, p.tail.neg));
+                if (tb + j < t_end) *dst = __float2bfloat16_rn(xielu_fast(__uint_as_float(r0[j]) + bias, pos, neg));
         }
         return;
     }
@@ -296,6 +296,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tm_w0, const __grid_cons
         const int q = warp & 3;
         const int n_local = q * 32 + lane;
         const int n = n_out0 + n_local;
+        const float bias = p.epilogue == EPI_TAIL_BF16 && p.tail.bias != nullptr && n < p.N ? p.tail.bias[n] : 0.f;      // (requested before the accumulators are there)
         if (num_kb > 0) {
             mbar_wait(tmem_full_bar, 0);
             tc_fence_after();
@@ -334,7 +335,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tm_w0, const __grid_cons
                     case EPI_GEGLU_BF16: if (NA == 2 && AB_FMT == 1) epi_loop<EPI_GEGLU_BF16, CH>(p, r0, r1, tb, n, t_end); break;
                     case EPI_SWIGLU_BF16: if (NA == 2 && AB_FMT == 1) epi_loop<EPI_SWIGLU_BF16, CH>(p, r0, r1, tb, n, t_end); break;
                     case EPI_RELU2_BF16: if (NA == 1 && AB_FMT == 1) epi_loop<EPI_RELU2_BF16, CH>(p, r0, r1, tb, n, t_end); break;
-                    case EPI_TAIL_BF16: if (NA == 1 && AB_FMT == 1) epi_loop<EPI_TAIL_BF16, CH>(p, r0, r1, tb, n, t_end); break;
+                    case EPI_TAIL_BF16: if (NA == 1 && AB_FMT == 1) epi_loop<EPI_TAIL_BF16, CH>(p, r0, r1, tb, n, t_end, bias); break;
                     case EPI_RS_PUSH_F32: epi_loop<EPI_RS_PUSH_F32, CH>(p, r0, r1, tb, n, t_end); break;
                 }
             }

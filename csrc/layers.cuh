@@ -176,14 +176,20 @@ struct DeltaArgs {
     float unit_eps, q_scale;
 };
 constexpr int DELTA_CHUNK = 64;
+// Workspaces of the chunked form, in the layouts in which they are read into shared memory.  Dp: D rounded up to 64 or 128; S: slices of 16 value
+// columns; pairs of bf16 parts are value and remainder.
+constexpr int DELTA_ROW = DELTA_CHUNK + 8;      // row of a 64 x 64 matrix
 struct DeltaChunks {
     const int* chunk;         // [n_chunks][2], as in ScanChunks
     const int* first;         // [n_seg + 1]
-    void* states;             // [n_chunks, H, 2, D, V] bf16: the state a chunk starts from, value and remainder
-    void* solve;              // [n_chunks, H, 2, 64, 64] bf16: the chunk's triangular inverse, value and remainder
-    void* u;                  // [2, T, H * V] bf16: what every token writes, value and remainder
-    float* gates;             // [n_chunks, H, 64, 4]: cumulative log2 decay, 1 / |k|, beta
-    int n_chunks, T;
+    void* states;             // [n_chunks, H, S][2][Dp][16] bf16: the state a chunk starts from
+    void* keys;               // [n_chunks, H / hpg][64][Dp + 8] bf16
+    void* solve;              // [n_chunks, H][2][64][DELTA_ROW] bf16: the chunk's triangular inverse
+    void* weights;            // [n_chunks, H][2][64][DELTA_ROW] bf16: what a token's output takes of every write up to its own
+    void* u;                  // [n_chunks, H, S][2][64][16] bf16: what every token writes
+    float* gates;             // [n_chunks, H][64 x 4 | 64]: write strength, the same times decay from the chunk's start / |k|, decay to its end / |k|,
+                              //                             decay of the whole chunk | decay from the start times scale / |q|
+    int n_chunks, pad;
 };
 int delta_scan(const DeltaArgs& a, cudaStream_t s);
 int delta_decode(const DeltaArgs& a, const ConvArgs* conv, cudaStream_t s);        // one token per segment; conv: q, k, v point into conv->x

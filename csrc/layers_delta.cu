@@ -9,7 +9,8 @@
 //
 // Chunks: with L the cumulative log decay inside a chunk, the writes solve a unit lower triangular system,
 //   (I + A) u = beta (v - exp(L) S_start^T k),   A_ts = beta_t exp(L_t - L_s) (k_t . k_s),  s < t
-// whose inverse does not depend on the state: it is formed for all chunks at once (solve), the state then runs over the chunks (state), and
+// whose inverse does not depend on the state: it is formed for all chunks at once (solve), as are the weights of the outputs; the state then
+// runs over the chunks (state), and
 //   o_t = exp(L_t) S_start^T q_t + sum_{s <= t} exp(L_t - L_s) (q_t . k_s) u_s
 // again for all chunks at once (out).  Exponents are never positive.  Rows behind the convolution are bf16 operands as they are; the factors
 // that make q and k unit vectors join the fp32 token weights.  Weights, inverse, writes and states are fp32 and enter the tensor cores as two
@@ -286,7 +287,7 @@ int delta_decode(const DeltaArgs& a, const ConvArgs* cv, cudaStream_t s) {
 }
 
 // ---- chunks --------------------------------------------------------------------------------------------------------------------------------
-constexpr int DC = DELTA_CHUNK, DLT = DC + 8;
+constexpr int DC = DELTA_CHUNK, DLT = DELTA_ROW;
 typedef __nv_bfloat16 bf16;
 
 // sums of squares of the rows of a [DC][DP + 8] tile, PT threads per row; every thread of a row gets its sum
@@ -309,26 +310,47 @@ __device__ __forceinline__ float row_squares(const bf16* tile) {
     return s;
 }
 
-// The inverse of I + A, in 16-row blocks: the diagonal ones by substitution (a lane per column), then the blocks below them by distance,
-// T_ij = -T_ii sum_m A_im T_mj; all in fp32.  64 threads share a block, four outputs each.
+constexpr int DGATES = DC * 4 + DC;             // floats of a chunk's gates
+template <int DP> __device__ __forceinline__ bf16* chunk_keys(const DeltaArgs& a, const DeltaChunks& c, int ch, int h) {
+    return reinterpret_cast<bf16*>(c.keys) + ((size_t)ch * (a.H / a.hpg) + h / a.hpg) * DC * (DP + 8);
+}
+__device__ __forceinline__ bf16* chunk_matrix(void* base, const DeltaArgs& a, int ch, int h) { return reinterpret_cast<bf16*>(base) + ((size_t)ch * a.H + h) * 2 * DC * DLT; }
+__device__ __forceinline__ float* chunk_gates(const DeltaArgs& a, const DeltaChunks& c, int ch, int h) { return c.gates + ((size_t)ch * a.H + h) * DGATES; }
+constexpr int DV = 16, DLV = DV + 8;            // value columns of a slice, and their row in shared memory
+__device__ __forceinline__ size_t chunk_slice(const DeltaArgs& a, int ch, int h, int slice) { return ((size_t)ch * a.H + h) * ((a.V + DV - 1) / DV) + slice; }
+// N 16-byte pieces to shared memory with cp.async, NTH threads
+template <int N, int NTH>
+__device__ __forceinline__ void copy_pieces(void* dst, const void* src) {
+#pragma unroll
+    for (int i = 0; i < (N + NTH - 1) / NTH; ++i)
+        if (i * NTH + NTH - 1 < N || i * NTH + (int)threadIdx.x < N) cp_async16(reinterpret_cast<uint4*>(dst) + i * NTH + threadIdx.x, reinterpret_cast<const uint4*>(src) + i * NTH + threadIdx.x, true);
+}
+
+// Everything of a chunk that does not depend on the state: gates, the keys' tile, the weights of the outputs, and the inverse of I + A in fp32:
+// its 16-row diagonal blocks by substitution (a lane per column), then what lies below them by blocks of 16 and of 32,
+//   [P 0; R Q]^-1 = [P^-1 0; -Q^-1 R P^-1 Q^-1]
 constexpr int DAP = DC + 4;
 template <int DP>
 struct DeltaSolveCfg {
-    static constexpr size_t SMEM = (size_t)(2 * DC * DAP + 3 * 16 * 20 + 3 * DC) * 4 + (size_t)DC * (DP + 8) * 2;
+    static constexpr int QT = DC * (DP + 8) * 2 > DC * DAP * 4 ? DC * (DP + 8) * 2 : DC * DAP * 4;      // the inverse takes the place of the queries
+    static constexpr size_t SMEM = (size_t)DC * (DP + 8) * 2 + QT + (size_t)(DC * DAP + 4 * DC) * 4;
 };
 template <int DP>
 __global__ void __launch_bounds__(256) delta_chunk_solve_kernel(const DeltaArgs a, const DeltaChunks cc) {
     constexpr int LDK = DP + 8;
     extern __shared__ __align__(16) uint8_t dc_smem[];
     bf16* sk = reinterpret_cast<bf16*>(dc_smem);                          // [DC][LDK]
-    float* A = reinterpret_cast<float*>(sk + DC * LDK);                   // [DC][DAP]
-    float* Ti = A + DC * DAP;                                             // [DC][DAP]
-    float* X = Ti + DC * DAP;                                             // [3][16][20]
-    float *sL = X + 3 * 16 * 20, *srk = sL + DC, *sb = srk + DC;
+    bf16* sq = sk + DC * LDK;                                             // [DC][LDK]
+    float* Ti = reinterpret_cast<float*>(sq);                             // [DC][DAP]
+    float* A = reinterpret_cast<float*>(reinterpret_cast<uint8_t*>(sq) + DeltaSolveCfg<DP>::QT);      // [DC][DAP]
+    float* X = A + 32;                                                    // [32][DAP], above the blocks of A that are used
+    float *sL = A + DC * DAP, *srk = sL + DC, *srq = srk + DC, *sb = srq + DC;
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, ch = blockIdx.x, h = blockIdx.y;
     pdl_wait();
     const int t0 = cc.chunk[2 * ch], n = cc.chunk[2 * ch + 1];
-    chunk_tile<bf16, DC, DP, 256>(a.k, a.ldk, (size_t)(h / a.hpg) * a.D, t0, n, a.D, 0, sk);
+    const size_t qk0 = (size_t)(h / a.hpg) * a.D;
+    chunk_tile<bf16, DC, DP, 256>(a.k, a.ldk, qk0, t0, n, a.D, 0, sk);
+    chunk_tile<bf16, DC, DP, 256>(a.q, a.ldq, qk0, t0, n, a.D, 0, sq);
     cp_commit();
     if (tid < DC) {
         float L = tid < n ? delta_log_decay(a, t0 + tid, h) * LOG2E_F : 0.f;
@@ -342,110 +364,146 @@ __global__ void __launch_bounds__(256) delta_chunk_solve_kernel(const DeltaArgs 
     }
     cp_wait<0>();
     __syncthreads();
-    const float carry = sL[31];
-    const float ss = row_squares<DP, 4>(sk);
-    if ((tid & 3) == 0) srk[tid >> 2] = 1.f / sqrtf(ss + a.unit_eps);
-    __syncthreads();
-    if (tid < DC) {
-        const float L = sL[tid] + (tid >= 32 ? carry : 0.f);
-        if (tid >= 32) sL[tid] = L;
-        reinterpret_cast<float4*>(cc.gates)[((size_t)ch * a.H + h) * DC + tid] = make_float4(L, srk[tid], sb[tid], 0.f);
+    const float carry = sL[31], kk = row_squares<DP, 4>(sk), qq = row_squares<DP, 4>(sq);
+    if ((tid & 3) == 0) {
+        srk[tid >> 2] = 1.f / sqrtf(kk + a.unit_eps);
+        srq[tid >> 2] = a.q_scale / sqrtf(qq + a.unit_eps);
     }
     __syncthreads();
-    // A: lower triangle, 16 x 16 blocks
-    for (int idx = warp; idx < 10; idx += 8) {
-        const int mt = idx < 1 ? 0 : idx < 3 ? 1 : idx < 6 ? 2 : 3, kb = idx - mt * (mt + 1) / 2;
+    if (tid >= 32 && tid < DC) sL[tid] += carry;
+    __syncthreads();
+    if (tid < DC) {
+        const float L = sL[tid], end = sL[DC - 1], b = sb[tid], rk = srk[tid], from = exp2f(L);
+        float* g = chunk_gates(a, cc, ch, h);
+        reinterpret_cast<float4*>(g)[tid] = make_float4(b, b * from * rk, exp2f(end - L) * rk, exp2f(end));
+        g[4 * DC + tid] = from * srq[tid];
+    }
+    if (h % a.hpg == 0) {
+        bf16* out = chunk_keys<DP>(a, cc, ch, h);
+        for (int i = tid; i < DC * LDK / 8; i += 256) reinterpret_cast<uint4*>(out)[i] = reinterpret_cast<const uint4*>(sk)[i];
+    }
+    // lower triangle in 16 x 16 blocks: A (ten blocks) and the weights (ten more)
+    bf16* wout = chunk_matrix(cc.weights, a, ch, h);
+    for (int idx = warp; idx < 20; idx += 8) {
+        const bool is_w = idx >= 10;
+        const int i = is_w ? idx - 10 : idx, mt = i < 1 ? 0 : i < 3 ? 1 : i < 6 ? 2 : 3, kb = i - mt * (mt + 1) / 2;
+        const bf16* left = is_w ? sq : sk;
         float p[2][4] = {};
 #pragma unroll
         for (int ks = 0; ks < DP / 16; ++ks) {
             uint32_t af[4], bf[4];
-            ldsm_x4(af, sk + (mt * 16 + (lane & 15)) * LDK + ks * 16 + (lane >> 4) * 8);
+            ldsm_x4(af, left + (mt * 16 + (lane & 15)) * LDK + ks * 16 + (lane >> 4) * 8);
             ldsm_x4(bf, sk + (kb * 16 + (lane & 7) + (lane >> 4) * 8) * LDK + ks * 16 + ((lane >> 3) & 1) * 8);
             mma16816(p[0], af, bf[0], bf[1]);
             mma16816(p[1], af, bf[2], bf[3]);
         }
+        const int ta = mt * 16 + (lane >> 2), s0 = kb * 16 + (lane & 3) * 2;
+        const float* row = is_w ? srq : srk;
+        float La[2] = {sL[ta], sL[ta + 8]}, fa[2] = {row[ta], row[ta + 8]};
+        if (!is_w) { fa[0] *= sb[ta]; fa[1] *= sb[ta + 8]; }
 #pragma unroll
-        for (int b = 0; b < 2; ++b)
+        for (int b = 0; b < 2; ++b) {
+            const int s = s0 + b * 8;
+            const float2 Ls = *reinterpret_cast<const float2*>(sL + s), fs = *reinterpret_cast<const float2*>(srk + s);
 #pragma unroll
-            for (int e = 0; e < 4; ++e) {
-                const int t = mt * 16 + (lane >> 2) + (e >> 1) * 8, s = kb * 16 + b * 8 + (lane & 3) * 2 + (e & 1);
-                A[t * DAP + s] = s < t ? p[b][e] * (sb[t] * srk[t] * srk[s] * exp2f(sL[t] - sL[s])) : 0.f;
-            }
-    }
-    __syncthreads();
-    if (warp < 4) {
-        if (lane < 16) {
-            const float* Ad = A + (warp * 16) * DAP + warp * 16;
-            float x[16];
-#pragma unroll
-            for (int i = 0; i < 16; ++i) {
-                float v = i == lane ? 1.f : 0.f;
-#pragma unroll
-                for (int m = 0; m < i; ++m) v = fmaf(-Ad[i * DAP + m], x[m], v);
-                x[i] = v;
-            }
-#pragma unroll
-            for (int i = 0; i < 16; ++i) Ti[(warp * 16 + i) * DAP + warp * 16 + lane] = x[i];
-        }
-    } else {
-        for (int i = tid - 128; i < DC * DC; i += 128) {
-            const int r = i / DC, c = i - r * DC;
-            if (c >> 4 > r >> 4) Ti[r * DAP + c] = 0.f;
-        }
-    }
-    __syncthreads();
-    const int grp = tid >> 6, r = (tid & 63) >> 2, c4 = (tid & 3) * 4;
-#pragma unroll 1
-    for (int dist = 1; dist < 4; ++dist) {
-        const int i = dist + grp, j = grp;
-        float x[4] = {0.f, 0.f, 0.f, 0.f};
-        auto mac = [&](const float* row, const float* mat, int ld) {       // x += row (16) * mat (16 x 4 columns)
-#pragma unroll
-            for (int m = 0; m < 16; m += 4) {
-                const float4 w = *reinterpret_cast<const float4*>(row + m);
-                const float wv[4] = {w.x, w.y, w.z, w.w};
-#pragma unroll
-                for (int q = 0; q < 4; ++q) {
-                    const float4 b = *reinterpret_cast<const float4*>(mat + (m + q) * ld);
-                    x[0] = fmaf(wv[q], b.x, x[0]);
-                    x[1] = fmaf(wv[q], b.y, x[1]);
-                    x[2] = fmaf(wv[q], b.z, x[2]);
-                    x[3] = fmaf(wv[q], b.w, x[3]);
+            for (int half = 0; half < 2; ++half) {
+                const int t = ta + half * 8, seen = t + (is_w ? 1 : 0);
+                const float x = s < seen ? p[b][half * 2] * (fa[half] * fs.x * exp2f(La[half] - Ls.x)) : 0.f;
+                const float y = s + 1 < seen ? p[b][half * 2 + 1] * (fa[half] * fs.y * exp2f(La[half] - Ls.y)) : 0.f;
+                if (is_w) {
+                    uint32_t hi, lo;
+                    split_bf16(x, y, hi, lo);
+                    *reinterpret_cast<uint32_t*>(wout + t * DLT + s) = hi;
+                    *reinterpret_cast<uint32_t*>(wout + (DC + t) * DLT + s) = lo;
+                } else {
+                    *reinterpret_cast<float2*>(A + t * DAP + s) = make_float2(x, y);
                 }
             }
-        };
-        if (i < 4) {
-#pragma unroll 1
-            for (int m = j; m < i; ++m) mac(A + (i * 16 + r) * DAP + m * 16, Ti + m * 16 * DAP + j * 16 + c4, DAP);
-            *reinterpret_cast<float4*>(X + (grp * 16 + r) * 20 + c4) = make_float4(x[0], x[1], x[2], x[3]);
+        }
+    }
+    __syncthreads();
+    if (warp < 4 && lane < 16) {
+        const float* Ad = A + (warp * 16) * DAP + warp * 16;
+        float x[16];
+#pragma unroll
+        for (int i = 0; i < 16; ++i) {
+            float v = i == lane ? 1.f : 0.f;
+#pragma unroll
+            for (int m = 0; m < i; ++m) v = fmaf(-Ad[i * DAP + m], x[m], v);
+            x[i] = v;
+        }
+#pragma unroll
+        for (int i = 0; i < 16; ++i) Ti[(warp * 16 + i) * DAP + warp * 16 + lane] = x[i];
+    }
+    __syncthreads();
+    // x += row (16) * mat (16 x 4 columns)
+    auto mac = [](float (&x)[4], const float* row, const float* mat, int ld) {
+#pragma unroll
+        for (int m = 0; m < 16; m += 4) {
+            const float4 w = *reinterpret_cast<const float4*>(row + m);
+            const float wv[4] = {w.x, w.y, w.z, w.w};
+#pragma unroll
+            for (int q = 0; q < 4; ++q) {
+                const float4 b = *reinterpret_cast<const float4*>(mat + (m + q) * ld);
+                x[0] = fmaf(wv[q], b.x, x[0]);
+                x[1] = fmaf(wv[q], b.y, x[1]);
+                x[2] = fmaf(wv[q], b.z, x[2]);
+                x[3] = fmaf(wv[q], b.w, x[3]);
+            }
+        }
+    };
+    {   // blocks (1, 0) and (3, 2): 64 threads each
+        const int i = 2 * (tid >> 6) + 1, r = (tid & 63) >> 2, c4 = (tid & 3) * 4;
+        float x[4] = {0.f, 0.f, 0.f, 0.f};
+        if (tid < 128) {
+            mac(x, A + (i * 16 + r) * DAP + (i - 1) * 16, Ti + (i - 1) * 16 * DAP + (i - 1) * 16 + c4, DAP);
+            *reinterpret_cast<float4*>(X + ((tid >> 6) * 16 + r) * DAP + c4) = make_float4(x[0], x[1], x[2], x[3]);
+        } else {               // what lies above the diagonal of the two 32-row blocks
+            const int j = tid - 128, b = j >> 6;
+            *reinterpret_cast<float4*>(Ti + (b * 32 + ((j & 63) >> 2)) * DAP + b * 32 + 16 + c4) = make_float4(0.f, 0.f, 0.f, 0.f);
         }
         __syncthreads();
-        if (i < 4) {
+        if (tid < 128) {
             x[0] = x[1] = x[2] = x[3] = 0.f;
-            mac(Ti + (i * 16 + r) * DAP + i * 16, X + grp * 16 * 20 + c4, 20);
-            *reinterpret_cast<float4*>(Ti + (i * 16 + r) * DAP + j * 16 + c4) = make_float4(-x[0], -x[1], -x[2], -x[3]);
+            mac(x, Ti + (i * 16 + r) * DAP + i * 16, X + (tid >> 6) * 16 * DAP + c4, DAP);
+            *reinterpret_cast<float4*>(Ti + (i * 16 + r) * DAP + (i - 1) * 16 + c4) = make_float4(-x[0], -x[1], -x[2], -x[3]);
         }
         __syncthreads();
     }
-    bf16* out = reinterpret_cast<bf16*>(cc.solve) + ((size_t)ch * a.H + h) * 2 * DC * DC;
+    {   // the 32 x 32 block below
+        const int r = tid >> 3, c4 = (tid & 7) * 4;
+        float x[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+        for (int m = 0; m < 32; m += 16) mac(x, A + (32 + r) * DAP + m, Ti + m * DAP + c4, DAP);
+        *reinterpret_cast<float4*>(X + r * DAP + c4) = make_float4(x[0], x[1], x[2], x[3]);
+        __syncthreads();
+        x[0] = x[1] = x[2] = x[3] = 0.f;
+#pragma unroll
+        for (int m = 0; m < 32; m += 16)
+            if (m <= r) mac(x, Ti + (32 + r) * DAP + 32 + m, X + m * DAP + c4, DAP);
+        *reinterpret_cast<float4*>(Ti + (32 + r) * DAP + c4) = make_float4(-x[0], -x[1], -x[2], -x[3]);
+        __syncthreads();
+    }
+    bf16* out = chunk_matrix(cc.solve, a, ch, h);
 #pragma unroll
     for (int i = tid; i < DC * DC / 4; i += 256) {
         const int rr = i / (DC / 4), q = i % (DC / 4) * 4;
-        put_split(out + rr * DC + q, out + DC * DC + rr * DC + q, *reinterpret_cast<const float4*>(Ti + rr * DAP + q));
+        put_split(out + rr * DLT + q, out + (DC + rr) * DLT + q, q >> 4 > rr >> 4 ? make_float4(0.f, 0.f, 0.f, 0.f) : *reinterpret_cast<const float4*>(Ti + rr * DAP + q));
     }
     pdl_launch_dependents();
 }
 
-// The state over the chunks of a segment: a block keeps DV columns of one head's state in its accumulators.  Per chunk: products with the keys
-// (S^T k of all tokens), the triangular solve, the update; the next chunk's operands arrive meanwhile.
-constexpr int DV = 16, DLV = DV + 8;
+// The state over the chunks of a segment: a block keeps DV columns of one head's state in its accumulators.  Per chunk eight warps form the products
+// with the keys (S^T k of all tokens), solve the triangular system, and update the state; warp 0 brings the next chunk's operands and stores the
+// state the chunk starts from meanwhile.
 template <int DP>
 struct DeltaStateCfg {
     static constexpr int LDK = DP + 8;
     static constexpr size_t SMEM = (size_t)(2 * DC * LDK + 4 * DC * DLT + 2 * DC * DLV + 2 * DP * DLV + 4 * DC * DLV) * 2 + 2 * DC * 16;
 };
+__device__ __forceinline__ void state_barrier() { asm volatile("bar.sync 1, 288;" ::: "memory"); }
 template <int DP>
-__global__ void __launch_bounds__(256, 2) delta_chunk_state_kernel(const DeltaArgs a, const DeltaChunks cc) {
+__global__ void __launch_bounds__(288, 2) delta_chunk_state_kernel(const DeltaArgs a, const DeltaChunks cc) {
     constexpr int LDK = DP + 8, MT = DP / 16, WN = 8 / MT, NT = DV / 8 / WN;
     extern __shared__ __align__(16) uint8_t dc_smem[];
     bf16* sk = reinterpret_cast<bf16*>(dc_smem);          // [2][DC][LDK]
@@ -455,25 +513,38 @@ __global__ void __launch_bounds__(256, 2) delta_chunk_state_kernel(const DeltaAr
     bf16* sr = sS + 2 * DP * DLV;                         // [part][DC][DLV]
     bf16* su = sr + 2 * DC * DLV;                         // [part][DC][DLV]
     float4* sg = reinterpret_cast<float4*>(su + 2 * DC * DLV);      // [2][DC]
-    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, c2 = (lane & 3) * 2;
-    const int v0 = blockIdx.x * DV, h = blockIdx.y, seg = blockIdx.z, ncol = min(DV, a.V - v0);
+    const int lane = threadIdx.x & 31, warp = (threadIdx.x >> 5) - 1, g = lane >> 2, c2 = (lane & 3) * 2;
+    const int v0 = blockIdx.x * DV, h = blockIdx.y, seg = blockIdx.z;
     pdl_wait();
-    const int first = cc.first[seg], last = cc.first[seg + 1];
-    auto fetch = [&](int ch, int b) {
-        const int t0 = cc.chunk[2 * ch], n = cc.chunk[2 * ch + 1];
-        chunk_tile<bf16, DC, DP, 256>(a.k, a.ldk, (size_t)(h / a.hpg) * a.D, t0, n, a.D, 0, sk + b * DC * LDK);
-        chunk_tile<bf16, DC, DV, 256>(a.v, a.ldv, (size_t)h * a.V + v0, t0, n, ncol, 0, sv + b * DC * DLV);
-        const bf16* T = reinterpret_cast<const bf16*>(cc.solve) + ((size_t)ch * a.H + h) * 2 * DC * DC;
-#pragma unroll
-        for (int i = tid; i < 2 * DC * DC / 8; i += 256) cp_async16(sT + b * 2 * DC * DLT + (i / (DC / 8)) * DLT + i % (DC / 8) * 8, T + i * 8, true);
-        if (tid < DC) cp_async16(sg + b * DC + tid, cc.gates + (((size_t)ch * a.H + h) * DC + tid) * 4, true);
-        cp_commit();
-    };
-    if (first < last) fetch(first, 0);
+    const int first = cc.first[seg], last = cc.first[seg + 1], lo = a.seg[2 * seg], hi = a.seg[2 * seg + 1];
+    if (warp < 0) {
+        const int ncol = min(DV, a.V - v0);
+        for (int ch = first; ch <= last; ++ch) {          // (one step ahead of the other warps)
+            const int b = (ch - first) & 1, t0 = lo + (ch - first) * DC;
+            if (ch < last) {
+                copy_pieces<DC * LDK / 8, 32>(sk + b * DC * LDK, chunk_keys<DP>(a, cc, ch, h));
+                copy_pieces<2 * DC * DLT / 8, 32>(sT + b * 2 * DC * DLT, chunk_matrix(cc.solve, a, ch, h));
+                copy_pieces<DC, 32>(sg + b * DC, chunk_gates(a, cc, ch, h));
+                chunk_tile<bf16, DC, DV, 32>(a.v, a.ldv, (size_t)h * a.V + v0, t0, min(DC, hi - t0), ncol, 0, sv + b * DC * DLV);
+                cp_commit();
+            }
+            if (ch > first) {
+                uint4* out = reinterpret_cast<uint4*>(reinterpret_cast<bf16*>(cc.states) + chunk_slice(a, ch - 1, h, blockIdx.x) * 2 * DP * DV);
+#pragma unroll 8
+                for (int i = lane; i < 2 * DP * DV / 8; i += 32) out[i] = *reinterpret_cast<const uint4*>(sS + (i >> 1) * DLV + (i & 1) * 8);
+                state_barrier();
+                state_barrier();
+            }
+            cp_wait<0>();
+            if (ch < last) state_barrier();
+        }
+        pdl_launch_dependents();
+        return;
+    }
     const int smt = warp % MT, sn0 = (warp / MT) * NT;
     float S[NT][4];
     float* st = a.state + ((size_t)a.seg_slot[seg] * a.H + h) * a.D * a.V;
-    const bool fresh = a.pos[a.seg[2 * seg]] == 0;
+    const bool fresh = a.pos[lo] == 0;
     auto each_state = [&](auto f) {
 #pragma unroll
         for (int j = 0; j < NT; ++j)
@@ -484,9 +555,11 @@ __global__ void __launch_bounds__(256, 2) delta_chunk_state_kernel(const DeltaAr
             }
     };
     each_state([&](float& s, bool ok, const float* p) { s = ok && !fresh ? *p : 0.f; });
-    const int mt = warp & 3, nt = warp >> 2;              // this warp's 16 tokens x 8 columns
-    for (int ch = first; ch < last; ++ch) {
-        const int b = (ch - first) & 1, t0 = cc.chunk[2 * ch], n = cc.chunk[2 * ch + 1];
+    const int mt = warp & 3, nt = warp >> 2, row = mt * 16 + g, col = nt * 8 + c2;              // this warp's 16 tokens x 8 columns
+    bf16* uout = reinterpret_cast<bf16*>(cc.u) + chunk_slice(a, first, h, blockIdx.x) * 2 * DC * DV + row * DV + col;
+    const size_t ustep = chunk_slice(a, 1, 0, 0) * 2 * DC * DV;
+    for (int ch = first; ch < last; ++ch, uout += ustep) {
+        const int b = (ch - first) & 1;
         const bf16* ck = sk + b * DC * LDK;
         const bf16* cT = sT + b * 2 * DC * DLT;
         const float4* cg = sg + b * DC;
@@ -494,32 +567,15 @@ __global__ void __launch_bounds__(256, 2) delta_chunk_state_kernel(const DeltaAr
         for (int j = 0; j < NT; ++j)
 #pragma unroll
             for (int e = 0; e < 4; e += 2) {
-                uint32_t hi, lo;
-                split_bf16(S[j][e], S[j][e + 1], hi, lo);
+                uint32_t x, y;
+                split_bf16(S[j][e], S[j][e + 1], x, y);
                 bf16* p = sS + (smt * 16 + g + (e >> 1) * 8) * DLV + (sn0 + j) * 8 + c2;
-                *reinterpret_cast<uint32_t*>(p) = hi;
-                *reinterpret_cast<uint32_t*>(p + DP * DLV) = lo;
+                *reinterpret_cast<uint32_t*>(p) = x;
+                *reinterpret_cast<uint32_t*>(p + DP * DLV) = y;
             }
-        cp_wait<0>();
-        __syncthreads();
-        if (ch + 1 < last) fetch(ch + 1, b ^ 1);
-        {   // the state the chunk starts from, for the outputs
-            bf16* out = reinterpret_cast<bf16*>(cc.states) + ((size_t)ch * a.H + h) * 2 * a.D * a.V + v0;
-            if (a.V % 8 == 0) {
-                for (int i = tid; i < 2 * DP * (DV / 8); i += 256) {
-                    const int r = i / (DV / 8), c = i % (DV / 8) * 8, part = r / DP, d = r % DP;
-                    if (d < a.D && c < ncol) *reinterpret_cast<uint4*>(out + ((size_t)part * a.D + d) * a.V + c) = *reinterpret_cast<const uint4*>(sS + r * DLV + c);
-                }
-            } else {
-                for (int i = tid; i < 2 * DP * DV; i += 256) {
-                    const int r = i / DV, c = i % DV, part = r / DP, d = r % DP;
-                    if (d < a.D && c < ncol) out[((size_t)part * a.D + d) * a.V + c] = sS[r * DLV + c];
-                }
-            }
-        }
-        float4 gt[2] = {cg[mt * 16 + g], cg[mt * 16 + g + 8]};
+        state_barrier();
         {   // r = beta (v - decay S^T k)
-            float xh[4] = {}, xl[4] = {};
+            float xh[2][4] = {}, xl[2][4] = {};
 #pragma unroll
             for (int ks = 0; ks < DP / 32; ++ks) {
                 uint32_t bh[4], bl[4];
@@ -529,26 +585,28 @@ __global__ void __launch_bounds__(256, 2) delta_chunk_state_kernel(const DeltaAr
                 for (int j = 0; j < 2; ++j) {
                     uint32_t af[4];
                     ldsm_x4(af, ck + (mt * 16 + (lane & 15)) * LDK + (ks * 2 + j) * 16 + (lane >> 4) * 8);
-                    mma16816(xh, af, bh[2 * j], bh[2 * j + 1]);
-                    mma16816(xl, af, bl[2 * j], bl[2 * j + 1]);
+                    mma16816(xh[j], af, bh[2 * j], bh[2 * j + 1]);
+                    mma16816(xl[j], af, bl[2 * j], bl[2 * j + 1]);
                 }
             }
 #pragma unroll
             for (int half = 0; half < 2; ++half) {
-                const int o = (mt * 16 + g + half * 8) * DLV + nt * 8 + c2;
-                const float2 v = bf2_to_f2(*reinterpret_cast<const uint32_t*>(sv + b * DC * DLV + o));
-                const float w = exp2f(gt[half].x) * gt[half].y;
-                uint32_t hi, lo;
-                split_bf16(gt[half].z * (v.x - w * (xh[2 * half] + xl[2 * half])), gt[half].z * (v.y - w * (xh[2 * half + 1] + xl[2 * half + 1])), hi, lo);
-                *reinterpret_cast<uint32_t*>(sr + o) = hi;
-                *reinterpret_cast<uint32_t*>(sr + DC * DLV + o) = lo;
+                const int o = (row + half * 8) * DLV + col;
+                const float2 gt = *reinterpret_cast<const float2*>(cg + row + half * 8), v = bf2_to_f2(*reinterpret_cast<const uint32_t*>(sv + b * DC * DLV + o));
+                const float x = (xh[0][2 * half] + xh[1][2 * half]) + (xl[0][2 * half] + xl[1][2 * half]);
+                const float y = (xh[0][2 * half + 1] + xh[1][2 * half + 1]) + (xl[0][2 * half + 1] + xl[1][2 * half + 1]);
+                uint32_t p, q;
+                split_bf16(fmaf(gt.x, v.x, -gt.y * x), fmaf(gt.x, v.y, -gt.y * y), p, q);
+                *reinterpret_cast<uint32_t*>(sr + o) = p;
+                *reinterpret_cast<uint32_t*>(sr + DC * DLV + o) = q;
             }
         }
-        __syncthreads();
-        const float end = cg[DC - 1].x;
+        state_barrier();
         {   // u = T r
-            float u0[4] = {}, u1[4] = {}, u2[4] = {};
-            for (int ks = 0; ks <= mt >> 1; ++ks) {
+            float u[2][3][4] = {};
+#pragma unroll
+            for (int ks = 0; ks < 2; ++ks) {
+                if (ks > mt >> 1) break;
                 uint32_t bh[4], bl[4];
                 ldsm_x4_t(bh, sr + (ks * 32 + lane) * DLV + nt * 8);
                 ldsm_x4_t(bl, sr + (DC + ks * 32 + lane) * DLV + nt * 8);
@@ -558,42 +616,34 @@ __global__ void __launch_bounds__(256, 2) delta_chunk_state_kernel(const DeltaAr
                     const bf16* p = cT + (mt * 16 + (lane & 15)) * DLT + (ks * 2 + j) * 16 + (lane >> 4) * 8;
                     ldsm_x4(ah, p);
                     ldsm_x4(al, p + DC * DLT);
-                    mma16816(u0, ah, bh[2 * j], bh[2 * j + 1]);
-                    mma16816(u1, ah, bl[2 * j], bl[2 * j + 1]);
-                    mma16816(u2, al, bh[2 * j], bh[2 * j + 1]);
+                    mma16816(u[j][0], ah, bh[2 * j], bh[2 * j + 1]);
+                    mma16816(u[j][1], ah, bl[2 * j], bl[2 * j + 1]);
+                    mma16816(u[j][2], al, bh[2 * j], bh[2 * j + 1]);
                 }
             }
-            const size_t part = (size_t)cc.T * a.H * a.V;
+            float x[4];
+#pragma unroll
+            for (int e = 0; e < 4; ++e) x[e] = (u[0][0][e] + u[1][0][e]) + ((u[0][1][e] + u[1][1][e]) + (u[0][2][e] + u[1][2][e]));
+            uint32_t p, q;
 #pragma unroll
             for (int half = 0; half < 2; ++half) {
-                const int t = mt * 16 + g + half * 8, c = nt * 8 + c2;
-                const float x = u0[2 * half] + (u1[2 * half] + u2[2 * half]), y = u0[2 * half + 1] + (u1[2 * half + 1] + u2[2 * half + 1]);
-                uint32_t hi, lo;
-                split_bf16(x, y, hi, lo);
-                if (t < n && c < ncol) {
-                    bf16* p = reinterpret_cast<bf16*>(cc.u) + ((size_t)(t0 + t) * a.H + h) * a.V + v0 + c;
-                    if (a.V % 2 == 0) {
-                        *reinterpret_cast<uint32_t*>(p) = hi;
-                        *reinterpret_cast<uint32_t*>(p + part) = lo;
-                    } else {
-                        p[0] = __ushort_as_bfloat16((unsigned short)(hi & 0xffff));
-                        p[part] = __ushort_as_bfloat16((unsigned short)(lo & 0xffff));
-                        if (c + 1 < ncol) {
-                            p[1] = __ushort_as_bfloat16((unsigned short)(hi >> 16));
-                            p[part + 1] = __ushort_as_bfloat16((unsigned short)(lo >> 16));
-                        }
-                    }
-                }
-                const float w = exp2f(end - gt[half].x) * gt[half].y;
-                split_bf16(x * w, y * w, hi, lo);
-                *reinterpret_cast<uint32_t*>(su + t * DLV + c) = hi;
-                *reinterpret_cast<uint32_t*>(su + (DC + t) * DLV + c) = lo;
+                const int o = (row + half * 8) * DLV + col;
+                const float w = cg[row + half * 8].z;
+                split_bf16(x[2 * half] * w, x[2 * half + 1] * w, p, q);
+                *reinterpret_cast<uint32_t*>(su + o) = p;
+                *reinterpret_cast<uint32_t*>(su + DC * DLV + o) = q;
+            }
+            state_barrier();
+#pragma unroll
+            for (int half = 0; half < 2; ++half) {
+                split_bf16(x[2 * half], x[2 * half + 1], p, q);
+                *reinterpret_cast<uint32_t*>(uout + half * 8 * DV) = p;
+                *reinterpret_cast<uint32_t*>(uout + (DC + half * 8) * DV) = q;
             }
         }
-        __syncthreads();
         {   // S = decay S + sum k u^T
-            const float f = exp2f(end);
-            float lo4[NT][4] = {};
+            const float f = cg[0].w;
+            float rest[NT][2][4] = {};
 #pragma unroll
             for (int j = 0; j < NT; ++j)
 #pragma unroll
@@ -608,140 +658,139 @@ __global__ void __launch_bounds__(256, 2) delta_chunk_state_kernel(const DeltaAr
                     uint32_t bh[4], bl[4];
                     ldsm_x4_t(bh, su + (ks * 32 + lane) * DLV + (sn0 + j) * 8);
                     ldsm_x4_t(bl, su + (DC + ks * 32 + lane) * DLV + (sn0 + j) * 8);
-#pragma unroll
-                    for (int i = 0; i < 2; ++i) {
-                        mma16816(S[j], af[i], bh[2 * i], bh[2 * i + 1]);
-                        mma16816(lo4[j], af[i], bl[2 * i], bl[2 * i + 1]);
-                    }
+                    mma16816(S[j], af[0], bh[0], bh[1]);
+                    mma16816(rest[j][0], af[1], bh[2], bh[3]);
+                    mma16816(rest[j][1], af[0], bl[0], bl[1]);
+                    mma16816(rest[j][1], af[1], bl[2], bl[3]);
                 }
             }
 #pragma unroll
             for (int j = 0; j < NT; ++j)
 #pragma unroll
-                for (int e = 0; e < 4; ++e) S[j][e] += lo4[j][e];
+                for (int e = 0; e < 4; ++e) S[j][e] += rest[j][0][e] + rest[j][1][e];
         }
     }
     pdl_launch_dependents();
     each_state([&](float& s, bool ok, float* p) { if (ok) *p = s; });
 }
 
-// Outputs of a chunk: a warp takes 16 queries; token weights stay in registers (the accumulators of q k^T, weighted, are the operand of the
-// product with the writes).
+// Outputs of a chunk, 64 columns: what the state a chunk starts from answers to the queries, and the weighted writes.  A warp takes 16 queries and
+// half of the columns.
 constexpr int DO = 64, DLO = DO + 8;
 template <int DP>
 struct DeltaOutCfg {
     static constexpr int LDK = DP + 8;
-    static constexpr size_t SMEM = (size_t)(2 * DC * LDK + 2 * DP * DLO + 2 * DC * DLO) * 2 + DC * 16;
+    static constexpr size_t SMEM = (size_t)(DC * LDK + 2 * DC * DLT + 2 * DP * DLO + 2 * DC * DLO) * 2 + DC * 4;
 };
 template <int DP>
-__global__ void __launch_bounds__(128) delta_chunk_out_kernel(const DeltaArgs a, const DeltaChunks cc) {
-    constexpr int LDK = DP + 8, NP = DO / 16;
+__global__ void __launch_bounds__(256, 2) delta_chunk_out_kernel(const DeltaArgs a, const DeltaChunks cc) {
+    constexpr int LDK = DP + 8;
     extern __shared__ __align__(16) uint8_t dc_smem[];
     bf16* sq = reinterpret_cast<bf16*>(dc_smem);          // [DC][LDK]
-    bf16* sk = sq + DC * LDK;                             // [DC][LDK]
-    bf16* sS = sk + DC * LDK;                             // [part][DP][DLO]
+    bf16* sw = sq + DC * LDK;                             // [part][DC][DLT]
+    bf16* sS = sw + 2 * DC * DLT;                         // [part][DP][DLO]
     bf16* su = sS + 2 * DP * DLO;                         // [part][DC][DLO]
-    float4* sg = reinterpret_cast<float4*>(su + 2 * DC * DLO);      // [DC]
-    const int tid = threadIdx.x, lane = tid & 31, mt = tid >> 5, g = lane >> 2, c2 = (lane & 3) * 2, ch = blockIdx.x, h = blockIdx.y, v0 = blockIdx.z * DO;
+    float* se = reinterpret_cast<float*>(su + 2 * DC * DLO);        // [DC]
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, mt = warp & 3, hf = warp >> 2, ch = blockIdx.x, h = blockIdx.y, v0 = blockIdx.z * DO;
     pdl_wait();
-    const int t0 = cc.chunk[2 * ch], n = cc.chunk[2 * ch + 1], ncol = min(DO, a.V - v0);
-    const size_t qk0 = (size_t)(h / a.hpg) * a.D;
-    chunk_tile<bf16, DC, DP, 128>(a.q, a.ldq, qk0, t0, n, a.D, 0, sq);
-    chunk_tile<bf16, DC, DP, 128>(a.k, a.ldk, qk0, t0, n, a.D, 0, sk);
-    const bf16* S = reinterpret_cast<const bf16*>(cc.states) + ((size_t)ch * a.H + h) * 2 * a.D * a.V;
-    const bf16* u = reinterpret_cast<const bf16*>(cc.u);
+    const int t0 = cc.chunk[2 * ch], n = cc.chunk[2 * ch + 1], ncol = min(DO, a.V - v0), slices = (ncol + DV - 1) / DV;
+    const size_t sl = chunk_slice(a, ch, h, v0 / DV);
+    {   // 16-column slices, side by side; the two halves of a group of threads take the halves of a row
+        const uint4* S = reinterpret_cast<const uint4*>(reinterpret_cast<const bf16*>(cc.states) + sl * 2 * DP * DV) + tid;
+        bf16* dst = sS + (tid >> 1) * DLO + (tid & 1) * 8;
 #pragma unroll
-    for (int part = 0; part < 2; ++part) {
-        chunk_tile<bf16, DP, DO, 128>(S + (size_t)part * a.D * a.V, a.V, v0, 0, a.D, ncol, 0, sS + part * DP * DLO);
-        chunk_tile<bf16, DC, DO, 128>(u + (size_t)part * cc.T * a.H * a.V, a.H * a.V, (size_t)h * a.V + v0, t0, n, ncol, 0, su + part * DC * DLO);
+        for (int s = 0; s < DO / DV; ++s)
+            if (s < slices)
+#pragma unroll
+                for (int i = 0; i < 4 * DP / 256; ++i) cp_async16(dst + i * 128 * DLO + s * DV, S + s * 4 * DP + i * 256, true);
     }
-    if (tid < DC) cp_async16(sg + tid, cc.gates + (((size_t)ch * a.H + h) * DC + tid) * 4, true);
+    chunk_tile<bf16, DC, DP, 256>(a.q, a.ldq, (size_t)(h / a.hpg) * a.D, t0, n, a.D, 0, sq);
     cp_commit();
-    cp_wait<0>();
+    {
+        const uint4* U = reinterpret_cast<const uint4*>(reinterpret_cast<const bf16*>(cc.u) + sl * 2 * DC * DV) + tid;
+        bf16* dst = su + (tid >> 1) * DLO + (tid & 1) * 8;
+#pragma unroll
+        for (int s = 0; s < DO / DV; ++s)
+            if (s < slices) cp_async16(dst + s * DV, U + s * 4 * DC, true);
+    }
+    copy_pieces<2 * DC * DLT / 8, 256>(sw, chunk_matrix(cc.weights, a, ch, h));
+    if (tid < DC / 4) cp_async16(se + tid * 4, chunk_gates(a, cc, ch, h) + 4 * DC + tid * 4, true);
+    cp_commit();
+    cp_wait<1>();
     __syncthreads();
-    const float qq = row_squares<DP, 2>(sq);
-    if ((tid & 1) == 0) sg[tid >> 1].w = a.q_scale / sqrtf(qq + a.unit_eps);
-    __syncthreads();
-    if (mt * 16 < n) {
-        uint32_t qf[DP / 16][4];
+    const bool mine = mt * 16 < n && hf * 32 < ncol;
+    float acc[2][2][4] = {};
+    if (mine) {
 #pragma unroll
-        for (int ks = 0; ks < DP / 16; ++ks) ldsm_x4(qf[ks], sq + (mt * 16 + (lane & 15)) * LDK + ks * 16 + (lane >> 4) * 8);
-        float acc[NP][2][4] = {};
+        for (int ks = 0; ks < DP / 16; ++ks) {
+            uint32_t af[4];
+            ldsm_x4(af, sq + (mt * 16 + (lane & 15)) * LDK + ks * 16 + (lane >> 4) * 8);
 #pragma unroll
-        for (int ks = 0; ks < DP / 16; ++ks)
-#pragma unroll
-            for (int j = 0; j < NP; ++j) {
-                const bf16* p = sS + (ks * 16 + (lane & 15)) * DLO + j * 16 + (lane >> 4) * 8;
+            for (int j = 0; j < 2; ++j) {
+                const bf16* p = sS + (ks * 16 + (lane & 15)) * DLO + hf * 32 + j * 16 + (lane >> 4) * 8;
                 uint32_t bh[4], bl[4];
                 ldsm_x4_t(bh, p);
                 ldsm_x4_t(bl, p + DP * DLO);
 #pragma unroll
                 for (int b = 0; b < 2; ++b) {
-                    mma16816(acc[j][b], qf[ks], bh[2 * b], bh[2 * b + 1]);
-                    mma16816(acc[j][b], qf[ks], bl[2 * b], bl[2 * b + 1]);
-                }
-            }
-        const float4 g0 = sg[mt * 16 + g], g1 = sg[mt * 16 + g + 8];
-        const float e0 = exp2f(g0.x) * g0.w, e1 = exp2f(g1.x) * g1.w;
-#pragma unroll
-        for (int j = 0; j < NP; ++j)
-#pragma unroll
-            for (int b = 0; b < 2; ++b) { acc[j][b][0] *= e0; acc[j][b][1] *= e0; acc[j][b][2] *= e1; acc[j][b][3] *= e1; }
-#pragma unroll 1
-        for (int kb = 0; kb <= mt; ++kb) {
-            float p[2][4] = {};
-#pragma unroll
-            for (int ks = 0; ks < DP / 16; ++ks) {
-                uint32_t bf[4];
-                ldsm_x4(bf, sk + (kb * 16 + (lane & 7) + (lane >> 4) * 8) * LDK + ks * 16 + ((lane >> 3) & 1) * 8);
-                mma16816(p[0], qf[ks], bf[0], bf[1]);
-                mma16816(p[1], qf[ks], bf[2], bf[3]);
-            }
-            uint32_t hi[4], lo[4];
-#pragma unroll
-            for (int b = 0; b < 2; ++b) {
-                float w[4];
-#pragma unroll
-                for (int e = 0; e < 4; ++e) {
-                    const int t = mt * 16 + g + (e >> 1) * 8, s = kb * 16 + b * 8 + c2 + (e & 1);
-                    const float4 gs = sg[s];
-                    w[e] = s <= t ? p[b][e] * (exp2f((e < 2 ? g0.x : g1.x) - gs.x) * gs.y * (e < 2 ? g0.w : g1.w)) : 0.f;
-                }
-                split_bf16(w[0], w[1], hi[2 * b], lo[2 * b]);
-                split_bf16(w[2], w[3], hi[2 * b + 1], lo[2 * b + 1]);
-            }
-#pragma unroll
-            for (int j = 0; j < NP; ++j) {
-                const bf16* q = su + (kb * 16 + (lane & 15)) * DLO + j * 16 + (lane >> 4) * 8;
-                uint32_t bh[4], bl[4];
-                ldsm_x4_t(bh, q);
-                ldsm_x4_t(bl, q + DC * DLO);
-#pragma unroll
-                for (int b = 0; b < 2; ++b) {
-                    mma16816(acc[j][b], hi, bh[2 * b], bh[2 * b + 1]);
-                    mma16816(acc[j][b], hi, bl[2 * b], bl[2 * b + 1]);
-                    mma16816(acc[j][b], lo, bh[2 * b], bh[2 * b + 1]);
+                    mma16816(acc[j][b], af, bh[2 * b], bh[2 * b + 1]);
+                    mma16816(acc[j][b], af, bl[2 * b], bl[2 * b + 1]);
                 }
             }
         }
-#pragma unroll
-        for (int j = 0; j < NP; ++j)
-#pragma unroll
-            for (int b = 0; b < 2; ++b)
-#pragma unroll
-                for (int e = 0; e < 4; e += 2) {
-                    const int t = mt * 16 + g + (e >> 1) * 8, c = j * 16 + b * 8 + c2;
-                    if (t >= n || c >= ncol) continue;
-                    float* o = a.out + (size_t)(t0 + t) * a.ldo + h * a.V + v0 + c;
-                    if (((a.V | a.ldo) & 1) == 0) {
-                        *reinterpret_cast<float2*>(o) = make_float2(acc[j][b][e], acc[j][b][e + 1]);
-                    } else {
-                        o[0] = acc[j][b][e];
-                        if (c + 1 < ncol) o[1] = acc[j][b][e + 1];
-                    }
-                }
     }
+    cp_wait<0>();
+    __syncthreads();
     pdl_launch_dependents();
+    if (!mine) return;
+    const int row = mt * 16 + (lane >> 2);
+    const float e0 = se[row], e1 = se[row + 8];
+#pragma unroll
+    for (int j = 0; j < 2; ++j)
+#pragma unroll
+        for (int b = 0; b < 2; ++b) { acc[j][b][0] *= e0; acc[j][b][1] *= e0; acc[j][b][2] *= e1; acc[j][b][3] *= e1; }
+#pragma unroll
+    for (int kb = 0; kb < DC / 16; ++kb) {
+        if (kb > mt) break;
+        uint32_t ah[4], al[4];
+        const bf16* p = sw + (mt * 16 + (lane & 15)) * DLT + kb * 16 + (lane >> 4) * 8;
+        ldsm_x4(ah, p);
+        ldsm_x4(al, p + DC * DLT);
+#pragma unroll
+        for (int j = 0; j < 2; ++j) {
+            const bf16* q = su + (kb * 16 + (lane & 15)) * DLO + hf * 32 + j * 16 + (lane >> 4) * 8;
+            uint32_t bh[4], bl[4];
+            ldsm_x4_t(bh, q);
+            ldsm_x4_t(bl, q + DC * DLO);
+#pragma unroll
+            for (int b = 0; b < 2; ++b) {
+                mma16816(acc[j][b], ah, bh[2 * b], bh[2 * b + 1]);
+                mma16816(acc[j][b], ah, bl[2 * b], bl[2 * b + 1]);
+                mma16816(acc[j][b], al, bh[2 * b], bh[2 * b + 1]);
+            }
+        }
+    }
+    const bool pair = ((a.V | a.ldo) & 1) == 0;
+#pragma unroll
+    for (int half = 0; half < 2; ++half) {
+        const int t = row + half * 8;
+        if (t >= n) break;
+        float* o = a.out + (size_t)(t0 + t) * a.ldo + h * a.V + v0;
+#pragma unroll
+        for (int j = 0; j < 2; ++j)
+#pragma unroll
+            for (int b = 0; b < 2; ++b) {
+                const int c = hf * 32 + j * 16 + b * 8 + (lane & 3) * 2;
+                if (c >= ncol) continue;
+                const float x = acc[j][b][half * 2], y = acc[j][b][half * 2 + 1];
+                if (pair) {
+                    *reinterpret_cast<float2*>(o + c) = make_float2(x, y);
+                } else {
+                    o[c] = x;
+                    if (c + 1 < ncol) o[c + 1] = y;
+                }
+            }
+    }
 }
 
 template <int DP>
@@ -755,17 +804,17 @@ static int launch_delta_chunks(const DeltaArgs& a, const DeltaChunks& c, cudaStr
     if (first_use_on_device((const void*)k2)) DLP_CHECK_CUDA(cudaFuncSetAttribute(k2, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)sm2));
     if (first_use_on_device((const void*)k3)) DLP_CHECK_CUDA(cudaFuncSetAttribute(k3, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)sm3));
     DLP_CHECK_CUDA(launch_pdl(k1, dim3(c.n_chunks, a.H), dim3(256), sm1, s, a, c));
-    DLP_CHECK_CUDA(launch_pdl(k2, dim3((a.V + DV - 1) / DV, a.H, a.n_seg), dim3(256), sm2, s, a, c));
-    DLP_CHECK_CUDA(launch_pdl(k3, dim3(c.n_chunks, a.H, (a.V + DO - 1) / DO), dim3(128), sm3, s, a, c));
+    DLP_CHECK_CUDA(launch_pdl(k2, dim3((a.V + DV - 1) / DV, a.H, a.n_seg), dim3(288), sm2, s, a, c));
+    DLP_CHECK_CUDA(launch_pdl(k3, dim3(c.n_chunks, a.H, (a.V + DO - 1) / DO), dim3(256), sm3, s, a, c));
     return 0;
 }
 int delta_chunked(const DeltaArgs& a, const DeltaChunks& c, cudaStream_t s) {
     const int rc = check_delta(a, "delta_chunked");
     if (rc) return rc;
-    DLP_REQUIRE(c.chunk && c.first && c.states && c.solve && c.u && c.gates && c.n_chunks > 0 && c.T > 0, "delta_chunked: no chunk table");
+    DLP_REQUIRE(c.chunk && c.first && c.states && c.keys && c.solve && c.weights && c.u && c.gates && c.n_chunks > 0, "delta_chunked: no chunk table");
     DLP_REQUIRE(!a.rows_f32 && a.D <= 128 && (a.V + DO - 1) / DO <= 65535, "delta_chunked: bf16 rows, state of %d x %d", a.D, a.V);
-    DLP_REQUIRE(((reinterpret_cast<uintptr_t>(c.states) | reinterpret_cast<uintptr_t>(c.solve) | reinterpret_cast<uintptr_t>(c.u) | reinterpret_cast<uintptr_t>(c.gates)) & 15) == 0,
-                "delta_chunked: workspace alignment");
+    DLP_REQUIRE(((reinterpret_cast<uintptr_t>(c.states) | reinterpret_cast<uintptr_t>(c.keys) | reinterpret_cast<uintptr_t>(c.solve) | reinterpret_cast<uintptr_t>(c.weights) |
+                  reinterpret_cast<uintptr_t>(c.u) | reinterpret_cast<uintptr_t>(c.gates)) & 15) == 0, "delta_chunked: workspace alignment");
     return a.D <= 64 ? launch_delta_chunks<64>(a, c, s) : launch_delta_chunks<128>(a, c, s);
 }
 

@@ -43,25 +43,31 @@ __global__ void __launch_bounds__(128) latent_write_kernel(const LatentRows a) {
         sincosf((float)a.pos[t] * a.inv_freq[i], &s, &c);
         cs[i] = make_float2(c * a.rot_scale, s * a.rot_scale);
     }
-    float ss = 0.f;
-    for (int k = threadIdx.x; k < a.R; k += 128) ss = fmaf(x[k], x[k], ss);
-    const float rs = 1.f / sqrtf(block_sum(ss, red) / (float)a.R + a.eps);
-    __syncthreads();
-    const int sl = a.slot[t];
-    if (sl >= 0) {
-        WT* row = reinterpret_cast<WT*>(a.cache) + (size_t)sl * a.Rc;
-        for (int k = threadIdx.x; k < a.Rc; k += 128)
-            if (k < a.R || k >= a.R + a.rot) row[k] = (WT)(k < a.R ? x[k] * rs * a.w[k] : 0.f);
-        for (int i = threadIdx.x; i < np; i += 128) {
-            int u, v;
-            const float2 y = turned(x + a.R, i, a.rot, a.adjacent, cs[i], u, v);
-            row[a.R + u] = (WT)y.x;
-            row[a.R + v] = (WT)y.y;
+    const int parts = gridDim.y - 1;           // block 0: the cache row; the others: the queries (none: block 0 as well)
+    if (blockIdx.y == 0) {
+        float ss = 0.f;
+        for (int k = threadIdx.x; k < a.R; k += 128) ss = fmaf(x[k], x[k], ss);
+        const float rs = 1.f / sqrtf(block_sum(ss, red) / (float)a.R + a.eps);
+        __syncthreads();
+        const int sl = a.slot[t];
+        if (sl >= 0) {
+            WT* row = reinterpret_cast<WT*>(a.cache) + (size_t)sl * a.Rc;
+            for (int k = threadIdx.x; k < a.Rc; k += 128)
+                if (k < a.R || k >= a.R + a.rot) row[k] = (WT)(k < a.R ? x[k] * rs * a.w[k] : 0.f);
+            for (int i = threadIdx.x; i < np; i += 128) {
+                int u, v;
+                const float2 y = turned(x + a.R, i, a.rot, a.adjacent, cs[i], u, v);
+                row[a.R + u] = (WT)y.x;
+                row[a.R + v] = (WT)y.y;
+            }
         }
     }
-    if (a.q != nullptr) {
+    if (a.q != nullptr && (blockIdx.y > 0 || parts == 0)) {
+        __syncthreads();
         float* q = a.q + (size_t)t * a.ldq + a.Dq - a.rot;
-        for (int j = threadIdx.x; j < a.H * np; j += 128) {
+        const int n = a.H * np, part = parts > 0 ? blockIdx.y - 1 : 0, step = 128 * max(parts, 1);
+#pragma unroll 4
+        for (int j = part * 128 + threadIdx.x; j < n; j += step) {
             const int h = j / np, i = j - h * np;
             float* p = q + (size_t)h * a.Dq;
             int u, v;
@@ -76,7 +82,9 @@ int latent_write(const LatentRows& a, int T, int f32, cudaStream_t s) {
     DLP_REQUIRE(a.proj && a.w && a.slot && a.cache && a.R > 0 && a.rot >= 0 && a.rot % 2 == 0 && a.Rc >= a.R + a.rot && T > 0, "latent_write: bad argument");
     DLP_REQUIRE(a.rot == 0 || (a.pos && a.inv_freq && a.rot <= 8192 && (!a.q || (a.H > 0 && a.Dq >= a.rot && a.ldq >= a.H * a.Dq))), "latent_write: rotation of %d columns", a.rot);
     const size_t smem = (size_t)(a.rot / 2) * 8;
-    DLP_CHECK_CUDA(f32 ? launch_pdl(latent_write_kernel<float>, dim3(T), dim3(128), smem, s, a) : launch_pdl(latent_write_kernel<__nv_bfloat16>, dim3(T), dim3(128), smem, s, a));
+    const int parts = a.q && a.rot > 0 && T <= 64 ? (a.H * (a.rot / 2) + 255) / 256 : 0;         // few tokens: blocks of their own for the queries
+    const dim3 grid(T, 1 + (parts < 16 ? parts : 16));
+    DLP_CHECK_CUDA(f32 ? launch_pdl(latent_write_kernel<float>, grid, dim3(128), smem, s, a) : launch_pdl(latent_write_kernel<__nv_bfloat16>, grid, dim3(128), smem, s, a));
     return 0;
 }
 

@@ -17,7 +17,7 @@ from ..ops import layers as lops
 from ..ops.weights import DeviceWeight
 from ..gguf.constants import GGMLType
 from .engine import EngineCore, PagedKVCache, RecurrentState
-from .mixers import MIXERS, MLPS, Attention, Dense, Joined, LatentAttention, RoutedExperts, Rows, XieluMlp, pad_to
+from .mixers import MIXERS, MLPS, Attention, Delta, Dense, Joined, LatentAttention, RoutedExperts, Rows, XieluMlp, pad_to
 from .modeldir import ModelDir, open_model_dir
 from .weights import ModelWeights
 
@@ -210,7 +210,7 @@ class LayeredEngine(EngineCore):
         for part in [*mixers.values(), *mlps, *joined]:
             for name, n in part.buffers(M).items():
                 sizes[name] = max(sizes.get(name, 0), n)
-        types = {"proj": f32, "o": f32, "router": f32, "gate_w": f32, "ey": f32, "ys": f32, "q_up": f32, "v_first": f32, "delta_g": f32, "ids": torch.int32}
+        types = {"proj": f32, "o": f32, "router": f32, "gate_w": f32, "ey": f32, "ys": f32, "q_up": f32, "v_first": f32, **{n: f32 for n in Delta.WORKSPACES}, "ids": torch.int32}
         self._flat = {n: torch.zeros(sz, dtype=types.get(n, self.dtype), device=dev) for n, sz in sizes.items()}
         experts = [m for m in mlps if isinstance(m, RoutedExperts)]
         self.expert_plans = {n: ops.MoePlan(M * max(m.top for m in experts), n, dev) for n in {m.n for m in experts}}
@@ -233,9 +233,10 @@ class LayeredEngine(EngineCore):
         chunked = [m for m in mixers.values() if m.states and m.chunk]
         self._chunk_sizes = sorted({m.chunk for m in chunked})
         self.chunk_ws = None
-        if chunked and self.long_from <= M:
+        own = [m for m in chunked if not isinstance(m, Delta)]       # (the delta rule's workspaces are buffers)
+        if own and self.long_from <= M:
             n = lops.most_chunks(M, self._chunk_sizes[0])
-            self.chunk_ws = tuple(torch.zeros(n * max(m.H * m.D * w(m) for m in chunked), dtype=f32, device=dev) for w in (lambda m: m.V, lambda m: 1))
+            self.chunk_ws = tuple(torch.zeros(n * max(m.H * m.D * w(m) for m in own), dtype=f32, device=dev) for w in (lambda m: m.V, lambda m: 1))
         self._variant = (1,) * (len(self._latent_kinds) + len(self._att_kinds))      # key ranges per decode query: every kind of latent, then of windowed attention
         self._decode_batches: dict[tuple, Batch] = {}
 

@@ -204,6 +204,7 @@ class Delta(Mixer):
     """Gated delta rule: what the decayed state answers to a key is taken off the value before it is written; unit queries and keys behind short
     convolutions, shared by groups of heads; a norm per head and a gate behind it."""
     UNIT_EPS = 1e-6         # inside the root that makes a unit vector
+    WORKSPACES = tuple("delta_" + n for n in ("states", "keys", "solve", "weights", "u", "gates"))
 
     def __init__(self, m: dict, get, device, dtype, eps: float):
         self.H, self.G, self.D, self.V, self.taps = m["heads"], m["kv_heads"], m["dim"], m["vdim"], m["conv"]
@@ -228,8 +229,7 @@ class Delta(Mixer):
     def buffers(self, rows: int) -> dict[str, int]:
         out = {"o": rows * self.H * self.V, "xbc": rows * pad_to(self.channels, 8)}
         if self.chunk:
-            _, solve, u, gates = lops.delta_workspace(lops.most_chunks(rows, self.chunk), rows, self.H, self.D, self.V)
-            out |= {"delta_t": solve // 2, "delta_u": u // 2, "delta_g": gates // 4}
+            out |= {n: b // 4 for n, b in zip(self.WORKSPACES, lops.delta_workspace(lops.most_chunks(rows, self.chunk), self.H, self.G, self.D, self.V))}
         return out
 
     def mix(self, eng, run: int, proj: torch.Tensor, b) -> Rows:
@@ -248,7 +248,7 @@ class Delta(Mixer):
             for s in (b.short, b.long):
                 if s is not None:
                     lops.conv_rows(raw, self.conv_w, None, ring, s.range, s.slot, s.n, s.longest, b.pos, xbc)
-                    ws = (*s.chunks[self.chunk], eng.chunk_ws[0], *(eng.flat(n) for n in ("delta_t", "delta_u", "delta_g"))) if s is b.long and self.chunk else None
+                    ws = (*s.chunks[self.chunk], *(eng.flat(n) for n in self.WORKSPACES)) if s is b.long and self.chunk else None
                     scan(cols(xbc), s, chunks=ws)
         return Rows(o, HV, w2=self.norm, groups2=H, g=gate, gate=lops.GATE_SILU_AFTER)
 

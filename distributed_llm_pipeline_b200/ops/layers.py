@@ -97,7 +97,7 @@ class DeltaArgs(C.Structure):
 
 
 class DeltaChunks(C.Structure):
-    _fields_ = [(n, C.c_void_p) for n in ("chunk", "first", "states", "solve", "u", "gates")] + [("n_chunks", C.c_int32), ("T", C.c_int32)]
+    _fields_ = [(n, C.c_void_p) for n in ("chunk", "first", "states", "keys", "solve", "weights", "u", "gates")] + [("n_chunks", C.c_int32), ("pad", C.c_int32)]
 
 
 class LatentRows(C.Structure):
@@ -287,8 +287,8 @@ def delta(rows, heads_per_group: int, state: torch.Tensor, a, b, log_decay, dt_b
           single: bool = False):
     """Gated delta rule over the listed segments.  rows = (q, k, v): columns of the first head onwards, fp32 or bf16, behind convolution and activation;
     a, b [T, H]: raw step sizes (decay exp(log_decay * softplus(a + dt_bias))) and raw write strengths; q and k are made unit vectors per head
-    (unit_eps inside the root), q is scaled by D^-1/2.  chunks = (chunk table [n, 2], first chunk of every segment [n_seg + 1], workspaces: states,
-    inverses, writes, gates): 64-token chunks (DELTA_CHUNK) on the tensor cores; single, conv: as for `ssd`."""
+    (unit_eps inside the root), q is scaled by D^-1/2.  chunks = (chunk table [n, 2], first chunk of every segment [n_seg + 1], workspaces as
+    `delta_workspace` lists them): 64-token chunks (DELTA_CHUNK) on the tensor cores; single, conv: as for `ssd`."""
     _need_cuda(state, "delta")
     q, k, v = rows
     _, H, D, V = state.shape
@@ -296,20 +296,21 @@ def delta(rows, heads_per_group: int, state: torch.Tensor, a, b, log_decay, dt_b
                      int(q.dtype == torch.float32), heads_per_group, a.stride(0), b.stride(0), out.stride(0), H, D, V, n_seg, unit_eps, D ** -0.5)
     c = None
     if chunks is not None:
-        table, first, states, solve, u, gates = chunks
-        n, T = table.shape[0], out.shape[0]
-        need = delta_workspace(n, T, H, D, V)
-        if any(t.numel() * t.element_size() < x for t, x in zip((states, solve, u, gates), need)):
+        table, first, *ws = chunks
+        n = table.shape[0]
+        if any(t.numel() * t.element_size() < x for t, x in zip(ws, delta_workspace(n, H, H // heads_per_group, D, V))):
             raise ValueError("delta: workspace too small")
-        c = DeltaChunks(_p(table), _p(first), _p(states), _p(solve), _p(u), _p(gates), n, T)
+        c = DeltaChunks(_p(table), _p(first), *(_p(t) for t in ws), n, 0)
     _lib.check(_lib.load().dlp_layers_delta(C.byref(args), _ref(c), _ref(conv), 1 if c is not None else 2 if single else 0, api._stream()), "layers_delta")
     api._count(3 if c is not None else 1)
     return out
 
 
-def delta_workspace(n_chunks: int, T: int, H: int, D: int, V: int) -> tuple[int, int, int, int]:
-    """Bytes of the workspaces of `delta` in chunks: states, inverses, writes, gates."""
-    return n_chunks * H * D * V * 4, n_chunks * H * DELTA_CHUNK * DELTA_CHUNK * 4, T * H * V * 4, n_chunks * H * DELTA_CHUNK * 16
+def delta_workspace(n_chunks: int, H: int, G: int, D: int, V: int) -> tuple[int, ...]:
+    """Bytes of the workspaces of `delta` in chunks (G heads of queries and keys): states, keys, inverses, weights, writes, gates."""
+    dp, vp, c = (64 if D <= 64 else 128), -(-V // 16) * 16, DELTA_CHUNK
+    matrix = n_chunks * H * c * (c + 8) * 4
+    return n_chunks * H * dp * vp * 4, n_chunks * G * c * (dp + 8) * 2, matrix, matrix, n_chunks * H * c * vp * 4, n_chunks * H * c * 20
 
 
 def most_chunks(rows: int, size: int) -> int:

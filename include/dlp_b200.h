@@ -403,7 +403,8 @@ typedef struct {              /* gated delta rule (csrc/layers.cuh DeltaArgs) */
     const int32_t* seg; const int32_t* seg_slot; const int32_t* pos; float* out;
     int32_t ldq, ldk, ldv, rows_f32, hpg, lda, ldb, ldo, H, D, V, n_seg; float unit_eps, q_scale;
 } dlp_delta_args;
-typedef struct { const int32_t* chunk; const int32_t* first; void* states; void* solve; void* u; float* gates; int32_t n_chunks, T; } dlp_delta_chunks;      /* csrc/layers.cuh DeltaChunks */
+typedef struct { const int32_t* chunk; const int32_t* first; void* states; void* keys; void* solve; void* weights; void* u; float* gates;
+                 int32_t n_chunks, pad; } dlp_delta_chunks;      /* csrc/layers.cuh DeltaChunks */
 /* decode product, 1..4 rows: out_mode 0 = fp32, 2 = bf16 (dlp_layers_linear); in the activation type: 1 = GEGLU of interleaved (gate, up) rows,
  * 3 = max(., 0)^2, 4 = SwiGLU of interleaved rows */
 int dlp_layers_matvec(const dlp_row_stage* st, const void* w, int ldw, int N, void* out, int ldo, int out_mode, const dlp_out_tail* tail, int T, int f32, void* stream);

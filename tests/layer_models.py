@@ -122,7 +122,7 @@ CONFIGS = {
                                    biased_attention(4, 2, 16, 24, 0.3, 16, 9, yarn=None), delta(3, 3, 12, 10, 1), biased_attention(2, 2, 24, 24, 0.35, 8, 33, ff=20, base=500.0),
                                    low_rank_latent(3, 8, 2, 12, 17, 25, 0.5, 40)], eps=3e-4, emb=3.0),
     # delta rules only: one head, one group, long and short convolutions, states of every register-resident size and beyond
-    "deltas": rigalorn(64, 60, [delta(4, 1, 64, 48, 4, ff=40), delta(2, 2, 128, 128, 2, ff=64), delta(1, 1, 160, 40, 6), delta(2, 1, 300, 12, 3), delta(5, 5, 8, 7, 32, ff=24)], eps=1e-6),
+    "deltas": rigalorn(64, 60, [delta(4, 1, 64, 48, 4, ff=40), delta(2, 2, 128, 128, 2, ff=64), delta(1, 1, 160, 40, 6), delta(2, 1, 300, 12, 3), delta(5, 5, 8, 7, 32, ff=24)], eps=1e-3),
     # heads and latents for every form of the attentions: expanded keys of 64, 128 and 192, beyond them, latents above 512, more heads than a tile;
     # windows above a page and a key tile, one token, more than the sequence
     "windows": rigalorn(256, 320, [low_rank_latent(4, 48, 16, 64, 96, 96, 0.14, 70, ff=96), biased_attention(8, 2, 128, 64, 0.12, 64, 150, ff=128, yarn=(4.0, 40, 8.0, 0.5)),

@@ -120,6 +120,73 @@ def test_activations_behind_products(dt, T, K, F, kind):
 
 
 @pytest.mark.parametrize("dt", TYPES)
+@pytest.mark.parametrize("T", [1, 2, 4, 5, 40, 300])
+@pytest.mark.parametrize("K,N,n2,bias", [(72, 101, 37, True), (256, 300, 128, True), (256, 300, 160, False), (40, 51, 0, True), (512, 64, None, True), (64, 33, 32, False)])
+def test_bias_and_second_output_of_a_product(dt, T, K, N, n2, bias):
+    """A bias on everything, and the outputs from n2 on behind xIELU elsewhere; inputs on both sides of zero, far out and next to it."""
+    L, r = ops(), gen(K + N)
+    x, w, b = r(T, K).to(dt), r(N, K, scale=3 * K ** -0.5).to(dt), r(N, scale=2.0)
+    w[::5] *= 1e-3
+    b[::5] *= 1e-3
+    w[1::7] *= 6
+    act = (1.3, 0.9)
+    n = N if n2 is None else n2
+    out, out2 = torch.zeros(T, n + 3, device=DEV), torch.zeros(T, N - n + 5, dtype=dt, device=DEV)
+    xd, wd, bd = x.to(DEV), w.to(DEV), b.to(DEV)              # (a tail does not keep its tensors alive)
+    tail = L.out_tail(bd if bias else None, **({} if n2 is None else dict(n2=n2, out2=out2, act=act)))
+    if T <= 4:
+        L.matvec(L.row_stage(xd, K, K, 0.0), wd, out, T, tail=tail)
+    else:
+        L.linear(xd, wd, out, tail=tail)
+    z = x.to(F64) @ w.to(F64).T + (b.to(F64) if bias else 0)
+    tol = 6e-3 if dt == BF16 else 3e-6
+    assert n == 0 or rel(out[:, :n], z[:, :n]) < (1e-5 if dt == BF16 else 3e-6)
+    assert not out[:, n:].any() and not out2[:, N - n:].any()
+    if n < N:
+        want = z[:, n:] / 2 + torch.where(z[:, n:] > 0, act[0] * z[:, n:] ** 2, act[1] * (torch.expm1(z[:, n:].clamp(max=0)) - z[:, n:]))
+        assert rel(out2[:, :N - n], want) < tol
+
+
+@pytest.mark.parametrize("dt", TYPES)
+@pytest.mark.parametrize("T", [4, 8])
+def test_xielu_keeps_the_digits_of_small_values(dt, T):
+    L = ops()
+    z = (torch.logspace(-7, 1.5, 400) * torch.tensor([1.0, -1.0]).repeat(200))[:, None].expand(400, 8).to(dt).contiguous()
+    out = torch.zeros(T, 400, dtype=dt, device=DEV)
+    x, zd, tail = torch.eye(8)[:T].to(dt).to(DEV), z.to(DEV), L.out_tail(n2=0, out2=out, act=(0.4, 0.5))
+    if T <= 4:
+        L.matvec(L.row_stage(x, 8, 8, 0.0), zd, out, T, tail=tail)
+    else:
+        L.linear(x, zd, out, tail=tail)
+    v = z[:, 0].to(F64)
+    want = v / 2 + torch.where(v > 0, 0.4 * v * v, 0.5 * (torch.expm1(v.clamp(max=0)) - v))
+    err = (out.cpu().to(F64) - want) / want
+    assert float(err.abs().max()) < (5e-3 if dt == BF16 else 1e-6)
+
+
+@pytest.mark.parametrize("dt", TYPES)
+@pytest.mark.parametrize("T", [1, 2, 3, 4])
+@pytest.mark.parametrize("K,K2,N,kind", [(72, 40, 33, "plain"), (256, 512, 60, "mixer"), (100, 8, 17, "mixer"), (2048, 1024, 24, "norm")])
+def test_rows_with_a_tail(dt, T, K, K2, N, kind):
+    """Staged rows and, behind them, columns that join the product as they are."""
+    L, r = ops(), gen(K + K2)
+    Kp, eps = (K + 7) // 8 * 8, 1e-3
+    x, both, w = r(T, K), r(T, Kp + K2).to(dt), torch.zeros(N, Kp + K2, dtype=dt)
+    w[:, :K], w[:, Kp:] = r(N, K, scale=K ** -0.5).to(dt), r(N, K2, scale=K2 ** -0.5).to(dt)
+    g, w2 = r(T, K), r(K) + 1
+    v = x.to(F64)
+    bd, kw = both.to(DEV), {}
+    if kind != "plain":
+        v, kw = plain.rms(v, eps) * w2.to(F64), dict(w2=w2.to(DEV))
+    if kind == "mixer":
+        v, kw = v * plain.silu(g.to(F64)), dict(w2=kw["w2"], g=g.to(DEV), gate=L.GATE_SILU_AFTER)
+    xd, wd, out = x.to(DEV), w.to(DEV), torch.full((T, N), float("nan"), device=DEV)
+    L.matvec(L.row_stage(xd, K, Kp, eps, tail=bd[:, Kp:], **kw), wd, out, T)
+    want = v.to(dt).to(F64) @ w[:, :K].to(F64).T + both[:, Kp:].to(F64) @ w[:, Kp:].to(F64).T
+    assert rel(out, want) < (6e-3 if dt == BF16 else 3e-6)
+
+
+@pytest.mark.parametrize("dt", TYPES)
 @pytest.mark.parametrize("T", [1, 2, 4, 5, 40, 200])
 @pytest.mark.parametrize("K,F", [(72, 36), (256, 300)])
 def test_geglu(dt, T, K, F):
@@ -202,18 +269,20 @@ def test_hgrn2_segments_and_carried_state(form, H, D, V):
 
 # ---- latent attention ------------------------------------------------------------------------------------------------------------
 @pytest.mark.parametrize("dt", TYPES)
-@pytest.mark.parametrize("H,R,page,splits", [(1, 32, 16, 1), (5, 40, 16, 4), (20, 160, 64, 1), (3, 544, 64, 2), (50, 96, 16, 8), (16, 512, 64, 1)])
-def test_latent_attention(dt, H, R, page, splits):
+@pytest.mark.parametrize("H,R,P,page,splits,window", [(1, 32, 0, 16, 1, None), (5, 40, 0, 16, 4, None), (20, 160, 0, 64, 1, None), (3, 544, 0, 64, 2, None), (50, 96, 0, 16, 8, None), (16, 512, 0, 64, 1, None),
+                                                      (4, 96, 16, 16, 2, 19), (5, 40, 6, 16, 1, 70), (20, 512, 64, 64, 4, 33), (2, 64, 32, 32, 8, 1), (3, 530, 20, 16, 1, 100), (50, 128, 96, 64, 2, 150)])
+def test_latent_attention(dt, H, R, P, page, splits, window):
     """Portions of several requests over scattered pages; one key per query stands out: far back, on both sides of every page border,
-    the first token, the query's own position."""
+    the first token, the query's own position, just inside and outside the window.  With P the latent is followed by key columns that are no values."""
     L, r = ops(), gen(R)
-    Rc = (R + 31) // 32 * 32
+    V, R = R, R + P                     # R: all columns of a key, V: those of a value
+    Rc, Vc = (R + 31) // 32 * 32, (V + 31) // 32 * 32
     spans = [(0, 3), (4 * page - 2, 5), (page - 1, 1), (9 * page + 3, 2), (0, 70)]      # (cached before, new) of every request
     max_pages, perm = 12, torch.randperm(60, generator=torch.Generator().manual_seed(2))
     cache, bt = torch.zeros(60, 1, page, Rc), perm.view(5, 12).to(torch.int32)
     cache.view(-1, Rc)[:] = 1e4                      # rows nobody wrote
     scale, rows_q, want, tok_slot, pos, row0, rows = 0.25, [], [], [], [], [], []
-    bm, base = L.latent_tile_rows(H, sum(n for _, n in spans)), 0
+    bm, base = L.latent_tile_rows(H, sum(n for _, n in spans), Rc), 0
     for s, (p0, n) in enumerate(spans):
         k = torch.arange(p0 + n)
         c = torch.zeros(p0 + n, Rc)
@@ -225,13 +294,16 @@ def test_latent_attention(dt, H, R, page, splits):
         marks = sorted({0, p0, *[b + d for b in range(page, p0 + n, page) for d in (-1, 0)]})
         for t in range(n):
             for h in range(H):
-                j = ([m for m in marks if m <= p0 + t] + [p0 + t])[(t + h) % (len([m for m in marks if m <= p0 + t]) + 1)]
+                edges = [p0 + t - d for d in (0, window - 1, window, window + 1) if p0 + t - d >= 0] if window else [p0 + t]
+                seen = [m for m in marks if m <= p0 + t] + edges
+                j = seen[(t + h) % len(seen)]
                 q[t, h, :R] += c[j, :R].float() * (12 / scale / R)
         q = q.to(dt)
         rows_q.append(q)
         sc = torch.einsum("thr,jr->thj", q.to(F64), c.to(F64)) * scale
-        sc = sc.masked_fill(k[None, None] > (p0 + torch.arange(n))[:, None, None], -math.inf)
-        want.append(torch.softmax(sc, -1) @ c.to(F64))
+        i = (p0 + torch.arange(n))[:, None, None]
+        sc = sc.masked_fill((k > i) | (i - k >= (window or 1 << 30)), -math.inf)
+        want.append((torch.softmax(sc, -1) @ c.to(F64))[..., :V])
         tok_slot += [s] * n
         pos += list(range(p0, p0 + n))
         for i in range(0, n * H, bm):
@@ -240,23 +312,27 @@ def test_latent_attention(dt, H, R, page, splits):
         base += n * H
     q, T = torch.cat(rows_q).reshape(len(pos), H * Rc).to(DEV), len(pos)
     i32 = dict(dtype=torch.int32, device=DEV)
-    out = torch.zeros(T, H * Rc, dtype=dt, device=DEV)
-    ws = (torch.empty(splits * T * H * Rc, device=DEV), torch.empty(splits * T * H * 2, device=DEV))
+    out = torch.zeros(T, H * Vc, dtype=dt, device=DEV)
+    ws = (torch.empty(splits * T * H * Vc, device=DEV), torch.empty(splits * T * H * 2, device=DEV))
     L.latent_attention(q, cache.to(dt).to(DEV), bt.to(DEV), torch.tensor(tok_slot, **i32), torch.tensor(pos, **i32), torch.tensor(row0, **i32),
-                       torch.tensor(rows, **i32), len(row0), bm, H, T, scale, out, n_splits=splits, workspace=ws)
-    assert rel(out, torch.cat(want).reshape(T, -1)) < (6e-3 if dt == BF16 else 5e-6)
+                       torch.tensor(rows, **i32), len(row0), bm, H, T, scale, out, n_splits=splits, workspace=ws, **(dict(window=window) if window else {}))
+    assert rel(out.view(T, H, Vc)[..., :V], torch.cat(want)) < (6e-3 if dt == BF16 else 5e-6)
 
 
-@pytest.mark.parametrize("H,D,V,pos0,T", [(2, 64, 64, 0, 128), (3, 32, 48, 0, 300), (2, 128, 64, 77, 131), (1, 20, 128, 512, 130), (4, 128, 128, 1, 257)])
-def test_expanded_attention(H, D, V, pos0, T):
-    """The flash kernel on expanded rows: a key that stands out at tile edges, at the start, and at the query itself; later keys unseen."""
+@pytest.mark.parametrize("H,D,V,pos0,T,window", [(2, 64, 64, 0, 128, None), (3, 32, 48, 0, 300, None), (2, 128, 64, 77, 131, None), (1, 20, 128, 512, 130, None), (4, 128, 128, 1, 257, None),
+                                                 (2, 64, 64, 30, 300, 65), (2, 80, 64, 0, 290, 1), (1, 100, 100, 200, 140, 128), (2, 192, 128, 0, 300, None), (3, 144, 64, 33, 259, 70), (2, 192, 128, 400, 128, 129),
+                                                 (1, 160, 40, 0, 129, 1000)])
+def test_expanded_attention(H, D, V, pos0, T, window):
+    """The flash kernel on expanded rows: a key that stands out at tile edges, at the start, at the query itself, and at the window's edge; later
+    and earlier keys unseen."""
     L, r = ops(), gen(T)
     Dp, Vp, S, scale = (D + 63) // 64 * 64, (V + 63) // 64 * 64, pos0 + T, 0.17
     k, v, q, gate = r(S, H, D).to(BF16), r(S, H, V).to(BF16), r(T, H, D, scale=D ** -0.5), r(T, H)
     marks = [m for m in (0, 1, 63, 64, 127, 128, 255, 256, S - 1) if m < S]
     for t in range(T):
         for h in range(H):
-            j = marks[(t + h) % len(marks)]                  # also keys the query must not see
+            edges = [pos0 + t - d for d in (window - 1, window) if pos0 + t >= d] if window else []
+            j = (marks + edges)[(t + h) % (len(marks) + len(edges))]                  # also keys the query must not see
             q[t, h] += k[j, h].float() * (12 / scale / D)
     kv = torch.zeros(S, H * (Dp + Vp), dtype=BF16)
     kv[:, :H * Dp].view(S, H, Dp)[:, :, :D] = k
@@ -264,10 +340,11 @@ def test_expanded_attention(H, D, V, pos0, T):
     qp = torch.empty(T, H * Dp, dtype=BF16, device=DEV)
     L.head_rows(q.reshape(T, H * D).to(DEV), H, D, Dp, qp)
     out = torch.zeros(T, H * V + 3, dtype=BF16, device=DEV)
-    L.rows_attention(qp, kv.to(DEV), S, pos0, H, Dp, Vp, V, scale, out, gate=gate.to(DEV))
+    L.rows_attention(qp, kv.to(DEV), S, pos0, H, Dp, Vp, V, scale, out, gate=gate.to(DEV), **(dict(window=window) if window else {}))
     L.check_waits()
     s = torch.einsum("thd,jhd->htj", q.to(BF16).to(F64), k.to(F64)) * scale
-    s = s.masked_fill(torch.arange(S)[None, None] > (pos0 + torch.arange(T))[None, :, None], -math.inf)
+    i, j = (pos0 + torch.arange(T))[None, :, None], torch.arange(S)
+    s = s.masked_fill((j > i) | (i - j >= (window or 1 << 30)), -math.inf)
     want = torch.einsum("htj,jhv->thv", torch.softmax(s, -1), v.to(F64)) / (1 + torch.exp(-gate.to(F64)))[:, :, None]
     assert rel(out[:, :H * V], want.reshape(T, -1)) < 6e-3 and not out[:, H * V:].any()
 
@@ -297,6 +374,33 @@ def test_latent_write_and_embed(dt):
     table, h = r(11, 24).to(dt).to(DEV), torch.zeros(5, 20, device=DEV)
     L.embed(table, torch.tensor([0, 10, 3, 3, 9], dtype=torch.int32, device=DEV), h, 5)
     assert torch.equal(h, table[[0, 10, 3, 3, 9], :20].float())
+
+
+@pytest.mark.parametrize("dt", TYPES)
+@pytest.mark.parametrize("H,D,P,R", [(4, 48, 16, 96), (3, 12, 2, 25), (20, 128, 64, 512), (1, 7, 6, 33)])
+@pytest.mark.parametrize("T", [7, 90])
+def test_latent_rows_with_positions(dt, H, D, P, R, T):
+    """Norm of the latent, rotation of the key part behind it and of every head's query part in place; positions far out, a row without a place."""
+    L, r = ops(), gen(R)
+    Rc, amp = (R + P + 31) // 32 * 32, 1.21
+    proj, w, q = r(T, 5 + R + P), r(R), r(T, H * (D + P))
+    cache = torch.full((8, 1, 16, Rc), 7.0, device=DEV).to(dt)
+    slot, pos = torch.tensor([0, 15, 16, 63, -1, 31, 40] + list(range(64, T + 57))), torch.tensor([0, 1, 77, 500, 3, 4099, 30000] + list(range(7, T)))
+    slot[slot >= 128] = -1
+    f = torch.tensor([500.0 ** (-2 * i / P) for i in range(P // 2)], dtype=torch.float32)
+    i32, qd, fd = dict(dtype=torch.int32, device=DEV), q.to(DEV), f.to(DEV)
+    L.latent_write(proj.to(DEV)[:, 5:], w.to(DEV), 1e-4, R, slot.to(**i32), cache, T, rot=(pos.to(**i32), fd, amp), q=qd, heads=H)
+    c = plain.rms(proj[:, 5:5 + R].to(F64), 1e-4) * w.to(F64)
+    kr = amp * plain.rotate_pairs(proj[:, None, 5 + R:].to(F64), f.to(F64), pos)[:, 0]
+    qw = q.to(F64).view(T, H, D + P)
+    qw = torch.cat([qw[..., :D], amp * plain.rotate_pairs(qw[..., D:], f.to(F64), pos)], -1)
+    rows = cache.view(-1, Rc)
+    for t, s in enumerate(slot.tolist()):
+        tol = (5e-3 if dt == BF16 else 1e-6) + 1.2e-7 * int(pos[t])          # fp32 angles
+        assert rel(qd[t].view(H, -1), qw[t]) < 1e-6 + 1.2e-7 * int(pos[t])
+        if s >= 0:
+            assert rel(rows[s, :R], c[t]) < tol and rel(rows[s, R:R + P], kr[t]) < tol and not rows[s, R + P:].any()
+    assert int((rows == 7).all(1).sum()) == 128 - int((slot >= 0).sum())
 
 
 # ---- norms in front of the sublayers -------------------------------------------------------------------------------------------
@@ -655,6 +759,50 @@ def test_two_maps_fused_decode(H, G, D, V, chunk, page, splits):
     assert rel(got, c.want) < 1.5e-2
 
 
+@pytest.mark.parametrize("dt", TYPES)
+@pytest.mark.parametrize("fused", [False, True])
+@pytest.mark.parametrize("H,G,D,V", [(6, 2, 20, 12), (8, 4, 64, 48), (40, 1, 32, 128)])
+def test_mixed_values_and_scaled_angles(dt, fused, H, G, D, V):
+    """The first layer's values are kept as they are and a share of them joins the later ones' before they are cached; cosine and sine times a factor."""
+    if fused and dt == F32:
+        pytest.skip("bf16 only")
+    L, r = ops(), gen(H * D)
+    c = attention_case(H, G, D, V, 40, 0, 16, [(p, 1) for p in (0, 5, 15, 16, 90, 300)], dt, seed=4, q_norm=False)
+    m, T, share = c.m, c.T, 0.35
+    m.rot_scale = 1.3
+    row0, rows = c.tiles(1)
+    first = torch.full((T, G * V), float("nan"), device=DEV)
+    own = []
+    for layer, lam in enumerate((None, share)):
+        proj, kc, vc = r(T, (H + G) * D + G * V), c.kc.clone(), c.vc.clone()
+        v = proj[:, (H + G) * D:].to(F64)
+        own.append(v)
+        if fused:
+            L.gqa_decode(m, proj.to(DEV), kc, vc, c.bt, c.tok_slot, c.pos, (row0, rows, row0.numel()), 2, torch.zeros(T, H * V, dtype=BF16, device=DEV), T, mix=(first, lam))
+        else:
+            q = torch.zeros(T, H * m.Dc, device=DEV).to(dt)
+            L.gqa_prepare(m, proj.to(DEV), kc, vc, c.bt, c.tok_slot, c.pos, c.slot, q, T, mix=(first, lam))
+            want = 1.3 * plain.rotate_half(proj[:, :H * D].to(F64).view(T, H, D), m.rot, m.base, c.pos.cpu())
+            want[..., m.rot:] /= 1.3
+            assert rel(q.view(T, H, m.Dc)[..., :D], want) < (6e-3 if dt == BF16 else 5e-5)
+        assert rel(first, own[0]) < 1e-7
+        v = (v if lam is None else (1 - lam) * v + lam * own[0]).view(T, G, V)
+        k = 1.3 * plain.rotate_half(proj[:, H * D:(H + G) * D].to(F64).view(T, G, D), m.rot, m.base, c.pos.cpu())
+        k[..., m.rot:] /= 1.3
+        for t in range(T):
+            s = int(c.slot[t])
+            assert rel(vc[s // 16, :, s % 16, :V], v[t]) < (5e-3 if dt == BF16 else 1e-6) and rel(kc[s // 16, :, s % 16, :D], k[t]) < (6e-3 if dt == BF16 else 5e-5)
+
+
+@pytest.mark.parametrize("rot", [{"dims": 12, "base": 1e4, "scaling": {"factor": 8.0, "original": 64, "fast": 32.0, "slow": 1.0}}, {"dims": 64, "base": 5e5, "scaling": {"factor": 4.0, "original": 8192, "fast": 32, "slow": 1}},
+                                 {"dims": 32, "base": 100.0, "scaling": {"factor": 2.0, "original": 40, "fast": 1.0, "slow": 1.0}}, {"dims": 8, "base": 300.0}, {"dims": 2, "base": 1e4, "scaling": {"factor": 16.0,
+                                  "original": 4096, "fast": 8.0, "slow": 0.25}}, {"dims": 48, "base": 1e6, "scaling": {"factor": 1.0, "original": 10, "fast": 32.0, "slow": 1.0}}])
+def test_yarn_frequencies(rot):
+    from distributed_llm_pipeline_b200.models.mixers import rotation
+    (f, amp), (want, amp2) = rotation(rot), plain.yarn_rotation(rot)
+    assert rel(f, want) < 1e-12 and abs(amp - amp2) < 1e-12 and (amp == 1) == (rot.get("scaling", {"factor": 1})["factor"] == 1)
+
+
 @pytest.mark.parametrize("dims,base,scaling", [(12, 2.5e5, (8.0, 1.0, 4.0, 2048)), (64, 1e4, (4.0, 1.0, 4.0, 64)), (2, 500.0, None), (128, 1e6, (32.0, 0.5, 1.5, 8192))])
 def test_rotation_frequencies(dims, base, scaling):
     from distributed_llm_pipeline_b200.models.mixers import rotation_frequencies
@@ -667,7 +815,7 @@ def test_rotation_frequencies(dims, base, scaling):
 @pytest.mark.parametrize("dt", TYPES)
 @pytest.mark.parametrize("T", [1, 3, 4, 7, 60])
 @pytest.mark.parametrize("K,groups,pair,gate", [(384, 4, 96, 0), (2048, 16, 128, 0), (72, 6, 12, 0), (384, 1, 0, 1), (2048, 1, 0, 1), (60, 1, 0, 1), (128, 2, 0, 2), (4096, 8, 0, 2), (30, 3, 0, 2),
-                                                (256, 2, 128, 1), (40, 5, 8, 2)])
+                                                (256, 2, 128, 1), (40, 5, 8, 2), (384, 3, 0, 3), (2048, 16, 0, 3), (60, 5, 0, 3)])
 def test_rows_behind_a_mixer(dt, T, K, groups, pair, gate):
     """Difference of two maps, norm in groups, gate on either side of it, in front of a product."""
     L, r = ops(), gen(K + T)
@@ -683,8 +831,8 @@ def test_rows_behind_a_mixer(dt, T, K, groups, pair, gate):
     if gate == 2:
         v = v * plain.silu(gate_cols)
     v = plain.grouped_norm(v, w2.to(F64).repeat(K // w2.numel()), groups, eps)
-    if gate == 1:
-        v = v * plain.sigmoid(gate_cols)
+    if gate in (1, 3):
+        v = v * (plain.sigmoid if gate == 1 else plain.silu)(gate_cols)
     gd = g.to(DEV)[:, 4:4 + K] if gate else None
     xd, w2d, wd = x.to(DEV), w2.to(DEV), w.to(DEV)
     st = L.row_stage(xd, K, Kp, eps, w2=w2d, groups2=groups, pair=pair, lam=lam, g=gd, gate=gate)
@@ -774,15 +922,105 @@ def test_scalar_decay_segments_and_carried_state(form, H, hpg, D, V, rows, steps
             assert rel(state[slots[i]], want[i][1]) < tol
 
 
+def delta_case(H, G, D, V, lens, seed, rows):
+    """Rows, gates and what they must give.  Among random tokens: keys that return (their value is corrected, not added), a token that forgets
+    everything, stretches that forget nothing, tokens that write nothing or all."""
+    r = gen(seed)
+    x = [r(t, 2 * G * D + H * V) for t in lens]
+    a, b, bias, a_log = [r(t, H, scale=2.0) - 3 for t in lens], [r(t, H, scale=2.0) for t in lens], r(H), r(H)
+    for i, t in enumerate(lens):
+        x[i][3::5, G * D:2 * G * D] = x[i][0, G * D:2 * G * D]            # one key again and again
+        x[i][4::9, :G * D] = x[i][0, G * D:2 * G * D] * 3                 # and queries for it
+        a[i][40::97] = 60.0
+        a[i][50:90] = -60.0
+        b[i][1::6] = 40.0
+        b[i][2::6] = -40.0
+        x[i] = x[i].to(rows)
+    want = []
+    for i, t in enumerate(lens):
+        q, k, v = x[i].to(F64).split([G * D, G * D, H * V], 1)
+        q, k = (plain.unit(y.reshape(t, G, D)).repeat_interleave(H // G, 1) for y in (q, k))
+        f = torch.exp(-torch.exp(a_log.to(F64)) * plain.softplus(a[i].to(F64) + bias.to(F64)))
+        want.append(plain.delta_scan(q * D ** -0.5, k, v.reshape(t, H, V), f, plain.sigmoid(b[i].to(F64))))
+    return x, a, b, bias, -torch.exp(a_log), want
+
+
+@pytest.mark.parametrize("form,H,G,D,V,rows", [("scan", 3, 3, 20, 10, F32), ("scan", 4, 2, 64, 64, BF16), ("scan", 2, 1, 300, 12, F32), ("scan", 2, 2, 160, 40, BF16), ("scan", 2, 1, 128, 128, F32),
+                                               ("chunks", 3, 1, 20, 10, BF16), ("chunks", 4, 2, 64, 64, BF16), ("chunks", 2, 2, 128, 128, BF16), ("chunks", 2, 1, 100, 33, BF16), ("chunks", 1, 1, 8, 130, BF16),
+                                               ("chunks", 6, 2, 48, 72, BF16), ("single", 3, 3, 20, 12, F32), ("single", 4, 1, 64, 64, BF16), ("single", 2, 2, 128, 128, F32), ("single", 2, 1, 256, 72, F32)])
+def test_delta_rule_segments_and_carried_state(form, H, G, D, V, rows):
+    """Ragged segments, some continuing a state, in portions of several sizes against the whole sequence."""
+    L = ops()
+    lens = [297, 1, 2, 140, 64] if form != "single" else [60, 1, 2, 53, 17]
+    x, a, b, bias, log_decay, want = delta_case(H, G, D, V, lens, D + H, rows)
+    slots, i32 = [4, 0, 6, 2, 3], dict(dtype=torch.int32, device=DEV)
+    state = torch.full((7, H, D, V), float("nan"), device=DEV)              # a new sequence must not read what its slot held
+    got = [[] for _ in lens]
+    for cut in portions(lens, [1] * 60 if form == "single" else (33, 2, 1, 3, 17, 64, 5, 130, 100)):
+        cat = lambda src: torch.cat([src[i][lo:lo + n] for i, lo, n in cut]).to(DEV)
+        proj = cat(x)
+        ends = torch.tensor([n for _, _, n in cut]).cumsum(0).tolist()
+        segs = [(hi - n, hi) for (_, _, n), hi in zip(cut, ends)]
+        pos = torch.cat([torch.arange(lo, lo + n) for _, lo, n in cut]).to(**i32)
+        out, chunks = torch.zeros(len(pos), H * V + 2, device=DEV), None
+        if form == "chunks":
+            table, first = L.scan_chunk_table(segs, L.DELTA_CHUNK)
+            ws = [torch.full((n // 4,), float("nan"), device=DEV) for n in L.delta_workspace(len(table) // 2, H, G, D, V)]
+            chunks = (torch.tensor(table, **i32).view(-1, 2), torch.tensor(first, **i32), *ws)
+        L.delta((proj, proj[:, G * D:], proj[:, 2 * G * D:]), H // G, state, cat(a), cat(b), log_decay.to(DEV), bias.to(DEV), torch.tensor(segs, **i32),
+                torch.tensor([slots[i] for i, _, _ in cut], **i32), len(cut), pos, out, 1e-6, chunks=chunks, single=form == "single")
+        assert not out[:, H * V:].any()
+        for (i, _, _), o in zip(cut, out[:, :H * V].split([n for _, _, n in cut])):
+            got[i].append(o)
+    tol = 1e-5 if form != "chunks" else 2e-4          # (two bf16 parts of every fp32 operand)
+    for i in range(len(lens)):
+        n = sum(len(o) for o in got[i])
+        assert rel(torch.cat(got[i]), want[i][0][:n].reshape(n, -1)) < tol
+        if n == lens[i]:
+            assert rel(state[slots[i]], want[i][1]) < tol
+
+
+@pytest.mark.parametrize("H,G,D,V,taps", [(4, 2, 32, 32, 4), (3, 3, 20, 12, 1), (2, 1, 128, 64, 3), (6, 2, 64, 40, 6), (2, 1, 200, 8, 2)])
+def test_single_tokens_of_the_delta_rule_behind_a_convolution(H, G, D, V, taps):
+    """Convolution, gates and recurrence of single tokens in one launch, behind a portion that left state and ring; several sequences."""
+    L, r = ops(), gen(D + V)
+    ch = 2 * G * D + H * V
+    lens, slots, i32 = [25, 9, 14], [2, 0, 1], dict(dtype=torch.int32, device=DEV)
+    x, a, b = [r(t, ch) for t in lens], [r(t, H) - 2 for t in lens], [r(t, H) for t in lens]
+    w, bias, a_log = r(ch, taps, scale=taps ** -0.5), r(H), r(H)
+    state, ring = torch.full((3, H, D, V), float("nan"), device=DEV), torch.full((3, taps, ch), float("nan"), device=DEV)
+    wd, got = w.T.contiguous().to(DEV), [[] for _ in lens]
+    for cut in portions(lens, (1, 1, 5, 1, 1, 1, 1, 1, 1, 2, 1, 1, 1, 1, 1, 1, 1, 1, 1, 1, 1, 1)):
+        rows = torch.cat([torch.cat([x[i], a[i], b[i]], 1)[lo:lo + n] for i, lo, n in cut]).to(DEV)
+        xd, single = rows[:, :ch], all(n == 1 for _, _, n in cut)
+        ends = torch.tensor([n for _, _, n in cut]).cumsum(0).tolist()
+        segs, seg_slot = torch.tensor([(hi - n, hi) for (_, _, n), hi in zip(cut, ends)], **i32), torch.tensor([slots[i] for i, _, _ in cut], **i32)
+        pos = torch.cat([torch.arange(lo, lo + n) for _, lo, n in cut]).to(**i32)
+        out, src, kw = torch.zeros(len(pos), H * V, device=DEV), xd, {}
+        if single:
+            kw = dict(conv=L.conv_args(xd, wd, None, ring), single=True)
+        else:
+            src = L.conv_rows(xd, wd, None, ring, segs, seg_slot, len(cut), max(n for _, _, n in cut), pos, torch.zeros(len(pos), ch, device=DEV))
+        L.delta((src, src[:, G * D:], src[:, 2 * G * D:]), H // G, state, rows[:, ch:], rows[:, ch + H:], -torch.exp(a_log).to(DEV), bias.to(DEV), segs, seg_slot, len(cut), pos, out, 1e-6, **kw)
+        for (i, _, _), o in zip(cut, out.split([n for _, _, n in cut])):
+            got[i].append(o)
+    for i, t in enumerate(lens):
+        q, k, v = plain.silu(plain.causal_conv(x[i].to(F64), w.to(F64), torch.zeros(ch, dtype=F64))).split([G * D, G * D, H * V], 1)
+        q, k = (plain.unit(y.reshape(t, G, D)).repeat_interleave(H // G, 1) for y in (q, k))
+        f = torch.exp(-torch.exp(a_log.to(F64)) * plain.softplus(a[i].to(F64) + bias.to(F64)))
+        o, S = plain.delta_scan(q * D ** -0.5, k, v.reshape(t, H, V), f, plain.sigmoid(b[i].to(F64)))
+        assert rel(torch.cat(got[i]), o.reshape(t, -1)) < 1e-5 and rel(state[slots[i]], S) < 1e-5
+
+
 @pytest.mark.parametrize("dt", TYPES)
 @pytest.mark.parametrize("taps,ch", [(4, 256), (4, 37), (1, 20), (2, 130), (3, 64), (6, 48), (32, 10)])
 def test_convolution_of_portions(dt, taps, ch):
     """Portions down to one token against the whole sequence; the ring holds garbage when a sequence starts."""
     L, r = ops(), gen(taps + ch)
     lens, slots, i32 = [150, 1, 2, 70, 33], [4, 0, 6, 2, 3], dict(dtype=torch.int32, device=DEV)
-    x, w, b = [r(t, ch + 3) for t in lens], r(ch, taps), r(ch)
+    x, w, b = [r(t, ch + 3) for t in lens], r(ch, taps), r(ch) if ch % 2 == 0 else None
     ring = torch.full((7, taps, ch), float("nan"), device=DEV)
-    wd, bd, got = w.T.contiguous().to(DEV), b.to(DEV), [[] for _ in lens]
+    wd, bd, got = w.T.contiguous().to(DEV), b.to(DEV) if b is not None else None, [[] for _ in lens]
     for cut in portions(lens, (1, 2, 1, 1, 33, 2, 3, 64, 100)):
         rows = torch.cat([x[i][a:a + m] for i, a, m in cut]).to(DEV)
         ends = torch.tensor([m for _, _, m in cut]).cumsum(0).tolist()
@@ -794,7 +1032,7 @@ def test_convolution_of_portions(dt, taps, ch):
         for (i, _, _), o in zip(cut, out[:, :ch].split([m for _, _, m in cut])):
             got[i].append(o)
     for i in range(len(lens)):
-        want = plain.silu(plain.causal_conv(x[i][:, 3:].to(F64), w.to(F64), b.to(F64)))
+        want = plain.silu(plain.causal_conv(x[i][:, 3:].to(F64), w.to(F64), b.to(F64) if b is not None else torch.zeros(ch, dtype=F64)))
         assert rel(torch.cat(got[i]), want) < (5e-3 if dt == BF16 else 2e-6)
 
 
@@ -872,7 +1110,7 @@ def test_cuts_of_a_prompt(models, name, dtype):
 
 
 @pytest.mark.parametrize("dtype", ["bf16", "f32"])
-@pytest.mark.parametrize("name", ["odd", "wide", "single", "experts", "grouped", "loop", "broad", "hybrid", "scalar", "maps", "states"])
+@pytest.mark.parametrize("name", ["odd", "wide", "single", "experts", "grouped", "loop", "broad", "hybrid", "scalar", "maps", "states", "parallel", "deltas", "windows"])
 def test_mixed_batches_and_reused_slots(models, name, dtype):
     """Eleven unequal requests through four slots and a pool that holds about two of the long ones, in random portions beside single tokens."""
     from distributed_llm_pipeline_b200.serving.trace_runner import TraceRunner
@@ -907,7 +1145,7 @@ def test_mixed_batches_and_reused_slots(models, name, dtype):
 
 
 @pytest.mark.parametrize("dtype", ["bf16", "f32"])
-@pytest.mark.parametrize("name", ["odd", "experts", "grouped", "hybrid", "maps"])
+@pytest.mark.parametrize("name", ["odd", "experts", "grouped", "hybrid", "maps", "parallel", "deltas", "windows"])
 def test_long_decoding(models, name, dtype):
     """Hundreds of decoded tokens through captured graphs (several key-range splits), two sequences of different length together."""
     cfg, w, path = models[name]
@@ -921,12 +1159,12 @@ def test_long_decoding(models, name, dtype):
         lg = eng.step([(sids[0], [ids[0][200 + t]]), (sids[1], [ids[1][7 + t]])])
         got[0].append(lg[0])
         got[1].append(lg[1])
-    assert len(eng._graphs) >= (2 if name == "odd" else 1)
+    assert len(eng._graphs) >= (2 if name in ("odd", "windows") else 1)
     assert lm.error(torch.stack(got[0]), want[0][200:530]) < LIMIT[dtype]
     assert lm.error(torch.stack(got[1]), want[1][7:337]) < LIMIT[dtype]
 
 
-@pytest.mark.parametrize("name", ["odd", "attention", "experts", "loop", "hybrid", "scalar"])
+@pytest.mark.parametrize("name", ["odd", "attention", "experts", "loop", "hybrid", "scalar", "parallel", "windows"])
 def test_far_token_decides(models, name):
     """The head reads what one far token left: changing it must move the logits as in the plain model, from prompts and from decoding."""
     cfg, w, path = models[name]
@@ -946,7 +1184,7 @@ def test_far_token_decides(models, name):
         assert (d - want).abs().max() < 2e-3 * max(1e-1, float(want.abs().max())), place
 
 
-@pytest.mark.parametrize("name", ["odd", "wide", "recurrent", "experts", "grouped", "hybrid", "maps", "states"])
+@pytest.mark.parametrize("name", ["odd", "wide", "recurrent", "experts", "grouped", "hybrid", "maps", "states", "parallel", "deltas", "windows"])
 @pytest.mark.parametrize("dtype", ["bf16", "f32"])
 def test_greedy_generation_through_the_scheduler(models, name, dtype):
     from distributed_llm_pipeline_b200.serving.orchestrator import build_service
@@ -973,7 +1211,7 @@ def test_greedy_generation_through_the_scheduler(models, name, dtype):
         assert alone.output_ids == reqs[0].output_ids
 
 
-@pytest.mark.parametrize("name", ["odd", "experts", "hybrid"])
+@pytest.mark.parametrize("name", ["odd", "experts", "hybrid", "parallel"])
 def test_seeded_sampling_does_not_depend_on_the_batch(models, name):
     from distributed_llm_pipeline_b200.serving.orchestrator import build_service
     from distributed_llm_pipeline_b200.serving.sampler import SamplingParams
@@ -989,7 +1227,7 @@ def test_seeded_sampling_does_not_depend_on_the_batch(models, name):
     assert reqs[0].output_ids == a.output_ids
 
 
-@pytest.mark.parametrize("name", ["odd", "experts", "hybrid"])
+@pytest.mark.parametrize("name", ["odd", "experts", "hybrid", "parallel"])
 def test_state_copy_session_and_rollback(models, name, tmp_path):
     from distributed_llm_pipeline_b200.utils.session import load_sequence, save_sequence
     cfg, w, path = models[name]
@@ -1008,7 +1246,7 @@ def test_state_copy_session_and_rollback(models, name, tmp_path):
     assert (eng.memory_breakdown()["recurrent_state"] > 0) == (name != "experts")
 
 
-@pytest.mark.parametrize("name", ["wide", "experts", "grouped", "loop", "hybrid", "scalar", "maps", "states"])
+@pytest.mark.parametrize("name", ["wide", "experts", "grouped", "loop", "hybrid", "scalar", "maps", "states", "parallel", "deltas", "windows"])
 def test_residual_after_every_layer(models, name):
     cfg, w, path = models[name]
     ids = lm.tokens(cfg, 50)
@@ -1020,7 +1258,7 @@ def test_residual_after_every_layer(models, name):
         assert all(rel(got[i], after[i]) < tol for i in range(len(after)))
 
 
-@pytest.mark.parametrize("name", ["odd", "experts", "hybrid"])
+@pytest.mark.parametrize("name", ["odd", "experts", "hybrid", "parallel"])
 def test_trace_run_program(models, name, tmp_path):
     import json
     import os
@@ -1042,7 +1280,7 @@ def test_trace_run_program(models, name, tmp_path):
         assert not (tmp_path / "1.f32").exists()
 
 
-@pytest.mark.parametrize("name", ["odd", "experts", "hybrid"])
+@pytest.mark.parametrize("name", ["odd", "experts", "hybrid", "parallel"])
 def test_command_line(models, name):
     import os
     import subprocess

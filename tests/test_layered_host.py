@@ -124,6 +124,47 @@ def test_hybrid_config_is_checked(tmp_path):
             load_weights(p, "cpu")
 
 
+def test_parallel_config_is_checked(tmp_path):
+    cfg = lm.CONFIGS["parallel"]
+    p = lm.write(str(tmp_path / "m"), cfg, lm.weights(cfg))
+    d = open_model_dir(p).cfg
+    assert (d.n_layer, d.norm_type, d.rms_eps, d.embedding_scale, d.logit_scale, d.parallel_residual) == (7, "rms", 3e-4, 3.0, 1.0, True)
+    assert [s.mixer.get("v_mix") for s in d.layers if s.type == "attention"] == [False, "first", "later"]
+    for name in ("parallel", "deltas", "windows"):
+        c = lm.CONFIGS[name]
+        assert open_model_dir(lm.write(str(tmp_path / name), c, lm.weights(c))).cfg.n_params() == sum(t.numel() for t in lm.weights(c).values())
+    de, at, la = lm.delta, lm.biased_attention, lm.low_rank_latent
+    for bad in ([de(4, 3, 8, 8, 3)], [de(4, 2, 8, 8, 33)], [de(4, 2, 8, 8, 0)], [at(6, 4, 8, 8, 0.3, 8, 4)], [at(2, 2, 8, 8, 0.3, 10, 4)], [at(2, 2, 8, 8, 0.3, 3, 4)], [at(2, 2, 8, 8, 0.3, 8, 0)], [at(2, 2, 8, 8, "1", 8, 4)],
+                [at(2, 2, 8, 8, 0.3, 8, 4, yarn=(8.0, 64, 32.0))], [at(2, 2, 8, 8, 0.3, 8, 4, yarn=(0.0, 64, 32.0, 1.0))], [at(2, 2, 8, 8, 0.3, 8, 4), at(2, 1, 8, 8, 0.3, 8, 4)], [la(2, 8, 3, 8, 8, 8, 0.3, 4)],
+                [la(2, 8, 4, 8, 0, 8, 0.3, 4)], [{**la(2, 8, 4, 8, 8, 8, 0.3, 4), "type": "mamba2"}], [de(2, 2, 8, 8, 3, ff=0)], [{**de(2, 2, 8, 8, 3), "mlp": lm.shared_moe(4, 2, 8, 8)}]):
+        json.dump({**cfg, "layers": bad}, open(os.path.join(p, "config.json"), "w"))
+        with pytest.raises(ValueError):
+            open_model_dir(p)
+    bad = la(2, 8, 4, 8, 8, 8, 0.3, 4)
+    bad["mixer"]["rot"]["dims"] = 2
+    json.dump({**cfg, "layers": [bad]}, open(os.path.join(p, "config.json"), "w"))
+    with pytest.raises(ValueError):
+        open_model_dir(p)
+    w = lm.weights(cfg)
+    for name in ("l0.mix.q.b", "l0.mix.o", "l0.mlp.act", "l0.mlp.down", "l1.mix.dq", "l1.mix.dq.norm", "l1.mix.uq", "l1.mix.dkv", "l1.mix.dkv.norm", "l1.mlp.up", "l2.mix.g", "l2.mix.k.conv", "l2.mix.a", "l2.mix.dt_bias",
+                 "l2.mix.A_log", "l2.mix.norm", "l2.norm1", "l5.mix.v.b", "final.norm"):
+        lm.write(p, cfg, {**w, name: w[name][:-1]})
+        with pytest.raises(ValueError):
+            load_weights(p, "cpu")
+
+
+def test_joined_products_are_stacked_once(tmp_path):
+    """Mixer and feed-forward share their matrices' memory; a layer without a feed-forward keeps its own."""
+    cfg = lm.CONFIGS["parallel"]
+    w = load_weights(lm.write(str(tmp_path / "m"), cfg, lm.weights(cfg)), "cpu", dtype="f32")
+    for i, s in enumerate(cfg["layers"]):
+        lw = w.layers[i]
+        assert (lw.joined is not None) == (s["mlp"] is not None) and lw.mlp is None and lw.norm2 is None
+        if lw.joined is not None:
+            assert lw.joined.w_in is lw.mixer.w_in and lw.joined.w_out is lw.mixer.w_out and lw.proj_cols % 32 == 0
+            assert lw.mixer.w_in.N == lw.proj_cols + s["mlp"]["ff"] and lw.mixer.w_out.K >= s["mlp"]["ff"] + s["mixer"]["heads"] * s["mixer"]["vdim"]
+
+
 def test_loading_checks_shapes_and_can_be_cancelled(tmp_path):
     cfg = lm.CONFIGS["odd"]
     w = lm.weights(cfg)
@@ -158,7 +199,7 @@ def test_prompt_portions_and_single_tokens(model, name):
     assert len(eng.kv.free) == eng.kv.n_pages
 
 
-@pytest.mark.parametrize("name", ["odd", "experts", "hybrid", "scalar"])
+@pytest.mark.parametrize("name", ["odd", "experts", "hybrid", "scalar", "parallel"])
 def test_batches_larger_than_the_buffers_and_reuse(model, name):
     cfg, w, eng, _ = model(name, max_batch_tokens=24, n_pages=12)
     run = TraceRunner(eng)
@@ -221,7 +262,7 @@ def test_attention_only_models_can_roll_back(model, name):
     assert lm.error(eng.prefill(sid, ids[12:], all_logits=True), plain.forward(cfg, w, ids)[0][12:]) < TOL
 
 
-@pytest.mark.parametrize("name", ["odd", "experts", "hybrid"])
+@pytest.mark.parametrize("name", ["odd", "experts", "hybrid", "parallel"])
 def test_session_file(model, name, tmp_path):
     from distributed_llm_pipeline_b200.utils.session import load_sequence, save_sequence
     cfg, w, eng, _ = model(name)
@@ -287,7 +328,7 @@ def check_greedy(cfg, w, prompt, out, min_gap):
         assert row.max() - row[t] < min_gap, i
 
 
-@pytest.mark.parametrize("name", ["odd", "recurrent", "experts", "hybrid"])
+@pytest.mark.parametrize("name", ["odd", "recurrent", "experts", "hybrid", "parallel"])
 def test_scheduler_mixes_prompts_and_decoding(model, name):
     cfg, w, eng, _ = model(name, n_seqs=3)
     sched = Scheduler(eng, IdTokenizer(cfg["vocab"]), n_batch=16, n_slots=3)

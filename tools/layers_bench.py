@@ -1,6 +1,7 @@
 #!/usr/bin/env python
 """Throughput of layer-list models beside the closest GGUF model of equal size, and every kernel of both against its roofline
-(`bench.py --layers`): Talizen beside a Llama, Vozinex beside a Qwen3-MoE, Nifalorn beside a Vozinex (tools/layers_bench_nifalorn.py).
+(`bench.py --layers`): Talizen beside a Llama, Vozinex beside a Qwen3-MoE, Nifalorn beside a Vozinex (tools/layers_bench_nifalorn.py),
+Rigalorn beside a Nifalorn (tools/layers_bench_rigalorn.py).
 
 Random weights at sizes of real models' layers.  Model numbers are device-timed with CUDA events around whole forwards (prefill) and
 blocks of graph replays (decode); a step streams weights larger than L2.  Kernel numbers: a captured graph of launches that rotate
@@ -21,6 +22,7 @@ sys.path[:0] = [REPO, os.path.join(REPO, "tools")]
 import torch  # noqa: E402
 
 import layers_bench_nifalorn as hybrid  # noqa: E402
+import layers_bench_rigalorn as parallel  # noqa: E402
 
 DEV = "cuda:0"
 SIZES = {   # name: (width, heads, head size, latent rank, ff, layers)
@@ -499,24 +501,29 @@ def moe_kernel_numbers(size: str, T: int = 2048):
 
 def main(argv=None) -> dict:
     ap = argparse.ArgumentParser(description=__doc__.split("\n")[0])
-    ap.add_argument("--sizes", default=",".join([*SIZES, *MOE_SIZES, *hybrid.HYBRID_SIZES]))
+    ap.add_argument("--sizes", default=",".join([*SIZES, *MOE_SIZES, *hybrid.HYBRID_SIZES, *parallel.PARALLEL_SIZES]))
     ap.add_argument("--no-models", action="store_true", help="kernels only")
     ap.add_argument("--no-kernels", action="store_true", help="whole models only")
     a = ap.parse_args(argv)
-    res = {"metric": "layers_bench", "unit": "tok/s", "data": "synthetic (random weights and token ids)", "dtype": "bf16 (talizen, vozinex, nifalorn) / fp16 (llama, qwen3moe)", "sizes": {}}
+    res = {"metric": "layers_bench", "unit": "tok/s", "data": "synthetic (random weights and token ids)", "dtype": "bf16 (talizen, vozinex, nifalorn, rigalorn) / fp16 (llama, qwen3moe)", "sizes": {}}
     for size in a.sizes.split(","):
         moe = size in MOE_SIZES
-        if size in hybrid.HYBRID_SIZES:
-            names = ("width", "lightning_heads", "mamba2_heads", "heads", "kv_heads", "experts", "experts_per_token", "ff", "shared_ff", "layers", "chunk")
-            r = {"config": {**dict(zip(names, hybrid.HYBRID_SIZES[size])), "vocab": VOCAB}}
+        if size in hybrid.HYBRID_SIZES or size in parallel.PARALLEL_SIZES:
+            if size in hybrid.HYBRID_SIZES:
+                names = ("width", "lightning_heads", "mamba2_heads", "heads", "kv_heads", "experts", "experts_per_token", "ff", "shared_ff", "layers", "chunk")
+                values, models, kernels = hybrid.HYBRID_SIZES[size], (("nifalorn", hybrid.nifalorn), ("vozinex", hybrid.vozinex)), hybrid.kernel_numbers
+            else:
+                names = ("width", "heads", "kv_heads", "delta_kv_heads", "rot_dim", "q_rank", "kv_rank", "ff", "layers", "window")
+                values, models, kernels = parallel.PARALLEL_SIZES[size], (("rigalorn", parallel.rigalorn), ("nifalorn", parallel.nifalorn)), parallel.kernel_numbers
+            r = {"config": {**dict(zip(names, values)), "vocab": VOCAB}}
             if not a.no_models:
-                for name, make in (("nifalorn", hybrid.nifalorn), ("vozinex", hybrid.vozinex)):
+                for name, make in models:
                     w = make(size)
                     r[name] = {"weights_gb": round(w.nbytes() / 1e9, 3), **model_numbers(w)}
                     del w
                     torch.cuda.empty_cache()
             if not a.no_kernels:
-                r["kernels"], res["peaks"] = hybrid.kernel_numbers(size, graph_us, copies, peaks)
+                r["kernels"], res["peaks"] = kernels(size, graph_us, copies, peaks)
             res["sizes"][size] = r
             continue
         names = ("width", "heads", "kv_heads", "head_dim", "experts", "experts_per_token", "ff", "layers", "window", "keep_first") if moe else \

@@ -36,6 +36,9 @@ def weights(cfg, norm_b, vec, shapes):
     norm = Norm(torch.ones(E, device=DEV), torch.zeros(E, device=DEV) if norm_b else None)
     layers = {i: LayeredLayer(MIXERS[s.type](s.mixer, get(s.type), DEV, torch.bfloat16, 1e-5), norm, MLPS[s.mlp["kind"]](s.mlp, get("mlp"), DEV, torch.bfloat16, E), norm)
               for i, s in enumerate(cfg.layers)}
+    if cfg.parallel_residual:
+        for lw in layers.values():
+            lw.join()
     tab = [DeviceWeight(GGMLType.BF16, VOCAB, E, [mat(VOCAB, E)]) for _ in range(2)]
     return LayeredWeights(cfg, layers, range(len(layers)), 0, 1, tab[0], norm.w, tab[1], (0, VOCAB), None, out_norm_b=norm.b)
 
